@@ -130,6 +130,8 @@ class KVSpec:
     head_dim: int
     dtype: torch.dtype = torch.bfloat16
     fp8: bool = False    # e4m3 cache: a page row holds Hkv * D value bytes + one fp32 scale per kv head (padded to 16)
+    # latent cache: one row of this many values per layer run that serves as key and value alike (no V tensors)
+    latent_widths: Optional[List[int]] = None
 
     @property
     def row_width(self) -> int:
@@ -144,6 +146,8 @@ class KVSpec:
 
     @property
     def cell_bytes(self) -> int:
+        if self.latent_widths is not None:
+            return sum(self.latent_widths) * torch.empty((), dtype=self.dtype).element_size()
         return 2 * self.n_layers * self.row_width * torch.empty((), dtype=self.store_dtype).element_size()
 
 
@@ -171,13 +175,23 @@ def kv_rows_from_float(x: torch.Tensor, row_width: int) -> torch.Tensor:
 
 
 class KVPool:
-    """K and V as ``[layer, page, row]``; one row per token page (bf16 values, or the e4m3 layout of ``KVSpec``)."""
+    """K and V as ``[layer, page, row]``; one row per token page (bf16 values, or the e4m3 layout of ``KVSpec``).
+    Latent caches keep a list of ``[page, width]`` tensors in ``k``, one per layer run, and nothing in ``v``."""
 
     def __init__(self, spec: KVSpec, n_pages: int, device):
         self.spec = spec
         self.n_pages = n_pages
+        if spec.latent_widths is not None:
+            self.k = [torch.zeros(n_pages + 1, w, dtype=spec.dtype, device=device) for w in spec.latent_widths]
+            self.v = []
+            return
         self.k = torch.zeros(spec.n_layers, n_pages + 1, spec.row_width, dtype=spec.store_dtype, device=device)
         self.v = torch.zeros(spec.n_layers, n_pages + 1, spec.row_width, dtype=spec.store_dtype, device=device)
+
+    def write_latent(self, layer: int, locs: torch.Tensor, c: torch.Tensor) -> None:
+        """Rows ``c`` [T, <= width] of a latent cache; the padding columns stay zero."""
+        pool = self.k[layer]
+        pool[locs.long(), :c.shape[1]] = c.to(pool.dtype)
 
     def write(self, layer: int, locs: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> None:
         if self.spec.fp8:
@@ -191,7 +205,8 @@ class KVPool:
 
 @dataclass
 class StateSpec:
-    """Recurrent (Gated-DeltaNet) state per sequence row."""
+    """Recurrent state per sequence row: the last ``conv_width - 1`` inputs of a causal convolution and, for
+    Gated-DeltaNet layers, the temporal state (``n_heads`` 0: convolution inputs only)."""
     n_layers: int
     conv_dim: int
     conv_width: int

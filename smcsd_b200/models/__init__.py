@@ -1,4 +1,4 @@
-"""Model families: dense Llama-style decoders and Qwen3.5-style Gated-DeltaNet hybrids."""
+"""Model families: dense Llama-style decoders, Qwen3.5-style Gated-DeltaNet hybrids and Pasizen."""
 from __future__ import annotations
 
 import os
@@ -14,6 +14,8 @@ def build_model(spec, dtype=torch.bfloat16, device="cpu", tp_rank: int = 0, tp_s
     cfg = resolve_config(spec)
     if cfg.arch == "hybrid_gdn":
         from .hybrid_gdn import HybridGDNModel as Cls
+    elif cfg.arch == "pasizen":
+        from .pasizen import PasizenModel as Cls
     else:
         from .llama import LlamaModel as Cls
     m = Cls(cfg, dtype=dtype, device=device, tp_rank=tp_rank, tp_size=tp_size, max_positions=max_positions)

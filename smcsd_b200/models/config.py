@@ -1,9 +1,11 @@
 """Architecture descriptions: parsed from a HF ``config.json`` or built from presets.
 
-Two families are served, the ones the reference runs: dense Llama-style decoders and
+Three families are served.  Two are the ones the reference runs: dense Llama-style decoders and
 Qwen3.5-style hybrids that interleave Gated-DeltaNet layers with gated full attention
 (reference: README.md model list; parameter names checked against the HF
-implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).
+implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).  The third is Pasizen: latent attention without
+positions, a short convolution in front of every mixer, hyper-connected residual streams, PolyNorm or
+mixture-of-experts feed-forwards and layers that may be looped; its config.json spells every layer out.
 """
 from __future__ import annotations
 
@@ -13,9 +15,50 @@ from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
 
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention over a cached latent: ``kv_rank`` values per token, keys and values of all heads expanded from them."""
+    heads: int
+    dim: int                             # query / key size per head
+    vdim: int                            # value size per head
+    kv_rank: int
+    scale: float
+
+
+@dataclass(frozen=True)
+class GluSpec:
+    """Gated unit with clamped inputs (``limit``)."""
+    ff: int
+    limit: float
+
+
+@dataclass(frozen=True)
+class RouterSpec:
+    """Softmax router: the ``top`` best experts among those of the ``keep`` best of ``groups`` equal groups."""
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+
+
+@dataclass(frozen=True)
+class FeedForwardSpec:
+    kind: str                            # "dense" (PolyNorm) | "moe"
+    ff: int = 0
+    expert: Optional[GluSpec] = None
+    router: Optional[RouterSpec] = None
+    shared: Optional[GluSpec] = None
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: LatentAttentionSpec
+    mlp: Optional[FeedForwardSpec]
+
+
 @dataclass
 class ModelConfig:
-    arch: str = "llama"                  # "llama" | "hybrid_gdn"
+    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen"
     vocab_size: int = 32000
     hidden_size: int = 4096
     n_layers: int = 32
@@ -41,6 +84,11 @@ class ModelConfig:
     attn_output_gate: bool = False
     qk_norm: bool = False
     norm_plus_one: bool = False                    # RMSNorm weight stored as (w - 1)
+    # ---- layer-by-layer description (Pasizen) --------------------------------
+    layers: Optional[List[LayerSpec]] = None
+    loop: Optional[tuple] = None                   # (start, stop, times): these layers run ``times`` times in a row
+    streams: int = 1                               # hyper-connected copies of the residual stream
+    conv_taps: int = 1                             # short causal convolution in front of every mixer
     name: str = ""
 
     # ---- derived -------------------------------------------------------------
@@ -62,6 +110,16 @@ class ModelConfig:
         return self.layer_types[i]
 
     @property
+    def layer_runs(self) -> List[int]:
+        """Layer index of every layer run, in execution order (a looped layer appears once per pass; every pass owns
+        its own cache and state)."""
+        n = list(range(self.n_layers))
+        if not self.loop:
+            return n
+        a, b, times = self.loop
+        return n[:a] + n[a:b] * times + n[b:]
+
+    @property
     def attn_layers(self) -> List[int]:
         return [i for i in range(self.n_layers) if self.layer_type(i) == "full_attention"]
 
@@ -75,6 +133,8 @@ class ModelConfig:
 
     def param_count(self) -> int:
         d, f = self.hidden_size, self.ffn_size
+        if self.arch == "pasizen":
+            return self._layered_param_count()
         n = self.vocab_size * d * (1 if self.tie_embeddings else 2) + d
         for i in range(self.n_layers):
             n += 3 * d * f + 2 * d
@@ -87,13 +147,68 @@ class ModelConfig:
                 n += d * (2 * kd + vd) + d * vd + 2 * d * self.gdn_n_v_heads + vd * d
         return n
 
+    def _layered_param_count(self) -> int:
+        d, s = self.hidden_size, self.streams
+        n = 2 * self.vocab_size * d + self.max_position * d + d
+        glu = lambda g: 3 * g.ff * d
+        for L in self.layers:
+            m = L.mixer
+            n += d * (m.heads * (m.dim + m.vdim) + m.kv_rank) + m.kv_rank * (m.heads * (m.dim + m.vdim) + 1)
+            n += d * (1 + self.conv_taps) + 2 * s + s * s
+            if L.mlp is None:
+                continue
+            n += d + 2 * s + s * s
+            if L.mlp.kind == "dense":
+                n += 2 * d * L.mlp.ff + 4
+            else:
+                n += L.mlp.router.experts * (d + glu(L.mlp.expert)) + (glu(L.mlp.shared) if L.mlp.shared else 0)
+        return n
+
     # ---- construction ----------------------------------------------------------
+    @classmethod
+    def from_layered_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
+        """config.json of a Pasizen model: every layer with its mixer and feed-forward, the loop, the stream count."""
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            if e["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            m = e["mixer"]
+            mixer = LatentAttentionSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]))
+            f, mlp = e.get("mlp"), None
+            glu = lambda g: GluSpec(int(g["ff"]), float(g["limit"]))
+            if f is not None and f["kind"] == "dense":
+                mlp = FeedForwardSpec("dense", ff=int(f["ff"]))
+            elif f is not None and f["kind"] == "moe":
+                r, g = f["router"], f["router"].get("groups") or {"count": 1, "keep": 1}
+                router = RouterSpec(int(r["experts"]), int(r["top"]), int(g["count"]), int(g["keep"]))
+                if router.experts % router.groups or not 1 <= router.keep <= router.groups or \
+                        not 1 <= router.top <= router.keep * (router.experts // router.groups):
+                    raise ValueError(f"layer {i}: inconsistent router {router}")
+                mlp = FeedForwardSpec("moe", expert=glu(f["expert"]), router=router,
+                                      shared=glu(f["shared"]) if f.get("shared") else None)
+            elif f is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(LayerSpec(mixer, mlp))
+        lp = c.get("loop")
+        loop = (int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None
+        if loop and not (0 <= loop[0] <= loop[1] <= len(layers) and loop[2] >= 1):
+            raise ValueError(f"inconsistent loop {lp}")
+        eos = c.get("eos_token_id")
+        m0 = layers[0].mixer
+        return cls(arch="pasizen", vocab_size=int(c["vocab"]), hidden_size=int(c["width"]), n_layers=len(layers),
+                   n_heads=m0.heads, n_kv_heads=1, head_dim=m0.kv_rank, ffn_size=0, rms_eps=float(c["norm"]["eps"]),
+                   max_position=int(c["max_positions"]), layers=layers, loop=loop, streams=int(c["streams"]),
+                   conv_taps=int(c["canon"]["taps"]),
+                   eos_token_ids=[] if eos is None else ([eos] if isinstance(eos, int) else list(eos)))
+
     @classmethod
     def from_hf_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
         if "text_config" in c and isinstance(c["text_config"], dict):
             merged = dict(c["text_config"])
             merged.setdefault("architectures", c.get("architectures"))
             c = merged
+        if c.get("architecture") == "Pasizen":
+            return cls.from_layered_dict(c)
         archs = c.get("architectures") or []
         mt = (c.get("model_type") or "").lower()
         is_hybrid = "layer_types" in c and any(t == "linear_attention" for t in c["layer_types"])
@@ -194,6 +309,24 @@ def preset(name: str) -> ModelConfig:
                            layer_types=lt, gdn_n_k_heads=2, gdn_n_v_heads=4, gdn_head_k_dim=32,
                            gdn_head_v_dim=32, gdn_conv_width=4, partial_rotary=0.25, attn_output_gate=True,
                            qk_norm=True, norm_plus_one=True, rms_eps=1e-6, name="tiny-hybrid")
+    if n in ("pasizen-2048", "pasizen-1024"):
+        # random-init stand-ins with the layer sizes of a real small model, dense and expert layers alternating
+        d, H, ff = (2048, 16, 6144) if n.endswith("2048") else (1024, 8, 3072)
+        mixer = LatentAttentionSpec(heads=H, dim=128, vdim=128, kv_rank=256, scale=128 ** -0.5)
+        dense = LayerSpec(mixer, FeedForwardSpec("dense", ff=ff))
+        moe = LayerSpec(mixer, FeedForwardSpec("moe", expert=GluSpec(ff // 8, 7.0), router=RouterSpec(32, 4, 8, 4),
+                                               shared=GluSpec(ff // 4, 7.0)))
+        return ModelConfig(arch="pasizen", vocab_size=65536, hidden_size=d, n_layers=16, n_heads=H, n_kv_heads=1,
+                           head_dim=256, ffn_size=0, rms_eps=1e-6, max_position=16384, layers=[dense, moe] * 8,
+                           streams=4, conv_taps=4, name=n)
+    if n in ("tiny-pasizen",):
+        mixer = LatentAttentionSpec(heads=3, dim=40, vdim=24, kv_rank=48, scale=0.2)
+        dense = LayerSpec(mixer, FeedForwardSpec("dense", ff=200))
+        moe = LayerSpec(LatentAttentionSpec(2, 32, 56, 72, 0.15),
+                        FeedForwardSpec("moe", expert=GluSpec(40, 1.0), router=RouterSpec(8, 2, 4, 2), shared=GluSpec(72, 1.5)))
+        return ModelConfig(arch="pasizen", vocab_size=4096, hidden_size=136, n_layers=3, n_heads=3, n_kv_heads=1,
+                           head_dim=48, ffn_size=0, rms_eps=1e-6, max_position=2048, layers=[dense, moe, dense],
+                           loop=(1, 3, 2), streams=2, conv_taps=3, name="tiny-pasizen")
     raise KeyError(f"unknown preset {name!r}")
 
 

@@ -23,7 +23,7 @@ from typing import List, Optional
 import torch
 import torch.nn.functional as F
 
-from ..memory.pools import StateSpec
+from ..memory.pools import KVSpec, StateSpec
 from .config import ModelConfig
 from .layers import ExtendBatch, apply_rope, paged_attention_reference, rmsnorm, rope_table, swiglu
 from .llama import interleave_gate_up, split_gate_up
@@ -127,6 +127,9 @@ class HybridGDNModel:
         self.key_dim = self.gdn_k_heads * cfg.gdn_head_k_dim
         self.value_dim = self.gdn_v_heads * cfg.gdn_head_v_dim
         self.conv_dim = 2 * self.key_dim + self.value_dim
+
+    def kv_spec(self, dtype, fp8: bool = False) -> KVSpec:
+        return KVSpec(len(self.cfg.attn_layers), self.n_kv_heads, self.cfg.head_dim, dtype, fp8)
 
     def state_spec(self) -> StateSpec:
         c = self.cfg

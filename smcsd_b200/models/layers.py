@@ -122,3 +122,90 @@ def paged_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
 
 def swiglu(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return F.silu(gate.float()).mul(up.float()).to(gate.dtype)
+
+
+# ----------------------------------------------------------------------------- mechanisms of layered architectures
+def rms_unit(x: torch.Tensor, eps: float) -> torch.Tensor:
+    """fp32 ``x`` divided by its root mean square over the last dimension."""
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def short_conv(h: torch.Tensor, w: torch.Tensor, batch: ExtendBatch, history: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+    """Causal depthwise convolution of the new tokens of every sequence.  h [T, C] fp32, w [C, taps]; ``history``
+    [rows, C, taps - 1] holds the inputs before the first new token (oldest first) and is advanced in place."""
+    taps = w.shape[1]
+    out = torch.empty_like(h)
+    t0 = 0
+    for b, e in enumerate(batch.lens()):
+        if e == 0:
+            continue
+        r = rows[b]
+        seq = torch.cat([history[r].to(h.dtype), h[t0:t0 + e].t()], dim=1)          # [C, taps - 1 + e]
+        out[t0:t0 + e] = (seq.unfold(1, taps, 1) * w.to(h.dtype).unsqueeze(1)).sum(-1).t()
+        if taps > 1:
+            history[r] = seq[:, -(taps - 1):].to(history.dtype)
+        t0 += e
+    return out
+
+
+def latent_attention_reference(q: torch.Tensor, pool: torch.Tensor, block_table: torch.Tensor, batch: ExtendBatch,
+                               scale: float) -> torch.Tensor:
+    """Causal attention in latent space: q [T, H, R] (queries already multiplied by the key expansion), cached latents
+    ``pool`` [pages, >= R] read through the block table as keys and as values.  Returns fp32 [T, H, R]."""
+    T, H, R = q.shape
+    out = torch.empty(T, H, R, dtype=torch.float32, device=q.device)
+    pref = batch.prefix_lens_host if batch.prefix_lens_host is not None else batch.prefix_lens.tolist()
+    t0 = 0
+    for b, (p, e) in enumerate(zip(pref, batch.lens())):
+        if e == 0:
+            continue
+        L = p + e
+        c = pool[block_table[batch.rows[b].long(), :L].long()][:, :R].float()
+        s = torch.einsum("ehr,lr->hel", q[t0:t0 + e].float(), c) * scale
+        causal = torch.arange(L, device=q.device).unsqueeze(0) <= (p + torch.arange(e, device=q.device)).unsqueeze(1)
+        s = s.masked_fill(~causal, float("-inf"))
+        out[t0:t0 + e] = torch.einsum("hel,lr->ehr", torch.softmax(s, dim=-1), c)
+        t0 += e
+    return out
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """coef[0] N(z) + coef[1] N(z^2) + coef[2] N(z^3) + coef[3], N dividing a row by its root mean square (fp32)."""
+    z = z.float()
+    return coef[0] * rms_unit(z, eps) + coef[1] * rms_unit(z * z, eps) + coef[2] * rms_unit(z * z * z, eps) + coef[3]
+
+
+GLU_SIGMOID_SLOPE = 1.702
+
+
+def clamped_glu(gate: torch.Tensor, up: torch.Tensor, limit: float) -> torch.Tensor:
+    g = gate.float().clamp(max=limit)
+    u = up.float().clamp(-limit, limit)
+    return g * torch.sigmoid(GLU_SIGMOID_SLOPE * g) * (u + 1.0)
+
+
+def route_grouped(z: torch.Tensor, top: int, groups: int, keep: int):
+    """Router logits [T, E] -> (expert ids [T, top], weights [T, top]): softmax over all experts, the ``top`` best among
+    the experts of the ``keep`` groups with the largest single score, weights renormalised to one."""
+    s = torch.softmax(z.float(), dim=-1)
+    T, E = s.shape
+    if keep < groups:
+        g = s.view(T, groups, E // groups).amax(dim=-1)
+        drop = torch.ones(T, groups, dtype=torch.bool, device=z.device)
+        drop.scatter_(1, g.topk(keep, dim=-1).indices, False)
+        cand = s.masked_fill(drop.repeat_interleave(E // groups, dim=1), -1.0)
+    else:
+        cand = s
+    idx = cand.topk(top, dim=-1).indices
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(-1, keepdim=True) + 1e-20)
+
+
+def hyper_read(x: torch.Tensor, w_in: torch.Tensor) -> torch.Tensor:
+    """Sublayer input of the hyper-connected streams x [T, S, d]: sum_s w_in[s] x_s."""
+    return torch.einsum("tsd,s->td", x, w_in)
+
+
+def hyper_write(x: torch.Tensor, y: torch.Tensor, w_mix: torch.Tensor, w_out: torch.Tensor) -> torch.Tensor:
+    """New streams x_t' = sum_s w_mix[s, t] x_s + w_out[t] y."""
+    return torch.einsum("tsd,su->tud", x, w_mix) + w_out.view(1, -1, 1) * y.unsqueeze(1)

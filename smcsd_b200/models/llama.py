@@ -18,6 +18,7 @@ from typing import List, Optional
 
 import torch
 
+from ..memory.pools import KVSpec
 from .config import ModelConfig
 from .layers import ExtendBatch, apply_rope, paged_attention_reference, rmsnorm, rope_table, swiglu
 from .loader import Checkpoint, strip_prefixes
@@ -227,6 +228,9 @@ class LlamaModel:
         self.final_norm = torch.ones_like(self.final_norm)
         self._folded = True
         return self
+
+    def kv_spec(self, dtype, fp8: bool = False) -> KVSpec:
+        return KVSpec(self.cfg.n_layers, self.n_kv_heads, self.cfg.head_dim, dtype, fp8)
 
     # recurrent-state hooks (no-ops for dense models)
     has_state = False

@@ -22,7 +22,7 @@ import torch
 from ..config import EngineArgs
 from ..io_types import (GenerateRequest, ParticleOutput, ProfileReq, RequestOutput, RpcReq, RpcResp,
                         validate_request)
-from ..memory.pools import BlockTable, KVPool, KVSpec, PageAllocator, StatePool, cobudget_pages
+from ..memory.pools import BlockTable, KVPool, PageAllocator, StatePool, cobudget_pages
 from ..models import build_model
 from ..utils import debug as smc_debug
 from ..utils import profiling
@@ -129,8 +129,7 @@ class SMCScheduler:
         if kv8 and (tp_size > 1 or pp_size > 1 or any(m.cfg.arch != "llama" for m in (self.target, self.draft))):
             # the e4m3 cache is read by the fused attention step of the dense chain (and by the PyTorch oracle)
             raise ValueError("kv_cache_dtype='fp8_e4m3' needs dense models, tp_size=1 and no particle parallelism")
-        kv_t = KVSpec(len(self.target.cfg.attn_layers), self.target.n_kv_heads, self.target.cfg.head_dim, self.dtype, kv8)
-        kv_d = KVSpec(len(self.draft.cfg.attn_layers), self.draft.n_kv_heads, self.draft.cfg.head_dim, self.dtype, kv8)
+        kv_t, kv_d = self.target.kv_spec(self.dtype, kv8), self.draft.kv_spec(self.dtype, kv8)
         n_rows = n_slots + n_parent_rows
         spec_t, spec_d = self.target.state_spec(), self.draft.state_spec()
         state_bytes = sum(s.row_bytes * n_rows for s in (spec_t, spec_d) if s)
