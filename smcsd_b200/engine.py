@@ -226,6 +226,14 @@ class SMCEngine:
             self.shutdown()
             raise RuntimeError("a scheduler process died; engine shut down")
 
+    def feed(self, entries, end=()):
+        """Feed given tokens instead of sampling: ``entries`` = [(id, tokens, wanted offsets)] run as one batch, each
+        continuing what earlier calls left under its id; ``end`` names the ids to release afterwards.  Returns the fp32
+        logits [wanted, vocab] of the target (in-process scheduler only)."""
+        if self._sched is None:
+            raise RuntimeError("feed() needs an in-process scheduler")
+        return self._sched.feed(entries, end)
+
     # ------------------------------------------------------------------ control
     def _rpc_roundtrip(self, msg, timeout: float = 600.0) -> List[Any]:
         if self._sched is not None:

@@ -17,6 +17,8 @@ CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "libsmcsd_b200.so")
 OBJ_DIR = os.path.join(HERE, "build")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
+# Sources whose fp32 arithmetic serves 32-bit runs: compiled with IEEE division, square root and exponentials.
+PRECISE = {"gemm_f32.cu", "hyper.cu", "latent_attention.cu", "moe.cu"}
 
 
 def sources():
@@ -46,13 +48,14 @@ def build(verbose: bool = False, force: bool = False) -> str:
         return OUT
     os.makedirs(OBJ_DIR, exist_ok=True)
     nvcc = nvcc_path()
-    flags = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "--use_fast_math", "-I", CSRC] + ARCH
+    flags = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-I", CSRC] + ARCH
     if verbose:
         flags += ["-Xptxas", "-v"]
 
     def compile_one(src: str) -> str:
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
-        cmd = [nvcc] + flags + ["-c", src, "-o", obj]
+        fast = [] if os.path.basename(src) in PRECISE else ["--use_fast_math"]
+        cmd = [nvcc] + flags + fast + ["-c", src, "-o", obj]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if verbose or r.returncode != 0:
             sys.stderr.write(f"$ {' '.join(cmd)}\n{r.stdout}{r.stderr}\n")

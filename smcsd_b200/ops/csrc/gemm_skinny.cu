@@ -21,6 +21,11 @@
 // tcgen05.mma.kind::f8f6f4 (K = 32 per instruction, fp32 accumulation) and the epilogues scale every value by the
 // weight row's scale and the token's activation scale.  Tiles, ring and descriptors are the same bytes as for bf16.
 //
+// Several products in one launch (GroupLink): "batched" runs one product per group (for instance per attention head) with
+// its own weight rows and its own column ranges of the activations and of the output; "tiled" takes its token tiles from
+// a table in device memory (group, first row, end row), so that the rows of every expert of a mixture-of-experts layer
+// meet that expert's weights without the host knowing the counts.
+//
 // Every mbarrier wait is bounded; on a timeout the CTA raises a status bit, drains its
 // outstanding copies, frees its tensor memory and returns.
 #include <string.h>
@@ -54,8 +59,20 @@ struct TpLink {
   int* arrive;                         // local arrival counter of this call site (self-resetting)
 };
 
+// Several products of one shape in one launch.
+struct GroupLink {
+  int mode;                 // 0: off, 1: batched (groups x all M rows), 2: tiled (rows of a group given by the table)
+  int groups;
+  int w_rows;               // weight rows between groups
+  int x_cols, out_cols;     // activation / output columns between groups (batched)
+  const int4* tiles;        // tiled: {group, first row, end row, -}; entries past the used ones have first == end
+  int max_tiles, bn;        // tiled: table length, rows per tile (the token-tile width the table was made for)
+  int act;                  // gated epilogue: 0 silu(g) * u, 1 clamped: min(g, limit) * sigmoid(slope g) * (clamp(u) + 1)
+  float limit, slope;
+};
+
 struct GemmParams {
-  int N, K, M;          // weight rows, reduction length, token rows
+  int N, K, M;          // weight rows (of a group), reduction length, token rows
   int kblocks;          // ceil(K / 64)
   int m_tiles;          // token tiles (grid x = weight slabs * m_tiles)
   int stages;           // 3 selects the lean build of the 128-token tile (host-side choice only)
@@ -82,7 +99,17 @@ struct GemmParams {
   int fp8;
   const float* w_scale;
   const float* x_scale;
+  GroupLink grp;
 };
+
+__device__ __forceinline__ float gated_unit(const GroupLink& a, float g, float u) {
+  if (a.act == 1) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.0f + __expf(-a.slope * g)) * (u + 1.0f);
+  }
+  return g / (1.0f + __expf(-g)) * u;
+}
 
 template <int BN, int EPI, bool LEAN>
 struct GemmCfg {
@@ -118,10 +145,31 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // token tiles of one weight slab are neighbours in launch order, so the slab is fetched from HBM once and
   // the other token tiles find it in L2
-  const int n_tile = blockIdx.x / p.m_tiles, split = blockIdx.y, m_tile = blockIdx.x % p.m_tiles;
+  int n_tile = blockIdx.x / p.m_tiles, m0 = (blockIdx.x % p.m_tiles) * BN, m_lim = p.M;
+  const int split = blockIdx.y;
+  int x_col0 = 0, w_row0 = 0;
+  size_t out_off = 0;
   // Let the next kernel of the stream start its prologue (and its weight prefetch) right away;
   // it still waits for this grid to finish before it touches anything this grid writes.
   if (p.pdl) pdl_launch_dependents();
+  if (p.grp.mode != 0) {
+    const int slabs = (p.N + C::BM - 1) / C::BM;
+    int g;
+    if (p.grp.mode == 1) {
+      g = n_tile / slabs;
+      n_tile -= g * slabs;
+      x_col0 = g * p.grp.x_cols;
+      out_off = (size_t)g * p.grp.out_cols;
+    } else {
+      if (p.pdl) pdl_wait_prior_grid();              // the table is the work of an earlier kernel of this stream
+      const int4 t = p.grp.tiles[blockIdx.x / slabs];
+      n_tile = blockIdx.x % slabs;
+      g = t.x; m0 = t.y; m_lim = t.z;
+      if (g < 0 || g >= p.grp.groups || m0 < 0 || m0 >= m_lim || m_lim > p.M) return;      // unused table entry
+    }
+    w_row0 = g * p.grp.w_rows;
+  }
+  w_row0 += n_tile * C::BM;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < nst; ++s) {
@@ -161,7 +209,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
       const int pre = nkb < nst ? nkb : nst;
       for (int i = 0; i < pre; ++i) {
         mbar_expect_tx(&full[i], C::STAGE_BYTES);
-        tma_load_2d(smem + i * C::STAGE_BYTES, &tmW, &full[i], (kb_begin + i) * bk, n_tile * C::BM, pol_w);
+        tma_load_2d(smem + i * C::STAGE_BYTES, &tmW, &full[i], (kb_begin + i) * bk, w_row0, pol_w);
       }
       if (p.pdl) pdl_wait_prior_grid();
       if (p.tp.ag_flag != nullptr) {
@@ -175,7 +223,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
         fence_proxy_async_all();
       }
       for (int i = 0; i < pre; ++i)
-        tma_load_2d(smem + i * C::STAGE_BYTES + C::A_BYTES, &tmX, &full[i], (kb_begin + i) * bk, m_tile * BN,
+        tma_load_2d(smem + i * C::STAGE_BYTES + C::A_BYTES, &tmX, &full[i], x_col0 + (kb_begin + i) * bk, m0,
                     pol_x);
       *sh_issued = pre;
       // stage index and phase advance by counting (the ring depth is a launch parameter: no division per k-block)
@@ -188,8 +236,8 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
           break;
         }
         mbar_expect_tx(&full[s], C::STAGE_BYTES);
-        tma_load_2d(smem + s * C::STAGE_BYTES, &tmW, &full[s], (kb_begin + i) * bk, n_tile * C::BM, pol_w);
-        tma_load_2d(smem + s * C::STAGE_BYTES + C::A_BYTES, &tmX, &full[s], (kb_begin + i) * bk, m_tile * BN,
+        tma_load_2d(smem + s * C::STAGE_BYTES, &tmW, &full[s], (kb_begin + i) * bk, w_row0, pol_w);
+        tma_load_2d(smem + s * C::STAGE_BYTES + C::A_BYTES, &tmX, &full[s], x_col0 + (kb_begin + i) * bk, m0,
                     pol_x);
         *sh_issued = i + 1;
       }
@@ -229,17 +277,17 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
     if (p.ssq_in != nullptr) {
       if (p.pdl) pdl_wait_prior_grid();
       for (int c = tid2; c < BN; c += 64) {
-        const int m = m_tile * BN + c;
+        const int m = m0 + c;
         float ss = 0.f;
-        if (m < p.M)
+        if (m < m_lim)
           for (int q = 0; q < p.ssq_parts; ++q) ss += p.ssq_in[(size_t)q * p.ssq_ld + (size_t)m * p.ssq_mstride];
         s_rstd[c] = rsqrtf(ss * p.norm_inv_d + p.norm_eps);
       }
     } else if (FP8 && p.x_scale != nullptr) {
       if (p.pdl) pdl_wait_prior_grid();
       for (int c = tid2; c < BN; c += 64) {
-        const int m = m_tile * BN + c;
-        s_rstd[c] = m < p.M ? p.x_scale[(size_t)m * p.ssq_mstride] : 1.f;
+        const int m = m0 + c;
+        s_rstd[c] = m < m_lim ? p.x_scale[(size_t)m * p.ssq_mstride] : 1.f;
       }
     } else {
       for (int c = tid2; c < BN; c += 64) s_rstd[c] = 1.f;
@@ -265,7 +313,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
     const int row_in_tile = warp * 32 + lane;
     const int n = n_tile * C::BM + row_in_tile;
     const uint32_t taddr = tmem_base + ((uint32_t)(warp * 32) << 16);
-    const int m_base = m_tile * BN;
+    const int m_base = m0;
     float wsc = 1.f;                                   // FP8: scale of this weight row
     if constexpr (FP8) wsc = n < p.N ? p.w_scale[n] : 1.f;
     if constexpr (EPI == EPI_SWIGLU_BF16) {
@@ -288,10 +336,10 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int m = m_base + c0 + j;
-            if (m < p.M && ch * 2 < p.N) {
+            if (m < m_lim && ch * 2 < p.N) {
               const float g = __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
               const float u = sbuf[row_in_tile * LD + c0 + j] * s_rstd[c0 + j];
-              out[(size_t)m * p.ldo + ch] = __float2bfloat16(g / (1.0f + __expf(-g)) * u);
+              out[(size_t)m * p.ldo + ch] = __float2bfloat16(gated_unit(p.grp, g, u));
             }
           }
         }
@@ -317,7 +365,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
       __syncthreads();
       int parity = 0;
 #pragma unroll 1
-      for (int c0 = 0; c0 < BN && m_base + c0 < p.M; c0 += 16) {
+      for (int c0 = 0; c0 < BN && m_base + c0 < m_lim; c0 += 16) {
         uint32_t r[16];
         tmem_ld_32x32b_x16(taddr + c0, r);
         tmem_ld_wait();
@@ -332,7 +380,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
       RowPartial* parts = reinterpret_cast<RowPartial*>(p.out);
       const int n_slabs = (p.N + C::BM - 1) / C::BM;
       for (int c = threadIdx.x; c < BN; c += 128)
-        if (m_base + c < p.M) parts[(size_t)(m_base + c) * n_slabs + n_tile] = s_rp[c];
+        if (m_base + c < m_lim) parts[(size_t)(m_base + c) * n_slabs + n_tile] = s_rp[c];
     } else {
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 16) {
@@ -343,12 +391,12 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int m = m_base + c0 + j;
-            if (m < p.M) {
+            if (m < m_lim) {
               if constexpr (EPI == EPI_PARTIAL_F32) {
                 reinterpret_cast<float*>(p.out)[((size_t)split * p.M + m) * p.N + n] =
                     __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
               } else {
-                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + n] =
+                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + out_off + n] =
                     __float2bfloat16(__uint_as_float(r[j]) * wsc * s_rstd[c0 + j]);
               }
             }
@@ -380,8 +428,8 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
     if (!any_failed) {
       const float* sbuf = reinterpret_cast<const float*>(smem);
       const int n = n_tile * C::BM + (int)threadIdx.x;
-      const int m_base = m_tile * BN;
-      float* out = reinterpret_cast<float*>(p.out);
+      const int m_base = m0;
+      float* out = reinterpret_cast<float*>(p.out) + out_off;
       // tokens are dealt round-robin to the CTAs of the cluster; ranks are summed in a fixed order.
       // All remote loads of a batch of tokens are issued before the first add, so their
       // latencies overlap instead of queueing up behind one another.
@@ -389,7 +437,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
       for (uint32_t s = 0; s < 8; ++s) rbase[s] = s < S ? dsmem_map(smem_u32(sbuf) + threadIdx.x * 4u, s) : 0u;
       constexpr int UN = 4;
-      for (int c0 = split; c0 < BN && m_base + c0 < p.M; c0 += (int)S * UN) {
+      for (int c0 = split; c0 < BN && m_base + c0 < m_lim; c0 += (int)S * UN) {
         float v[UN][8];
         float prev[UN];
         float sq[UN];
@@ -398,7 +446,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
         for (int u = 0; u < UN; ++u) {
           const int c = c0 + u * (int)S;
-          const bool live = c < BN && m_base + c < p.M;
+          const bool live = c < BN && m_base + c < m_lim;
 #pragma unroll
           for (uint32_t s = 0; s < 8; ++s)
             v[u][s] = (live && s < S) ? ld_dsmem_f32_at(rbase[s] + (uint32_t)c * (C::BM * 4u)) : 0.f;
@@ -410,7 +458,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
         for (int u = 0; u < UN; ++u) {
           const int c = c0 + u * (int)S;
-          if (c < BN && m_base + c < p.M && n < p.N) {
+          if (c < BN && m_base + c < m_lim && n < p.N) {
             float acc = 0.f;
 #pragma unroll
             for (uint32_t s = 0; s < 8; ++s) acc += v[u][s];
@@ -445,9 +493,9 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 #pragma unroll
             for (int u = 0; u < UN; ++u) {
               const int c = c0 + u * (int)S;
-              if (c < BN && m_base + c < p.M && ch * 2 < p.N) {
+              if (c < BN && m_base + c < m_lim && ch * 2 < p.N) {
                 const float g = prev[u], up = s_pair[u][threadIdx.x];
-                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(g / (1.0f + __expf(-g)) * up);
+                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(gated_unit(p.grp, g, up));
               }
             }
           }
@@ -464,7 +512,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
             __syncthreads();
             if (threadIdx.x < UN) {
               const int c = c0 + (int)threadIdx.x * (int)S;
-              if (c < BN && m_base + c < p.M)
+              if (c < BN && m_base + c < m_lim)
                 p.ssq_out[(size_t)n_tile * p.ssq_ld + m_base + c] =
                     s_red[threadIdx.x][0] + s_red[threadIdx.x][1] + s_red[threadIdx.x][2] + s_red[threadIdx.x][3];
             }
@@ -675,7 +723,8 @@ struct Fp8Link { const float* w_scale; const float* x_scale; };      // e4m3 ope
 
 static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int M, int ldx, int ldo, int splits,
                       int epi, int* status, int pdl, const smc::TpLink* tp, const NormLink* nl, cudaStream_t stream,
-                      const smc::SampleArgs* samp = nullptr, const Fp8Link* f8 = nullptr) {
+                      const smc::SampleArgs* samp = nullptr, const Fp8Link* f8 = nullptr,
+                      const smc::GroupLink* grp = nullptr) {
   using namespace smc;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int es = f8 != nullptr ? 1 : 2;                 // element size in bytes
@@ -688,8 +737,15 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
   if ((epi == EPI_SWIGLU_BF16 || epi == EPI_SWIGLU_SPLIT) && (N % 128) != 0) return -22;
   if (epi == EPI_RS_F32 && (tp == nullptr || tp->tp < 1 || tp->tp > 8 || tp->rows_per_rank < 1)) return -24;
   if (epi == EPI_LMHEAD && (samp == nullptr || splits != 1 || M > 256)) return -26;
-  const int bn = bn_for(M, N, clustered);
+  const int gmode = grp != nullptr ? grp->mode : 0, groups = gmode != 0 ? grp->groups : 1;
+  if (gmode != 0 && (tp != nullptr || nl != nullptr || f8 != nullptr || samp != nullptr || groups < 1)) return -31;
+  if (gmode == 1 && (grp->x_cols * es) % 16 != 0) return -20;
+  if (gmode == 2 && (grp->tiles == nullptr || grp->max_tiles < 1)) return -32;
+  if (gmode == 1 && (epi == EPI_SWIGLU_BF16 || epi == EPI_SWIGLU_SPLIT || epi == EPI_PARTIAL_F32)) return -33;
+  if (gmode == 2 && epi == EPI_PARTIAL_F32) return -33;
+  const int bn = gmode == 2 ? grp->bn : bn_for(M, N * (gmode == 1 ? groups : 1), clustered);
   GemmParams p;
+  if (grp != nullptr) p.grp = *grp; else memset(&p.grp, 0, sizeof(p.grp));
   p.N = N; p.K = K; p.M = M;
   p.kblocks = f8 != nullptr ? (K + 127) / 128 : (K + 63) / 64;
   p.fp8 = f8 != nullptr; p.w_scale = f8 ? f8->w_scale : nullptr; p.x_scale = f8 ? f8->x_scale : nullptr;
@@ -709,18 +765,19 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
     if (p.ssq_out != nullptr && epi != EPI_RESID_F32) return -25;
   }
   CUtensorMap tmW, tmX;
-  int rc = cached_tmap(&tmW, W, N, K, K, 128, es);
+  int rc = cached_tmap(&tmW, W, gmode ? (long long)(groups - 1) * grp->w_rows + N : N, K, K, 128, es);
   if (rc) return rc;
-  rc = cached_tmap(&tmX, X, M, K, ldx, bn, es);
+  rc = cached_tmap(&tmX, X, M, gmode == 1 ? (long long)(groups - 1) * grp->x_cols + K : K, ldx, bn, es);
   if (rc) return rc;
-  p.m_tiles = (M + bn - 1) / bn;
+  p.m_tiles = gmode == 2 ? 1 : (M + bn - 1) / bn;
+  const int n_units = gmode == 2 ? grp->max_tiles : groups;       // launch columns per slab besides the token tiles
   {
     // ring depth: 128-token tiles drop to three stages where two CTAs per SM pay off (see GemmCfg)
-    const long long tiles = (long long)((N + 127) / 128) * p.m_tiles * p.splits;
+    const long long tiles = (long long)((N + 127) / 128) * n_units * p.m_tiles * p.splits;
     p.stages = bn <= 32 ? 5 : 4;
     if (bn == 128 && (clustered || tiles > 148)) p.stages = 3;
   }
-  dim3 grid(((N + 127) / 128) * p.m_tiles, p.splits, 1);
+  dim3 grid(((N + 127) / 128) * n_units * p.m_tiles, p.splits, 1);
   if (p.fp8) {
     switch (epi) {
       case EPI_BF16: return dispatch_bn_fp8<EPI_BF16>(bn, tmW, tmX, p, grid, stream);
@@ -823,5 +880,16 @@ SMC_API int smc_lm_head_sample(const void* W, const void* X, int V, int K, int M
                                     logp_out, logz_out, pdl));
   return 0;
 }
+
+// Several products in one launch (see GroupLink).  Batched: out[:, g * out_cols ..] = X[:, g * x_cols ..] W_g^T for every
+// group g, W_g = rows [g * w_rows, g * w_rows + N) of W.  Tiled: rows [first, end) of X (one table entry per tile of bn
+// rows) meet W_g of the entry's group.  Gated epilogues (epi 2) take the activation from the link, grouped or not.
+SMC_API int smc_gemm_grouped(const void* W, const void* X, void* out, int N, int K, int M, int ldx, int ldo, int splits,
+                             int epi, int* status, int pdl, const smc::GroupLink* grp, cudaStream_t stream) {
+  if (grp == nullptr) return -34;
+  return gemm_entry(W, X, out, N, K, M, ldx, ldo, splits, epi, status, pdl, nullptr, nullptr, stream, nullptr, nullptr, grp);
+}
+
+SMC_API int smc_group_link_size() { return (int)sizeof(smc::GroupLink); }
 
 SMC_API int smc_tp_link_size() { return (int)sizeof(smc::TpLink); }

@@ -603,3 +603,138 @@ def gdn_chunked_supported(dk: int, dv: int) -> bool:
 
 
 _KERNELS_PER_CALL["smc_gdn_step"] = 2
+
+
+# ----------------------------------------------------------------------------- layered architectures
+_VP, _I, _F = C.c_void_p, C.c_int, C.c_float
+
+
+class Ragged(C.Structure):
+    """Work list of a step over sequences of unequal length (csrc/ragged.cuh)."""
+    _fields_ = [(n, _VP) for n in ("seq_row", "seq_prefix", "seq_off", "seq_len", "blk_seq", "blk_start")] + \
+               [(n, _I) for n in ("n_seq", "n_blk", "E", "B")]
+
+
+class HyperArgs(C.Structure):
+    _fields_ = [("x", _VP), ("S", _I), ("d", _I), ("ids", _VP), ("positions", _VP), ("embed", _VP), ("pos", _VP), ("vocab", _I),
+                ("max_pos", _I), ("y", _VP), ("ldy", _I), ("ye", _VP), ("ldye", _I), ("top", _I), ("route_slot", _VP),
+                ("route_w", _VP), ("w_mix", _VP), ("w_out", _VP), ("w_in", _VP), ("norm_w", _VP), ("eps", _F), ("n_out", _VP),
+                ("xa", _VP), ("ldxa", _I), ("conv_w", _VP), ("hist", _VP), ("rows", _VP), ("taps", _I), ("n_rows", _I),
+                ("status", _VP), ("pdl", _I)]
+
+
+class LatentArgs(C.Structure):
+    _fields_ = [("q", _VP), ("pool", _VP), ("out", _VP), ("block_table", _VP), ("bt_stride", _I), ("bt_rows", _I), ("n_pages", _I),
+                ("H", _I), ("ldc", _I), ("scale", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
+class GroupLink(C.Structure):
+    """Several products in one GEMM launch (csrc/gemm_skinny.cu); mode 0 only selects the gated epilogue's activation."""
+    _fields_ = [(n, _I) for n in ("mode", "groups", "w_rows", "x_cols", "out_cols")] + [("tiles", _VP)] + \
+               [(n, _I) for n in ("max_tiles", "bn", "act")] + [("limit", _F), ("slope", _F)]
+
+
+GROUP_BATCHED, GROUP_TILED = 1, 2
+ACT_SILU, ACT_CLAMPED = 0, 1
+
+
+def layered_lib():
+    L = lib()
+    if not getattr(L, "_layered_declared", False):
+        vp, i, f = _VP, _I, _F
+        L.smc_gemm_grouped.argtypes = [vp, vp, vp, i, i, i, i, i, i, i, vp, i, vp, vp]
+        L.smc_gemm_f32.argtypes = [vp, vp, vp, i, i, i, i, i, i, i, i, i, i, vp, i, i, vp]
+        L.smc_hyper_step.argtypes = [vp, i, i, vp]
+        L.smc_short_conv.argtypes = [vp, vp, i, vp, vp, i, i, i, vp, vp, i, i, vp]
+        L.smc_poly_norm.argtypes = [vp, i, vp, f, vp, i, i, i, i, i, vp]
+        L.smc_clamped_glu_f32.argtypes = [vp, i, vp, i, i, i, f, f, i, i, vp]
+        L.smc_route.argtypes = [vp, i, vp, i, i, i, i, i, i, vp, vp, i, i, vp]
+        L.smc_dispatch.argtypes = [vp, i, i, i, i, vp, vp, vp, i, vp, i, vp]
+        L.smc_gather_rows.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, vp]
+        L.smc_latent_new.argtypes = [vp, i, i, i, vp, f, vp, i, vp, i, i, vp, i, vp, i, i, vp]
+        L.smc_latent_attn.argtypes = [vp, i, vp]
+        for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_clamped_glu_f32",
+                  "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn"):
+            getattr(L, n).restype = C.c_int
+        for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
+                       (GroupLink, "smc_group_link_size")):
+            assert C.sizeof(cls) == getattr(L, n)(), f"{cls.__name__} layout mismatch"
+        L._layered_declared = True
+    return L
+
+
+def ptr(t: Optional[torch.Tensor]) -> Optional[int]:
+    """Address for a structure field."""
+    return None if t is None else t.data_ptr()
+
+
+def gemm_grouped(W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, *, N: int, M: int, splits: int, epi: int, link: GroupLink,
+                 status: torch.Tensor, pdl: bool = False) -> None:
+    """Batched or tiled products (``link``) on the tensor cores: N weight rows per group, M activation rows in all."""
+    _check(layered_lib().smc_gemm_grouped(_p(W), _p(X), _p(out), N, W.shape[-1], M, X.stride(0), out.stride(0), splits, epi,
+                                          _p(status), int(pdl), C.byref(link), _stream()), "smc_gemm_grouped")
+
+
+def gemm_f32(W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, *, N: int, M: int, link: Optional[GroupLink] = None,
+             ldx: Optional[int] = None, pdl: bool = False) -> None:
+    """fp32 product on the CUDA cores, same grouped forms."""
+    g = link if link is not None else GroupLink()
+    _check(layered_lib().smc_gemm_f32(_p(W), _p(X), _p(out), N, W.shape[-1], M, X.stride(0) if ldx is None else ldx, out.stride(0),
+                                      g.mode, g.groups, g.w_rows, g.x_cols, g.out_cols, g.tiles, g.max_tiles, int(pdl), _stream()),
+           "smc_gemm_f32")
+
+
+def hyper_step(a: HyperArgs, T: int, f32: bool) -> None:
+    _check(layered_lib().smc_hyper_step(C.byref(a), T, int(f32), _stream()), "smc_hyper_step")
+
+
+def short_conv(n: torch.Tensor, xa: torch.Tensor, w: torch.Tensor, hist: torch.Tensor, r: Ragged, *, status: torch.Tensor,
+               f32: bool, pdl: bool = False) -> None:
+    """xa = n + causal depthwise convolution of n; hist [rows, d, taps - 1] advances."""
+    _check(layered_lib().smc_short_conv(_p(n), _p(xa), xa.stride(0), _p(w), _p(hist), hist.shape[0], w.shape[0], w.shape[1],
+                                        C.byref(r), _p(status), int(f32), int(pdl), _stream()), "smc_short_conv")
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, *, ff: int, M: int, eps: float, f32: bool,
+              pdl: bool = False) -> None:
+    _check(layered_lib().smc_poly_norm(_p(z), z.stride(0), _p(coef), eps, _p(out), out.stride(0), ff, M, int(f32), int(pdl),
+                                       _stream()), "smc_poly_norm")
+
+
+def clamped_glu_f32(gu: torch.Tensor, out: torch.Tensor, *, ff: int, blk: int, limit: float, slope: float, M: int,
+                    pdl: bool = False) -> None:
+    _check(layered_lib().smc_clamped_glu_f32(_p(gu), gu.stride(0), _p(out), out.stride(0), ff, blk, limit, slope, M, int(pdl),
+                                             _stream()), "smc_clamped_glu_f32")
+
+
+def route(h: torch.Tensor, wr: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor, *, d: int, top: int, groups: int, keep: int,
+          T: int, f32: bool, pdl: bool = False) -> None:
+    """Expert choice of T tokens: fp32 logits, softmax over all experts, best groups, best experts, weights summing to one."""
+    _check(layered_lib().smc_route(_p(h), d, _p(wr), wr.stride(0), wr.shape[0], top, groups, keep, T, _p(idx), _p(wgt), int(f32),
+                                   int(pdl), _stream()), "smc_route")
+
+
+def dispatch(idx: torch.Tensor, slot: torch.Tensor, src: torch.Tensor, tiles: torch.Tensor, *, n: int, top: int, experts: int,
+             rows: int, max_tiles: int, status: torch.Tensor, pdl: bool = False) -> None:
+    """Slots of the n (token, k) pairs sorted by expert, and the tile table of the grouped GEMMs (``rows`` per tile)."""
+    _check(layered_lib().smc_dispatch(_p(idx), n, top, experts, rows, _p(slot), _p(src), _p(tiles), max_tiles, _p(status), int(pdl),
+                                      _stream()), "smc_dispatch")
+
+
+def gather_rows(x: torch.Tensor, src: torch.Tensor, out: torch.Tensor, *, n: int, n_src: int, status: torch.Tensor,
+                pdl: bool = False) -> None:
+    es = x.element_size()
+    _check(layered_lib().smc_gather_rows(_p(x), x.stride(0) * es, _p(src), _p(out), out.stride(0) * es, out.shape[1] * es, n, n_src,
+                                         _p(status), int(pdl), _stream()), "smc_gather_rows")
+
+
+def latent_new(proj: torch.Tensor, q: Optional[torch.Tensor], pool: torch.Tensor, c_norm: torch.Tensor, cache_locs: torch.Tensor, *,
+               nq: int, R: int, eps: float, M: int, status: torch.Tensor, f32: bool, pdl: bool = False) -> None:
+    """New tokens' projections: query columns to ``q``, normalised latent columns to their cache pages."""
+    _check(layered_lib().smc_latent_new(_p(proj), proj.stride(0), nq, R, _p(c_norm), eps, _p(q), q.stride(0) if q is not None else 0,
+                                        _p(pool), pool.stride(0), pool.shape[0] - 1, _p(cache_locs), M, _p(status), int(f32), int(pdl),
+                                        _stream()), "smc_latent_new")
+
+
+def latent_attention(a: LatentArgs, f32: bool) -> None:
+    _check(layered_lib().smc_latent_attn(C.byref(a), int(f32), _stream()), "smc_latent_attn")

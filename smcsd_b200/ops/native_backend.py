@@ -18,6 +18,7 @@ import torch
 from ..models.layers import ExtendBatch
 from ..runtime.slot_state import CycleInputs, CycleOutputs
 from . import native as K
+from .ragged import Portion, pack_ragged
 
 
 # Shared-prefix group pass on the tcgen05 kernel instead of the mma.sync one (SMC_ATTN_TC): 0 never, 1 for forwards of
@@ -33,6 +34,11 @@ def _env_int(name: str, default: int) -> int:
 def _env_flag(name: str, default: bool) -> bool:
     v = os.environ.get(name)
     return default if v is None else v.strip().lower() in ("1", "true", "yes", "on")
+
+
+def _samples_in_head(nm) -> bool:
+    """Chains whose lm_head can sample / score in its epilogue (no logits in memory)."""
+    return type(nm) is NativeLlama or getattr(nm, "fused_lm_sample", False)
 
 
 class NativeLlama:
@@ -472,9 +478,9 @@ class NativeState:
                            st.seed, st.counters, st.group_log_Z, self.job_dst, self.job_src)
         max_jobs = self.n_groups * (st.N - 1)
         for pool in st.state_pools:
-            K.state_copy(pool.conv, pool.conv.shape[0], pool.n_rows, st.counters, self.job_dst, self.job_src, max_jobs)
-            K.state_copy(pool.temporal, pool.temporal.shape[0], pool.n_rows, st.counters, self.job_dst, self.job_src,
-                         max_jobs)
+            for t in (pool.conv, pool.temporal):
+                if t.numel():                          # convolution-only states have no temporal part
+                    K.state_copy(t, t.shape[0], pool.n_rows, st.counters, self.job_dst, self.job_src, max_jobs)
 
 
 class NativeRunner:
@@ -511,7 +517,8 @@ class NativeRunner:
         # capture caps (SMC_DRAFT_GRAPH_MAX_BS / SMC_DRAFT_GRAPH_MAX_CONTEXT): larger batches or contexts launch eagerly
         self.graph_max_bs = int(a.graph_max_bs)
         self.graph_max_context = int(a.graph_max_context)
-        self.T_draft, self.T_target, self.alpha = float(a.draft_temperature), float(a.target_temperature), float(a.power_alpha)
+        # greedy proposals (draft temperature 0) are the limit the samplers reach with a tiny temperature
+        self.T_draft, self.T_target, self.alpha = max(float(a.draft_temperature), 1e-5), float(a.target_temperature), float(a.power_alpha)
         self.defer = bool(a.defer_bonus)
         # A/B switches (environment > argument > default on).  Switching a fused step off routes it to the PyTorch
         # implementation of the same step; such cycles launch eagerly, like the reference's downgrade of its graph
@@ -547,6 +554,9 @@ class NativeRunner:
                     setattr(self, name, PersistentLlama(nm.m, nm.kv, nm.bt, 128, self.status))
 
     def _wrap(self, model, kv, bt, max_tokens, max_logit_rows, splits, pdl, state=None):
+        if model.cfg.arch == "pasizen":
+            from .native_pasizen import NativePasizen
+            return NativePasizen(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, state=state)
         if model.cfg.arch != "llama":
             from .native_hybrid import NativeHybrid
             return NativeHybrid(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, runner=self,
@@ -575,6 +585,7 @@ class NativeRunner:
     # ---- prefill ---------------------------------------------------------------------------------------
     PREFILL_BLOCK = 16
     PREFILL_MAX_TOKENS = 4096
+    EXTEND_LOGIT_ROWS = 64               # rows per lm_head pass when logits of given tokens are asked for
     PREFILL_MAX_TOKENS_TP = 1024         # token capacity of the tensor-parallel prompt chain (symmetric-heap buffers)
 
     def _prefill_chain(self, which: str):
@@ -586,6 +597,9 @@ class NativeRunner:
             if isinstance(base, NativeLlama):
                 nm = NativeLlama(base.m, base.kv, base.bt, self.PREFILL_MAX_TOKENS, 8, base.attn_splits, self.status,
                                  self.pdl)
+            elif getattr(base, "ragged", False):
+                nm = type(base)(base.m, base.kv, base.bt, self.PREFILL_MAX_TOKENS, self.EXTEND_LOGIT_ROWS, base.attn_splits,
+                                self.status, self.pdl, state=base.state)
             elif type(base).__name__ == "NativeHybrid":
                 nm = type(base)(base.m, base.kv, base.bt, self.PREFILL_MAX_TOKENS, 8, base.attn_splits, self.status,
                                 self.pdl, runner=self, state=base.state)
@@ -605,13 +619,15 @@ class NativeRunner:
         decode kernels with token-tile GEMMs.  Gated-DeltaNet layers of hybrid models walk each prompt once, token
         by token, with the state held in registers.  Tensor-parallel targets and over-long batches take the plain
         PyTorch forward.  Dense prompts longer than the chains' token capacity run in several passes over
-        consecutive blocks (earlier passes have already cached their keys)."""
+        consecutive blocks (earlier passes have already cached their keys).  Chains with a ragged work list take the
+        prompts as they are (``_ragged_pass``)."""
         B = self.PREFILL_BLOCK
         lens = [len(it.input_ids) for it in items]
         n_blocks = [(L + B - 1) // B for L in lens]
         T = sum(n_blocks) * B
         tgt, drf = self._prefill_chain("target"), self._prefill_chain("draft")
-        stateful = any(getattr(nm.m, "has_state", False) for nm in (tgt, drf) if nm is not None)
+        is_ragged = lambda nm: getattr(nm, "ragged", False)
+        stateful = any(getattr(nm.m, "has_state", False) and not is_ragged(nm) for nm in (tgt, drf) if nm is not None)
         if tgt is None or drf is None or (T > self.PREFILL_MAX_TOKENS and stateful) or len(items) > 256:
             native, worker.native = worker.native, None
             try:
@@ -649,7 +665,8 @@ class NativeRunner:
         worker.io_bytes["h2d"] += T * 16
         bs = sum(n_blocks)
         for nm in (tgt, drf):
-            nm.set_context(max(lens), bs)
+            if not is_ragged(nm):
+                nm.set_context(max(lens), bs)
 
         def seqs_for(nm, short: int):
             # prompts as variable-length rows for the recurrent layers (None for dense models)
@@ -663,7 +680,7 @@ class NativeRunner:
                              "off": pin(torch.tensor(offs, dtype=torch.int32)),
                              "len": pin(torch.tensor([max(L - short, 0) for L in lens], dtype=torch.int32)),
                              "n": len(items), "max": max(lens)}}
-        cb = max(1, min(nm.T for nm in (tgt, drf)) // B)     # blocks per pass
+        cb = max(1, min(nm.T for nm in (tgt, drf) if not is_ragged(nm)) // B) if not (is_ragged(tgt) and is_ragged(drf)) else 0
         last = torch.tensor(last_rows, dtype=torch.long, device=dev)
 
         def grab(nm, idx):
@@ -678,6 +695,10 @@ class NativeRunner:
             return {"x": nm.final_hidden(idx), "ssq": None, "normed": nm.final_hidden(idx)}
 
         def run(nm, short: int, want_hidden: bool):
+            if is_ragged(nm):
+                x = self._ragged_pass(nm, [Portion(it.row, 0, it.input_ids[:L - short]) for it, L in zip(items, lens)],
+                                      [[L - short - 1] if want_hidden else [] for L in lens])
+                return {"n": len(items), "x": x, "ssq": None, "normed": lambda: x} if want_hidden else None
             if bs <= cb:
                 nm.forward(ids, pos, locs, rows, pref, bs, B, two_pass=True, **seqs_for(nm, short))
                 parts = [grab(nm, last)] if want_hidden else []
@@ -708,6 +729,92 @@ class NativeRunner:
         worker.io_bytes["d2h"] += 4 * len(items)
         return x0.to(torch.int32)
 
+    def _ragged_pass(self, nm, portions, want) -> Optional[torch.Tensor]:
+        """Run portions of sequences through a ragged chain; returns the final rows of the wanted tokens (``want``: offsets
+        inside each portion), portion by portion, or None when nothing is wanted."""
+        base, total = [], 0
+        for w in want:
+            base.append(total)
+            total += len(w)
+        out = torch.empty(total, nm.xa.shape[1], dtype=nm.xa.dtype, device=self.device) if total else None
+        slots = [{o: b + i for i, o in enumerate(w)} for w, b in zip(want, base)]
+        for plan in pack_ragged(portions, nm.T, nm.BLOCK, nm.bt):
+            nm.forward_plan(plan)
+            hit = [(t, slots[p][o]) for t, (p, o) in enumerate(plan.tokens) if o in slots[p]]
+            if hit:
+                src, dst = torch.tensor(hit, dtype=torch.long).t().contiguous().pin_memory().to(self.device, non_blocking=True)
+                out[dst] = nm.final_hidden(src)
+        return out
+
+    def _block_pass(self, nm, portions, want) -> Optional[torch.Tensor]:
+        """The same for chains that run fixed blocks: portions are cut into blocks of PREFILL_BLOCK tokens (the last one
+        padded), as many per launch chain as its buffers hold; the recurrent layers of hybrids walk each portion once."""
+        B, dev = self.PREFILL_BLOCK, self.device
+        cap = max(1, nm.T // B)
+        pin = lambda v, dt=torch.int32: torch.tensor(v, dtype=dt).pin_memory().to(dev, non_blocking=True)
+        out = [None] * sum(len(w) for w in want)
+        base, total = [], 0
+        for w in want:
+            base.append(total)
+            total += len(w)
+        cells = [(p, b) for p, q in enumerate(portions) for b in range(0, len(q.ids), B)]
+        for c0 in range(0, len(cells), cap):
+            part = cells[c0:c0 + cap]
+            ids, pos, cols, rows_of, ok, rows, pref, where = [], [], [], [], [], [], [], {}
+            runs = []                                  # (row, token offset, count) of each portion inside this pass
+            for p, b in part:
+                q = portions[p]
+                n, t = min(B, len(q.ids) - b), len(ids)
+                start = q.prefix + b
+                ids += list(q.ids[b:b + n]) + [0] * (B - n)
+                pos += list(range(start, start + n)) + [start + n - 1] * (B - n)
+                cols += list(range(start, start + n)) + [0] * (B - n)
+                rows_of += [q.row] * B
+                ok += [True] * n + [False] * (B - n)
+                rows.append(q.row)
+                pref.append(start)
+                for i in range(n):
+                    where[(p, b + i)] = t + i
+                if runs and runs[-1][0] == q.row:
+                    runs[-1][2] += n
+                else:
+                    runs.append([q.row, t, n])
+            locs = torch.where(pin(ok, torch.bool), nm.bt[pin(rows_of, torch.long), pin(cols, torch.long)],
+                               torch.zeros((), dtype=torch.int32, device=dev))
+            kw = {}
+            if getattr(nm.m, "has_state", False):
+                kw["seqs"] = {"rows": pin([r[0] for r in runs]), "off": pin([r[1] for r in runs]), "len": pin([r[2] for r in runs]),
+                              "n": len(runs), "max": max(r[2] for r in runs)}
+            nm.set_context(max(portions[p].prefix + len(portions[p].ids) for p, _ in part), len(part))
+            nm.forward(pin(ids), pin(pos), locs, pin(rows), pin(pref), len(part), B, two_pass=True, **kw)
+            hit = [(where[(p, o)], base[p] + i) for p, w in enumerate(want) for i, o in enumerate(w) if (p, o) in where]
+            if hit:
+                x = nm.final_hidden(pin([t for t, _ in hit], torch.long))
+                for row, (_, i) in zip(x, hit):
+                    out[i] = row
+        return torch.stack(out) if out else None
+
+    def extend(self, portions, want, which: str = "target") -> torch.Tensor:
+        """Feed given tokens: every portion continues its sequence's cache and state, all portions are one batch.  Returns
+        the fp32 logits [wanted, vocab] of the tokens ``want`` names (offsets inside each portion)."""
+        nm = self._prefill_chain(which)
+        if nm is None or nm.m.tp_size > 1:
+            raise NotImplementedError("feeding given tokens needs an unsharded kernel chain")
+        x = (self._ragged_pass if getattr(nm, "ragged", False) else self._block_pass)(nm, portions, want)
+        n, V, step = (0 if x is None else x.shape[0]), nm.c.vocab_size, nm.logits.shape[0]
+        out = torch.empty(n, V, dtype=torch.float32, device=self.device)
+        for i in range(0, n, step):
+            rows = x[i:i + step].contiguous()
+            if hasattr(nm, "project"):
+                nm.project(rows, rows.shape[0])
+            else:
+                K.gemm_skinny(nm.m.lm_head, rows, nm.logits, M=rows.shape[0], splits=1, epi=K.EPI_STORE_F32,
+                              ldo=nm.logits.stride(0), status=self.status)
+            lg = nm.logits[:rows.shape[0], :V]
+            cap = float(nm.c.logit_softcap)
+            out[i:i + step] = torch.tanh(lg / cap) * cap if cap > 0 else lg
+        return out
+
     def _sample_x0(self, nm, hidden, worker) -> torch.Tensor:
         """x0 of every prompt: a draw from softmax(alpha * logits / T_target) of the last prompt token.  Dense chains
         project and sample with the fused lm_head kernel (no logits in memory, noise keyed by the running count of
@@ -733,7 +840,7 @@ class NativeRunner:
                          cycle_counter=self._x0_counter_tp, call_id=4096, tok_out=tok, logp_out=lp, logz_out=None,
                          epoch=self._x0_epoch)
             return tok
-        if type(nm) is NativeLlama and self.fused_sampling and self.fused_lm_head and n <= 256:
+        if _samples_in_head(nm) and self.fused_sampling and self.fused_lm_head and n <= 256:
             dev = self.device
             if getattr(self, "_x0_counter", None) is None:
                 self._x0_counter = torch.zeros(1, dtype=torch.int64, device=dev)
@@ -840,7 +947,7 @@ class NativeRunner:
             self._verify_torch(nm, ids, pos, locs, rows, prefix, bs, E)
         else:
             nm.forward(ids, pos, locs, rows, prefix, bs, E)
-            if lm_rows > 0 and self.fused_sampling and self.fused_lm_head and type(nm) is NativeLlama and lm_rows <= 256:
+            if lm_rows > 0 and self.fused_sampling and self.fused_lm_head and _samples_in_head(nm) and lm_rows <= 256:
                 # sampling / scoring inside the lm_head epilogue: no logits in memory, one merge launch
                 nm.lm_head_sample(lm_rows, lm_off, lm_step, temperature=temperature, alpha=alpha, tokens_in=tokens_in,
                                   seed=self.seed, cycle_counter=self._counters, call_id=call_id, tok_out=tok_out,

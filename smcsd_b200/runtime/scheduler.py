@@ -23,13 +23,16 @@ from ..config import EngineArgs
 from ..io_types import (GenerateRequest, ParticleOutput, ProfileReq, RequestOutput, RpcReq, RpcResp,
                         validate_request)
 from ..memory.pools import BlockTable, KVPool, PageAllocator, StatePool, cobudget_pages
-from ..models import build_model
+from ..models import build_model, resolve_config
 from ..utils import debug as smc_debug
 from ..utils import profiling
+from .feeder import TokenFeeder
 from .slot_state import HostSnapshot, SlotState
 from .worker import PrefillItem, SMCWorker
 
 log = logging.getLogger("smcsd_b200.scheduler")
+
+NATIVE_F32_ARCHS = ("pasizen",)       # architectures whose kernel chain also runs in 32-bit
 
 
 @dataclass
@@ -81,6 +84,10 @@ class SMCScheduler:
         backend = a.backend
         if backend == "auto":
             backend = "native" if on_cuda and self.dtype == torch.bfloat16 else "torch"
+            archs = [m.cfg.arch if m is not None else resolve_config(path).arch
+                     for m, path in ((target, a.model_path), (draft, a.draft_model_path))]
+            if on_cuda and self.dtype == torch.float32 and all(x in NATIVE_F32_ARCHS for x in archs):
+                backend = "native"
         self.backend = backend
         if os.environ.get("SMC_SYNC_DEBUG") == "1" and on_cuda:
             torch.cuda.set_sync_debug_mode("warn")
@@ -120,6 +127,13 @@ class SMCScheduler:
             if os.environ.get("SMC_FP8_DRAFT", "0") == "1":
                 self.draft.quantization = "fp8"
         self.context_len = int(a.context_length or min(self.target.cfg.max_position, 16384))
+        for m in (self.target, self.draft):
+            # learned position rows end at max_position, and the latent cache and its state are not shared over ranks
+            if m.cfg.arch == "pasizen" and self.context_len > m.cfg.max_position:
+                raise ValueError(f"context_length {self.context_len} exceeds the {m.cfg.max_position} learned positions of "
+                                 f"{m.cfg.name or 'the model'}")
+            if m.cfg.arch == "pasizen" and pp_size > 1:
+                raise NotImplementedError("particle-parallel groups do not support latent caches")
         # ---- memory -----------------------------------------------------------
         N, G = self.n_local, a.gamma + 1
         self.max_groups = a.max_running_requests
@@ -178,6 +192,7 @@ class SMCScheduler:
         self._log_alloc_retries = os.environ.get("SMC_LOG_ALLOC_RETRIES") == "1" and self.device.type == "cuda"
         self._alloc_retries_seen = 0
         self.paused = False
+        self.feeder = TokenFeeder(self)     # sequences fed with given tokens (replay, scoring)
         self.pending: Deque = deque()       # snapshots awaiting host post-processing
         self.outbox: List = []
         self.final_gen = torch.Generator().manual_seed(seed * 31 + 5)
@@ -554,13 +569,13 @@ class SMCScheduler:
         if os.environ.get("SMC_STRICT_MEM_CHECK", os.environ.get("SGLANG_ENABLE_STRICT_MEM_CHECK_DURING_IDLE", "1")) \
                 not in ("1", "true", "True"):
             return
-        free = self.alloc.available()
+        free = self.alloc.available() + self.feeder.held_pages
         if free != self.alloc.size:
             raise RuntimeError(f"KV page leak: {self.alloc.size - free} pages still held while idle")
         if len(self.state.free_slots) != self.state.max_slots:
             raise RuntimeError("slot leak while idle")
-        if self.reserved_pages != 0:
-            raise RuntimeError(f"page reservation leak: {self.reserved_pages}")
+        if self.reserved_pages != self.feeder.held_pages:
+            raise RuntimeError(f"page reservation leak: {self.reserved_pages - self.feeder.held_pages}")
 
     def cycle_timing(self, last: int = 0, reset: bool = False) -> dict:
         """Device time of the recorded decode cycles (CUDA events; needs SMC_TIME_CYCLES=1)."""
@@ -669,6 +684,10 @@ class SMCScheduler:
             self.alloc.free(pages)
             self.bt.free_parent_row(row)
         return out
+
+    def feed(self, entries, end=()):
+        """One step of given tokens (see ``TokenFeeder.step``)."""
+        return self.feeder.step(entries, end)
 
     def handle_rpc(self, req: RpcReq) -> RpcResp:
         try:

@@ -28,6 +28,16 @@ class PrefillItem:
     input_ids: List[int]
 
 
+@dataclass
+class ExtendItem:
+    """Given tokens that continue a sequence (block-table / state row) already holding ``prefix`` tokens; ``want`` are the
+    offsets among them whose logits are asked for."""
+    row: int
+    prefix: int
+    input_ids: List[int]
+    want: List[int]
+
+
 class SMCWorker:
     def __init__(self, args: EngineArgs, target, draft, kv_target: KVPool, kv_draft: KVPool,
                  block_table: BlockTable, allocator: PageAllocator,
@@ -90,6 +100,25 @@ class SMCWorker:
             self.draft.forward_torch(dbatch, self.kv_d, self.bt.table, self.state_d)
         self.io_bytes["d2h"] += 4 * len(items)
         return x0.to(torch.int32)
+
+    def extend(self, items: Sequence[ExtendItem]) -> torch.Tensor:
+        """One batch of given tokens through the target: portions of prompts beside single tokens.  Pages are already in
+        the block table.  Returns fp32 logits [wanted, vocab] in the order of the items and of their ``want``."""
+        if self.native is not None:
+            from ..ops.ragged import Portion
+            return self.native.extend([Portion(it.row, it.prefix, it.input_ids) for it in items], [it.want for it in items])
+        dev, lens = self.device, [len(it.input_ids) for it in items]
+        ids = torch.tensor([t for it in items for t in it.input_ids], dtype=torch.int64, device=dev)
+        pos = torch.cat([torch.arange(it.prefix, it.prefix + n, device=dev) for it, n in zip(items, lens)])
+        locs = torch.cat([self.bt.table[it.row, it.prefix:it.prefix + n] for it, n in zip(items, lens)])
+        rows = torch.tensor([it.row for it in items], dtype=torch.int32, device=dev)
+        pref = [it.prefix for it in items]
+        batch = ExtendBatch(ids, pos, locs, rows, torch.tensor(pref, dtype=torch.int32, device=dev), extend_len=0, extend_lens=lens,
+                            prefix_lens_host=pref)
+        hid = self.target.forward_torch(batch, self.kv_t, self.bt.table, self.state_t)
+        off = [sum(lens[:i]) for i in range(len(items))]
+        at = [o + w for o, it in zip(off, items) for w in it.want]
+        return self.target.logits_torch(hid[torch.tensor(at, dtype=torch.long, device=dev)])
 
     # ------------------------------------------------------------------ decode
     def decode_cycle(self, cin: CycleInputs) -> CycleOutputs:
