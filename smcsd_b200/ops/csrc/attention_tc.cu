@@ -25,9 +25,6 @@
 #include "common.cuh"
 #include "tmap_host.h"
 
-#include <mutex>
-#include <unordered_map>
-
 namespace smc {
 
 constexpr int TC_MAX_STAGES = 8;
@@ -489,31 +486,6 @@ template <int D>
 static size_t tc_smem_bytes() {
   constexpr int BK = TcCfg<D>::BK, ST = TcCfg<D>::STAGES;
   return (size_t)(D / 64) * 128 * 128 + (size_t)ST * 2 * (D / 64) * BK * 128 + (size_t)2 * (BK / 64) * 128 * 128 + 1024;
-}
-
-// Tensor maps of the K / V pools ([pages + 1, Hkv * D] bf16, box = 64 columns x 64 pages), cached per pool.
-struct PoolMapKey {
-  const void* base; long long rows, cols;
-  bool operator==(const PoolMapKey& o) const { return base == o.base && rows == o.rows && cols == o.cols; }
-};
-struct PoolMapHash {
-  size_t operator()(const PoolMapKey& k) const {
-    return std::hash<const void*>()(k.base) ^ (std::hash<long long>()(k.rows) * 1315423911u) ^ std::hash<long long>()(k.cols);
-  }
-};
-static int pool_tmap(CUtensorMap* tm, const void* base, long long rows, long long cols) {
-  static std::unordered_map<PoolMapKey, CUtensorMap, PoolMapHash> cache;
-  static std::mutex mu;
-  std::lock_guard<std::mutex> lock(mu);
-  const PoolMapKey key{base, rows, cols};
-  auto it = cache.find(key);
-  if (it != cache.end()) { *tm = it->second; return 0; }
-  const int rc = make_tmap(tm, base, rows, cols, cols, 64);
-  if (rc == 0) {
-    if (cache.size() > 4096) cache.clear();
-    cache.emplace(key, *tm);
-  }
-  return rc;
 }
 
 }  // namespace smc

@@ -6,7 +6,7 @@
 //                   root mean square (and weighted) into the token's cache page
 //   latent_attn     causal attention over the paged rows, one (token, head) per CTA, four warps over the keys: the form
 //                   32-bit runs use; the tensor-core form is in latent_attention_tc.cu
-#include "ragged.cuh"
+#include "latent_attention.cuh"
 
 namespace smc {
 
@@ -36,18 +36,6 @@ __global__ void __launch_bounds__(256) latent_new_kernel(const float* proj, int 
   }
   for (int i = threadIdx.x; i < R; i += blockDim.x) pool[(size_t)page * ldc + i] = from_f32<AT>(c[i] * inv * c_norm[i]);
 }
-
-struct LatentArgs {
-  const void* q;            // [T, H * ldc] queries in latent space (columns beyond R are zero)
-  const void* pool;         // [pages + 1, ldc]
-  void* out;                // [T, H * ldc]
-  const int* block_table;
-  int bt_stride, bt_rows, n_pages, H, ldc;
-  float scale;
-  Ragged r;
-  int* status;
-  int pdl;
-};
 
 template <int NR, typename AT>      // NR = ldc / 32 values per lane
 __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {

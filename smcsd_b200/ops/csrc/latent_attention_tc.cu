@@ -1,0 +1,495 @@
+// Latent attention on the 5th-generation tensor cores (tcgen05 + tensor memory).
+//
+// All heads of a token attend to the same cached rows of R values (R padded to panels of 64), so the query rows of a block
+// of tokens - row = token * heads + head, up to 128 per CTA - form one M = 128 operand, and a tile of 64 cached rows serves
+// as keys and as values from the same shared-memory bytes:
+//     S = Q C^T        UMMA 128 x 64 x R, C taken K-major
+//     softmax          one query row per thread, causal limit per row, P as bf16 into a SWIZZLE_128B tile
+//     O += P C         UMMA 128 x R x 64 accumulating in tensor memory, C taken MN-major
+// Two score buffers (64 columns each) and up to 384 output columns live in tensor memory; wider latents split their output
+// columns over two CTAs that both compute the scores.  The exponent reference of a row only moves when its maximum grew by
+// more than 2^8; only then is its part of O rescaled in tensor memory.
+// Cached rows live one page per token: a tile of 64 consecutive pages is fetched with one TMA box per panel, a scattered one
+// is gathered by four loader warps with 16-byte cp.async copies into the same swizzled layout.  Key ranges may be split over
+// CTAs (few sequences, long contexts): every split parks its unnormalised rows in fp32 and a second kernel merges them.
+// The work list (ragged.cuh) mixes prompts, portions of prompts and single tokens; query rows never mix sequences.
+// Every mbarrier wait is bounded; a timeout raises a status bit and every role unwinds.
+#include "latent_attention.cuh"
+#include "tmap_host.h"
+
+namespace smc {
+
+constexpr int LT_BK = 64;                       // cached rows per tile
+constexpr int LT_LOADERS = 4;
+constexpr int LT_THREADS = (5 + LT_LOADERS) * 32;   // warps 0..3 softmax, 4 MMA, 5..8 loaders
+constexpr int LT_PANEL_Q = 128 * 128;           // bytes of one [128 rows][64 values] panel
+constexpr int LT_PANEL_C = LT_BK * 128;
+constexpr int LT_O_COL = 2 * LT_BK;             // first output column in tensor memory
+constexpr int LT_MAX_STAGES = 8;
+
+// NPAN: panels of 64 values per cached row.  Ring depth within 227 KB next to the Q tile and two P tiles.
+template <int NPAN> struct LtCfg {
+  static constexpr int VSPLIT = NPAN > 6 ? 2 : 1;                    // CTAs sharing the output columns
+  static constexpr int OPAN = (NPAN + VSPLIT - 1) / VSPLIT;          // output panels per CTA (the second may have fewer)
+  static constexpr int FIXED = NPAN * LT_PANEL_Q + 2 * LT_PANEL_Q;
+  static constexpr int FIT = (231000 - 1024 - FIXED) / (NPAN * LT_PANEL_C);
+  static constexpr int STAGES = FIT > LT_MAX_STAGES ? LT_MAX_STAGES : FIT;
+  static constexpr int LAG = STAGES > 2 ? STAGES - 2 : 0;            // gathered tiles in flight behind the newest
+  static constexpr int SMEM = FIXED + STAGES * NPAN * LT_PANEL_C + 1024;
+  static_assert(STAGES >= 1, "a tile must fit");
+};
+
+struct LatentTcParams {
+  const __nv_bfloat16* pool;     // [pages + 1, ldc]
+  __nv_bfloat16* out;            // [T * H, ldc]
+  float* part;                   // [KS, T * H, ldc] (KS > 1)
+  float* part_ml;                // [KS, T * H, 2]: reference exponent (log2 units), sum
+  const int* block_table;
+  int bt_stride, bt_rows, n_pages, H, ldc, KS, MT, T;
+  float scale_log2;
+  Ragged r;
+  int* status;
+  int pdl;
+};
+
+struct LtShared {
+  uint64_t q_full, c_full[LT_MAX_STAGES], c_empty[LT_MAX_STAGES], s_full[2], s_empty[2], p_full[2], p_empty[2];
+  uint32_t tmem_slot;
+  volatile int abort;
+};
+
+__device__ __forceinline__ bool lt_wait(LtShared& S, int* status, uint64_t* bar, uint32_t parity) {
+  if (mbar_try_wait(bar, parity)) return true;
+  if (S.abort) return false;
+  const long long t0 = clock64();
+  for (;;) {
+    for (int i = 0; i < 64; ++i)
+      if (mbar_try_wait(bar, parity)) return true;
+    if (S.abort) return false;
+    if (clock64() - t0 > SMC_SPIN_CYCLES) {
+      atomicOr(status, SMC_ERR_BARRIER_TIMEOUT);
+      S.abort = 1;
+      return false;
+    }
+  }
+}
+
+__device__ __forceinline__ float lt_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ uint32_t lt_pack(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+template <int NPAN>
+__global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTcParams p, const __grid_constant__ CUtensorMap tmC,
+                                                                  const __grid_constant__ CUtensorMap tmQ) {
+  using C = LtCfg<NPAN>;
+  constexpr int STAGES = C::STAGES, LAG = C::LAG, CPR = NPAN * 8, KPW = LT_BK / LT_LOADERS, C_BYTES = NPAN * LT_PANEL_C;
+  extern __shared__ uint8_t lt_raw[];
+  __shared__ LtShared S;
+  const uint32_t raw = smem_u32(lt_raw);
+  uint8_t* q_s = lt_raw + (((raw + 1023u) & ~1023u) - raw);
+  uint8_t* c_s = q_s + NPAN * LT_PANEL_Q;
+  uint8_t* p_s = c_s + STAGES * C_BYTES;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  if (threadIdx.x == 0) {
+    mbar_init(&S.q_full, 1);
+    for (int s = 0; s < STAGES; ++s) {
+      mbar_init(&S.c_full[s], LT_LOADERS);
+      mbar_init(&S.c_empty[s], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&S.s_full[i], 1);
+      mbar_init(&S.s_empty[i], 4);
+      mbar_init(&S.p_full[i], 4);
+      mbar_init(&S.p_empty[i], 1);
+    }
+    S.abort = 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&tmC);
+    tma_prefetch_desc(&tmQ);
+  }
+  if (warp == 4) {
+    tmem_alloc(&S.tmem_slot, 512);
+    tmem_relinquish();
+  }
+  if (p.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+
+  // ---- this CTA's rows and keys --------------------------------------------------------------------------------------
+  const int vs = blockIdx.x % C::VSPLIT, mt = (blockIdx.x / C::VSPLIT) % p.MT, blk = blockIdx.x / (C::VSPLIT * p.MT), ks = blockIdx.y;
+  RaggedBlock b = ragged_block(p.r, blk);
+  if (b.row < 0 || b.row >= p.bt_rows || b.prefix < 0 || b.prefix + b.len > p.bt_stride || b.off < 0 || b.off + b.len > p.T) {
+    if (threadIdx.x == 0) atomicOr(p.status, SMC_ERR_BOUNDS);
+    b.n = 0;
+    b.row = 0;
+  }
+  const int row0 = mt * 128, n_rows = min(128, max(0, b.n) * p.H - row0);      // <= 0: nothing to do
+  const int g_row0 = (b.off + b.start) * p.H + row0;                           // in the [T * H] query rows
+  const int pos0 = b.prefix + b.start;                                         // position of the block's first token
+  const int lim_min = pos0 + row0 / p.H + 1;                                   // keys the tile's first row sees
+  const int n_keys = n_rows > 0 ? pos0 + (row0 + n_rows - 1) / p.H + 1 : 0;
+  int per = (n_keys + p.KS - 1) / p.KS;
+  per = (per + LT_BK - 1) / LT_BK * LT_BK;
+  const int kb = ks * per, ke = min(n_keys, kb + per);
+  const int n_tiles = ke > kb ? (ke - kb + LT_BK - 1) / LT_BK : 0;
+  const int vpan = vs * C::OPAN, n_opan = min(C::OPAN, NPAN - vpan);           // this CTA's output panels
+
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = S.tmem_slot;
+  const uint32_t tO = tmem_base + LT_O_COL;
+
+  if (warp >= 5) {
+    // ================================================================= loaders
+    const int lw = warp - 5;
+    const uint64_t pol = l2_policy_evict_last();      // other row tiles and splits read the same rows
+    if (lw == 0 && lane == 0 && n_tiles > 0) {
+      mbar_expect_tx(&S.q_full, NPAN * LT_PANEL_Q);
+      for (int pan = 0; pan < NPAN; ++pan) tma_load_2d(q_s + pan * LT_PANEL_Q, &tmQ, &S.q_full, pan * 64, g_row0, pol);
+    }
+    const int* bt = p.block_table + (size_t)b.row * p.bt_stride;
+    // every loader warp reads all 64 page ids of a tile (lane l: keys l and l + 32), so all take the same path
+    auto page_of = [&](int tile, int half) {
+      const int key = kb + tile * LT_BK + half * 32 + lane;
+      int page = 0;
+      if (tile < n_tiles && key < ke) {
+        page = bt[key];
+        if (page < 0 || page > p.n_pages) { atomicOr(p.status, SMC_ERR_BOUNDS); page = 0; }
+      }
+      return page;
+    };
+    constexpr int PD = 4;                             // page ids are fetched this many tiles ahead
+    int issued = 0;
+    uint32_t gathered = 0;                            // bit (j & 31): tile j went through cp.async (arrival still owed)
+    int pg[PD][2];
+#pragma unroll
+    for (int u = 0; u < PD; ++u) {
+      pg[u][0] = page_of(u, 0);
+      pg[u][1] = page_of(u, 1);
+    }
+    bool go = true;
+    for (int j0 = 0; go && j0 < n_tiles; j0 += PD) {
+#pragma unroll
+      for (int u = 0; u < PD; ++u) {
+        const int j = j0 + u;
+        if (j >= n_tiles) break;
+        const int st = j % STAGES, use = j / STAGES;
+        const bool ok = use < 1 || lt_wait(S, p.status, &S.c_empty[st], (uint32_t)(use - 1) & 1u);
+        if (!__all_sync(0xffffffffu, ok)) { go = false; break; }
+        const int pa = pg[u][0], pb = pg[u][1];
+        pg[u][0] = page_of(j + PD, 0);
+        pg[u][1] = page_of(j + PD, 1);
+        const int base = __shfl_sync(0xffffffffu, pa, 0), key_end = kb + (j + 1) * LT_BK;
+        const bool asc = __all_sync(0xffffffffu, pa == base + lane && pb == base + 32 + lane);
+        // descending pages reverse the keys inside the tile, which is fine where every row sees all of them
+        const bool desc = __all_sync(0xffffffffu, pa == base - lane && pb == base - 32 - lane) && base >= LT_BK && key_end <= lim_min;
+        const bool run = key_end <= ke && base >= 1 && (asc || desc);
+        uint8_t* c_ptr = c_s + (size_t)st * C_BYTES;
+        if (run) {
+          if (lane == 0) {
+            if (lw == 0) {
+              mbar_expect_tx(&S.c_full[st], C_BYTES);
+              for (int pan = 0; pan < NPAN; ++pan)
+                tma_load_2d(c_ptr + pan * LT_PANEL_C, &tmC, &S.c_full[st], pan * 64, asc ? base : base - (LT_BK - 1), pol);
+            } else {
+              mbar_arrive(&S.c_full[st]);
+            }
+          }
+          gathered &= ~(1u << (j & 31));
+        } else {
+          const uint32_t c_t = smem_u32(c_ptr);
+          const int mine = lw < 2 ? pa : pb;          // this warp's 16 keys sit in lanes (lw & 1) * 16 ..
+#pragma unroll 4
+          for (int idx = lane; idx < KPW * CPR; idx += 32) {
+            const int kl = idx / CPR, c = idx % CPR, key = lw * KPW + kl;
+            const int pgi = __shfl_sync(0xffffffffu, mine, (lw & 1) * 16 + kl);
+            const uint32_t dst = c_t + (uint32_t)((c >> 3) * LT_PANEL_C + key * 128 + (((c & 7) ^ (key & 7)) << 4));
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(p.pool + (size_t)pgi * p.ldc + c * 8) : "memory");
+          }
+          gathered |= 1u << (j & 31);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");       // one group per tile (empty for a TMA tile)
+        if (j >= LAG && ((gathered >> ((j - LAG) & 31)) & 1u)) {   // gathered tile j - LAG has landed: hand it over
+          asm volatile("cp.async.wait_group %0;" ::"n"(LAG) : "memory");
+          fence_proxy_async();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&S.c_full[(j - LAG) % STAGES]);
+        }
+        ++issued;
+      }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    fence_proxy_async();
+    __syncwarp();
+    if (lane == 0)
+      for (int t = max(0, issued - LAG); t < issued; ++t)
+        if ((gathered >> (t & 31)) & 1u) mbar_arrive(&S.c_full[t % STAGES]);
+    // TMA copies still in flight after an abort must land before the CTA ends
+    if (S.abort && lw == 0 && lane == 0) {
+      if (n_tiles > 0) (void)mbar_wait(&S.q_full, 0);
+      for (int t = max(0, issued - STAGES); t < issued; ++t)
+        if (!((gathered >> (t & 31)) & 1u)) (void)mbar_wait(&S.c_full[t % STAGES], (uint32_t)(t / STAGES) & 1u);
+    }
+  } else if (warp == 4) {
+    // ================================================================= MMA issuer (one thread)
+    if (elect_one()) {
+      constexpr uint32_t idesc_s = umma_idesc_bf16(128, LT_BK);
+      const uint32_t q_addr = smem_u32(q_s), p_addr = smem_u32(p_s), c_addr0 = smem_u32(c_s);
+      auto issue_s = [&](int j) -> bool {
+        const int st = j % STAGES;
+        if (!lt_wait(S, p.status, &S.c_full[st], (uint32_t)(j / STAGES) & 1u)) return false;
+        if (j >= 2 && !lt_wait(S, p.status, &S.s_empty[j & 1], (uint32_t)((j >> 1) - 1) & 1u)) return false;
+        tc_fence_after();
+        const uint32_t c_addr = c_addr0 + (uint32_t)st * C_BYTES;
+#pragma unroll
+        for (int pan = 0; pan < NPAN; ++pan)
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_bf16_ss(tmem_base + (uint32_t)(j & 1) * LT_BK, umma_desc_k_sw128(q_addr + pan * LT_PANEL_Q) + 2 * k,
+                         umma_desc_k_sw128(c_addr + pan * LT_PANEL_C) + 2 * k, idesc_s, (pan | k) ? 1u : 0u);
+        umma_commit(&S.s_full[j & 1]);
+        return true;
+      };
+      bool ok = n_tiles > 0 && lt_wait(S, p.status, &S.q_full, 0) && issue_s(0);
+      for (int j = 0; ok && j < n_tiles; ++j) {
+        if (STAGES > 1 && j + 1 < n_tiles && !issue_s(j + 1)) break;     // next tile's scores overlap this tile's softmax
+        if (!lt_wait(S, p.status, &S.p_full[j & 1], (uint32_t)(j >> 1) & 1u)) break;
+        tc_fence_after();
+        const int st = j % STAGES;
+        const uint32_t pj = p_addr + (uint32_t)(j & 1) * LT_PANEL_Q;
+        const uint32_t v_addr = c_addr0 + (uint32_t)st * C_BYTES + (uint32_t)vpan * LT_PANEL_C;
+        for (int g = 0; g < n_opan; g += 4) {                            // at most 256 output columns per instruction
+          const uint32_t idesc_o = umma_idesc_bf16(128, min(4, n_opan - g) * 64) | (1u << 16);   // B operand is MN-major
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_bf16_ss(tO + (uint32_t)g * 64u, umma_desc_k_sw128(pj) + 2 * k,
+                         umma_desc_mn_sw128(v_addr + g * LT_PANEL_C + k * 2048, LT_PANEL_C), idesc_o, (j | k) ? 1u : 0u);
+        }
+        umma_commit(&S.c_empty[st]);
+        umma_commit(&S.p_empty[j & 1]);                                  // also: O holds the sum over tiles 0..j
+        if (STAGES == 1 && j + 1 < n_tiles && !issue_s(j + 1)) break;
+      }
+    }
+    __syncwarp();
+  } else {
+    // ================================================================= softmax (one query row per thread)
+    const int r = warp * 32 + lane;
+    const uint32_t lane_off = ((uint32_t)(warp * 32)) << 16;
+    const bool real = r < n_rows;
+    const int lim = real ? pos0 + (row0 + r) / p.H + 1 : ke;             // keys [0, lim) are visible (spare rows: unmasked)
+    float m_ref = -INFINITY, l = 0.f;                                    // exponent reference (log2 domain), running sum
+    bool alive = true;
+    const bool idle = warp * 32 >= n_rows;                               // no real row in this warp: keep the protocol only
+    for (int j = 0; j < n_tiles; ++j) {
+      const int nv = min(lim, ke) - kb - j * LT_BK;                      // visible keys of this tile (may be <= 0)
+      if (!__all_sync(0xffffffffu, lt_wait(S, p.status, &S.s_full[j & 1], (uint32_t)(j >> 1) & 1u))) { alive = false; break; }
+      tc_fence_after();
+      uint32_t x[LT_BK];
+      if (!idle) {
+        const uint32_t ts = tmem_base + (uint32_t)(j & 1) * LT_BK + lane_off;
+#pragma unroll
+        for (int c0 = 0; c0 < LT_BK; c0 += 16) tmem_ld_32x32b_x16(ts + c0, *reinterpret_cast<uint32_t(*)[16]>(&x[c0]));
+        tmem_ld_wait();
+      }
+      tc_fence_before();                              // the scores are in registers: the buffer can take tile j + 2
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&S.s_empty[j & 1]);
+      float mx = -INFINITY;
+      const bool full = __all_sync(0xffffffffu, nv >= LT_BK);
+      bool grow = false;
+      if (!idle) {
+        if (full) {
+#pragma unroll
+          for (int i = 0; i < LT_BK; ++i) mx = fmaxf(mx, __uint_as_float(x[i]));
+        } else {
+#pragma unroll
+          for (int i = 0; i < LT_BK; ++i)
+            if (i < nv) mx = fmaxf(mx, __uint_as_float(x[i]));
+        }
+        mx *= p.scale_log2;
+        grow = mx > m_ref + 8.f;                      // also true on the row's first visible key (m_ref = -inf)
+      }
+      if (j >= 1 && __any_sync(0xffffffffu, grow)) {
+        // PV of tile j - 1 must have completed before O is rescaled in tensor memory
+        if (!__all_sync(0xffffffffu, lt_wait(S, p.status, &S.p_empty[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1u))) { alive = false; break; }
+        tc_fence_after();
+        const float alpha = grow ? exp2f(m_ref - mx) : 1.f;
+        for (int c0 = 0; c0 < n_opan * 64; c0 += 16) {
+          uint32_t o[16];
+          tmem_ld_32x32b_x16(tO + lane_off + c0, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+          tmem_st_32x32b_x16(tO + lane_off + c0, o);
+        }
+        tmem_st_wait();
+        l *= alpha;
+      }
+      if (grow) m_ref = mx;
+      // P buffer j & 1 was last read by PV of tile j - 2
+      if (!__all_sync(0xffffffffu, j < 2 || lt_wait(S, p.status, &S.p_empty[j & 1], (uint32_t)((j - 2) >> 1) & 1u))) { alive = false; break; }
+      uint8_t* prow = p_s + (j & 1) * LT_PANEL_Q + r * 128;
+      if (idle) {
+        if (j < 2) {                                  // rows without a query stay zero in both buffers
+#pragma unroll
+          for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(prow + (c << 4)) = make_uint4(0u, 0u, 0u, 0u);
+        }
+      } else {
+        float s0 = 0.f, s1 = 0.f;
+        const float ref = m_ref == -INFINITY ? 0.f : m_ref;
+#pragma unroll
+        for (int c0 = 0; c0 < LT_BK; c0 += 16) {
+          uint32_t pk[8];
+#pragma unroll
+          for (int i = 0; i < 16; i += 2) {
+            float p0 = lt_ex2(fmaf(__uint_as_float(x[c0 + i]), p.scale_log2, -ref));
+            float p1 = lt_ex2(fmaf(__uint_as_float(x[c0 + i + 1]), p.scale_log2, -ref));
+            if (!full) {
+              p0 = c0 + i < nv ? p0 : 0.f;
+              p1 = c0 + i + 1 < nv ? p1 : 0.f;
+            }
+            s0 += p0;
+            s1 += p1;
+            pk[i >> 1] = lt_pack(p0, p1);
+          }
+          const int cc = c0 >> 3;                     // two 16-byte chunks of this row's 128 bytes
+          *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+          *reinterpret_cast<uint4*>(prow + (((cc + 1) ^ (r & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+        }
+        l += s0 + s1;
+      }
+      tc_fence_before();
+      fence_proxy_async();                            // P must be visible to the tensor core
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&S.p_full[j & 1]);
+    }
+    // the last PV has completed when its P buffer is released: read O once
+    if (alive && n_tiles > 0)
+      alive = __all_sync(0xffffffffu, lt_wait(S, p.status, &S.p_empty[(n_tiles - 1) & 1], (uint32_t)((n_tiles - 1) >> 1) & 1u));
+    tc_fence_after();
+    const bool write = real && alive && !S.abort;
+    const size_t gr = (size_t)g_row0 + r;
+    if (n_tiles > 0 && alive && !idle) {
+      const float inv = l > 0.f ? 1.0f / l : 0.f;
+      float* po = p.part + ((size_t)ks * p.T * p.H + gr) * p.ldc + vpan * 64;
+      __nv_bfloat16* oo = p.out + gr * p.ldc + vpan * 64;
+      for (int c0 = 0; c0 < n_opan * 64; c0 += 16) {
+        uint32_t o[16];
+        tmem_ld_32x32b_x16(tO + lane_off + c0, o);
+        tmem_ld_wait();
+        if (write) {
+          if (p.KS > 1) {
+#pragma unroll
+            for (int i = 0; i < 16; i += 4)
+              *reinterpret_cast<uint4*>(po + c0 + i) = make_uint4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+          } else {
+            uint32_t pk[8];
+#pragma unroll
+            for (int i = 0; i < 16; i += 2) pk[i >> 1] = lt_pack(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
+            *reinterpret_cast<uint4*>(oo + c0) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+            *reinterpret_cast<uint4*>(oo + c0 + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+          }
+        }
+      }
+    }
+    if (p.KS > 1 && write && vs == 0) {
+      float* ml = p.part_ml + ((size_t)ks * p.T * p.H + gr) * 2;
+      ml[0] = m_ref;
+      ml[1] = l;
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 4) tmem_dealloc(tmem_base, 512);
+}
+
+// Merge of the key splits: one CTA per query row.
+__global__ void __launch_bounds__(128) latent_merge_kernel(const float* part, const float* part_ml, __nv_bfloat16* out, int rows,
+                                                           int ldc, int KS, int pdl) {
+  if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  const size_t row = blockIdx.x;
+  float m = -INFINITY;
+  for (int s = 0; s < KS; ++s) m = fmaxf(m, part_ml[((size_t)s * rows + row) * 2]);
+  float l = 0.f;
+  for (int s = 0; s < KS; ++s) {
+    const float* ml = part_ml + ((size_t)s * rows + row) * 2;
+    if (ml[1] > 0.f) l = fmaf(ml[1], exp2f(ml[0] - m), l);
+  }
+  const float inv = 1.0f / l;
+  for (int c = threadIdx.x * 4; c < ldc; c += 512) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < KS; ++s) {
+      const float* ml = part_ml + ((size_t)s * rows + row) * 2;
+      if (ml[1] > 0.f) {
+        const float f = exp2f(ml[0] - m) * inv;
+        const float4 v = load4(part + ((size_t)s * rows + row) * ldc + c);
+        a.x = fmaf(f, v.x, a.x); a.y = fmaf(f, v.y, a.y); a.z = fmaf(f, v.z, a.z); a.w = fmaf(f, v.w, a.w);
+      }
+    }
+    store4(out + row * ldc + c, a);
+  }
+}
+
+template <int NPAN>
+static int latent_tc_launch(LatentTcParams& p, const CUtensorMap& tmC, const CUtensorMap& tmQ, cudaStream_t st) {
+  using C = LtCfg<NPAN>;
+  static bool configured = false;
+  if (!configured) {
+    CUDA_CHECK_RET(cudaFuncSetAttribute(latent_tc_kernel<NPAN>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
+    configured = true;
+  }
+  return launch_pdl(latent_tc_kernel<NPAN>, dim3((unsigned)(p.r.n_blk * p.MT * C::VSPLIT), (unsigned)p.KS), dim3(LT_THREADS),
+                    (size_t)C::SMEM, st, p.pdl, p, tmC, tmQ);
+}
+
+}  // namespace smc
+
+// Largest padded latent width the tensor-core kernel takes.
+SMC_API int smc_latent_tc_max_width() { return 512; }
+
+// Key splits for `tiles` row tiles (blocks x 128-row tiles) over about `keys` cached rows: one wave of CTAs, at least 128
+// keys per split, powers of two so that a growing context re-plans rarely.
+SMC_API int smc_latent_tc_splits(int tiles, int ldc, int keys) {
+  const int v = ldc > 384 ? 2 : 1;
+  int ks = 1;
+  while (ks < 32 && (long long)tiles * v * ks * 2 <= 148 && keys / (ks * 2) >= 128) ks *= 2;
+  return ks;
+}
+
+// a: as for smc_latent_attn (bf16).  tokens: query tokens in all; blk_rows: rows (tokens x heads) of the longest block;
+// KS > 1 needs part [KS, tokens * H, ldc] and part_ml [KS, tokens * H, 2] fp32.
+SMC_API int smc_latent_attn_tc(const smc::LatentArgs* a, int tokens, int blk_rows, int KS, float* part, float* part_ml,
+                               cudaStream_t st) {
+  using namespace smc;
+  if (a->r.n_blk <= 0) return 0;
+  if (a->ldc % 64 || a->ldc > 512 || KS < 1 || KS > 32 || (KS > 1 && (part == nullptr || part_ml == nullptr))) return -99;
+  LatentTcParams p;
+  p.pool = (const __nv_bfloat16*)a->pool; p.out = (__nv_bfloat16*)a->out; p.part = part; p.part_ml = part_ml;
+  p.block_table = a->block_table; p.bt_stride = a->bt_stride; p.bt_rows = a->bt_rows; p.n_pages = a->n_pages;
+  p.H = a->H; p.ldc = a->ldc; p.KS = KS; p.MT = (blk_rows + 127) / 128; p.T = tokens;
+  p.scale_log2 = a->scale * 1.4426950408889634f;
+  p.r = a->r; p.status = a->status; p.pdl = a->pdl;
+  CUtensorMap tmC, tmQ;
+  int rc = pool_tmap(&tmC, a->pool, (long long)a->n_pages + 1, a->ldc);
+  if (rc == 0) rc = make_tmap(&tmQ, a->q, (long long)tokens * a->H, a->ldc, a->ldc, 128);
+  if (rc) return rc;
+  switch (a->ldc / 64) {
+    case 1: rc = latent_tc_launch<1>(p, tmC, tmQ, st); break;
+    case 2: rc = latent_tc_launch<2>(p, tmC, tmQ, st); break;
+    case 3: rc = latent_tc_launch<3>(p, tmC, tmQ, st); break;
+    case 4: rc = latent_tc_launch<4>(p, tmC, tmQ, st); break;
+    case 5: rc = latent_tc_launch<5>(p, tmC, tmQ, st); break;
+    case 6: rc = latent_tc_launch<6>(p, tmC, tmQ, st); break;
+    case 7: rc = latent_tc_launch<7>(p, tmC, tmQ, st); break;
+    case 8: rc = latent_tc_launch<8>(p, tmC, tmQ, st); break;
+  }
+  if (rc || KS == 1) return rc;
+  return launch_pdl(latent_merge_kernel, dim3((unsigned)(tokens * a->H)), dim3(128), 0, st, p.pdl, (const float*)part,
+                    (const float*)part_ml, p.out, tokens * a->H, p.ldc, KS, p.pdl);
+}

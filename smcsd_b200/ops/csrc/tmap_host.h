@@ -4,6 +4,9 @@
 #include <cuda.h>
 #include <cuda_runtime.h>
 
+#include <mutex>
+#include <unordered_map>
+
 namespace smc {
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
@@ -50,6 +53,31 @@ inline int make_tmap_u8(CUtensorMap* tm, const void* base, long long rows, long 
                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   return r == CUDA_SUCCESS ? 0 : -2 - (int)r;
+}
+
+// Tensor maps of page pools ([pages + 1, row] bf16, box = 64 columns x 64 pages), cached per pool.
+struct PoolMapKey {
+  const void* base; long long rows, cols;
+  bool operator==(const PoolMapKey& o) const { return base == o.base && rows == o.rows && cols == o.cols; }
+};
+struct PoolMapHash {
+  size_t operator()(const PoolMapKey& k) const {
+    return std::hash<const void*>()(k.base) ^ (std::hash<long long>()(k.rows) * 1315423911u) ^ std::hash<long long>()(k.cols);
+  }
+};
+inline int pool_tmap(CUtensorMap* tm, const void* base, long long rows, long long cols) {
+  static std::unordered_map<PoolMapKey, CUtensorMap, PoolMapHash> cache;
+  static std::mutex mu;
+  std::lock_guard<std::mutex> lock(mu);
+  const PoolMapKey key{base, rows, cols};
+  auto it = cache.find(key);
+  if (it != cache.end()) { *tm = it->second; return 0; }
+  const int rc = make_tmap(tm, base, rows, cols, cols, 64);
+  if (rc == 0) {
+    if (cache.size() > 4096) cache.clear();
+    cache.emplace(key, *tm);
+  }
+  return rc;
 }
 
 }  // namespace smc

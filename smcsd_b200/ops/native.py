@@ -653,6 +653,11 @@ def layered_lib():
         L.smc_gather_rows.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, vp]
         L.smc_latent_new.argtypes = [vp, i, i, i, vp, f, vp, i, vp, i, i, vp, i, vp, i, i, vp]
         L.smc_latent_attn.argtypes = [vp, i, vp]
+        L.smc_latent_attn_tc.argtypes = [vp, i, i, i, vp, vp, vp]
+        L.smc_latent_attn_tc.restype = C.c_int
+        L.smc_latent_tc_splits.argtypes = [i, i, i]
+        L.smc_latent_tc_splits.restype = C.c_int
+        L.smc_latent_tc_max_width.restype = C.c_int
         for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_clamped_glu_f32",
                   "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn"):
             getattr(L, n).restype = C.c_int
@@ -738,3 +743,17 @@ def latent_new(proj: torch.Tensor, q: Optional[torch.Tensor], pool: torch.Tensor
 
 def latent_attention(a: LatentArgs, f32: bool) -> None:
     _check(layered_lib().smc_latent_attn(C.byref(a), int(f32), _stream()), "smc_latent_attn")
+
+
+def latent_tc_splits(tiles: int, width: int, keys: int) -> int:
+    """Key splits of the tensor-core latent attention for ``tiles`` row tiles over about ``keys`` cached rows."""
+    return layered_lib().smc_latent_tc_splits(tiles, width, int(keys))
+
+
+def latent_attention_tc(a: LatentArgs, *, tokens: int, blk_rows: int, splits: int = 1, part: Optional[torch.Tensor] = None,
+                        part_ml: Optional[torch.Tensor] = None) -> None:
+    """bf16 latent attention on the tensor cores; ``splits`` > 1 parks partial rows in part / part_ml and merges them."""
+    _check(layered_lib().smc_latent_attn_tc(C.byref(a), tokens, blk_rows, splits, _p(part), _p(part_ml), _stream()),
+           "smc_latent_attn_tc")
+    global launch_count
+    launch_count += splits > 1

@@ -11,6 +11,7 @@ captured in a graph.
 """
 from __future__ import annotations
 
+import os
 from typing import Dict, List, Optional
 
 import torch
@@ -21,9 +22,14 @@ from . import native as K
 from .ragged import RaggedPlan, uniform_struct
 
 
+def _env_flag(name: str, default: bool) -> bool:
+    v = os.environ.get(name)
+    return default if v is None else v.strip().lower() in ("1", "true", "yes", "on")
+
+
 class NativePasizen:
     ragged = True
-    BLOCK = 16                            # tokens per block of the work list
+    BLOCK = 64                            # tokens per block of the work list
 
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
@@ -73,8 +79,9 @@ class NativePasizen:
             self._room("gu", max([pairs * 2 * round_up(f.expert.ff, GU_BLOCK) for f in moe] +
                                  [T * 2 * round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared], default=0), torch.float32)
         self.logits = torch.empty(max_logit_rows, self.V, dtype=torch.float32, device=self.dev)
-        # attention split over key ranges: parked states, allocated when a plan first needs them
-        self._parts: Optional[torch.Tensor] = None
+        # attention split over key ranges: parked rows, allocated when a plan first needs them
+        self._parts = self._parts_ml = torch.empty(0, dtype=torch.float32, device=self.dev)
+        self.attn_tc = not self.f32 and _env_flag("SMC_LATENT_TC", True)
         self._steps = self._build_steps()
 
     # ---- buffers ------------------------------------------------------------------------
@@ -120,10 +127,18 @@ class NativePasizen:
     def set_context(self, ctx: int, bs: int, Es=(1, 2)) -> tuple:
         """Record the context-length hint; returns what it decides about the launch grids (part of a graph's identity)."""
         self.ctx_hint = int(ctx)
-        return tuple(self._ks(bs, E) for E in Es)
+        shapes = sorted({(L.mixer.heads, round_up(L.mixer.kv_rank, 64)) for L in self.c.layers})
+        return tuple(self._ks(bs * ((E + self.BLOCK - 1) // self.BLOCK), min(E, self.BLOCK), H, Rp) for E in Es for H, Rp in shapes)
 
-    def _ks(self, bs: int, E: int) -> int:
-        return 1
+    def _ks(self, n_blk: int, tokens: int, H: int, Rp: int) -> int:
+        """Key splits of one layer's attention: ``n_blk`` blocks of at most ``tokens`` tokens."""
+        if not self.attn_tc or Rp > K.latent_tc_max_width():
+            return 1
+        ks = K.latent_tc_splits(n_blk * ((tokens * H + 127) // 128), Rp, self.ctx_hint)
+        cap = max(1, int(self.attn_splits))
+        while ks > cap:
+            ks //= 2
+        return ks
 
     def _cluster(self, N: int, Kd: int, M: int) -> int:
         key = (N, Kd, M)
@@ -161,7 +176,7 @@ class NativePasizen:
         K.gemm_grouped(W, X, act, N=ff2, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, link=link, status=self.status, pdl=self.pdl)
 
     # ---- sublayers ----------------------------------------------------------------------
-    def _mixer(self, s: dict, T: int, locs: torch.Tensor, work: "K.Ragged", ks: int) -> None:
+    def _mixer(self, s: dict, T: int, locs: torch.Tensor, work: "K.Ragged", longest: int) -> None:
         L, run = s["L"], s["run"]
         m, pdl = L.spec.mixer, self.pdl
         H, D8, R, Rp = m.heads, round_up(m.dim, 8), m.kv_rank, round_up(m.kv_rank, 64)
@@ -176,7 +191,16 @@ class NativePasizen:
         a = K.LatentArgs(q=K.ptr(lat), pool=K.ptr(pool), out=K.ptr(ctx), block_table=K.ptr(self.bt), bt_stride=self.bt.stride(0),
                          bt_rows=self.bt.shape[0], n_pages=pool.shape[0] - 1, H=H, ldc=Rp, scale=m.scale, r=work,
                          status=K.ptr(self.status), pdl=int(pdl))
-        K.latent_attention(a, self.f32)
+        if self.attn_tc and Rp <= K.latent_tc_max_width():
+            tokens = min(longest, self.BLOCK)
+            ks = self._ks(work.n_blk, tokens, H, Rp)
+            if ks > 1 and self._parts.numel() < ks * T * H * Rp:
+                self._parts = torch.empty(ks * T * H * Rp, dtype=torch.float32, device=self.dev)
+            if ks > 1 and self._parts_ml.numel() < ks * T * H * 2:
+                self._parts_ml = torch.empty(ks * T * H * 2, dtype=torch.float32, device=self.dev)
+            K.latent_attention_tc(a, tokens=T, blk_rows=tokens * H, splits=ks, part=self._parts, part_ml=self._parts_ml)
+        else:
+            K.latent_attention(a, self.f32)
         self._per_head(L.wuv, ctx, vo, T, H, Rp, m.vdim)
         self._gemm(L.wo, vo, self._rows("y", T, self.d), T)
 
@@ -217,7 +241,7 @@ class NativePasizen:
             self._gemm(L.s_down, sa, self._rows("y", T, self.d), T)
 
     # ---- forward ------------------------------------------------------------------------
-    def _run(self, ids, positions, locs, T: int, work: "K.Ragged", single_rows: Optional[torch.Tensor], ks: int) -> torch.Tensor:
+    def _run(self, ids, positions, locs, T: int, work: "K.Ragged", single_rows: Optional[torch.Tensor], longest: int) -> torch.Tensor:
         assert T <= self.T and self.state is not None
         for s in self._steps:
             a, kind = s["args"], s["kind"]
@@ -238,7 +262,7 @@ class NativePasizen:
                 if not folded:
                     K.short_conv(self.n, self.xa, s["L"].conv_w, self.state.conv[s["run"]], work, status=self.status, f32=self.f32,
                                  pdl=self.pdl)
-                self._mixer(s, T, locs, work, ks)
+                self._mixer(s, T, locs, work, longest)
             elif kind == "ff":
                 (self._dense if s["L"].spec.mlp.kind == "dense" else self._experts)(s, T)
         return self.xa
@@ -246,12 +270,12 @@ class NativePasizen:
     def forward(self, ids, positions, cache_locs, rows, prefix_lens, bs: int, E: int, two_pass: bool = False) -> torch.Tensor:
         """bs sequences of E new tokens each."""
         work = uniform_struct(rows, prefix_lens, bs, E, self.BLOCK)
-        return self._run(ids, positions, cache_locs, bs * E, work, rows if E == 1 else None, self._ks(bs, E))
+        return self._run(ids, positions, cache_locs, bs * E, work, rows if E == 1 else None, E)
 
     def forward_plan(self, plan: RaggedPlan) -> torch.Tensor:
         self.ctx_hint = plan.max_keys
         return self._run(plan.ids, plan.positions, plan.locs, plan.T, plan.struct, plan.rows if plan.single else None,
-                         self._ks(plan.struct.n_blk, 1 if plan.single else self.BLOCK))
+                         plan.longest)
 
     # ---- head ---------------------------------------------------------------------------
     def final_hidden(self, rows_idx: torch.Tensor) -> torch.Tensor:

@@ -26,6 +26,7 @@ class Portion:
 class RaggedPlan:
     T: int
     single: bool                          # every sequence brings exactly one token
+    longest: int                          # most tokens any sequence brings
     max_keys: int                         # longest context any token sees
     ids: torch.Tensor
     positions: torch.Tensor
@@ -81,5 +82,5 @@ def pack_ragged(portions: Sequence[Portion], capacity: int, block: int, block_ta
         locs = block_table[t_row.long(), t_pos.long()].contiguous()
         st = K.Ragged(seq_row=K.ptr(rows), seq_prefix=K.ptr(prefix), seq_off=K.ptr(soff), seq_len=K.ptr(slen), blk_seq=K.ptr(bseq),
                       blk_start=K.ptr(bstart), n_seq=n_seq, n_blk=n_blk, E=0, B=block)
-        yield RaggedPlan(off, all(n == 1 for _, _, n in seqs), max(c[1] + c[3] for c in seq_cols), t_ids, t_pos, locs, rows, st,
+        yield RaggedPlan(off, all(n == 1 for _, _, n in seqs), max(c[3] for c in seq_cols), max(c[1] + c[3] for c in seq_cols), t_ids, t_pos, locs, rows, st,
                          (host, d), tokens)

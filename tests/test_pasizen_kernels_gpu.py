@@ -172,7 +172,7 @@ def test_poly_norm(f32, ff):
     _close(out, O.poly_norm(z.double(), coef.double(), 1e-3), 1e-5 if f32 else 1e-2)
 
 
-def _work(K, seqs, block=16):
+def _work(K, seqs, block=64):
     """Ragged work list of (row, prefix, length) sequences."""
     rows, pref, lens = zip(*seqs)
     off = [sum(lens[:i]) for i in range(len(lens))]
@@ -295,6 +295,44 @@ def test_latent_attention(f32, H, R, seqs):
     K.latent_attention(a, f32)
     _close(out, _latent_ref(bt, pool, q, H, Rp, seqs, R ** -0.5), 1e-5 if f32 else 1e-2)
     assert int(st) == 0
+
+
+def _page_order(bt, seqs, kind):
+    """Pages of every sequence renumbered: consecutive ascending, consecutive descending, or left scattered."""
+    if kind == "scattered":
+        return bt
+    out, at = torch.zeros_like(bt), 1
+    for row, p, n in seqs:
+        ids = torch.arange(at, at + p + n, dtype=torch.int32, device=bt.device)
+        out[row, :p + n] = ids if kind == "up" else ids.flip(0)
+        at += p + n
+    return out
+
+
+TC_SEQS = SEQS + [[(0, 0, 200)], [(2, 63, 2), (3, 64, 65), (1, 127, 1), (5, 128, 3)], [(4, 900, 130), (6, 1, 1)]]
+
+
+@pytest.mark.parametrize("splits", [1, 2, 8])
+@pytest.mark.parametrize("pages", ["scattered", "up", "down"])
+@pytest.mark.parametrize("H,R", [(8, 64), (3, 48), (5, 180), (16, 256), (7, 320), (20, 384), (2, 448), (16, 512)])
+@pytest.mark.parametrize("seqs", TC_SEQS)
+def test_latent_attention_on_tensor_cores(seqs, H, R, pages, splits):
+    """Row tiles that straddle tokens, key tiles at every causal edge, prompts beside single tokens, merged key splits;
+    a query that singles out the first key, the last cached key, its own key and the next (invisible) one."""
+    K = _k()
+    s, (row, p, n) = len(seqs) - 1, seqs[-1]
+    far = [(s, n - 1, 0), (s, 0, p)] + ([(s, n // 2, p + n // 2 + 1)] if n > 2 else []) + ([(0, 0, seqs[0][1] - 1)] if seqs[0][1] else [])
+    bt, pool, q, Rp = _latent_case(K, torch.bfloat16, H, R, seqs, far=far)
+    bt = _page_order(bt, seqs, pages)
+    T = q.shape[0]
+    out, st = torch.zeros_like(q), _status()
+    part, ml = torch.full((splits * T * H * Rp,), float("nan"), device=DEV), torch.full((splits * T * H * 2,), float("nan"), device=DEV)
+    work, keep = _work(K, seqs)
+    a = K.LatentArgs(q=K.ptr(q), pool=K.ptr(pool), out=K.ptr(out), block_table=K.ptr(bt), bt_stride=bt.stride(0), bt_rows=bt.shape[0],
+                     n_pages=pool.shape[0] - 1, H=H, ldc=Rp, scale=R ** -0.5, r=work, status=K.ptr(st))
+    K.latent_attention_tc(a, tokens=T, blk_rows=min(64, max(x[2] for x in seqs)) * H, splits=splits, part=part, part_ml=ml)
+    assert int(st) == 0
+    _close(out, _latent_ref(bt, pool, q, H, Rp, seqs, R ** -0.5), 1.5e-2)
 
 
 @pytest.mark.parametrize("f32", [False, True])
