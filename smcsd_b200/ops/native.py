@@ -745,6 +745,11 @@ def latent_attention(a: LatentArgs, f32: bool) -> None:
     _check(layered_lib().smc_latent_attn(C.byref(a), int(f32), _stream()), "smc_latent_attn")
 
 
+def latent_tc_max_width() -> int:
+    """Widest (padded) latent row the tensor-core kernel takes."""
+    return layered_lib().smc_latent_tc_max_width()
+
+
 def latent_tc_splits(tiles: int, width: int, keys: int) -> int:
     """Key splits of the tensor-core latent attention for ``tiles`` row tiles over about ``keys`` cached rows."""
     return layered_lib().smc_latent_tc_splits(tiles, width, int(keys))
