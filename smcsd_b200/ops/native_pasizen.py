@@ -78,7 +78,8 @@ class NativePasizen:
         if self.f32:
             self._room("gu", max([pairs * 2 * round_up(f.expert.ff, GU_BLOCK) for f in moe] +
                                  [T * 2 * round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared], default=0), torch.float32)
-        self.logits = torch.empty(max_logit_rows, self.V, dtype=torch.float32, device=self.dev)
+        # the samplers read rows of float4
+        self.logits = torch.empty(max_logit_rows, round_up(self.V, 4), dtype=torch.float32, device=self.dev)
         # attention split over key ranges: parked rows, allocated when a plan first needs them
         self._parts = self._parts_ml = torch.empty(0, dtype=torch.float32, device=self.dev)
         self.attn_tc = not self.f32 and _env_flag("SMC_LATENT_TC", True)
