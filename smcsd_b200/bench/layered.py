@@ -1,0 +1,265 @@
+"""Prefill and decode of Pasizen beside a dense Llama-style model of equal size, whole forwards and kernel by kernel.
+
+    python -m smcsd_b200.bench.layered --width 2048            (or: python bench.py --layered 2048,1024)
+
+Both models run random weights through their kernel chains: the same width, heads, layer count, head and feed-forward
+weights per layer; the dense model caches as many bytes per token as its KV heads take.  A forward is captured in a CUDA
+graph and timed with CUDA events (weights of all layers exceed L2; the cached keys come on top).  For the kernel table every
+launch of one forward is recorded and the launches of one kind - the same kernel in all layers, so that the weights rotate -
+are captured and timed together.  Fraction = (the larger of bytes / measured copy bandwidth and FLOPs / measured bf16 rate)
+/ measured time.
+"""
+from __future__ import annotations
+
+import argparse
+import ctypes
+import json
+from collections import OrderedDict
+from typing import Dict, List, Tuple
+
+import torch
+
+from ..models.config import FeedForwardSpec, GluSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RouterSpec
+from ..utils.roofline import measured_peaks
+
+VOCAB = 32768
+
+
+def pasizen_config(width: int, layers: int, kv_rank: int, experts: bool) -> ModelConfig:
+    H, ff = width // 128, 3 * width
+    mixer = LatentAttentionSpec(heads=H, dim=128, vdim=128, kv_rank=kv_rank, scale=128 ** -0.5)
+    dense = LayerSpec(mixer, FeedForwardSpec("dense", ff=ff))
+    moe = LayerSpec(mixer, FeedForwardSpec("moe", expert=GluSpec(ff // 8, 7.0), router=RouterSpec(32, 4, 8, 4), shared=GluSpec(ff // 6, 7.0)))
+    return ModelConfig(arch="pasizen", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=H, n_kv_heads=1, head_dim=kv_rank,
+                       ffn_size=0, rms_eps=1e-6, max_position=8192, layers=[moe if experts else dense] * layers, streams=4,
+                       conv_taps=4, name=f"pasizen-{width}-{'experts' if experts else 'dense'}")
+
+
+def dense_config(width: int, layers: int) -> ModelConfig:
+    """The closest existing family: gate / up / down of the same number of weights as the two PolyNorm matrices."""
+    return ModelConfig(arch="llama", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=width // 128,
+                       n_kv_heads=max(1, width // 512), head_dim=128, ffn_size=2 * width, rms_eps=1e-6, max_position=8192,
+                       name=f"llama-{width}")
+
+
+class Rig:
+    """One model with its chain, caches filled with noise, and step inputs."""
+
+    def __init__(self, cfg: ModelConfig, bs: int, ctx: int, prompt: int, n_prompts: int):
+        from ..memory.pools import KVPool, StatePool
+        from ..models import build_model
+        from ..ops.native_backend import NativeLlama
+        from ..ops.native_pasizen import NativePasizen
+        dev = self.dev = torch.device("cuda", 0)
+        self.cfg, self.bs, self.ctx, self.prompt, self.n_prompts = cfg, bs, ctx, prompt, n_prompts
+        m = self.m = build_model(cfg, torch.bfloat16, dev, seed=3)
+        span = max(ctx + 1, prompt)
+        rows = max(bs, n_prompts)
+        kv = self.kv = KVPool(m.kv_spec(torch.bfloat16), rows * span, dev)
+        for t in list(kv.k) + list(kv.v):
+            t.normal_(0, 0.5)
+        perm = (torch.randperm(rows * span, generator=torch.Generator().manual_seed(1)) + 1).to(torch.int32)
+        self.bt = perm.view(rows, span).to(dev).contiguous()               # scattered pages: the worst case for both
+        self.status = torch.zeros(1, dtype=torch.int32, device=dev)
+        T = n_prompts * prompt
+        if cfg.arch == "pasizen":
+            spec = m.state_spec()
+            self.state = StatePool(spec, rows, dev)
+            make = lambda t, lr: NativePasizen(m, kv, self.bt, t, lr, 16, self.status, True, state=self.state)
+        else:
+            make = lambda t, lr: NativeLlama(m, kv, self.bt, t, lr, 16, self.status, True)
+        self.dec, self.pre = make(bs, bs), make(T, 8)
+        g = torch.Generator().manual_seed(2)
+        i32 = lambda v: torch.as_tensor(v, dtype=torch.int32).to(dev)
+        self.ids = i32(torch.randint(0, VOCAB, (bs,), generator=g))
+        self.pos, self.rows, self.pref = i32([ctx] * bs), i32(list(range(bs))), i32([ctx] * bs)
+        self.locs = self.bt[:bs, ctx].contiguous()
+        self.p_ids = torch.randint(0, VOCAB, (T,), generator=g).tolist()
+        self.dec.set_context(ctx + 1, bs, (1,))
+        if cfg.arch == "pasizen":
+            from ..ops.ragged import Portion, pack_ragged
+            portions = [Portion(r, 0, self.p_ids[r * prompt:(r + 1) * prompt]) for r in range(n_prompts)]
+            self.plan = next(pack_ragged(portions, T, self.pre.BLOCK, self.bt))
+        else:
+            B = 16
+            nb = prompt // B
+            self.p_args = (i32(self.p_ids), i32(list(range(prompt)) * n_prompts), self.bt[:n_prompts, :prompt].reshape(-1).contiguous(),
+                           i32([r for r in range(n_prompts) for _ in range(nb)]), i32([j * B for _ in range(n_prompts) for j in range(nb)]))
+            self.pre.set_context(prompt, n_prompts * nb)
+
+    def decode(self) -> None:
+        self.dec.forward(self.ids, self.pos, self.locs, self.rows, self.pref, self.bs, 1)
+
+    def prefill(self) -> None:
+        if self.cfg.arch == "pasizen":
+            self.pre.forward_plan(self.plan)
+        else:
+            self.pre.forward(*self.p_args, self.n_prompts * self.prompt // 16, 16, two_pass=True)
+
+
+def timed(fn, reps: int = 20) -> float:
+    """Microseconds per call, captured in a graph (so that host launch time is out)."""
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        fn()
+    torch.cuda.current_stream().wait_stream(side)
+    torch.cuda.synchronize()
+    gr = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(gr):
+        fn()
+    for _ in range(3):
+        gr.replay()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(reps):
+        gr.replay()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / reps * 1e3
+
+
+# ---------------------------------------------------------------------------------- kernel by kernel
+RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
+            "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc")
+
+
+def record(fn) -> List[Tuple[str, tuple, dict]]:
+    """Every kernel call of one forward (structures copied: the chain reuses them)."""
+    from ..ops import native as K
+    calls, saved = [], {}
+
+    def keep(x):
+        return type(x).from_buffer_copy(x) if isinstance(x, ctypes.Structure) else x
+    for name in RECORDED:
+        real = saved[name] = getattr(K, name)
+
+        def wrapped(*a, _real=real, _name=name, **kw):
+            calls.append((_name, tuple(keep(x) for x in a), {k: keep(v) for k, v in kw.items()}))
+            return _real(*a, **kw)
+        setattr(K, name, wrapped)
+    try:
+        fn()
+        torch.cuda.synchronize()
+    finally:
+        for name, real in saved.items():
+            setattr(K, name, real)
+    return calls
+
+
+def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: int) -> Tuple[str, float, float]:
+    """(kind, bytes, FLOPs) of a recorded call; ``keys``: cached rows an average token attends to; ``seqs``: sequences."""
+    cfg = rig.cfg
+    d = cfg.hidden_size
+    if name in ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped"):
+        W, X, out = a[:3]
+        M, N, Kd = kw["M"], (kw["N"] if "N" in kw else W.shape[0]), W.shape[-1]
+        link = kw.get("link")
+        groups = link.groups if link is not None and link.mode == 1 else 1
+        wbytes = W.numel() * 2
+        if link is not None and link.mode == 2:                # experts that some token chose (uniform choices)
+            wbytes = wbytes * (1.0 - (1.0 - 1.0 / link.groups) ** M)
+        flops = 2.0 * M * N * Kd * groups
+        epi = kw["epi"]
+        per_out = {1: 2, 2: 1, 3: 4, 4: 8}[epi]                # bytes per product (gated pairs leave half a bf16 value each)
+        kind = f"gemm {N}x{Kd}" + (f" x{groups} heads" if groups > 1 else "") + (" experts" if link is not None and link.mode == 2 else "")
+        return kind, wbytes + M * Kd * 2 * groups + M * N * groups * per_out, flops
+    if name == "latent_attention_tc":
+        s = a[0]
+        fl = 2.0 * 2 * T * s.H * keys * s.ldc
+        return "attention", T * s.H * s.ldc * 4 + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.ldc * 2, fl
+    if name == "attention_fused":
+        H, Hkv, D = kw["Hq"], kw["Hkv"], kw["D"]
+        fl = 2.0 * 2 * T * H * keys * D
+        return "attention", T * H * D * 6 + seqs * (rig.ctx if T == rig.bs else rig.prompt) * Hkv * D * 4, fl
+    if name == "hyper_step":
+        s = a[0]
+        S = s.S
+        by = T * d * (4 * S * (1 + (s.w_in is not None)) + 4 * (s.y is not None) + 4 * s.top + 4 * (s.n_out is not None) + 2 * (s.xa is not None))
+        return "streams + norm" + (" + conv" if s.conv_w else "") + (" + experts" if s.top else ""), by, 0.0
+    sizes = {"add_rmsnorm": T * d * 10, "short_conv": T * d * 6, "rope_kv_write": T * (cfg.q_size + 2 * cfg.kv_size) * 6}
+    if name == "poly_norm":
+        return "PolyNorm", T * kw["ff"] * 6, 0.0
+    if name == "latent_new":
+        return "latent_new", T * (kw["nq"] * 6 + kw["R"] * 6), 0.0
+    if name == "gather_rows":
+        return "gather_rows", kw["n"] * a[2].shape[1] * 4, 0.0
+    if name == "route":
+        return "route", T * kw["d"] * 4 + a[1].numel() * 2, 2.0 * T * kw["d"] * a[1].shape[0]
+    if name == "dispatch":
+        return "dispatch", kw["n"] * 12, 0.0
+    return name, float(sizes[name]), 0.0
+
+
+def kernel_table(rig: Rig, fn, T: int, keys: float, seqs: int) -> List[dict]:
+    from ..ops import native as K
+    hbm, tflops, _ = measured_peaks()
+    kinds: Dict[str, dict] = OrderedDict()
+    for name, a, kw in record(fn):
+        kind, by, fl = work_of(rig, name, a, kw, T, keys, seqs)
+        k = kinds.setdefault(kind, {"kernel": kind, "calls": [], "bytes": by, "flops": fl})
+        k["calls"].append((getattr(K, name), a, kw))
+    out = []
+    for k in kinds.values():
+        calls = k.pop("calls")
+        us = timed(lambda: [f(*a, **kw) for f, a, kw in calls], reps=8) / len(calls)
+        floor = max(k["bytes"] / (hbm * 1e3), k["flops"] / (tflops * 1e6))
+        out.append({**k, "launches": len(calls), "us": round(us, 2), "floor_us": round(floor, 2), "fraction": round(floor / us, 3)})
+    return out
+
+
+def run(width: int, layers: int = 12, bs: int = 8, ctx: int = 1024, prompt: int = 1024, n_prompts: int = 4, kv_rank: int = 256,
+        tables: bool = True) -> dict:
+    import gc
+    rec = {"width": width, "layers": layers, "decode": {"sequences": bs, "context": ctx}, "prefill": {"prompts": n_prompts, "tokens": prompt},
+           "kv_rank": kv_rank, "pages": "scattered", "weights": "random, bf16", "models": []}
+    for cfg in (dense_config(width, layers), pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)):
+        rig = Rig(cfg, bs, ctx, prompt, n_prompts)
+        T = n_prompts * prompt
+        dec, pre = timed(rig.decode), timed(rig.prefill, reps=8)
+        one = {"model": cfg.name, "weight_mb": rig.m.weight_bytes() / 1e6, "decode_us": round(dec, 1), "decode_tok_s": round(bs / dec * 1e6),
+               "prefill_us": round(pre, 1), "prefill_tok_s": round(T / pre * 1e6)}
+        if tables:
+            one["decode_kernels"] = kernel_table(rig, rig.decode, bs, ctx + 1, bs)
+            one["prefill_kernels"] = kernel_table(rig, rig.prefill, T, (prompt + 1) / 2, n_prompts)
+        one["device_status"] = int(rig.status.item())
+        rec["models"].append(one)
+        del rig
+        gc.collect()
+        torch.cuda.empty_cache()
+    return rec
+
+
+def show(rec: dict) -> str:
+    lines = [f"width {rec['width']}, {rec['layers']} layers, kv_rank {rec['kv_rank']}; decode {rec['decode']}, prefill {rec['prefill']}, "
+             f"pages {rec['pages']}"]
+    for m in rec["models"]:
+        lines.append(f"{m['model']}: {m['weight_mb']:.0f} MB  decode {m['decode_us']} us ({m['decode_tok_s']} tok/s)  prefill "
+                     f"{m['prefill_us']} us ({m['prefill_tok_s']} tok/s)  status {m['device_status']}")
+        for part in ("decode_kernels", "prefill_kernels"):
+            for k in m.get(part, []):
+                lines.append(f"  {part[:7]:8}{k['kernel']:34}{k['launches']:4} x {k['us']:9.2f} us  floor {k['floor_us']:8.2f}  {k['fraction']:.3f}")
+    return "\n".join(lines)
+
+
+def main(argv=None) -> None:
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--width", type=int, default=2048)
+    ap.add_argument("--layers", type=int, default=12)
+    ap.add_argument("--bs", type=int, default=8)
+    ap.add_argument("--ctx", type=int, default=1024)
+    ap.add_argument("--prompt", type=int, default=1024)
+    ap.add_argument("--kv-rank", type=int, default=256)
+    ap.add_argument("--no-tables", action="store_true")
+    ap.add_argument("--json", default=None)
+    ns = ap.parse_args(argv)
+    rec = run(ns.width, ns.layers, ns.bs, ns.ctx, ns.prompt, kv_rank=ns.kv_rank, tables=not ns.no_tables)
+    print(show(rec))
+    if ns.json:
+        with open(ns.json, "w") as f:
+            json.dump(rec, f)
+
+
+if __name__ == "__main__":
+    main()

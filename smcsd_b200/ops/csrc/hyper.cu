@@ -69,8 +69,12 @@ template <int VEC, typename T> __device__ __forceinline__ void stc(T* p, const C
   else *p = from_f32<T>(c.v[0]);
 }
 
-template <int S_T, typename AT, int VEC>
-__global__ void __launch_bounds__(256) hyper_step_kernel(const HyperArgs a) {
+// CONV: 0 no folded convolution, 1 taps and history in registers (up to 4 taps, two column groups per thread), 2 any.
+constexpr int HYPER_CONV_GROUPS = 2, HYPER_CONV_HL = 3;
+
+template <int S_T, typename AT, int VEC, int CONV>
+__global__ void __launch_bounds__(CONV == 1 ? 512 : 256) hyper_step_kernel(const HyperArgs a) {
+  constexpr int NV = CONV == 1 ? HYPER_CONV_GROUPS : HYPER_MAXV;
   __shared__ float red[32];
   __shared__ float s_mix[HYPER_MAX_STREAMS * HYPER_MAX_STREAMS], s_out[HYPER_MAX_STREAMS], s_in[HYPER_MAX_STREAMS];
   const int S = S_T > 0 ? S_T : a.S, d = a.d, t = blockIdx.x;
@@ -81,7 +85,39 @@ __global__ void __launch_bounds__(256) hyper_step_kernel(const HyperArgs a) {
     s_out[threadIdx.x] = a.ids == nullptr ? a.w_out[threadIdx.x] : 0.f;
     s_in[threadIdx.x] = a.w_in != nullptr ? a.w_in[threadIdx.x] : 1.f;
   }
+  constexpr int CG = CONV == 1 ? NV : 1, CH = CONV == 1 ? HYPER_CONV_HL : 1;
+  float cw[CG][VEC][CH + 1], hv[CG][VEC][CH];
+  const int hl = a.taps - 1;
+  if constexpr (CONV == 1) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k)
+#pragma unroll
+        for (int j = 0; j <= CH; ++j) cw[i][k][j] = (c < d && j <= hl) ? a.conv_w[(size_t)(c + k) * (hl + 1) + j] : 0.f;
+    }
+  }
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  int row = 0;
+  if constexpr (CONV != 0) {
+    row = a.rows[t];
+    if (row < 0 || row >= a.n_rows) {
+      if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
+      row = -1;
+    }
+  }
+  if constexpr (CONV == 1) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k)
+#pragma unroll
+        for (int j = 0; j < CH; ++j)
+          hv[i][k][j] = (c < d && j < hl && row >= 0) ? a.hist[((size_t)row * d + c + k) * hl + j] : 0.f;
+    }
+  }
   __syncthreads();
   float* x = a.x + (size_t)t * S * d;
   const AT *er = nullptr, *pr = nullptr;
@@ -96,10 +132,10 @@ __global__ void __launch_bounds__(256) hyper_step_kernel(const HyperArgs a) {
     pr = reinterpret_cast<const AT*>(a.pos) + (size_t)p * d;
   }
   const bool write_x = a.w_in != nullptr;
-  Cols<VEC> u[HYPER_MAXV];
+  Cols<VEC> u[NV];
   float ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < HYPER_MAXV; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
     if (c < d) {
       Cols<VEC> xs[SM], acc;
@@ -155,16 +191,8 @@ __global__ void __launch_bounds__(256) hyper_step_kernel(const HyperArgs a) {
     }
   }
   const float inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)d + a.eps);
-  int row = 0;
-  if (a.conv_w != nullptr) {
-    row = a.rows[t];
-    if (row < 0 || row >= a.n_rows) {
-      if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
-      row = -1;
-    }
-  }
 #pragma unroll
-  for (int i = 0; i < HYPER_MAXV; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
     if (c < d) {
       const Cols<VEC> w = ldc<VEC>(a.norm_w + c);
@@ -172,8 +200,25 @@ __global__ void __launch_bounds__(256) hyper_step_kernel(const HyperArgs a) {
 #pragma unroll
       for (int k = 0; k < VEC; ++k) n.v[k] = u[i].v[k] * inv * w.v[k];
       if (a.n_out != nullptr) stc<VEC>(a.n_out + (size_t)t * d + c, n);
-      if (a.conv_w != nullptr && row >= 0) {
-        const int hl = a.taps - 1;
+      if constexpr (CONV == 1) {
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+          float* hp = a.hist + ((size_t)max(row, 0) * d + c + k) * hl;
+          float o = 0.f;
+#pragma unroll
+          for (int j = 0; j < CH; ++j) o = fmaf(cw[i][k][j], hv[i][k][j], o);      // zero beyond the history
+#pragma unroll
+          for (int j = 0; j <= CH; ++j)
+            if (j == hl) o = fmaf(cw[i][k][j], n.v[k], o);
+          if (row >= 0) {
+#pragma unroll
+            for (int j = 0; j < CH; ++j)
+              if (j < hl) hp[j] = j + 1 < hl ? hv[i][k][j + 1 < CH ? j + 1 : j] : n.v[k];
+            n.v[k] += o;
+          }
+        }
+      }
+      if (CONV == 2 && row >= 0) {
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
           const float* cw = a.conv_w + (size_t)(c + k) * a.taps;
@@ -256,8 +301,18 @@ static int hyper_launch(const HyperArgs& a, int T, cudaStream_t st) {
   const int groups = (a.d + per - 1) / per;
   int threads = groups <= 64 ? 64 : groups <= 128 ? 128 : 256;
   if (groups > threads * HYPER_MAXV) return -91;
-  if (vec) return launch_pdl(hyper_step_kernel<S_T, AT, 4>, dim3(T), dim3(threads), 0, st, a.pdl, a);
-  return launch_pdl(hyper_step_kernel<S_T, AT, 1>, dim3(T), dim3(threads), 0, st, a.pdl, a);
+#define SMC_HYPER(V, CV) return launch_pdl(hyper_step_kernel<S_T, AT, V, CV>, dim3(T), dim3(threads), 0, st, a.pdl, a)
+  if (a.conv_w == nullptr) {
+    if (vec) SMC_HYPER(4, 0);
+    SMC_HYPER(1, 0);
+  }
+  if (vec && a.taps <= HYPER_CONV_HL + 1 && groups <= 512 * HYPER_CONV_GROUPS) {
+    if (groups > threads * HYPER_CONV_GROUPS) threads = 512;
+    SMC_HYPER(4, 1);
+  }
+  if (vec) SMC_HYPER(4, 2);
+  SMC_HYPER(1, 2);
+#undef SMC_HYPER
 }
 
 template <typename AT>

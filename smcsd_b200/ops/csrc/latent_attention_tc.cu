@@ -11,7 +11,8 @@
 // more than 2^8; only then is its part of O rescaled in tensor memory.
 // Cached rows live one page per token: a tile of 64 consecutive pages is fetched with one TMA box per panel, a scattered one
 // is gathered by four loader warps with 16-byte cp.async copies into the same swizzled layout.  Key ranges may be split over
-// CTAs (few sequences, long contexts): every split parks its unnormalised rows in fp32 and a second kernel merges them.
+// the CTAs of a thread-block cluster (few sequences, long contexts): every split parks its unnormalised rows in its own shared
+// memory and the CTAs merge them through distributed shared memory, each a share of the rows.
 // The work list (ragged.cuh) mixes prompts, portions of prompts and single tokens; query rows never mix sequences.
 // Every mbarrier wait is bounded; a timeout raises a status bit and every role unwinds.
 #include "latent_attention.cuh"
@@ -26,6 +27,7 @@ constexpr int LT_PANEL_Q = 128 * 128;           // bytes of one [128 rows][64 va
 constexpr int LT_PANEL_C = LT_BK * 128;
 constexpr int LT_O_COL = 2 * LT_BK;             // first output column in tensor memory
 constexpr int LT_MAX_STAGES = 8;
+constexpr int LT_MAX_SPLITS = 8;                // CTAs of a cluster
 
 // NPAN: panels of 64 values per cached row.  Ring depth within 227 KB next to the Q tile and two P tiles.
 template <int NPAN> struct LtCfg {
@@ -36,14 +38,13 @@ template <int NPAN> struct LtCfg {
   static constexpr int STAGES = FIT > LT_MAX_STAGES ? LT_MAX_STAGES : FIT;
   static constexpr int LAG = STAGES > 2 ? STAGES - 2 : 0;            // gathered tiles in flight behind the newest
   static constexpr int SMEM = FIXED + STAGES * NPAN * LT_PANEL_C + 1024;
-  static_assert(STAGES >= 1, "a tile must fit");
+  static constexpr int OLD = OPAN * 64 + 1;                          // row pitch of the parked rows (floats)
+  static_assert(STAGES >= 1 && 128 * OLD * 4 + 1024 <= SMEM, "a tile and the parked rows must fit");
 };
 
 struct LatentTcParams {
   const __nv_bfloat16* pool;     // [pages + 1, ldc]
   __nv_bfloat16* out;            // [T * H, ldc]
-  float* part;                   // [KS, T * H, ldc] (KS > 1)
-  float* part_ml;                // [KS, T * H, 2]: reference exponent (log2 units), sum
   const int* block_table;
   int bt_stride, bt_rows, n_pages, H, ldc, KS, MT, T;
   float scale_log2;
@@ -56,6 +57,7 @@ struct LtShared {
   uint64_t q_full, c_full[LT_MAX_STAGES], c_empty[LT_MAX_STAGES], s_full[2], s_empty[2], p_full[2], p_empty[2];
   uint32_t tmem_slot;
   volatile int abort;
+  float m[128], l[128];          // key splits: reference exponent (log2 units) and sum of every row
 };
 
 __device__ __forceinline__ bool lt_wait(LtShared& S, int* status, uint64_t* bar, uint32_t parity) {
@@ -374,65 +376,63 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       alive = __all_sync(0xffffffffu, lt_wait(S, p.status, &S.p_empty[(n_tiles - 1) & 1], (uint32_t)((n_tiles - 1) >> 1) & 1u));
     tc_fence_after();
     const bool write = real && alive && !S.abort;
-    const size_t gr = (size_t)g_row0 + r;
+    if (p.KS > 1) {
+      S.m[r] = write ? m_ref : -INFINITY;
+      S.l[r] = write ? l : 0.f;                       // 0: this split holds nothing for the row
+    }
     if (n_tiles > 0 && alive && !idle) {
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      float* po = p.part + ((size_t)ks * p.T * p.H + gr) * p.ldc + vpan * 64;
-      __nv_bfloat16* oo = p.out + gr * p.ldc + vpan * 64;
+      float* po = reinterpret_cast<float*>(q_s) + r * C::OLD;       // operands and tiles are no longer needed
+      __nv_bfloat16* oo = p.out + ((size_t)g_row0 + r) * p.ldc + vpan * 64;
       for (int c0 = 0; c0 < n_opan * 64; c0 += 16) {
         uint32_t o[16];
         tmem_ld_32x32b_x16(tO + lane_off + c0, o);
         tmem_ld_wait();
-        if (write) {
-          if (p.KS > 1) {
+        if (p.KS > 1) {
 #pragma unroll
-            for (int i = 0; i < 16; i += 4)
-              *reinterpret_cast<uint4*>(po + c0 + i) = make_uint4(o[i], o[i + 1], o[i + 2], o[i + 3]);
-          } else {
-            uint32_t pk[8];
+          for (int i = 0; i < 16; ++i) po[c0 + i] = __uint_as_float(o[i]);
+        } else if (write) {
+          uint32_t pk[8];
 #pragma unroll
-            for (int i = 0; i < 16; i += 2) pk[i >> 1] = lt_pack(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
-            *reinterpret_cast<uint4*>(oo + c0) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
-            *reinterpret_cast<uint4*>(oo + c0 + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
-          }
+          for (int i = 0; i < 16; i += 2) pk[i >> 1] = lt_pack(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
+          *reinterpret_cast<uint4*>(oo + c0) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+          *reinterpret_cast<uint4*>(oo + c0 + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
         }
       }
-    }
-    if (p.KS > 1 && write && vs == 0) {
-      float* ml = p.part_ml + ((size_t)ks * p.T * p.H + gr) * 2;
-      ml[0] = m_ref;
-      ml[1] = l;
     }
   }
   tc_fence_before();
   __syncthreads();
   if (warp == 4) tmem_dealloc(tmem_base, 512);
-}
-
-// Merge of the key splits: one CTA per query row.
-__global__ void __launch_bounds__(128) latent_merge_kernel(const float* part, const float* part_ml, __nv_bfloat16* out, int rows,
-                                                           int ldc, int KS, int pdl) {
-  if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
-  const size_t row = blockIdx.x;
-  float m = -INFINITY;
-  for (int s = 0; s < KS; ++s) m = fmaxf(m, part_ml[((size_t)s * rows + row) * 2]);
-  float l = 0.f;
-  for (int s = 0; s < KS; ++s) {
-    const float* ml = part_ml + ((size_t)s * rows + row) * 2;
-    if (ml[1] > 0.f) l = fmaf(ml[1], exp2f(ml[0] - m), l);
-  }
-  const float inv = 1.0f / l;
-  for (int c = threadIdx.x * 4; c < ldc; c += 512) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < KS; ++s) {
-      const float* ml = part_ml + ((size_t)s * rows + row) * 2;
-      if (ml[1] > 0.f) {
-        const float f = exp2f(ml[0] - m) * inv;
-        const float4 v = load4(part + ((size_t)s * rows + row) * ldc + c);
-        a.x = fmaf(f, v.x, a.x); a.y = fmaf(f, v.y, a.y); a.z = fmaf(f, v.z, a.z); a.w = fmaf(f, v.w, a.w);
+  if (p.KS > 1) {
+    // merge: CTA `ks` of the cluster takes rows ks, ks + KS, ..; a warp per row
+    cluster_sync();
+    for (int r = ks + warp * p.KS; r < n_rows; r += p.KS * (LT_THREADS / 32)) {
+      float ms = -INFINITY, ls = 0.f;
+      if (lane < p.KS) {
+        ls = ld_dsmem_f32(smem_u32(&S.l[r]), (uint32_t)lane);
+        if (ls > 0.f) ms = ld_dsmem_f32(smem_u32(&S.m[r]), (uint32_t)lane);
+      }
+      const float mm = warp_max(ms);
+      float f = ls > 0.f ? exp2f(ms - mm) : 0.f;
+      f *= 1.0f / warp_sum(ls * f);
+      const uint32_t base = smem_u32(reinterpret_cast<float*>(q_s) + r * C::OLD);
+      __nv_bfloat16* oo = p.out + ((size_t)g_row0 + r) * p.ldc + vpan * 64;
+      for (int c = lane * 2; c < n_opan * 64; c += 64) {
+        float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+        for (int q = 0; q < LT_MAX_SPLITS; ++q) {
+          const float fq = __shfl_sync(0xffffffffu, f, q);
+          if (q < p.KS && fq > 0.f) {
+            const uint32_t rem = dsmem_map(base + (uint32_t)c * 4u, (uint32_t)q);
+            a0 = fmaf(fq, ld_dsmem_f32_at(rem), a0);
+            a1 = fmaf(fq, ld_dsmem_f32_at(rem + 4u), a1);
+          }
+        }
+        *reinterpret_cast<uint32_t*>(oo + c) = lt_pack(a0, a1);
       }
     }
-    store4(out + row * ldc + c, a);
+    cluster_sync();                                   // nobody leaves while its rows may still be read
   }
 }
 
@@ -444,8 +444,27 @@ static int latent_tc_launch(LatentTcParams& p, const CUtensorMap& tmC, const CUt
     CUDA_CHECK_RET(cudaFuncSetAttribute(latent_tc_kernel<NPAN>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
     configured = true;
   }
-  return launch_pdl(latent_tc_kernel<NPAN>, dim3((unsigned)(p.r.n_blk * p.MT * C::VSPLIT), (unsigned)p.KS), dim3(LT_THREADS),
-                    (size_t)C::SMEM, st, p.pdl, p, tmC, tmQ);
+  cudaLaunchAttribute attr[2];
+  int na = 0;
+  if (p.pdl) {
+    attr[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[na++].val.programmaticStreamSerializationAllowed = 1;
+  }
+  if (p.KS > 1) {
+    attr[na].id = cudaLaunchAttributeClusterDimension;
+    attr[na].val.clusterDim.x = 1;
+    attr[na].val.clusterDim.y = (unsigned)p.KS;
+    attr[na++].val.clusterDim.z = 1;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)(p.r.n_blk * p.MT * C::VSPLIT), (unsigned)p.KS);
+  cfg.blockDim = dim3(LT_THREADS);
+  cfg.dynamicSmemBytes = C::SMEM;
+  cfg.stream = st;
+  cfg.attrs = attr;
+  cfg.numAttrs = na;
+  CUDA_CHECK_RET(cudaLaunchKernelEx(&cfg, latent_tc_kernel<NPAN>, (const LatentTcParams)p, tmC, tmQ));
+  return 0;
 }
 
 }  // namespace smc
@@ -453,24 +472,23 @@ static int latent_tc_launch(LatentTcParams& p, const CUtensorMap& tmC, const CUt
 // Largest padded latent width the tensor-core kernel takes.
 SMC_API int smc_latent_tc_max_width() { return 512; }
 
-// Key splits for `tiles` row tiles (blocks x 128-row tiles) over about `keys` cached rows: one wave of CTAs, at least 128
-// keys per split, powers of two so that a growing context re-plans rarely.
+// Key splits for `tiles` row tiles (blocks x 128-row tiles) over about `keys` cached rows: one wave of CTAs, at least
+// LT_BK keys per split, powers of two so that a growing context re-plans rarely.
 SMC_API int smc_latent_tc_splits(int tiles, int ldc, int keys) {
   const int v = ldc > 384 ? 2 : 1;
   int ks = 1;
-  while (ks < 32 && (long long)tiles * v * ks * 2 <= 148 && keys / (ks * 2) >= 128) ks *= 2;
+  while (ks < smc::LT_MAX_SPLITS && (long long)tiles * v * ks * 2 <= 148 && keys / (ks * 2) >= smc::LT_BK) ks *= 2;
   return ks;
 }
 
 // a: as for smc_latent_attn (bf16).  tokens: query tokens in all; blk_rows: rows (tokens x heads) of the longest block;
-// KS > 1 needs part [KS, tokens * H, ldc] and part_ml [KS, tokens * H, 2] fp32.
-SMC_API int smc_latent_attn_tc(const smc::LatentArgs* a, int tokens, int blk_rows, int KS, float* part, float* part_ml,
-                               cudaStream_t st) {
+// KS: key splits, at most eight.
+SMC_API int smc_latent_attn_tc(const smc::LatentArgs* a, int tokens, int blk_rows, int KS, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_blk <= 0) return 0;
-  if (a->ldc % 64 || a->ldc > 512 || KS < 1 || KS > 32 || (KS > 1 && (part == nullptr || part_ml == nullptr))) return -99;
+  if (a->ldc % 64 || a->ldc > 512 || KS < 1 || KS > LT_MAX_SPLITS) return -99;
   LatentTcParams p;
-  p.pool = (const __nv_bfloat16*)a->pool; p.out = (__nv_bfloat16*)a->out; p.part = part; p.part_ml = part_ml;
+  p.pool = (const __nv_bfloat16*)a->pool; p.out = (__nv_bfloat16*)a->out;
   p.block_table = a->block_table; p.bt_stride = a->bt_stride; p.bt_rows = a->bt_rows; p.n_pages = a->n_pages;
   p.H = a->H; p.ldc = a->ldc; p.KS = KS; p.MT = (blk_rows + 127) / 128; p.T = tokens;
   p.scale_log2 = a->scale * 1.4426950408889634f;
@@ -480,16 +498,14 @@ SMC_API int smc_latent_attn_tc(const smc::LatentArgs* a, int tokens, int blk_row
   if (rc == 0) rc = make_tmap(&tmQ, a->q, (long long)tokens * a->H, a->ldc, a->ldc, 128);
   if (rc) return rc;
   switch (a->ldc / 64) {
-    case 1: rc = latent_tc_launch<1>(p, tmC, tmQ, st); break;
-    case 2: rc = latent_tc_launch<2>(p, tmC, tmQ, st); break;
-    case 3: rc = latent_tc_launch<3>(p, tmC, tmQ, st); break;
-    case 4: rc = latent_tc_launch<4>(p, tmC, tmQ, st); break;
-    case 5: rc = latent_tc_launch<5>(p, tmC, tmQ, st); break;
-    case 6: rc = latent_tc_launch<6>(p, tmC, tmQ, st); break;
-    case 7: rc = latent_tc_launch<7>(p, tmC, tmQ, st); break;
-    case 8: rc = latent_tc_launch<8>(p, tmC, tmQ, st); break;
+    case 1: return latent_tc_launch<1>(p, tmC, tmQ, st);
+    case 2: return latent_tc_launch<2>(p, tmC, tmQ, st);
+    case 3: return latent_tc_launch<3>(p, tmC, tmQ, st);
+    case 4: return latent_tc_launch<4>(p, tmC, tmQ, st);
+    case 5: return latent_tc_launch<5>(p, tmC, tmQ, st);
+    case 6: return latent_tc_launch<6>(p, tmC, tmQ, st);
+    case 7: return latent_tc_launch<7>(p, tmC, tmQ, st);
+    case 8: return latent_tc_launch<8>(p, tmC, tmQ, st);
   }
-  if (rc || KS == 1) return rc;
-  return launch_pdl(latent_merge_kernel, dim3((unsigned)(tokens * a->H)), dim3(128), 0, st, p.pdl, (const float*)part,
-                    (const float*)part_ml, p.out, tokens * a->H, p.ldc, KS, p.pdl);
+  return -99;
 }

@@ -67,35 +67,66 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const float* gu, int l
 }
 
 // ---------------------------------------------------------------- router
-// A CTA takes TM tokens; a warp takes an expert's weight row and multiplies it with all of them.  Then one warp per token
-// runs the softmax and the two selections.
-template <typename AT>
-__global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const AT* wr, int ldw,
-                                                    int E, int top, int groups, int keep, int T, int TM,
-                                                    int* idx, float* wgt, int pdl) {
+// A CTA takes TM tokens; a warp takes four experts at a time, so that a value read from shared memory meets four weight rows
+// and their loads overlap.  Then one warp per token runs the softmax and the two selections.
+template <typename AT, int TM>
+__global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const AT* wr, int ldw, int E, int top, int groups,
+                                                    int keep, int T, int* idx, float* wgt, int pdl) {
   extern __shared__ float rt_smem[];
-  float* sh = rt_smem;                         // [TM][d]
-  float* sl = sh + (size_t)TM * d;             // [TM][E] logits, then scores
-  float* sg = sl + TM * E;                     // [TM][groups] best score of every group; -1: not kept
+  const int d4 = (d + 3) & ~3;
+  float* sh = rt_smem;                         // [TM][d4]
+  float* sl = sh + (size_t)TM * d4;            // [TM][E] logits, then scores
+  float* sg = sl + TM * E;                     // [TM][groups] best score of every group
   float* sw = sg + TM * groups;                // [TM][top]
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int t0 = blockIdx.x * TM, nt = min(TM, T - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  for (int i = threadIdx.x; i < nt * d; i += blockDim.x) sh[i] = h[(size_t)t0 * d + i];
+  const bool vec = (d & 3) == 0 && (ldw & 3) == 0;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < TM * d; i += blockDim.x * 4)
+      store4(sh + i, i < nt * d ? load4(h + (size_t)t0 * d + i) : make_float4(0.f, 0.f, 0.f, 0.f));
+  } else {
+    for (int i = threadIdx.x; i < TM * d4; i += blockDim.x) {
+      const int m = i / d4, c = i - m * d4;
+      sh[i] = m < nt && c < d ? h[(size_t)(t0 + m) * d + c] : 0.f;
+    }
+  }
   __syncthreads();
-  for (int e = warp; e < E; e += nw) {
-    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    const AT* w = wr + (size_t)e * ldw;
-    for (int c = lane; c < d; c += 32) {
-      const float v = to_f32<AT>(w[c]);
+  constexpr int EG = 4;
+  for (int e0 = warp * EG; e0 < E; e0 += nw * EG) {
+    float acc[EG][TM];
 #pragma unroll
-      for (int m = 0; m < 8; ++m)
-        if (m < nt) acc[m] = fmaf(v, sh[m * d + c], acc[m]);
+    for (int q = 0; q < EG; ++q)
+#pragma unroll
+      for (int m = 0; m < TM; ++m) acc[q][m] = 0.f;
+    if (vec) {
+#pragma unroll 2
+      for (int c = lane * 4; c < d; c += 128) {
+        float4 w[EG];
+#pragma unroll
+        for (int q = 0; q < EG; ++q) w[q] = load4(wr + (size_t)min(e0 + q, E - 1) * ldw + c);
+#pragma unroll
+        for (int m = 0; m < TM; ++m) {
+          const float4 v = load4(sh + (size_t)m * d + c);
+#pragma unroll
+          for (int q = 0; q < EG; ++q)
+            acc[q][m] = fmaf(w[q].x, v.x, fmaf(w[q].y, v.y, fmaf(w[q].z, v.z, fmaf(w[q].w, v.w, acc[q][m]))));
+        }
+      }
+    } else {
+      for (int c = lane; c < d; c += 32)
+#pragma unroll
+        for (int q = 0; q < EG; ++q) {
+          const float w = to_f32<AT>(wr[(size_t)min(e0 + q, E - 1) * ldw + c]);
+#pragma unroll
+          for (int m = 0; m < TM; ++m) acc[q][m] = fmaf(w, sh[(size_t)m * d4 + c], acc[q][m]);
+        }
     }
 #pragma unroll
-    for (int m = 0; m < 8; ++m)
-      if (m < nt) {
-        const float s = warp_sum(acc[m]);
-        if (lane == 0) sl[m * E + e] = s;
+    for (int q = 0; q < EG; ++q)
+#pragma unroll
+      for (int m = 0; m < TM; ++m) {
+        const float s = warp_sum(acc[q][m]);
+        if (lane == 0 && e0 + q < E) sl[m * E + e0 + q] = s;
       }
   }
   __syncthreads();
@@ -257,17 +288,22 @@ SMC_API int smc_route(const float* h, int d, const void* wr, int ldw, int E, int
   using namespace smc;
   if (T <= 0) return 0;
   if (E < 1 || top < 1 || groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups)) return -95;
-  int TM = T > 296 ? 8 : 1;
-  auto bytes = [&](int tm) { return (size_t)tm * (d + E + groups + top) * sizeof(float); };
-  while (TM > 1 && bytes(TM) > 100 * 1024) TM >>= 1;
+  auto bytes = [&](int tm) { return (size_t)tm * (((d + 3) & ~3) + E + groups + top) * sizeof(float); };
+  const bool wide = T > 296 && bytes(8) <= 200 * 1024;      // eight tokens per CTA once there are enough of them
+  const int TM = wide ? 8 : 1;
   if (bytes(TM) > 200 * 1024) return -96;
-  const void* k = f32 ? (const void*)route_kernel<float> : (const void*)route_kernel<__nv_bfloat16>;
-  CUDA_CHECK_RET(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
   const dim3 grid((T + TM - 1) / TM);
-  if (f32) return launch_pdl(route_kernel<float>, grid, dim3(256), bytes(TM), st, pdl, h, d, (const float*)wr, ldw, E, top, groups,
-                             keep, T, TM, idx, wgt, pdl);
-  return launch_pdl(route_kernel<__nv_bfloat16>, grid, dim3(256), bytes(TM), st, pdl, h, d, (const __nv_bfloat16*)wr, ldw, E, top,
-                    groups, keep, T, TM, idx, wgt, pdl);
+#define SMC_ROUTE(AT, N)                                                                                                    \
+  {                                                                                                                         \
+    CUDA_CHECK_RET(cudaFuncSetAttribute(route_kernel<AT, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));     \
+    return launch_pdl(route_kernel<AT, N>, grid, dim3(256), bytes(TM), st, pdl, h, d, (const AT*)wr, ldw, E, top, groups,   \
+                      keep, T, idx, wgt, pdl);                                                                              \
+  }
+  if (f32 && wide) SMC_ROUTE(float, 8)
+  if (f32) SMC_ROUTE(float, 1)
+  if (wide) SMC_ROUTE(__nv_bfloat16, 8)
+  SMC_ROUTE(__nv_bfloat16, 1)
+#undef SMC_ROUTE
 }
 
 // idx [n] expert of every (token, k) pair -> slot [n], src [n] (token of every slot), tiles [max_tiles].

@@ -653,7 +653,7 @@ def layered_lib():
         L.smc_gather_rows.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, vp]
         L.smc_latent_new.argtypes = [vp, i, i, i, vp, f, vp, i, vp, i, i, vp, i, vp, i, i, vp]
         L.smc_latent_attn.argtypes = [vp, i, vp]
-        L.smc_latent_attn_tc.argtypes = [vp, i, i, i, vp, vp, vp]
+        L.smc_latent_attn_tc.argtypes = [vp, i, i, i, vp]
         L.smc_latent_attn_tc.restype = C.c_int
         L.smc_latent_tc_splits.argtypes = [i, i, i]
         L.smc_latent_tc_splits.restype = C.c_int
@@ -755,10 +755,6 @@ def latent_tc_splits(tiles: int, width: int, keys: int) -> int:
     return layered_lib().smc_latent_tc_splits(tiles, width, int(keys))
 
 
-def latent_attention_tc(a: LatentArgs, *, tokens: int, blk_rows: int, splits: int = 1, part: Optional[torch.Tensor] = None,
-                        part_ml: Optional[torch.Tensor] = None) -> None:
-    """bf16 latent attention on the tensor cores; ``splits`` > 1 parks partial rows in part / part_ml and merges them."""
-    _check(layered_lib().smc_latent_attn_tc(C.byref(a), tokens, blk_rows, splits, _p(part), _p(part_ml), _stream()),
-           "smc_latent_attn_tc")
-    global launch_count
-    launch_count += splits > 1
+def latent_attention_tc(a: LatentArgs, *, tokens: int, blk_rows: int, splits: int = 1) -> None:
+    """bf16 latent attention on the tensor cores; ``splits`` key ranges run as a thread-block cluster and merge on chip."""
+    _check(layered_lib().smc_latent_attn_tc(C.byref(a), tokens, blk_rows, splits, _stream()), "smc_latent_attn_tc")

@@ -80,8 +80,6 @@ class NativePasizen:
                                  [T * 2 * round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared], default=0), torch.float32)
         # the samplers read rows of float4
         self.logits = torch.empty(max_logit_rows, round_up(self.V, 4), dtype=torch.float32, device=self.dev)
-        # attention split over key ranges: parked rows, allocated when a plan first needs them
-        self._parts = self._parts_ml = torch.empty(0, dtype=torch.float32, device=self.dev)
         self.attn_tc = not self.f32 and _env_flag("SMC_LATENT_TC", True)
         self._steps = self._build_steps()
 
@@ -195,11 +193,7 @@ class NativePasizen:
         if self.attn_tc and Rp <= K.latent_tc_max_width():
             tokens = min(longest, self.BLOCK)
             ks = self._ks(work.n_blk, tokens, H, Rp)
-            if ks > 1 and self._parts.numel() < ks * T * H * Rp:
-                self._parts = torch.empty(ks * T * H * Rp, dtype=torch.float32, device=self.dev)
-            if ks > 1 and self._parts_ml.numel() < ks * T * H * 2:
-                self._parts_ml = torch.empty(ks * T * H * 2, dtype=torch.float32, device=self.dev)
-            K.latent_attention_tc(a, tokens=T, blk_rows=tokens * H, splits=ks, part=self._parts, part_ml=self._parts_ml)
+            K.latent_attention_tc(a, tokens=T, blk_rows=tokens * H, splits=ks)
         else:
             K.latent_attention(a, self.f32)
         self._per_head(L.wuv, ctx, vo, T, H, Rp, m.vdim)

@@ -326,11 +326,10 @@ def test_latent_attention_on_tensor_cores(seqs, H, R, pages, splits):
     bt = _page_order(bt, seqs, pages)
     T = q.shape[0]
     out, st = torch.zeros_like(q), _status()
-    part, ml = torch.full((splits * T * H * Rp,), float("nan"), device=DEV), torch.full((splits * T * H * 2,), float("nan"), device=DEV)
     work, keep = _work(K, seqs)
     a = K.LatentArgs(q=K.ptr(q), pool=K.ptr(pool), out=K.ptr(out), block_table=K.ptr(bt), bt_stride=bt.stride(0), bt_rows=bt.shape[0],
                      n_pages=pool.shape[0] - 1, H=H, ldc=Rp, scale=R ** -0.5, r=work, status=K.ptr(st))
-    K.latent_attention_tc(a, tokens=T, blk_rows=min(64, max(x[2] for x in seqs)) * H, splits=splits, part=part, part_ml=ml)
+    K.latent_attention_tc(a, tokens=T, blk_rows=min(64, max(x[2] for x in seqs)) * H, splits=splits)
     assert int(st) == 0
     _close(out, _latent_ref(bt, pool, q, H, Rp, seqs, R ** -0.5), 1.5e-2)
 
