@@ -4,13 +4,15 @@
 // of tokens - row = token * heads + head, up to 128 per CTA - form one M = 128 operand, and a tile of 64 cached rows serves
 // as keys and as values from the same shared-memory bytes:
 //     S = Q C^T        UMMA 128 x 64 x R, C taken K-major
-//     softmax          one query row per thread, causal limit per row, P as bf16 into a SWIZZLE_128B tile
+//     softmax          two threads per query row (both take the row's maximum, each exponentiates half of the tile's
+//                      columns), causal limit per row, P as bf16 into a SWIZZLE_128B tile
 //     O += P C         UMMA 128 x R x 64 accumulating in tensor memory, C taken MN-major
 // Two score buffers (64 columns each) and up to 384 output columns live in tensor memory; wider latents split their output
 // columns over two CTAs that both compute the scores.  The exponent reference of a row only moves when its maximum grew by
 // more than 2^8; only then is its part of O rescaled in tensor memory.
 // Cached rows live one page per token: a tile of 64 consecutive pages is fetched with one TMA box per panel, a scattered one
-// is gathered by four loader warps with 16-byte cp.async copies into the same swizzled layout.  Key ranges may be split over
+// is gathered by four loader warps with 16-byte cp.async copies into the same swizzled layout (TMA gathers of four rows each
+// measured 1.5 times slower); the copies arrive on the tile's mbarrier by themselves, so loaders never wait for one to land.  Key ranges may be split over
 // the CTAs of a thread-block cluster (few sequences, long contexts): every split parks its unnormalised rows in its own shared
 // memory and the CTAs merge them through distributed shared memory, each a share of the rows.
 // The work list (ragged.cuh) mixes prompts, portions of prompts and single tokens; query rows never mix sequences.
@@ -22,11 +24,11 @@ namespace smc {
 
 constexpr int LT_BK = 64;                       // cached rows per tile
 constexpr int LT_LOADERS = 4;
-constexpr int LT_THREADS = (5 + LT_LOADERS) * 32;   // warps 0..3 softmax, 4 MMA, 5..8 loaders
+constexpr int LT_THREADS = (9 + LT_LOADERS) * 32;   // warps 0..7 softmax (4..7: the upper half of the columns), 8 MMA, 9.. loaders
 constexpr int LT_PANEL_Q = 128 * 128;           // bytes of one [128 rows][64 values] panel
 constexpr int LT_PANEL_C = LT_BK * 128;
 constexpr int LT_O_COL = 2 * LT_BK;             // first output column in tensor memory
-constexpr int LT_MAX_STAGES = 8;
+constexpr int LT_MAX_STAGES = 6;
 constexpr int LT_MAX_SPLITS = 8;                // CTAs of a cluster
 
 // NPAN: panels of 64 values per cached row.  Ring depth within 227 KB next to the Q tile and two P tiles.
@@ -36,10 +38,11 @@ template <int NPAN> struct LtCfg {
   static constexpr int FIXED = NPAN * LT_PANEL_Q + 2 * LT_PANEL_Q;
   static constexpr int FIT = (231000 - 1024 - FIXED) / (NPAN * LT_PANEL_C);
   static constexpr int STAGES = FIT > LT_MAX_STAGES ? LT_MAX_STAGES : FIT;
-  static constexpr int LAG = STAGES > 2 ? STAGES - 2 : 0;            // gathered tiles in flight behind the newest
   static constexpr int SMEM = FIXED + STAGES * NPAN * LT_PANEL_C + 1024;
   static constexpr int OLD = OPAN * 64 + 1;                          // row pitch of the parked rows (floats)
-  static_assert(STAGES >= 1 && 128 * OLD * 4 + 1024 <= SMEM, "a tile and the parked rows must fit");
+  static constexpr int STATS = FIXED + STAGES * NPAN * LT_PANEL_C - 2048;   // row statistics, at the end of the P buffers
+  static constexpr int TMEM_COLS = OPAN <= 2 ? 256 : 512;
+  static_assert(STAGES >= 1 && 128 * OLD * 4 <= STATS, "a tile and the parked rows must fit");
 };
 
 struct LatentTcParams {
@@ -57,7 +60,6 @@ struct LtShared {
   uint64_t q_full, c_full[LT_MAX_STAGES], c_empty[LT_MAX_STAGES], s_full[2], s_empty[2], p_full[2], p_empty[2];
   uint32_t tmem_slot;
   volatile int abort;
-  float m[128], l[128];          // key splits: reference exponent (log2 units) and sum of every row
 };
 
 __device__ __forceinline__ bool lt_wait(LtShared& S, int* status, uint64_t* bar, uint32_t parity) {
@@ -90,25 +92,27 @@ template <int NPAN>
 __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTcParams p, const __grid_constant__ CUtensorMap tmC,
                                                                   const __grid_constant__ CUtensorMap tmQ) {
   using C = LtCfg<NPAN>;
-  constexpr int STAGES = C::STAGES, LAG = C::LAG, CPR = NPAN * 8, KPW = LT_BK / LT_LOADERS, C_BYTES = NPAN * LT_PANEL_C;
+  constexpr int STAGES = C::STAGES, CPR = NPAN * 8, KPW = LT_BK / LT_LOADERS, C_BYTES = NPAN * LT_PANEL_C;
   extern __shared__ uint8_t lt_raw[];
   __shared__ LtShared S;
   const uint32_t raw = smem_u32(lt_raw);
   uint8_t* q_s = lt_raw + (((raw + 1023u) & ~1023u) - raw);
   uint8_t* c_s = q_s + NPAN * LT_PANEL_Q;
   uint8_t* p_s = c_s + STAGES * C_BYTES;
+  float* st_m = reinterpret_cast<float*>(q_s + C::STATS);   // [128] reference exponents (log2 units), [128] sums of a key split,
+  float* st_l = st_m + 128;                                 // [2][128] sums of the two halves of the columns; P is idle by then
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   if (threadIdx.x == 0) {
     mbar_init(&S.q_full, 1);
     for (int s = 0; s < STAGES; ++s) {
-      mbar_init(&S.c_full[s], LT_LOADERS);
+      mbar_init(&S.c_full[s], LT_LOADERS * 32);
       mbar_init(&S.c_empty[s], 1);
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&S.s_full[i], 1);
-      mbar_init(&S.s_empty[i], 4);
-      mbar_init(&S.p_full[i], 4);
+      mbar_init(&S.s_empty[i], 8);
+      mbar_init(&S.p_full[i], 8);
       mbar_init(&S.p_empty[i], 1);
     }
     S.abort = 0;
@@ -116,8 +120,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
     tma_prefetch_desc(&tmC);
     tma_prefetch_desc(&tmQ);
   }
-  if (warp == 4) {
-    tmem_alloc(&S.tmem_slot, 512);
+  if (warp == 8) {
+    tmem_alloc(&S.tmem_slot, C::TMEM_COLS);
     tmem_relinquish();
   }
   if (p.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
@@ -147,9 +151,9 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
   const uint32_t tmem_base = S.tmem_slot;
   const uint32_t tO = tmem_base + LT_O_COL;
 
-  if (warp >= 5) {
+  if (warp >= 9) {
     // ================================================================= loaders
-    const int lw = warp - 5;
+    const int lw = warp - 9;
     const uint64_t pol = l2_policy_evict_last();      // other row tiles and splits read the same rows
     if (lw == 0 && lane == 0 && n_tiles > 0) {
       mbar_expect_tx(&S.q_full, NPAN * LT_PANEL_Q);
@@ -167,9 +171,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       return page;
     };
     constexpr int PD = 4;                             // page ids are fetched this many tiles ahead
-    int issued = 0;
-    uint32_t gathered = 0;                            // bit (j & 31): tile j went through cp.async (arrival still owed)
-    int pg[PD][2];
+    int issued = 0, pg[PD][2];
 #pragma unroll
     for (int u = 0; u < PD; ++u) {
       pg[u][0] = page_of(u, 0);
@@ -194,51 +196,37 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
         const bool run = key_end <= ke && base >= 1 && (asc || desc);
         uint8_t* c_ptr = c_s + (size_t)st * C_BYTES;
         if (run) {
-          if (lane == 0) {
-            if (lw == 0) {
-              mbar_expect_tx(&S.c_full[st], C_BYTES);
-              for (int pan = 0; pan < NPAN; ++pan)
-                tma_load_2d(c_ptr + pan * LT_PANEL_C, &tmC, &S.c_full[st], pan * 64, asc ? base : base - (LT_BK - 1), pol);
-            } else {
-              mbar_arrive(&S.c_full[st]);
-            }
+          if (lw == 0 && lane == 0) {
+            mbar_expect_tx(&S.c_full[st], C_BYTES);
+            for (int pan = 0; pan < NPAN; ++pan)
+              tma_load_2d(c_ptr + pan * LT_PANEL_C, &tmC, &S.c_full[st], pan * 64, asc ? base : base - (LT_BK - 1), pol);
+          } else {
+            mbar_arrive(&S.c_full[st]);
           }
-          gathered &= ~(1u << (j & 31));
         } else {
           const uint32_t c_t = smem_u32(c_ptr);
           const int mine = lw < 2 ? pa : pb;          // this warp's 16 keys sit in lanes (lw & 1) * 16 ..
-#pragma unroll 4
-          for (int idx = lane; idx < KPW * CPR; idx += 32) {
-            const int kl = idx / CPR, c = idx % CPR, key = lw * KPW + kl;
+#pragma unroll
+          for (int i = 0; i < KPW * CPR / 32; ++i) {
+            const int idx = i * 32 + lane, kl = idx / CPR, c = idx % CPR, key = lw * KPW + kl;
             const int pgi = __shfl_sync(0xffffffffu, mine, (lw & 1) * 16 + kl);
             const uint32_t dst = c_t + (uint32_t)((c >> 3) * LT_PANEL_C + key * 128 + (((c & 7) ^ (key & 7)) << 4));
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(p.pool + (size_t)pgi * p.ldc + c * 8) : "memory");
           }
-          gathered |= 1u << (j & 31);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");       // one group per tile (empty for a TMA tile)
-        if (j >= LAG && ((gathered >> ((j - LAG) & 31)) & 1u)) {   // gathered tile j - LAG has landed: hand it over
-          asm volatile("cp.async.wait_group %0;" ::"n"(LAG) : "memory");
-          fence_proxy_async();
-          __syncwarp();
-          if (lane == 0) mbar_arrive(&S.c_full[(j - LAG) % STAGES]);
+          // this thread's arrival follows its copies
+          asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(smem_u32(&S.c_full[st])) : "memory");
         }
         ++issued;
       }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    fence_proxy_async();
-    __syncwarp();
-    if (lane == 0)
-      for (int t = max(0, issued - LAG); t < issued; ++t)
-        if ((gathered >> (t & 31)) & 1u) mbar_arrive(&S.c_full[t % STAGES]);
+    asm volatile("cp.async.wait_all;" ::: "memory");
     // TMA copies still in flight after an abort must land before the CTA ends
+    __syncwarp();
     if (S.abort && lw == 0 && lane == 0) {
       if (n_tiles > 0) (void)mbar_wait(&S.q_full, 0);
-      for (int t = max(0, issued - STAGES); t < issued; ++t)
-        if (!((gathered >> (t & 31)) & 1u)) (void)mbar_wait(&S.c_full[t % STAGES], (uint32_t)(t / STAGES) & 1u);
+      for (int t = max(0, issued - STAGES); t < issued; ++t) (void)mbar_wait(&S.c_full[t % STAGES], (uint32_t)(t / STAGES) & 1u);
     }
-  } else if (warp == 4) {
+  } else if (warp == 8) {
     // ================================================================= MMA issuer (one thread)
     if (elect_one()) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(128, LT_BK);
@@ -247,6 +235,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
         const int st = j % STAGES;
         if (!lt_wait(S, p.status, &S.c_full[st], (uint32_t)(j / STAGES) & 1u)) return false;
         if (j >= 2 && !lt_wait(S, p.status, &S.s_empty[j & 1], (uint32_t)((j >> 1) - 1) & 1u)) return false;
+        fence_proxy_async();                          // gathered rows were written through the generic proxy
         tc_fence_after();
         const uint32_t c_addr = c_addr0 + (uint32_t)st * C_BYTES;
 #pragma unroll
@@ -280,49 +269,54 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
     }
     __syncwarp();
   } else {
-    // ================================================================= softmax (one query row per thread)
-    const int r = warp * 32 + lane;
-    const uint32_t lane_off = ((uint32_t)(warp * 32)) << 16;
+    // ================================================================= softmax (two threads per query row)
+    constexpr int HB = LT_BK / 2;                                        // columns this thread exponentiates
+    const int half = warp >> 2, r = (warp & 3) * 32 + lane;
+    const uint32_t lane_off = ((uint32_t)((warp & 3) * 32)) << 16;
     const bool real = r < n_rows;
     const int lim = real ? pos0 + (row0 + r) / p.H + 1 : ke;             // keys [0, lim) are visible (spare rows: unmasked)
     float m_ref = -INFINITY, l = 0.f;                                    // exponent reference (log2 domain), running sum
     bool alive = true;
-    const bool idle = warp * 32 >= n_rows;                               // no real row in this warp: keep the protocol only
+    const bool idle = (warp & 3) * 32 >= n_rows;                         // no real row in this warp: keep the protocol only
     for (int j = 0; j < n_tiles; ++j) {
       const int nv = min(lim, ke) - kb - j * LT_BK;                      // visible keys of this tile (may be <= 0)
       if (!__all_sync(0xffffffffu, lt_wait(S, p.status, &S.s_full[j & 1], (uint32_t)(j >> 1) & 1u))) { alive = false; break; }
       tc_fence_after();
-      uint32_t x[LT_BK];
+      uint32_t x[HB];
+      float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      const bool full = __all_sync(0xffffffffu, nv >= LT_BK);
       if (!idle) {
         const uint32_t ts = tmem_base + (uint32_t)(j & 1) * LT_BK + lane_off;
+        uint32_t y[HB];                               // the other half: only its maximum is needed here
 #pragma unroll
-        for (int c0 = 0; c0 < LT_BK; c0 += 16) tmem_ld_32x32b_x16(ts + c0, *reinterpret_cast<uint32_t(*)[16]>(&x[c0]));
+        for (int c0 = 0; c0 < HB; c0 += 16) {
+          tmem_ld_32x32b_x16(ts + half * HB + c0, *reinterpret_cast<uint32_t(*)[16]>(&x[c0]));
+          tmem_ld_32x32b_x16(ts + (half ^ 1) * HB + c0, *reinterpret_cast<uint32_t(*)[16]>(&y[c0]));
+        }
         tmem_ld_wait();
+        if (full) {
+#pragma unroll
+          for (int i = 0; i < HB; ++i) m4[i & 3] = fmaxf(m4[i & 3], fmaxf(__uint_as_float(x[i]), __uint_as_float(y[i])));
+        } else {
+          const int nx = nv - half * HB, ny = nv - (half ^ 1) * HB;
+#pragma unroll
+          for (int i = 0; i < HB; ++i) {
+            if (i < nx) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(x[i]));
+            if (i < ny) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(y[i]));
+          }
+        }
       }
       tc_fence_before();                              // the scores are in registers: the buffer can take tile j + 2
       __syncwarp();
       if (lane == 0) mbar_arrive(&S.s_empty[j & 1]);
-      float mx = -INFINITY;
-      const bool full = __all_sync(0xffffffffu, nv >= LT_BK);
-      bool grow = false;
-      if (!idle) {
-        if (full) {
-#pragma unroll
-          for (int i = 0; i < LT_BK; ++i) mx = fmaxf(mx, __uint_as_float(x[i]));
-        } else {
-#pragma unroll
-          for (int i = 0; i < LT_BK; ++i)
-            if (i < nv) mx = fmaxf(mx, __uint_as_float(x[i]));
-        }
-        mx *= p.scale_log2;
-        grow = mx > m_ref + 8.f;                      // also true on the row's first visible key (m_ref = -inf)
-      }
+      const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * p.scale_log2;
+      const bool grow = mx > m_ref + 8.f;             // also true on the row's first visible key (m_ref = -inf)
       if (j >= 1 && __any_sync(0xffffffffu, grow)) {
         // PV of tile j - 1 must have completed before O is rescaled in tensor memory
         if (!__all_sync(0xffffffffu, lt_wait(S, p.status, &S.p_empty[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1u))) { alive = false; break; }
         tc_fence_after();
         const float alpha = grow ? exp2f(m_ref - mx) : 1.f;
-        for (int c0 = 0; c0 < n_opan * 64; c0 += 16) {
+        for (int c0 = half * 32; c0 < n_opan * 64; c0 += (c0 & 16) ? 48 : 16) {     // this half's 32 columns of every panel
           uint32_t o[16];
           tmem_ld_32x32b_x16(tO + lane_off + c0, o);
           tmem_ld_wait();
@@ -340,31 +334,32 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       if (idle) {
         if (j < 2) {                                  // rows without a query stay zero in both buffers
 #pragma unroll
-          for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(prow + (c << 4)) = make_uint4(0u, 0u, 0u, 0u);
+          for (int c = 0; c < 4; ++c) *reinterpret_cast<uint4*>(prow + ((half * 4 + c) << 4)) = make_uint4(0u, 0u, 0u, 0u);
         }
       } else {
-        float s0 = 0.f, s1 = 0.f;
+        float s4[4] = {0.f, 0.f, 0.f, 0.f};
         const float ref = m_ref == -INFINITY ? 0.f : m_ref;
+        const int nx = nv - half * HB;
 #pragma unroll
-        for (int c0 = 0; c0 < LT_BK; c0 += 16) {
+        for (int c0 = 0; c0 < HB; c0 += 16) {
           uint32_t pk[8];
 #pragma unroll
           for (int i = 0; i < 16; i += 2) {
             float p0 = lt_ex2(fmaf(__uint_as_float(x[c0 + i]), p.scale_log2, -ref));
             float p1 = lt_ex2(fmaf(__uint_as_float(x[c0 + i + 1]), p.scale_log2, -ref));
             if (!full) {
-              p0 = c0 + i < nv ? p0 : 0.f;
-              p1 = c0 + i + 1 < nv ? p1 : 0.f;
+              p0 = c0 + i < nx ? p0 : 0.f;
+              p1 = c0 + i + 1 < nx ? p1 : 0.f;
             }
-            s0 += p0;
-            s1 += p1;
+            s4[i & 2] += p0;
+            s4[(i & 2) + 1] += p1;
             pk[i >> 1] = lt_pack(p0, p1);
           }
-          const int cc = c0 >> 3;                     // two 16-byte chunks of this row's 128 bytes
+          const int cc = (half * HB + c0) >> 3;       // two 16-byte chunks of this row's 128 bytes
           *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
           *reinterpret_cast<uint4*>(prow + (((cc + 1) ^ (r & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
         }
-        l += s0 + s1;
+        l += (s4[0] + s4[1]) + (s4[2] + s4[3]);
       }
       tc_fence_before();
       fence_proxy_async();                            // P must be visible to the tensor core
@@ -376,15 +371,18 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       alive = __all_sync(0xffffffffu, lt_wait(S, p.status, &S.p_empty[(n_tiles - 1) & 1], (uint32_t)((n_tiles - 1) >> 1) & 1u));
     tc_fence_after();
     const bool write = real && alive && !S.abort;
-    if (p.KS > 1) {
-      S.m[r] = write ? m_ref : -INFINITY;
-      S.l[r] = write ? l : 0.f;                       // 0: this split holds nothing for the row
+    st_l[128 + half * 128 + r] = l;
+    asm volatile("bar.sync 1, 256;" ::: "memory");    // the eight softmax warps
+    l = st_l[128 + r] + st_l[256 + r];
+    if (p.KS > 1 && half == 0) {
+      st_m[r] = write ? m_ref : -INFINITY;
+      st_l[r] = write ? l : 0.f;                       // 0: this split holds nothing for the row
     }
     if (n_tiles > 0 && alive && !idle) {
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       float* po = reinterpret_cast<float*>(q_s) + r * C::OLD;       // operands and tiles are no longer needed
       __nv_bfloat16* oo = p.out + ((size_t)g_row0 + r) * p.ldc + vpan * 64;
-      for (int c0 = 0; c0 < n_opan * 64; c0 += 16) {
+      for (int c0 = half * 32; c0 < n_opan * 64; c0 += (c0 & 16) ? 48 : 16) {
         uint32_t o[16];
         tmem_ld_32x32b_x16(tO + lane_off + c0, o);
         tmem_ld_wait();
@@ -403,15 +401,15 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 4) tmem_dealloc(tmem_base, 512);
+  if (warp == 8) tmem_dealloc(tmem_base, C::TMEM_COLS);
   if (p.KS > 1) {
     // merge: CTA `ks` of the cluster takes rows ks, ks + KS, ..; a warp per row
     cluster_sync();
     for (int r = ks + warp * p.KS; r < n_rows; r += p.KS * (LT_THREADS / 32)) {
       float ms = -INFINITY, ls = 0.f;
       if (lane < p.KS) {
-        ls = ld_dsmem_f32(smem_u32(&S.l[r]), (uint32_t)lane);
-        if (ls > 0.f) ms = ld_dsmem_f32(smem_u32(&S.m[r]), (uint32_t)lane);
+        ls = ld_dsmem_f32(smem_u32(st_l + r), (uint32_t)lane);
+        if (ls > 0.f) ms = ld_dsmem_f32(smem_u32(st_m + r), (uint32_t)lane);
       }
       const float mm = warp_max(ms);
       float f = ls > 0.f ? exp2f(ms - mm) : 0.f;
