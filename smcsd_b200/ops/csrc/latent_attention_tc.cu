@@ -163,11 +163,10 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
     // every loader warp reads all 64 page ids of a tile (lane l: keys l and l + 32), so all take the same path
     auto page_of = [&](int tile, int half) {
       const int key = kb + tile * LT_BK + half * 32 + lane;
-      int page = 0;
-      if (tile < n_tiles && key < ke) {
-        page = bt[key];
-        if (page < 0 || page > p.n_pages) { atomicOr(p.status, SMC_ERR_BOUNDS); page = 0; }
-      }
+      return tile < n_tiles && key < ke ? bt[key] : 0;
+    };
+    auto checked = [&](int page) {                    // at the point of use: a check at the load would wait for it
+      if (page < 0 || page > p.n_pages) { atomicOr(p.status, SMC_ERR_BOUNDS); page = 0; }
       return page;
     };
     constexpr int PD = 4;                             // page ids are fetched this many tiles ahead
@@ -186,7 +185,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
         const int st = j % STAGES, use = j / STAGES;
         const bool ok = use < 1 || lt_wait(S, p.status, &S.c_empty[st], (uint32_t)(use - 1) & 1u);
         if (!__all_sync(0xffffffffu, ok)) { go = false; break; }
-        const int pa = pg[u][0], pb = pg[u][1];
+        const int pa = checked(pg[u][0]), pb = checked(pg[u][1]);
         pg[u][0] = page_of(j + PD, 0);
         pg[u][1] = page_of(j + PD, 1);
         const int base = __shfl_sync(0xffffffffu, pa, 0), key_end = kb + (j + 1) * LT_BK;
@@ -403,32 +402,37 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
   __syncthreads();
   if (warp == 8) tmem_dealloc(tmem_base, C::TMEM_COLS);
   if (p.KS > 1) {
-    // merge: CTA `ks` of the cluster takes rows ks, ks + KS, ..; a warp per row
+    // merge: CTA `ks` of the cluster takes rows ks, ks + KS, ..; a warp per (row, panel)
     cluster_sync();
-    for (int r = ks + warp * p.KS; r < n_rows; r += p.KS * (LT_THREADS / 32)) {
-      float ms = -INFINITY, ls = 0.f;
+    const int mine = n_rows > ks ? (n_rows - ks + p.KS - 1) / p.KS : 0;
+    for (int t = warp; t < mine * n_opan; t += LT_THREADS / 32) {
+      const int r = ks + (t / n_opan) * p.KS, c = (t % n_opan) * 64 + lane * 2;
+      const uint32_t base = smem_u32(reinterpret_cast<float*>(q_s) + r * C::OLD + c);
+      float v0[LT_MAX_SPLITS], v1[LT_MAX_SPLITS], ms = -INFINITY, ls = 0.f;
+#pragma unroll
+      for (int q = 0; q < LT_MAX_SPLITS; ++q)
+        if (q < p.KS) {
+          const uint32_t rem = dsmem_map(base, (uint32_t)q);
+          v0[q] = ld_dsmem_f32_at(rem);
+          v1[q] = ld_dsmem_f32_at(rem + 4u);
+        }
       if (lane < p.KS) {
         ls = ld_dsmem_f32(smem_u32(st_l + r), (uint32_t)lane);
-        if (ls > 0.f) ms = ld_dsmem_f32(smem_u32(st_m + r), (uint32_t)lane);
+        ms = ld_dsmem_f32(smem_u32(st_m + r), (uint32_t)lane);
       }
-      const float mm = warp_max(ms);
+      const float mm = warp_max(ls > 0.f ? ms : -INFINITY);
       float f = ls > 0.f ? exp2f(ms - mm) : 0.f;
       f *= 1.0f / warp_sum(ls * f);
-      const uint32_t base = smem_u32(reinterpret_cast<float*>(q_s) + r * C::OLD);
-      __nv_bfloat16* oo = p.out + ((size_t)g_row0 + r) * p.ldc + vpan * 64;
-      for (int c = lane * 2; c < n_opan * 64; c += 64) {
-        float a0 = 0.f, a1 = 0.f;
+      float a0 = 0.f, a1 = 0.f;
 #pragma unroll
-        for (int q = 0; q < LT_MAX_SPLITS; ++q) {
-          const float fq = __shfl_sync(0xffffffffu, f, q);
-          if (q < p.KS && fq > 0.f) {
-            const uint32_t rem = dsmem_map(base + (uint32_t)c * 4u, (uint32_t)q);
-            a0 = fmaf(fq, ld_dsmem_f32_at(rem), a0);
-            a1 = fmaf(fq, ld_dsmem_f32_at(rem + 4u), a1);
-          }
+      for (int q = 0; q < LT_MAX_SPLITS; ++q) {
+        const float fq = __shfl_sync(0xffffffffu, f, q);
+        if (q < p.KS && fq > 0.f) {                   // a split without keys for the row left nothing behind
+          a0 = fmaf(fq, v0[q], a0);
+          a1 = fmaf(fq, v1[q], a1);
         }
-        *reinterpret_cast<uint32_t*>(oo + c) = lt_pack(a0, a1);
       }
+      *reinterpret_cast<uint32_t*>(p.out + ((size_t)g_row0 + r) * p.ldc + vpan * 64 + c) = lt_pack(a0, a1);
     }
     cluster_sync();                                   // nobody leaves while its rows may still be read
   }
