@@ -156,6 +156,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
     const int lw = warp - 9;
     const uint64_t pol = l2_policy_evict_last();      // other row tiles and splits read the same rows
     if (lw == 0 && lane == 0 && n_tiles > 0) {
+      // whole boxes of 128 rows: what the rows behind the queries contain only reaches their own outputs
       mbar_expect_tx(&S.q_full, NPAN * LT_PANEL_Q);
       for (int pan = 0; pan < NPAN; ++pan) tma_load_2d(q_s + pan * LT_PANEL_Q, &tmQ, &S.q_full, pan * 64, g_row0, pol);
     }
@@ -336,27 +337,27 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
           for (int c = 0; c < 4; ++c) *reinterpret_cast<uint4*>(prow + ((half * 4 + c) << 4)) = make_uint4(0u, 0u, 0u, 0u);
         }
       } else {
-        float s4[4] = {0.f, 0.f, 0.f, 0.f};
         const float ref = m_ref == -INFINITY ? 0.f : m_ref;
-        const int nx = nv - half * HB;
+        if (!full) {                                  // keys the row does not see: exp2 of -inf
+          const int nx = nv - half * HB;
 #pragma unroll
-        for (int c0 = 0; c0 < HB; c0 += 16) {
-          uint32_t pk[8];
+          for (int i = 0; i < HB; ++i) x[i] = i < nx ? x[i] : 0xff800000u;
+        }
+        float s4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-          for (int i = 0; i < 16; i += 2) {
-            float p0 = lt_ex2(fmaf(__uint_as_float(x[c0 + i]), p.scale_log2, -ref));
-            float p1 = lt_ex2(fmaf(__uint_as_float(x[c0 + i + 1]), p.scale_log2, -ref));
-            if (!full) {
-              p0 = c0 + i < nx ? p0 : 0.f;
-              p1 = c0 + i + 1 < nx ? p1 : 0.f;
-            }
-            s4[i & 2] += p0;
-            s4[(i & 2) + 1] += p1;
-            pk[i >> 1] = lt_pack(p0, p1);
-          }
-          const int cc = (half * HB + c0) >> 3;       // two 16-byte chunks of this row's 128 bytes
-          *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
-          *reinterpret_cast<uint4*>(prow + (((cc + 1) ^ (r & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+        for (int i = 0; i < HB; ++i) {
+          const float e = lt_ex2(fmaf(__uint_as_float(x[i]), p.scale_log2, -ref));
+          s4[i & 3] += e;
+          x[i] = __float_as_uint(e);
+        }
+#pragma unroll
+        for (int c = 0; c < HB / 8; ++c) {            // 16-byte chunks of this row's 128 bytes
+          const int cc = half * (HB / 8) + c;
+          *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) =
+              make_uint4(lt_pack(__uint_as_float(x[c * 8]), __uint_as_float(x[c * 8 + 1])),
+                         lt_pack(__uint_as_float(x[c * 8 + 2]), __uint_as_float(x[c * 8 + 3])),
+                         lt_pack(__uint_as_float(x[c * 8 + 4]), __uint_as_float(x[c * 8 + 5])),
+                         lt_pack(__uint_as_float(x[c * 8 + 6]), __uint_as_float(x[c * 8 + 7])));
         }
         l += (s4[0] + s4[1]) + (s4[2] + s4[3]);
       }
