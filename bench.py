@@ -17,6 +17,7 @@ cycle with forced cross-GPU resampling, reported under ``fused``.
     python -m torch.distributed.run --nnodes=1 --nproc-per-node 8 --master-addr 127.0.0.1 \
         --master-port 29511 bench.py --gpus 8 --steps 40 --warmup 5
     python bench.py --impl reference        # prints why the reference cannot run here
+    python bench.py --layered 2048,1024     # another workload: Pasizen beside a dense model of equal size, kernel by kernel
 """
 from __future__ import annotations
 
@@ -113,6 +114,28 @@ def _run_fused_children(rank: int, steps: int, warm: int, dry_run: bool = False,
                                                                  f"ended with code {proc.returncode} without a record")}
 
 
+def layered_arm(args) -> int:
+    """Prefill and decode of Pasizen beside the dense family at the given widths (random weights); the kernel tables go to
+    stderr, the whole record is the JSON line."""
+    import torch
+
+    from smcsd_b200.bench import layered
+    from smcsd_b200.ops import native as K
+    from smcsd_b200.utils.profiling import ClockSampler
+    torch.cuda.set_device(0)
+    sampler, l0 = ClockSampler(0).start(), K.launch_count
+    recs = [layered.run(int(w), ctx=args.layered_ctx) for w in args.layered.split(",")]
+    for r in recs:
+        print(layered.show(r), file=sys.stderr)
+    pick = {m["model"]: m for r in recs for m in r["models"]}
+    main_model = pick[f"pasizen-{args.layered.split(',')[0]}-dense"]
+    print(json.dumps({"metric": "decode tokens/s (Pasizen layers, random weights)", "value": main_model["decode_tok_s"],
+                      "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+                      "timing": "CUDA events around graph replays; the weights of all layers exceed L2", "records": recs,
+                      "clocks": sampler.stop(), "gpu_launches": K.launch_count - l0}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -138,9 +161,14 @@ def main() -> int:
                     help="run the MAIN measurement with the e4m3 KV cache (the line's dtype says so; not the headline)")
     ap.add_argument("--no-fp8", action="store_true",
                     help="skip the extra W8A8 (e4m3) measurement reported under the 'fp8' key (one GPU only)")
+    ap.add_argument("--layered", default=None, metavar="WIDTHS",
+                    help="run the layer comparison of Pasizen and the dense family at these widths instead of the headline")
+    ap.add_argument("--layered-ctx", type=int, default=1024, help="cached tokens per sequence of the layer comparison's decode step")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.layered:
+        return layered_arm(args)
 
     import torch
     import torch.distributed as dist
