@@ -102,8 +102,9 @@ struct GemmParams {
   GroupLink grp;
 };
 
+template <bool GRP>
 __device__ __forceinline__ float gated_unit(const GroupLink& a, float g, float u) {
-  if (a.act == 1) {
+  if (GRP && a.act == 1) {
     g = fminf(g, a.limit);
     u = fminf(fmaxf(u, -a.limit), a.limit);
     return g / (1.0f + __expf(-a.slope * g)) * (u + 1.0f);
@@ -125,7 +126,7 @@ struct GemmCfg {
   static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 /*align*/ + 256 /*barriers*/;
 };
 
-template <int BN, int EPI, bool LEAN, bool FP8>
+template <int BN, int EPI, bool LEAN, bool FP8, bool GRP>
 __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW,
                                                          const __grid_constant__ CUtensorMap tmX,
                                                          const GemmParams p) {
@@ -152,7 +153,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
   // Let the next kernel of the stream start its prologue (and its weight prefetch) right away;
   // it still waits for this grid to finish before it touches anything this grid writes.
   if (p.pdl) pdl_launch_dependents();
-  if (p.grp.mode != 0) {
+  if (GRP && p.grp.mode != 0) {
     const int slabs = (p.N + C::BM - 1) / C::BM;
     int g;
     if (p.grp.mode == 1) {
@@ -339,7 +340,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
             if (m < m_lim && ch * 2 < p.N) {
               const float g = __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
               const float u = sbuf[row_in_tile * LD + c0 + j] * s_rstd[c0 + j];
-              out[(size_t)m * p.ldo + ch] = __float2bfloat16(gated_unit(p.grp, g, u));
+              out[(size_t)m * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p.grp, g, u));
             }
           }
         }
@@ -495,7 +496,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
               const int c = c0 + u * (int)S;
               if (c < BN && m_base + c < m_lim && ch * 2 < p.N) {
                 const float g = prev[u], up = s_pair[u][threadIdx.x];
-                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(gated_unit(p.grp, g, up));
+                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p.grp, g, up));
               }
             }
           }
@@ -548,11 +549,11 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
 }
 
 // ---------------------------------------------------------------- host side
-template <int BN, int EPI, bool LEAN = false, bool FP8 = false>
+template <int BN, int EPI, bool LEAN = false, bool FP8 = false, bool GRP = false>
 static int launch(const CUtensorMap& tmW, const CUtensorMap& tmX, const GemmParams& p, dim3 grid, cudaStream_t st) {
   using C = GemmCfg<BN, EPI, LEAN>;
   static bool configured = false;
-  auto kern = gemm_skinny_kernel<BN, EPI, LEAN, FP8>;
+  auto kern = gemm_skinny_kernel<BN, EPI, LEAN, FP8, GRP>;
   if (!configured) {
     CUDA_CHECK_RET(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES));
     configured = true;
@@ -597,15 +598,15 @@ static int dispatch_bn_fp8(int bn, const CUtensorMap& a, const CUtensorMap& b, c
   return -10;
 }
 
-template <int EPI>
+template <int EPI, bool GRP = false>
 static int dispatch_bn(int bn, const CUtensorMap& a, const CUtensorMap& b, const GemmParams& p, dim3 g, cudaStream_t st) {
   switch (bn) {
-    case 16: return launch<16, EPI>(a, b, p, g, st);
-    case 32: return launch<32, EPI>(a, b, p, g, st);
-    case 64: return launch<64, EPI>(a, b, p, g, st);
-    case 80: return launch<80, EPI>(a, b, p, g, st);
-    case 128: return p.stages == 3 ? launch<128, EPI, true>(a, b, p, g, st) : launch<128, EPI, false>(a, b, p, g, st);
-    case 256: return launch<256, EPI>(a, b, p, g, st);
+    case 16: return launch<16, EPI, false, false, GRP>(a, b, p, g, st);
+    case 32: return launch<32, EPI, false, false, GRP>(a, b, p, g, st);
+    case 64: return launch<64, EPI, false, false, GRP>(a, b, p, g, st);
+    case 80: return launch<80, EPI, false, false, GRP>(a, b, p, g, st);
+    case 128: return p.stages == 3 ? launch<128, EPI, true, false, GRP>(a, b, p, g, st) : launch<128, EPI, false, false, GRP>(a, b, p, g, st);
+    case 256: return launch<256, EPI, false, false, GRP>(a, b, p, g, st);
   }
   return -10;
 }
@@ -787,6 +788,15 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
       case EPI_SWIGLU_SPLIT: return dispatch_bn_fp8<EPI_SWIGLU_SPLIT>(bn, tmW, tmX, p, grid, stream);
     }
     return -30;
+  }
+  if (grp != nullptr) {                       // builds with the group logic compiled in
+    switch (epi) {
+      case EPI_BF16: return dispatch_bn<EPI_BF16, true>(bn, tmW, tmX, p, grid, stream);
+      case EPI_SWIGLU_BF16: return dispatch_bn<EPI_SWIGLU_BF16, true>(bn, tmW, tmX, p, grid, stream);
+      case EPI_STORE_F32: return dispatch_bn<EPI_STORE_F32, true>(bn, tmW, tmX, p, grid, stream);
+      case EPI_SWIGLU_SPLIT: return dispatch_bn<EPI_SWIGLU_SPLIT, true>(bn, tmW, tmX, p, grid, stream);
+    }
+    return -33;
   }
   switch (epi) {
     case EPI_PARTIAL_F32: return dispatch_bn<EPI_PARTIAL_F32>(bn, tmW, tmX, p, grid, stream);
