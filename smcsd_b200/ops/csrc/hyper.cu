@@ -15,7 +15,7 @@
 
 namespace smc {
 
-constexpr int HYPER_MAX_STREAMS = 8;
+constexpr int HYPER_MAX_STREAMS = 16;
 constexpr int HYPER_MAXV = 8;          // column groups per thread
 constexpr int CONV_MAX_TAPS = 8;
 

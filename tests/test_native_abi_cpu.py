@@ -35,3 +35,14 @@ def test_split_plans_are_bounded_and_monotone():
         prev = ks
     # more sequences or heads fill the GPU by themselves: fewer splits are planned, never more
     assert K.attention_tc_splits(64, 8, 16384, 128) <= K.attention_tc_splits(1, 8, 16384, 128)
+
+
+def test_layered_structures_match_the_library():
+    """Sizes are asserted when the layered entry points are declared; the split planner stays within the cluster limit."""
+    K.layered_lib()
+    for tiles in (1, 8, 37, 200):
+        prev = 0
+        for keys in (1, 64, 500, 4096, 65536):
+            ks = K.latent_tc_splits(tiles, 256, keys)
+            assert 1 <= ks <= 8 and ks >= prev and (ks == 1 or tiles * ks <= 148)
+            prev = ks

@@ -204,7 +204,7 @@ def test_short_conv_over_portions(taps, d):
         assert int(st) == 0 and hist[0].abs().sum() == 0
 
 
-@pytest.mark.parametrize("S,d,taps", [(1, 64, 4), (3, 328, 5), (5, 250, 2), (8, 136, 1), (4, 2048, 3)])
+@pytest.mark.parametrize("S,d,taps", [(1, 64, 4), (3, 328, 5), (5, 250, 2), (8, 136, 1), (11, 68, 4), (4, 2048, 3)])
 def test_stream_step_with_folded_convolution(S, d, taps):
     """Embedding start, update, single-token convolution and the final sum."""
     K = _k()
