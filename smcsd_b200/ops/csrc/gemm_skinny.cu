@@ -848,7 +848,7 @@ SMC_API int smc_gemm_skinny_norm(const void* W, const void* X, void* out, int N,
 }
 
 namespace smc {
-__global__ void __launch_bounds__(32) lm_sample_merge_kernel(SampleArgs a, const RowPartial* __restrict__ parts,
+__global__ void __launch_bounds__(32) lm_sample_merge_kernel(SampleArgs a, const RowPartial* parts,
                                                             int n_slabs, int* tok_out, float* logp_out,
                                                             float* logz_out, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }

@@ -14,10 +14,10 @@ namespace smc {
 constexpr int S1_THREADS = 256;
 
 __global__ void __launch_bounds__(S1_THREADS)
-sample_stage1_kernel(const float* __restrict__ logits, int splits, long long split_stride, long long row_stride, int V,
-                     float inv_temp, float alpha, const int* __restrict__ tokens_in, uint64_t seed,
-                     const long long* __restrict__ cycle_counter, int call_id, float softcap,
-                     RowPartial* __restrict__ parts, int pdl) {
+sample_stage1_kernel(const float* logits, int splits, long long split_stride, long long row_stride, int V,
+                     float inv_temp, float alpha, const int* tokens_in, uint64_t seed,
+                     const long long* cycle_counter, int call_id, float softcap,
+                     RowPartial* parts, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int row = blockIdx.x, chunk = blockIdx.y, nchunks = gridDim.y;
   const int per = (((V + nchunks - 1) / nchunks) + 3) & ~3;
@@ -97,11 +97,11 @@ sample_stage1_kernel(const float* __restrict__ logits, int splits, long long spl
   }
 }
 
-__global__ void sample_stage2_kernel(const RowPartial* __restrict__ parts, int nchunks, const float* __restrict__ logits,
+__global__ void sample_stage2_kernel(const RowPartial* parts, int nchunks, const float* logits,
                                      int splits, long long split_stride, long long row_stride, float inv_temp,
-                                     float alpha, float softcap, const int* __restrict__ tokens_in,
-                                     int* __restrict__ tok_out, float* __restrict__ logp_out,
-                                     float* __restrict__ logz_out, int rows, int pdl) {
+                                     float alpha, float softcap, const int* tokens_in,
+                                     int* tok_out, float* logp_out,
+                                     float* logz_out, int rows, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int row = blockIdx.x * blockDim.x + threadIdx.x;
   if (row < rows) {
