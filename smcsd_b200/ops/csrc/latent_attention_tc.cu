@@ -344,20 +344,19 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
           for (int i = 0; i < HB; ++i) x[i] = i < nx ? x[i] : 0xff800000u;
         }
         float s4[4] = {0.f, 0.f, 0.f, 0.f};
+        uint32_t w[HB / 2];
 #pragma unroll
-        for (int i = 0; i < HB; ++i) {
-          const float e = lt_ex2(fmaf(__uint_as_float(x[i]), p.scale_log2, -ref));
-          s4[i & 3] += e;
-          x[i] = __float_as_uint(e);
+        for (int i = 0; i < HB / 2; ++i) {
+          w[i] = lt_pack(lt_ex2(fmaf(__uint_as_float(x[2 * i]), p.scale_log2, -ref)),
+                         lt_ex2(fmaf(__uint_as_float(x[2 * i + 1]), p.scale_log2, -ref)));
+          // the sum is taken over the rounded weights: they add up to one, and a lone heavy key carries no rounding error
+          s4[(2 * i) & 3] += __uint_as_float(w[i] << 16);
+          s4[(2 * i + 1) & 3] += __uint_as_float(w[i] & 0xffff0000u);
         }
 #pragma unroll
         for (int c = 0; c < HB / 8; ++c) {            // 16-byte chunks of this row's 128 bytes
           const int cc = half * (HB / 8) + c;
-          *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) =
-              make_uint4(lt_pack(__uint_as_float(x[c * 8]), __uint_as_float(x[c * 8 + 1])),
-                         lt_pack(__uint_as_float(x[c * 8 + 2]), __uint_as_float(x[c * 8 + 3])),
-                         lt_pack(__uint_as_float(x[c * 8 + 4]), __uint_as_float(x[c * 8 + 5])),
-                         lt_pack(__uint_as_float(x[c * 8 + 6]), __uint_as_float(x[c * 8 + 7])));
+          *reinterpret_cast<uint4*>(prow + ((cc ^ (r & 7)) << 4)) = make_uint4(w[c * 4], w[c * 4 + 1], w[c * 4 + 2], w[c * 4 + 3]);
         }
         l += (s4[0] + s4[1]) + (s4[2] + s4[3]);
       }
