@@ -14,7 +14,7 @@ smcsd/model_executor/smc_model_runner.py:109-239.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import List, Optional, Tuple
 
 import torch
 
@@ -132,6 +132,8 @@ class KVSpec:
     fp8: bool = False    # e4m3 cache: a page row holds Hkv * D value bytes + one fp32 scale per kv head (padded to 16)
     # latent cache: one row of this many values per layer run that serves as key and value alike (no V tensors)
     latent_widths: Optional[List[int]] = None
+    # layers of unequal heads: (K, V) values of a page row per layer
+    row_widths: Optional[List[Tuple[int, int]]] = None
 
     @property
     def row_width(self) -> int:
@@ -148,6 +150,8 @@ class KVSpec:
     def cell_bytes(self) -> int:
         if self.latent_widths is not None:
             return sum(self.latent_widths) * torch.empty((), dtype=self.dtype).element_size()
+        if self.row_widths is not None:
+            return sum(k + v for k, v in self.row_widths) * torch.empty((), dtype=self.dtype).element_size()
         return 2 * self.n_layers * self.row_width * torch.empty((), dtype=self.store_dtype).element_size()
 
 
@@ -176,7 +180,8 @@ def kv_rows_from_float(x: torch.Tensor, row_width: int) -> torch.Tensor:
 
 class KVPool:
     """K and V as ``[layer, page, row]``; one row per token page (bf16 values, or the e4m3 layout of ``KVSpec``).
-    Latent caches keep a list of ``[page, width]`` tensors in ``k``, one per layer run, and nothing in ``v``."""
+    Latent caches keep a list of ``[page, width]`` tensors in ``k``, one per layer run, and nothing in ``v``; layers of
+    unequal heads keep such lists in both."""
 
     def __init__(self, spec: KVSpec, n_pages: int, device):
         self.spec = spec
@@ -184,6 +189,9 @@ class KVPool:
         if spec.latent_widths is not None:
             self.k = [torch.zeros(n_pages + 1, w, dtype=spec.dtype, device=device) for w in spec.latent_widths]
             self.v = []
+            return
+        if spec.row_widths is not None:
+            self.k, self.v = ([torch.zeros(n_pages + 1, w[i], dtype=spec.dtype, device=device) for w in spec.row_widths] for i in (0, 1))
             return
         self.k = torch.zeros(spec.n_layers, n_pages + 1, spec.row_width, dtype=spec.store_dtype, device=device)
         self.v = torch.zeros(spec.n_layers, n_pages + 1, spec.row_width, dtype=spec.store_dtype, device=device)
@@ -194,6 +202,10 @@ class KVPool:
         pool[locs.long(), :c.shape[1]] = c.to(pool.dtype)
 
     def write(self, layer: int, locs: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> None:
+        if self.spec.row_widths is not None:
+            for pool, x in ((self.k[layer], k), (self.v[layer], v)):
+                pool.index_copy_(0, locs.long(), x.reshape(x.shape[0], -1).to(pool.dtype))
+            return
         if self.spec.fp8:
             H, D = self.spec.n_kv_heads, self.spec.head_dim
             self.k[layer].index_copy_(0, locs.long(), kv_rows_from_float(k.reshape(k.shape[0], H, D), self.spec.row_width))
@@ -205,8 +217,10 @@ class KVPool:
 
 @dataclass
 class StateSpec:
-    """Recurrent state per sequence row: the last ``conv_width - 1`` inputs of a causal convolution and, for
-    Gated-DeltaNet layers, the temporal state (``n_heads`` 0: convolution inputs only)."""
+    """Recurrent state per sequence row: the last ``conv_width - 1`` inputs of a causal convolution (of a token shift, with
+    a width of 2) and, for Gated-DeltaNet layers, the temporal state (``n_heads`` 0: convolution inputs only).  Layers with
+    matrices of unequal sizes list them in ``matrices`` (heads, rows, columns); ``n_layers`` then counts the layers that
+    keep convolution inputs."""
     n_layers: int
     conv_dim: int
     conv_width: int
@@ -215,25 +229,45 @@ class StateSpec:
     head_v_dim: int
     conv_dtype: torch.dtype = torch.bfloat16
     state_dtype: torch.dtype = torch.float32
+    matrices: Optional[List[Tuple[int, int, int]]] = None
+
+    @property
+    def matrix_offsets(self) -> List[int]:
+        """First element of every matrix inside a row, and the row's length last (matrices start on 128-byte borders)."""
+        at = [0]
+        for h, r, c in self.matrices:
+            at.append(at[-1] + (h * r * c + 31) // 32 * 32)
+        return at
 
     @property
     def row_bytes(self) -> int:
         conv = self.conv_dim * (self.conv_width - 1) * torch.empty((), dtype=self.conv_dtype).element_size()
+        if self.matrices is not None:
+            return self.n_layers * conv + self.matrix_offsets[-1] * torch.empty((), dtype=self.state_dtype).element_size()
         temp = self.n_heads * self.head_k_dim * self.head_v_dim * torch.empty((), dtype=self.state_dtype).element_size()
         return self.n_layers * (conv + temp)
 
 
 class StatePool:
     """Conv window and temporal state per (layer, row).  Multi-token passes advance the state in place (SMC accepts
-    every token), so no per-position copies are kept."""
+    every token), so no per-position copies are kept.  Matrices of unequal sizes share one row, behind one another."""
 
     def __init__(self, spec: StateSpec, n_rows: int, device):
         self.spec = spec
         self.n_rows = n_rows
         self.conv = torch.zeros(spec.n_layers, n_rows, spec.conv_dim, spec.conv_width - 1,
                                 dtype=spec.conv_dtype, device=device)
+        if spec.matrices is not None:
+            self.temporal = torch.zeros(1, n_rows, spec.matrix_offsets[-1], dtype=spec.state_dtype, device=device)
+            return
         self.temporal = torch.zeros(spec.n_layers, n_rows, spec.n_heads, spec.head_k_dim, spec.head_v_dim,
                                     dtype=spec.state_dtype, device=device)
+
+    def matrix(self, i: int) -> torch.Tensor:
+        """View [rows, heads, matrix rows, matrix columns] of one layer's matrices."""
+        h, r, c = self.spec.matrices[i]
+        at = self.spec.matrix_offsets[i]
+        return self.temporal[0, :, at:at + h * r * c].unflatten(1, (h, r, c))
 
     def copy_rows(self, dst: torch.Tensor, src: torch.Tensor) -> None:
         """dst[i] <- src[i] for every layer (fan-out at materialize, resample copies)."""

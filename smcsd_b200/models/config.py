@@ -1,18 +1,22 @@
 """Architecture descriptions: parsed from a HF ``config.json`` or built from presets.
 
-Three families are served.  Two are the ones the reference runs: dense Llama-style decoders and
+Four families are served.  Two are the ones the reference runs: dense Llama-style decoders and
 Qwen3.5-style hybrids that interleave Gated-DeltaNet layers with gated full attention
 (reference: README.md model list; parameter names checked against the HF
-implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).  The third is Pasizen: latent attention without
-positions, a short convolution in front of every mixer, hyper-connected residual streams, PolyNorm or
-mixture-of-experts feed-forwards and layers that may be looped; its config.json spells every layer out.
+implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).  The others spell every layer out in config.json.
+Pasizen: latent attention without positions, a short convolution in front of every mixer, hyper-connected residual
+streams, PolyNorm or mixture-of-experts feed-forwards and layers that may be looped.  Makodra: generalized delta rule,
+token-shifted decaying memory and chunked attention in any order, with norms on the sublayers' outputs.
 """
 from __future__ import annotations
 
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Union
+
+
+UNLIMITED_POSITIONS = 1 << 20             # positions of architectures that compute them instead of looking them up
 
 
 @dataclass(frozen=True)
@@ -23,6 +27,28 @@ class LatentAttentionSpec:
     vdim: int                            # value size per head
     kv_rank: int
     scale: float
+
+
+@dataclass(frozen=True)
+class ChunkAttentionSpec:
+    """Grouped-query attention inside chunks of ``chunk`` positions: unit-rms queries and keys, a logarithmic distance
+    bias per head, a sink of score 0, optional mixing with the first such layer's values, a sigmoid output gate."""
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key size per head
+    vdim: int                            # value size per head
+    scale: float
+    chunk: int
+    v_mix: bool = False
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    """A memory matrix [dim, dim] per head: "general_delta" (diagonal decay plus a rank-one removal) or "wkv" (diagonal
+    decay, bonus for the current token, token-shifted inputs)."""
+    kind: str
+    heads: int
+    dim: int
 
 
 @dataclass(frozen=True)
@@ -43,7 +69,7 @@ class RouterSpec:
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    kind: str                            # "dense" (PolyNorm) | "moe"
+    kind: str                            # "dense" (PolyNorm) | "moe" | "swiglu"
     ff: int = 0
     expert: Optional[GluSpec] = None
     router: Optional[RouterSpec] = None
@@ -52,13 +78,13 @@ class FeedForwardSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentAttentionSpec
+    mixer: Union[LatentAttentionSpec, ChunkAttentionSpec, RecurrentSpec]
     mlp: Optional[FeedForwardSpec]
 
 
 @dataclass
 class ModelConfig:
-    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen"
+    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen" | "makodra"
     vocab_size: int = 32000
     hidden_size: int = 4096
     n_layers: int = 32
@@ -84,7 +110,7 @@ class ModelConfig:
     attn_output_gate: bool = False
     qk_norm: bool = False
     norm_plus_one: bool = False                    # RMSNorm weight stored as (w - 1)
-    # ---- layer-by-layer description (Pasizen) --------------------------------
+    # ---- layer-by-layer description (Pasizen, Makodra) -----------------------
     layers: Optional[List[LayerSpec]] = None
     loop: Optional[tuple] = None                   # (start, stop, times): these layers run ``times`` times in a row
     streams: int = 1                               # hyper-connected copies of the residual stream
@@ -135,6 +161,8 @@ class ModelConfig:
         d, f = self.hidden_size, self.ffn_size
         if self.arch == "pasizen":
             return self._layered_param_count()
+        if self.arch == "makodra":
+            return self._makodra_param_count()
         n = self.vocab_size * d * (1 if self.tie_embeddings else 2) + d
         for i in range(self.n_layers):
             n += 3 * d * f + 2 * d
@@ -164,7 +192,47 @@ class ModelConfig:
                 n += L.mlp.router.experts * (d + glu(L.mlp.expert)) + (glu(L.mlp.shared) if L.mlp.shared else 0)
         return n
 
+    def _makodra_param_count(self) -> int:
+        d, n = self.hidden_size, self.vocab_size * self.hidden_size + self.hidden_size
+        for L in self.layers:
+            m = L.mixer
+            n += d * (1 if L.mlp is None else 2 + 3 * L.mlp.ff)
+            if isinstance(m, ChunkAttentionSpec):
+                n += d * (m.heads * (m.dim + 2 * m.vdim) + m.kv_heads * (m.dim + m.vdim)) + 2 * m.heads + m.v_mix
+            else:                        # without the low-rank decay maps, whose rank only the weights tell
+                delta = m.kind == "general_delta"
+                n += m.heads * m.dim * ((6 if delta else 5) * d + 3) + (0 if delta else 5 * d)
+        return n
+
     # ---- construction ----------------------------------------------------------
+    @classmethod
+    def from_makodra_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
+        """config.json of a Makodra model: every layer with its mixer and feed-forward."""
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            m, f = e["mixer"], e.get("mlp")
+            if e["type"] == "attention":
+                mixer = ChunkAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                           int(m["mask"]["size"]), bool(m.get("v_mix", False)))
+                if mixer.heads % mixer.kv_heads or mixer.chunk < 1:
+                    raise ValueError(f"layer {i}: inconsistent attention {mixer}")
+            elif e["type"] in ("general_delta", "wkv"):
+                mixer = RecurrentSpec(e["type"], int(m["heads"]), int(m["dim"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            if f is not None and f["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(LayerSpec(mixer, None if f is None else FeedForwardSpec("swiglu", ff=int(f["ff"]))))
+        mixing = {(L.mixer.kv_heads, L.mixer.vdim) for L in layers if isinstance(L.mixer, ChunkAttentionSpec) and L.mixer.v_mix}
+        if len(mixing) > 1:
+            raise ValueError(f"layers that mix values need values of one shape, not {sorted(mixing)}")
+        eos = c.get("eos_token_id")
+        m0 = layers[0].mixer
+        return cls(arch="makodra", vocab_size=int(c["vocab"]), hidden_size=int(c["width"]), n_layers=len(layers), n_heads=m0.heads,
+                   n_kv_heads=getattr(m0, "kv_heads", m0.heads), head_dim=m0.dim, ffn_size=0, rms_eps=float(c["norm"]["eps"]),
+                   max_position=UNLIMITED_POSITIONS, tie_embeddings=True, logit_softcap=float(c.get("logit_softcap") or 0.0),
+                   layers=layers, eos_token_ids=[] if eos is None else ([eos] if isinstance(eos, int) else list(eos)))
+
     @classmethod
     def from_layered_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
         """config.json of a Pasizen model: every layer with its mixer and feed-forward, the loop, the stream count."""
@@ -209,6 +277,8 @@ class ModelConfig:
             c = merged
         if c.get("architecture") == "Pasizen":
             return cls.from_layered_dict(c)
+        if c.get("architecture") == "Makodra":
+            return cls.from_makodra_dict(c)
         archs = c.get("architectures") or []
         mt = (c.get("model_type") or "").lower()
         is_hybrid = "layer_types" in c and any(t == "linear_attention" for t in c["layer_types"])
@@ -327,6 +397,21 @@ def preset(name: str) -> ModelConfig:
         return ModelConfig(arch="pasizen", vocab_size=4096, hidden_size=136, n_layers=3, n_heads=3, n_kv_heads=1,
                            head_dim=48, ffn_size=0, rms_eps=1e-6, max_position=2048, layers=[dense, moe, dense],
                            loop=(1, 3, 2), streams=2, conv_taps=3, name="tiny-pasizen")
+    if n in ("makodra-2048", "makodra-1024"):
+        # random-init stand-ins with the layer sizes of a real small model: two recurrent layers to one attention layer
+        d, ff = (2048, 5632) if n.endswith("2048") else (1024, 2816)
+        H, mlp = d // 64, FeedForwardSpec("swiglu", ff=ff)
+        trio = [LayerSpec(RecurrentSpec("general_delta", H, 64), mlp), LayerSpec(RecurrentSpec("wkv", H, 64), mlp),
+                LayerSpec(ChunkAttentionSpec(d // 128, d // 512, 128, 128, 11.3, 1024, True), mlp)]
+        return ModelConfig(arch="makodra", vocab_size=65536, hidden_size=d, n_layers=15, n_heads=H, n_kv_heads=H, head_dim=64,
+                           ffn_size=0, rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, tie_embeddings=True, logit_softcap=30.0,
+                           layers=trio * 5, name=n)
+    if n in ("tiny-makodra",):
+        mlp = FeedForwardSpec("swiglu", ff=200)
+        return ModelConfig(arch="makodra", vocab_size=4096, hidden_size=136, n_layers=3, n_heads=3, n_kv_heads=3, head_dim=40,
+                           ffn_size=0, rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, tie_embeddings=True, logit_softcap=20.0,
+                           layers=[LayerSpec(RecurrentSpec("wkv", 3, 40), mlp), LayerSpec(ChunkAttentionSpec(4, 2, 24, 40, 3.0, 48, True), None),
+                                   LayerSpec(RecurrentSpec("general_delta", 5, 32), mlp)], name="tiny-makodra")
     raise KeyError(f"unknown preset {name!r}")
 
 

@@ -209,3 +209,87 @@ def hyper_read(x: torch.Tensor, w_in: torch.Tensor) -> torch.Tensor:
 def hyper_write(x: torch.Tensor, y: torch.Tensor, w_mix: torch.Tensor, w_out: torch.Tensor) -> torch.Tensor:
     """New streams x_t' = sum_s w_mix[s, t] x_s + w_out[t] y."""
     return torch.einsum("tsd,su->tud", x, w_mix) + w_out.view(1, -1, 1) * y.unsqueeze(1)
+
+
+# ---- positions, token shift and memory matrices
+def sinusoidal_positions(positions: torch.Tensor, d: int, base: float = 10000.0) -> torch.Tensor:
+    """fp32 [T, d]: entry 2i is sin(p base^(-2i/d)), entry 2i + 1 the cosine of the same angle."""
+    c = torch.arange(d, device=positions.device)
+    freq = base ** (-(c - c % 2).double() / d)
+    ang = positions.double().unsqueeze(1) * freq.unsqueeze(0)
+    return torch.where(c % 2 == 0, ang.sin(), ang.cos()).float()
+
+
+def token_shift(h: torch.Tensor, mu: torch.Tensor, batch: ExtendBatch, history: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
+    """h [T, d] fp32, mu [n, d] -> [T, n, d]: h + (h' - h) mu with h' the row of the token before.  ``history`` [rows, >= d, 1]
+    holds the row before the first new token and is advanced in place."""
+    d, t0 = h.shape[1], 0
+    prev = torch.empty_like(h)
+    for b, e in enumerate(batch.lens()):
+        if e == 0:
+            continue
+        r = rows[b]
+        prev[t0] = history[r, :d, 0].to(h.dtype)
+        prev[t0 + 1:t0 + e] = h[t0:t0 + e - 1]
+        history[r, :d, 0] = h[t0 + e - 1].to(history.dtype)
+        t0 += e
+    return h.unsqueeze(1) + (prev - h).unsqueeze(1) * mu
+
+
+DELTA_UNIT_EPS = 1e-6
+
+
+def delta_memory(state: torch.Tensor, r, w, k, v, a) -> torch.Tensor:
+    """Generalized delta rule of one sequence, token by token: with u = k / |k| and M the matrix before the token,
+    M <- diag(w) M - (a u) (u^T M) + k v^T, read out with r.  r, w, k, a [T, H, dk], v [T, H, dv]; ``state`` [H, dv, dk] fp32
+    holds M transposed and is advanced in place.  Returns [T, H, dv]."""
+    u = k * torch.rsqrt((k * k).sum(-1, keepdim=True) + DELTA_UNIT_EPS)
+    M, out = state.clone(), torch.empty_like(v)
+    for t in range(r.shape[0]):
+        gone = (M * u[t].unsqueeze(1)).sum(-1, keepdim=True)                  # [H, dv, 1]
+        M = M * w[t].unsqueeze(1) - gone * (a[t] * u[t]).unsqueeze(1) + v[t].unsqueeze(-1) * k[t].unsqueeze(1)
+        out[t] = (M * r[t].unsqueeze(1)).sum(-1)
+    state.copy_(M)
+    return out
+
+
+def bonus_memory(state: torch.Tensor, r, w, k, v, bonus) -> torch.Tensor:
+    """Decaying memory of one sequence: out = (M + diag(bonus) k v^T)^T r, then M <- diag(w) M + k v^T; layouts as in
+    ``delta_memory``, bonus [H, dk]."""
+    M, out = state.clone(), torch.empty_like(v)
+    for t in range(r.shape[0]):
+        kv = v[t].unsqueeze(-1) * k[t].unsqueeze(1)
+        out[t] = ((M + kv * bonus.unsqueeze(1)) * r[t].unsqueeze(1)).sum(-1)
+        M = M * w[t].unsqueeze(1) + kv
+    state.copy_(M)
+    return out
+
+
+def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
+                              batch: ExtendBatch, kv_heads: int, scale: float, r1: torch.Tensor, r2: torch.Tensor,
+                              chunk: int) -> torch.Tensor:
+    """Causal attention inside chunks of ``chunk`` positions with scores scale q.k - r1 ln(1 + r2 distance) and a sink of
+    score 0.  q [T, H, D]; pools [pages, kv_heads * width]; returns fp32 [T, H, value width]."""
+    T, H, D = q.shape
+    rep, V = H // kv_heads, v_pool.shape[1] // kv_heads
+    out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
+    pref = batch.prefix_lens_host if batch.prefix_lens_host is not None else batch.prefix_lens.tolist()
+    t0 = 0
+    for b, (p, e) in enumerate(zip(pref, batch.lens())):
+        if e == 0:
+            continue
+        lo, L = p // chunk * chunk, p + e
+        pages = block_table[batch.rows[b].long(), lo:L].long()
+        kk = k_pool[pages].view(L - lo, kv_heads, -1)[:, :, :D].float().repeat_interleave(rep, dim=1)
+        vv = v_pool[pages].view(L - lo, kv_heads, V).float().repeat_interleave(rep, dim=1)
+        i = torch.arange(p, L, device=q.device).unsqueeze(1)
+        j = torch.arange(lo, L, device=q.device).unsqueeze(0)
+        dist = (i - j).clamp(min=0).float()
+        s = torch.einsum("ehd,lhd->hel", q[t0:t0 + e].float(), kk) * scale
+        s = s - r1.view(H, 1, 1) * torch.log1p(r2.view(H, 1, 1) * dist)
+        s = s.masked_fill((j > i) | (i // chunk != j // chunk), float("-inf"))
+        top = s.amax(-1, keepdim=True).clamp(min=0.0)
+        ex = torch.exp(s - top)
+        out[t0:t0 + e] = torch.einsum("hel,lhv->ehv", ex / (torch.exp(-top) + ex.sum(-1, keepdim=True)), vv)
+        t0 += e
+    return out

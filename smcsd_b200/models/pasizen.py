@@ -25,24 +25,11 @@ from typing import Iterator, List, Optional
 import torch
 
 from ..memory.pools import KVSpec, StateSpec
-from .config import LayerSpec, ModelConfig
+from .config import LayerSpec
+from .layered import GU_BLOCK, LayeredModel, pad_to, round_up
 from .layers import (ExtendBatch, clamped_glu, hyper_read, hyper_write, latent_attention_reference, poly_norm, rms_unit,
                      route_grouped, short_conv)
 from .llama import interleave_gate_up, split_gate_up
-from .loader import Checkpoint
-
-GU_BLOCK = 64
-
-
-def round_up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
-
-
-def pad_to(w: torch.Tensor, *shape: int) -> torch.Tensor:
-    """Zero-padded copy of ``w`` with the given (not smaller) shape."""
-    out = torch.zeros(*shape, dtype=w.dtype, device=w.device)
-    out[tuple(slice(0, n) for n in w.shape)] = w
-    return out
 
 
 @dataclass
@@ -82,19 +69,8 @@ class PasizenLayerWeights:
                 yield from vars(v).values()
 
 
-class PasizenModel:
-    has_state = True
-
-    def __init__(self, cfg: ModelConfig, dtype=torch.bfloat16, device="cpu", tp_rank: int = 0, tp_size: int = 1,
-                 max_positions: Optional[int] = None):
-        if tp_size != 1:
-            raise ValueError("Pasizen models run with tp_size=1")
-        self.cfg, self.dtype, self.device = cfg, dtype, torch.device(device)
-        self.tp_rank, self.tp_size, self.tp_group = 0, 1, None
-        self.n_heads, self.n_kv_heads = cfg.n_heads, 1
-        self.layers: List[PasizenLayerWeights] = []
-        self.embed = self.pos = self.lm_head = self.final_norm = None
-        self.runs = cfg.layer_runs
+class PasizenModel(LayeredModel):
+    family = "Pasizen"
 
     # ---- cache and state ---------------------------------------------------------------
     def kv_spec(self, dtype, fp8: bool = False) -> KVSpec:
@@ -107,16 +83,6 @@ class PasizenModel:
         return StateSpec(len(self.runs), self.cfg.hidden_size, self.cfg.conv_taps, 0, 0, 0, conv_dtype=torch.float32)
 
     # ---- parameters --------------------------------------------------------------------
-    def all_tensors(self) -> Iterator[torch.Tensor]:
-        for t in (self.embed, self.pos, self.lm_head, self.final_norm):
-            if t is not None:
-                yield t
-        for L in self.layers:
-            yield from L.tensors()
-
-    def weight_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.all_tensors())
-
     def _assemble(self, get) -> "PasizenModel":
         """Fill the packed layout from ``get(name, *shape)``, which returns a tensor by its checkpoint name."""
         c, dt, dev = self.cfg, self.dtype, self.device
@@ -165,19 +131,6 @@ class PasizenModel:
                         L.s_gu, L.s_down = glu(p + "mlp.shared.", f.shared.ff)
             self.layers.append(L)
         return self
-
-    def load_hf(self, path: str) -> "PasizenModel":
-        ck = Checkpoint(path)
-
-        def get(name, *shape):
-            t = ck.get(name)
-            if tuple(t.shape) != tuple(shape):
-                raise ValueError(f"{name}: shape {tuple(t.shape)} in the checkpoint, {tuple(shape)} by the configuration")
-            return t
-        try:
-            return self._assemble(get)
-        finally:
-            ck.close()
 
     def init_random(self, seed: int = 0, std: float = 0.02) -> "PasizenModel":
         g = torch.Generator(device=self.device)
@@ -239,11 +192,6 @@ class PasizenModel:
             out = out + self._glu(x, L.s_gu, L.s_down, f.shared.limit)
         return out
 
-    def _act(self, h: torch.Tensor) -> torch.Tensor:
-        """fp32 rows in the activation dtype, padded to the GEMM operand width."""
-        d8 = round_up(h.shape[1], 8)
-        return pad_to(h.to(self.dtype), h.shape[0], d8) if d8 != h.shape[1] else h.to(self.dtype)
-
     def forward_torch(self, batch: ExtendBatch, kv, block_table: torch.Tensor, state=None, per_run=None) -> torch.Tensor:
         """Post-norm hidden rows of the new tokens; ``per_run`` (a list) collects the summed streams after every layer run."""
         if state is None:
@@ -263,6 +211,3 @@ class PasizenModel:
             if per_run is not None:
                 per_run.append(x.sum(1))
         return self._act(rms_unit(x.sum(1), c.rms_eps) * self.final_norm)
-
-    def logits_torch(self, hidden: torch.Tensor) -> torch.Tensor:
-        return (hidden @ self.lm_head.t()).float()

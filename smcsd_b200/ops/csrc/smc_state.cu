@@ -368,7 +368,8 @@ SMC_API int smc_state_copy(void* state, long long layer_stride_bytes, long long 
   if (max_jobs <= 0 || n_layers <= 0) return 0;
   if (row_bytes & 15) return -61;
   int chunks = (int)((row_bytes / 16 + 255) / 256);
-  if (chunks > 16) chunks = 16;
+  const int most = n_layers == 1 ? 256 : 16;      // all layers' matrices in one row: the row alone fills the machine
+  if (chunks > most) chunks = most;
   smc::state_copy_kernel<<<dim3(max_jobs, n_layers, chunks), 256, 0, st>>>((uint8_t*)state, layer_stride_bytes, row_bytes,
                                                                         counters, job_dst, job_src, n_rows);
   return (int)cudaGetLastError();

@@ -17,7 +17,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..models.layers import GLU_SIGMOID_SLOPE
-from ..models.pasizen import GU_BLOCK, round_up
+from ..models.layered import GU_BLOCK, round_up
 from . import native as K
 from .ragged import RaggedPlan, uniform_struct
 

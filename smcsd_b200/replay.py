@@ -22,7 +22,7 @@ def open_engine(model: str, dtype: str, max_tokens: int, device: str = "auto"):
     from .models.config import resolve_config
     cfg = resolve_config(model)
     return SMCEngine(model, model, n_particles=1, gamma=1, dtype=dtype, device=device, max_running_requests=MAX_SEQUENCES,
-                     max_total_tokens=max_tokens, context_length=cfg.max_position, skip_tokenizer_init=True, in_process=True)
+                     max_total_tokens=max_tokens, context_length=min(cfg.max_position, max_tokens), skip_tokenizer_init=True, in_process=True)
 
 
 def replay(engine, lines, out_dir: str, reply) -> None:

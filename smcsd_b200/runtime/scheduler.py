@@ -32,7 +32,7 @@ from .worker import PrefillItem, SMCWorker
 
 log = logging.getLogger("smcsd_b200.scheduler")
 
-NATIVE_F32_ARCHS = ("pasizen",)       # architectures whose kernel chain also runs in 32-bit
+NATIVE_F32_ARCHS = ("pasizen", "makodra")       # architectures whose kernel chain also runs in 32-bit
 
 
 @dataclass
@@ -132,8 +132,8 @@ class SMCScheduler:
             if m.cfg.arch == "pasizen" and self.context_len > m.cfg.max_position:
                 raise ValueError(f"context_length {self.context_len} exceeds the {m.cfg.max_position} learned positions of "
                                  f"{m.cfg.name or 'the model'}")
-            if m.cfg.arch == "pasizen" and pp_size > 1:
-                raise NotImplementedError("particle-parallel groups do not support latent caches")
+            if m.cfg.arch in ("pasizen", "makodra") and pp_size > 1:
+                raise NotImplementedError("particle-parallel groups do not support caches with a row width per layer")
         # ---- memory -----------------------------------------------------------
         N, G = self.n_local, a.gamma + 1
         self.max_groups = a.max_running_requests
