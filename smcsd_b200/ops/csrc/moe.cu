@@ -1,6 +1,6 @@
 // Feed-forward pieces around the GEMMs of layered architectures:
 //   poly_norm       a N(z) + b N(z^2) + c N(z^3) + e, N dividing the token's row by its root mean square
-//   clamped_glu     min(g, limit) sigmoid(slope g) (clamp(u) + 1) on stored gate / up rows (32-bit runs; the bf16 path has
+//   gated_unit      min(g, limit) sigmoid(slope g) (clamp(u) + shift) on stored gate / up rows (32-bit runs; the bf16 path has
 //                   it in the GEMM epilogue)
 //   route           router logits, softmax over all experts, best groups, best experts, renormalised weights
 //   dispatch        slots of the (token, expert) pairs sorted by expert, and the table of token tiles the grouped GEMMs use
@@ -53,16 +53,16 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const float* z, int ldz,
   }
 }
 
-// ---------------------------------------------------------------- clamped gated unit on stored rows
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const float* gu, int ldg, float* out,
-                                                          int ldo, int ff, int blk, float limit, float slope, int M, int pdl) {
+// ---------------------------------------------------------------- gated unit on stored rows (an infinite limit: none)
+__global__ void __launch_bounds__(256) gated_unit_kernel(const float* gu, int ldg, float* out, int ldo, int ff, int blk, float limit,
+                                                         float slope, float shift, int M, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const long long n = (long long)M * ff;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const int m = (int)(i / ff), c = (int)(i % ff), q = c / blk, r = c - q * blk;
     const float* row = gu + (size_t)m * ldg + (size_t)q * 2 * blk + r;
     const float g = fminf(row[0], limit), u = fminf(fmaxf(row[blk], -limit), limit);
-    out[(size_t)m * ldo + c] = g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+    out[(size_t)m * ldo + c] = g / (1.0f + expf(-slope * g)) * (u + shift);
   }
 }
 
@@ -273,13 +273,13 @@ SMC_API int smc_poly_norm(const float* z, int ldz, const float* coef, float eps,
   return launch_pdl(poly_norm_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, st, pdl, z, ldz, coef, eps, (__nv_bfloat16*)out, ldo, ff, pdl);
 }
 
-SMC_API int smc_clamped_glu_f32(const float* gu, int ldg, float* out, int ldo, int ff, int blk, float limit, float slope,
-                                int M, int pdl, cudaStream_t st) {
+SMC_API int smc_gated_unit_f32(const float* gu, int ldg, float* out, int ldo, int ff, int blk, float limit, float slope,
+                               float shift, int M, int pdl, cudaStream_t st) {
   using namespace smc;
   if (M <= 0) return 0;
   const long long n = ((long long)M * ff + 255) / 256;
-  return launch_pdl(clamped_glu_kernel, dim3((unsigned)(n < 2368 ? n : 2368)), dim3(256), 0, st, pdl, gu, ldg, out, ldo, ff, blk,
-                    limit, slope, M, pdl);
+  return launch_pdl(gated_unit_kernel, dim3((unsigned)(n < 2368 ? n : 2368)), dim3(256), 0, st, pdl, gu, ldg, out, ldo, ff, blk,
+                    limit, slope, shift, M, pdl);
 }
 
 // h fp32 [T, d] packed; wr [E, ldw]; idx / wgt [T, top].

@@ -628,6 +628,31 @@ class LatentArgs(C.Structure):
                 ("H", _I), ("ldc", _I), ("scale", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
+class PostNormArgs(C.Structure):
+    _fields_ = [("x", _VP), ("d", _I), ("ids", _VP), ("positions", _VP), ("embed", _VP), ("freq", _VP), ("vocab", _I), ("y", _VP),
+                ("ldy", _I), ("w", _VP), ("eps", _F), ("w_final", _VP), ("xa", _VP), ("ldxa", _I), ("mu", _VP), ("mix", _VP),
+                ("hist", _VP), ("rows", _VP), ("n_mix", _I), ("ldh", _I), ("n_rows", _I), ("status", _VP), ("pdl", _I)]
+
+
+class HeadsNewArgs(C.Structure):
+    _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "H", "G", "D", "V", "dim")] + \
+               [("eps", _F), ("q", _VP), ("kpool", _VP), ("vpool", _VP), ("n_pages", _I), ("locs", _VP), ("lam", _F), ("v_first", _VP),
+                ("gives", _I), ("status", _VP), ("pdl", _I)]
+
+
+class ChunkAttnArgs(C.Structure):
+    _fields_ = [("q", _VP), ("kpool", _VP), ("vpool", _VP), ("out", _VP), ("gate", _VP), ("ldg", _I), ("block_table", _VP)] + \
+               [(n, _I) for n in ("bt_stride", "bt_rows", "n_pages", "H", "G", "D", "V", "chunk")] + \
+               [("scale", _F), ("r1", _VP), ("r2", _VP), ("sink", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
+class ScanArgs(C.Structure):
+    _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "r_off", "k_off", "v_off", "g_off", "a_off")] + \
+               [("z", _VP), ("ldz", _I), ("w0", _VP), ("a_bias", _VP), ("bonus", _VP), ("onorm", _VP), ("state", _VP),
+                ("row_stride", C.c_longlong), ("n_rows", _I), ("out", _VP), ("ldo", _I), ("H", _I), ("D", _I), ("eps", _F),
+                ("unit_eps", _F), ("log_decay", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
 class GroupLink(C.Structure):
     """Several products in one GEMM launch (csrc/gemm_skinny.cu); mode 0 only selects the gated epilogue's activation."""
     _fields_ = [(n, _I) for n in ("mode", "groups", "w_rows", "x_cols", "out_cols")] + [("tiles", _VP)] + \
@@ -647,7 +672,7 @@ def layered_lib():
         L.smc_hyper_step.argtypes = [vp, i, i, vp]
         L.smc_short_conv.argtypes = [vp, vp, i, vp, vp, i, i, i, vp, vp, i, i, vp]
         L.smc_poly_norm.argtypes = [vp, i, vp, f, vp, i, i, i, i, i, vp]
-        L.smc_clamped_glu_f32.argtypes = [vp, i, vp, i, i, i, f, f, i, i, vp]
+        L.smc_gated_unit_f32.argtypes = [vp, i, vp, i, i, i, f, f, f, i, i, vp]
         L.smc_route.argtypes = [vp, i, vp, i, i, i, i, i, i, vp, vp, i, i, vp]
         L.smc_dispatch.argtypes = [vp, i, i, i, i, vp, vp, vp, i, vp, i, vp]
         L.smc_gather_rows.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, vp]
@@ -658,11 +683,22 @@ def layered_lib():
         L.smc_latent_tc_splits.argtypes = [i, i, i]
         L.smc_latent_tc_splits.restype = C.c_int
         L.smc_latent_tc_max_width.restype = C.c_int
-        for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_clamped_glu_f32",
-                  "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn"):
+        L.smc_post_norm_step.argtypes = [vp, i, i, vp]
+        L.smc_token_shift.argtypes = [vp, i, vp, i, vp, i, vp, i, i, vp, vp, i, i, vp]
+        L.smc_heads_new.argtypes = [vp, i, i, vp]
+        L.smc_chunk_attn.argtypes = [vp, i, vp]
+        L.smc_chunk_attn_tc.argtypes = [vp, vp]
+        L.smc_memory_scan.argtypes = [vp, i, i, vp]
+        L.smc_tanh_rows.argtypes = [vp, i, vp, i, i, i, i, i, vp]
+        for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_gated_unit_f32",
+                  "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn", "smc_post_norm_step",
+                  "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_tc", "smc_chunk_attn_tc_max_width",
+                  "smc_memory_scan", "smc_tanh_rows"):
             getattr(L, n).restype = C.c_int
         for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
-                       (GroupLink, "smc_group_link_size")):
+                       (GroupLink, "smc_group_link_size"), (PostNormArgs, "smc_post_norm_args_size"),
+                       (HeadsNewArgs, "smc_heads_new_args_size"), (ChunkAttnArgs, "smc_chunk_attn_args_size"),
+                       (ScanArgs, "smc_scan_args_size")):
             assert C.sizeof(cls) == getattr(L, n)(), f"{cls.__name__} layout mismatch"
         L._layered_declared = True
     return L
@@ -706,10 +742,11 @@ def poly_norm(z: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, *, ff: int
                                        _stream()), "smc_poly_norm")
 
 
-def clamped_glu_f32(gu: torch.Tensor, out: torch.Tensor, *, ff: int, blk: int, limit: float, slope: float, M: int,
-                    pdl: bool = False) -> None:
-    _check(layered_lib().smc_clamped_glu_f32(_p(gu), gu.stride(0), _p(out), out.stride(0), ff, blk, limit, slope, M, int(pdl),
-                                             _stream()), "smc_clamped_glu_f32")
+def gated_unit_f32(gu: torch.Tensor, out: torch.Tensor, *, ff: int, blk: int, limit: float, slope: float, shift: float, M: int,
+                   pdl: bool = False) -> None:
+    """min(g, limit) sigmoid(slope g) (clamp(u, limit) + shift) on gate / up columns interleaved in blocks of ``blk``."""
+    _check(layered_lib().smc_gated_unit_f32(_p(gu), gu.stride(0), _p(out), out.stride(0), ff, blk, limit, slope, shift, M, int(pdl),
+                                            _stream()), "smc_gated_unit_f32")
 
 
 def route(h: torch.Tensor, wr: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor, *, d: int, top: int, groups: int, keep: int,
@@ -758,3 +795,43 @@ def latent_tc_splits(tiles: int, width: int, keys: int) -> int:
 def latent_attention_tc(a: LatentArgs, *, tokens: int, blk_rows: int, splits: int = 1) -> None:
     """bf16 latent attention on the tensor cores; ``splits`` key ranges run as a thread-block cluster and merge on chip."""
     _check(layered_lib().smc_latent_attn_tc(C.byref(a), tokens, blk_rows, splits, _stream()), "smc_latent_attn_tc")
+
+
+def post_norm_step(a: PostNormArgs, T: int, f32: bool) -> None:
+    """x <- x + y / rms(y) w (or the embedding start, or the final norm), x in the activation type, folded token shift."""
+    _check(layered_lib().smc_post_norm_step(C.byref(a), T, int(f32), _stream()), "smc_post_norm_step")
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, mix: torch.Tensor, hist: torch.Tensor, r: Ragged, *, ldm: int, status: torch.Tensor,
+                f32: bool, pdl: bool = False) -> None:
+    """mix [T, n, ldm] = x + (row before - x) mu[s]; x fp32 [T, d], hist [rows, ldh] advances."""
+    _check(layered_lib().smc_token_shift(_p(x), mu.shape[1], _p(mu), mu.shape[0], _p(mix), ldm, _p(hist), hist.stride(0), hist.shape[0],
+                                         C.byref(r), _p(status), int(f32), int(pdl), _stream()), "smc_token_shift")
+
+
+def heads_new(a: HeadsNewArgs, T: int, f32: bool) -> None:
+    """New tokens' queries, keys and values: unit rms per head, mixed values, cache pages."""
+    _check(layered_lib().smc_heads_new(C.byref(a), T, int(f32), _stream()), "smc_heads_new")
+
+
+def chunk_attention(a: ChunkAttnArgs, f32: bool) -> None:
+    _check(layered_lib().smc_chunk_attn(C.byref(a), int(f32), _stream()), "smc_chunk_attn")
+
+
+def chunk_attention_tc(a: ChunkAttnArgs) -> None:
+    """The same in bf16 on the tensor cores, for blocks of up to 64 tokens."""
+    _check(layered_lib().smc_chunk_attn_tc(C.byref(a), _stream()), "smc_chunk_attn_tc")
+
+
+def chunk_tc_max_width() -> int:
+    """Widest head the tensor-core form takes."""
+    return layered_lib().smc_chunk_attn_tc_max_width()
+
+
+def memory_scan(a: ScanArgs, delta: bool, f32: bool) -> None:
+    """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu)."""
+    _check(layered_lib().smc_memory_scan(C.byref(a), int(delta), int(f32), _stream()), "smc_memory_scan")
+
+
+def tanh_rows(x: torch.Tensor, out: torch.Tensor, *, n: int, M: int, f32: bool, pdl: bool = False) -> None:
+    _check(layered_lib().smc_tanh_rows(_p(x), x.stride(0), _p(out), out.stride(0), n, M, int(f32), int(pdl), _stream()), "smc_tanh_rows")

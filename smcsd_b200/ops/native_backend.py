@@ -557,6 +557,9 @@ class NativeRunner:
         if model.cfg.arch == "pasizen":
             from .native_pasizen import NativePasizen
             return NativePasizen(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, state=state)
+        if model.cfg.arch == "makodra":
+            from .native_makodra import NativeMakodra
+            return NativeMakodra(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, state=state)
         if model.cfg.arch != "llama":
             from .native_hybrid import NativeHybrid
             return NativeHybrid(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, runner=self,

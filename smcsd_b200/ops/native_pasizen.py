@@ -11,42 +11,22 @@ captured in a graph.
 """
 from __future__ import annotations
 
-import os
-from typing import Dict, List, Optional
+from typing import List, Optional
 
 import torch
 
 from ..models.layers import GLU_SIGMOID_SLOPE
 from ..models.layered import GU_BLOCK, round_up
 from . import native as K
-from .ragged import RaggedPlan, uniform_struct
+from .native_layered import NativeLayered, env_flag
 
 
-def _env_flag(name: str, default: bool) -> bool:
-    v = os.environ.get(name)
-    return default if v is None else v.strip().lower() in ("1", "true", "yes", "on")
-
-
-class NativePasizen:
-    ragged = True
-    BLOCK = 64                            # tokens per block of the work list
-
+class NativePasizen(NativeLayered):
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
-        self.m, self.kv, self.bt, self.state = model, kv, block_table, state
-        self.c = c = model.cfg
-        self.T, self.status, self.pdl, self.attn_splits = max_tokens, status, pdl, attn_splits
-        self.f32 = model.dtype == torch.float32
-        if model.dtype not in (torch.float32, torch.bfloat16):
-            raise ValueError("the Pasizen kernel chain runs in bfloat16 or float32")
-        self.dt = model.dtype
-        self.d, self.d8, self.S = c.hidden_size, round_up(c.hidden_size, 8), c.streams
-        self.V = model.lm_head.shape[0]
-        self.fused_lm_sample = not self.f32
-        self.dev = model.device
-        self.ctx_hint = 0
-        self._lm_parts = None
-        self._splits: Dict = {}
+        super().__init__(model, kv, block_table, max_tokens, max_logit_rows, attn_splits, status, pdl, state)
+        c = self.c
+        self.S = c.streams
         mixers = [L.mixer for L in c.layers]
         mlps = [L.mlp for L in c.layers if L.mlp is not None]
         dense, moe = [f for f in mlps if f.kind == "dense"], [f for f in mlps if f.kind == "moe"]
@@ -54,9 +34,6 @@ class NativePasizen:
         T = max_tokens
         self.x = torch.zeros(T, self.S, self.d, dtype=torch.float32, device=self.dev)
         self.n = torch.zeros(T, self.d, dtype=torch.float32, device=self.dev)
-        self.xa = torch.zeros(T, self.d8, dtype=self.dt, device=self.dev)
-        # flat buffers, viewed per layer with that layer's own row width
-        self._flat: Dict[str, torch.Tensor] = {}
         self._room("proj", T * most(m.heads * round_up(m.dim, 8) + m.kv_rank for m in mixers), torch.float32)
         self._room("q", T * most(m.heads * round_up(m.dim, 8) for m in mixers), self.dt)
         self._room("lat", T * most(m.heads * round_up(m.kv_rank, 64) for m in mixers), self.dt)
@@ -78,17 +55,8 @@ class NativePasizen:
         if self.f32:
             self._room("gu", max([pairs * 2 * round_up(f.expert.ff, GU_BLOCK) for f in moe] +
                                  [T * 2 * round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared], default=0), torch.float32)
-        # the samplers read rows of float4
-        self.logits = torch.empty(max_logit_rows, round_up(self.V, 4), dtype=torch.float32, device=self.dev)
-        self.attn_tc = not self.f32 and _env_flag("SMC_LATENT_TC", True)
+        self.attn_tc = not self.f32 and env_flag("SMC_LATENT_TC", True)
         self._steps = self._build_steps()
-
-    # ---- buffers ------------------------------------------------------------------------
-    def _room(self, name: str, numel: int, dtype) -> None:
-        self._flat[name] = torch.zeros(max(int(numel), 8), dtype=dtype, device=self.dev)
-
-    def _rows(self, name: str, rows: int, width: int) -> torch.Tensor:
-        return self._flat[name][:rows * width].view(rows, width)
 
     def _build_steps(self) -> List[dict]:
         """The sublayers of every layer run in execution order, each with the prepared arguments of the stream step that
@@ -139,21 +107,7 @@ class NativePasizen:
             ks //= 2
         return ks
 
-    def _cluster(self, N: int, Kd: int, M: int) -> int:
-        key = (N, Kd, M)
-        if key not in self._splits:
-            self._splits[key] = K.gemm_cluster_splits(N, Kd, M)
-        return self._splits[key]
-
     # ---- products -----------------------------------------------------------------------
-    def _gemm(self, W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, M: int) -> None:
-        """out (fp32) = X W^T."""
-        if self.f32:
-            K.gemm_f32(W, X, out, N=W.shape[0], M=M, pdl=self.pdl)
-        else:
-            K.gemm_skinny(W, X, out, M=M, splits=self._cluster(W.shape[0], W.shape[1], M), epi=K.EPI_STORE_F32,
-                          ldo=out.stride(0), status=self.status, pdl=self.pdl)
-
     def _per_head(self, W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, M: int, H: int, x_cols: int, out_cols: int) -> None:
         """Head h: out[:, h * out_cols ..] = X[:, h * x_cols ..] W_h^T, in the activation type."""
         link = K.GroupLink(mode=K.GROUP_BATCHED, groups=H, w_rows=out_cols, x_cols=x_cols, out_cols=out_cols)
@@ -164,15 +118,8 @@ class NativePasizen:
 
     def _glu_gemm(self, W: torch.Tensor, X: torch.Tensor, act: torch.Tensor, M: int, limit: float, link: "K.GroupLink") -> None:
         """act = clamped gated unit of the interleaved gate / up product."""
-        ff2 = W.shape[-2]
         link.act, link.limit, link.slope = K.ACT_CLAMPED, limit, GLU_SIGMOID_SLOPE
-        if self.f32:
-            gu = self._rows("gu", M, ff2)
-            K.gemm_f32(W, X, gu, N=ff2, M=M, link=link, pdl=self.pdl)
-            K.clamped_glu_f32(gu, act, ff=ff2 // 2, blk=GU_BLOCK, limit=limit, slope=GLU_SIGMOID_SLOPE, M=M, pdl=self.pdl)
-            return
-        splits = K.gemm_swiglu_splits(ff2, W.shape[-1], M) if link.mode == 0 else 1
-        K.gemm_grouped(W, X, act, N=ff2, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, link=link, status=self.status, pdl=self.pdl)
+        self._gated_gemm(W, X, act, M, GU_BLOCK, link, shift=1.0)
 
     # ---- sublayers ----------------------------------------------------------------------
     def _mixer(self, s: dict, T: int, locs: torch.Tensor, work: "K.Ragged", longest: int) -> None:
@@ -261,40 +208,3 @@ class NativePasizen:
             elif kind == "ff":
                 (self._dense if s["L"].spec.mlp.kind == "dense" else self._experts)(s, T)
         return self.xa
-
-    def forward(self, ids, positions, cache_locs, rows, prefix_lens, bs: int, E: int, two_pass: bool = False) -> torch.Tensor:
-        """bs sequences of E new tokens each."""
-        work = uniform_struct(rows, prefix_lens, bs, E, self.BLOCK)
-        return self._run(ids, positions, cache_locs, bs * E, work, rows if E == 1 else None, E)
-
-    def forward_plan(self, plan: RaggedPlan) -> torch.Tensor:
-        self.ctx_hint = plan.max_keys
-        return self._run(plan.ids, plan.positions, plan.locs, plan.T, plan.struct, plan.rows if plan.single else None,
-                         plan.longest)
-
-    # ---- head ---------------------------------------------------------------------------
-    def final_hidden(self, rows_idx: torch.Tensor) -> torch.Tensor:
-        return self.xa[rows_idx]
-
-    def project(self, X: torch.Tensor, rows: int, ldx: Optional[int] = None) -> torch.Tensor:
-        """fp32 logits of ``rows`` final rows X (pitch ``ldx``), left in the chain's logits buffer."""
-        W, out = self.m.lm_head, self.logits
-        if self.f32:
-            K.gemm_f32(W, X, out, N=W.shape[0], M=rows, ldx=ldx, pdl=self.pdl)
-        else:
-            K.gemm_skinny(W, X, out, M=rows, splits=1, epi=K.EPI_STORE_F32, ldx=ldx, ldo=out.stride(0), status=self.status,
-                          pdl=self.pdl)
-        return out
-
-    def lm_head(self, rows: int, row_offset: int = 0, row_step: int = 1) -> torch.Tensor:
-        return self.project(self.xa[row_offset:], rows, self.d8 * row_step)
-
-    def lm_head_sample(self, rows: int, row_offset: int, row_step: int, *, temperature: float, alpha: float, tokens_in, seed: int,
-                       cycle_counter, call_id: int, tok_out, logp_out, logz_out) -> None:
-        V = self.c.vocab_size
-        if self._lm_parts is None or self._lm_parts.numel() < K.lm_parts_bytes(rows, V):
-            self._lm_parts = torch.empty(K.lm_parts_bytes(max(rows, self.logits.shape[0]), V), dtype=torch.uint8, device=self.dev)
-        K.lm_head_sample(self.m.lm_head, self.xa[row_offset:], M=rows, V=V, ldx=self.d8 * row_step, status=self.status,
-                         temperature=temperature, alpha=alpha, softcap=0.0, tokens_in=tokens_in, seed=seed,
-                         cycle_counter=cycle_counter, call_id=call_id, parts=self._lm_parts, tok_out=tok_out, logp_out=logp_out,
-                         logz_out=logz_out, pdl=self.pdl)

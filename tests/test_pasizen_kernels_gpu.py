@@ -120,7 +120,7 @@ def test_expert_products_and_weighted_sum(f32, T, top, E, d, ff):
     if f32:
         g32 = torch.zeros(n, 2 * ff, device=DEV)
         K.gemm_f32(gu, xe, g32, N=2 * ff, M=n, link=link)
-        K.clamped_glu_f32(g32, ea, ff=ff, blk=64, limit=0.8, slope=GLU_SIGMOID_SLOPE, M=n)
+        K.gated_unit_f32(g32, ea, ff=ff, blk=64, limit=0.8, slope=GLU_SIGMOID_SLOPE, shift=1.0, M=n)
         K.gemm_f32(down, ea, ye, N=d, M=n, link=link2)
     else:
         K.gemm_grouped(gu, xe, ea, N=2 * ff, M=n, splits=1, epi=K.EPI_SWIGLU_BF16, link=link, status=st)
