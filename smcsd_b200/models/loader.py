@@ -69,7 +69,7 @@ def save_safetensors(tensors: Dict[str, torch.Tensor], path: str, metadata: Opti
     blobs = []
     for name, t in tensors.items():
         t = t.detach().contiguous().cpu()
-        raw = t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _DTYPE_NAMES[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + len(raw)]}
         off += len(raw)
         blobs.append(raw)

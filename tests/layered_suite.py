@@ -1,11 +1,14 @@
-"""Checks of a Pasizen engine against the float64 oracle, shared by the CPU and the GPU tests.  ``ctx`` supplies the device,
-the dtype, the tolerance and the share of rows that may exceed it (bf16 expert choices can fall the other way)."""
+"""Checks of a layer-by-layer family's engine against its float64 oracle, shared by the CPU and the GPU tests of all such
+families.  ``ctx`` supplies the family (its oracle and its test models), the device, the dtype, the tolerance and the share of
+rows that may exceed it (bf16 expert choices can fall the other way)."""
 from dataclasses import dataclass
+from typing import Any
 
 import torch
 
-import pasizen_oracle as O
-from pasizen_models import far_effect, row_error, save_model, tokens
+import pasizen_models
+import pasizen_oracle
+from pasizen_models import far_effect, row_error, tokens
 
 
 @dataclass
@@ -14,13 +17,15 @@ class Ctx:
     dtype: str
     tol: float
     slack: float = 0.0                    # share of rows allowed beyond tol
+    models: Any = pasizen_models
+    oracle: Any = pasizen_oracle
 
 
 def engine(ctx, folder, max_tokens=2000, **kw):
     from smcsd_b200 import SMCEngine
     from smcsd_b200.models import resolve_config
     base = dict(n_particles=1, gamma=1, dtype=ctx.dtype, device=ctx.device, max_running_requests=4, max_total_tokens=max_tokens,
-                context_length=resolve_config(folder).max_position, skip_tokenizer_init=True, in_process=True)
+                context_length=min(resolve_config(folder).max_position, 4096), skip_tokenizer_init=True, in_process=True)
     base.update(kw)
     return SMCEngine(folder, base.pop("draft", folder), **base)
 
@@ -50,11 +55,11 @@ def feed_in_cuts(eng, rid, ids, cuts):
 
 def whole_portions_and_decoding(ctx, tmp_path, name):
     """One sequence whole, in portions of several sizes (two tokens at the least), and token by token."""
-    folder, cfg, W = save_model(tmp_path / name, name)
+    folder, cfg, W = ctx.models.save_model(tmp_path / name, name)
     ids = tokens(cfg, 150)
-    ref = O.forward(cfg, W, ids)
+    ref = ctx.oracle.forward(cfg, W, ids)
     eng = engine(ctx, folder)
-    effect = far_effect(lambda x: O.forward(cfg, W, x), cfg, ids, ref)
+    effect = far_effect(lambda x: ctx.oracle.forward(cfg, W, x), cfg, ids, ref)
     assert effect > 0.05
     for cuts in ([150], [2, 3, 64, 65, 16], [63, 2, 64, 21], [1] * 20 + [2] * 20 + [90], [118] + [1] * 32):
         got = feed_in_cuts(eng, "a", ids, cuts)
@@ -68,12 +73,12 @@ def whole_portions_and_decoding(ctx, tmp_path, name):
 def mixed_batches(ctx, tmp_path, name):
     """Unequal requests in one batch, each as if alone; sequences pause; rows and pages are freed and used again in a pool
     that holds one generation of requests only."""
-    folder, cfg, W = save_model(tmp_path / name, name, seed=3)
+    folder, cfg, W = ctx.models.save_model(tmp_path / name, name, seed=3)
     lens = {"a": 130, "b": 40, "c": 70, "d": 5}
     eng = engine(ctx, folder, max_tokens=sum(lens.values()) + 3)
     for gen in range(3):
         ids = {k: tokens(cfg, n, seed=10 * gen + i) for i, (k, n) in enumerate(lens.items())}
-        ref = {k: O.forward(cfg, W, v) for k, v in ids.items()}
+        ref = {k: ctx.oracle.forward(cfg, W, v) for k, v in ids.items()}
         at, got = {k: 0 for k in ids}, {k: [] for k in ids}
         plan = [{"a": 64, "b": 1}, {"b": 2, "c": 66}, {"a": 1, "b": 30, "c": 1, "d": 3}, {"a": 62, "d": 1}, {"a": 1, "b": 5, "c": 1, "d": 1},
                 {"a": 2, "b": 2, "c": 2}]
@@ -93,7 +98,7 @@ def mixed_batches(ctx, tmp_path, name):
 
 def long_decoding(ctx, tmp_path, name, n=330):
     """Hundreds of single-token steps behind a short prompt, three sequences at once at different lengths."""
-    folder, cfg, W = save_model(tmp_path / name, name, seed=5)
+    folder, cfg, W = ctx.models.save_model(tmp_path / name, name, seed=5)
     seqs = {k: tokens(cfg, n + i, seed=20 + i) for i, k in enumerate("xyz")}
     eng = engine(ctx, folder)
     got = {k: [] for k in seqs}
@@ -105,7 +110,7 @@ def long_decoding(ctx, tmp_path, name, n=330):
         for i, k in enumerate(seqs):
             got[k].append(out[i:i + 1])
     for i, k in enumerate(seqs):
-        check(ctx, torch.cat(got[k]), O.forward(cfg, W, seqs[k])[1 + i:], (name, k))
+        check(ctx, torch.cat(got[k]), ctx.oracle.forward(cfg, W, seqs[k])[1 + i:], (name, k))
     eng.feed([], list(seqs))
     idle(eng)
 
@@ -113,7 +118,7 @@ def long_decoding(ctx, tmp_path, name, n=330):
 def greedy_generation(ctx, tmp_path, name, gammas=(1, 3), **kw):
     """Greedy output of ``generate``: every token is the oracle's argmax given the tokens before it, or within the tolerance
     of it.  The proposal is the model itself at temperature 0, so the text is the target's own greedy text."""
-    folder, cfg, W = save_model(tmp_path / name, name, seed=7)
+    folder, cfg, W = ctx.models.save_model(tmp_path / name, name, seed=7)
     prompts = [tokens(cfg, n, seed=40 + n) for n in (1, 9, 70)]
     outs = {}
     for gamma in gammas:
@@ -123,9 +128,32 @@ def greedy_generation(ctx, tmp_path, name, gammas=(1, 3), **kw):
             for p, r in zip(prompts, res):
                 ids = r["output_ids"]
                 assert len(ids) == 21
-                lg = O.forward(cfg, W, p + ids[:-1])[len(p) - 1:]
+                lg = ctx.oracle.forward(cfg, W, p + ids[:-1])[len(p) - 1:]
                 gap = (lg.max(-1).values - lg.gather(1, torch.tensor(ids).unsqueeze(1))[:, 0]) / lg.std()
                 assert (gap <= 4 * ctx.tol).float().mean() >= 1 - ctx.slack, (name, gamma, defer, gap.max().item())
             outs[gamma, defer] = [r["output_ids"] for r in res]
             idle(eng)
     return outs
+
+
+def chunk_edges(ctx, tmp_path, cfg, size, n):
+    """One attention layer alone: a changed token moves exactly the rows of its own chunk behind it, whether they come with
+    the prompt or are decoded, and the first rows of every chunk (few keys beside the sink) are right."""
+    folder, cfg, W = ctx.models.save_model(tmp_path / "edges", cfg, seed=4)
+    eng = engine(ctx, folder)
+    ids = tokens(cfg, n, seed=6)
+    ref = ctx.oracle.forward(cfg, W, ids)
+    base = feed_in_cuts(eng, "a", ids, [n])
+    check(ctx, base, ref)
+    for j in (0, size - 2, size - 1, size, 2 * size - 1, 2 * size):
+        other = list(ids)
+        other[j] = (ids[j] + 1) % cfg["vocab"]
+        lo, hi = j, min(n, (j // size + 1) * size)
+        for cuts in ([n], [j + 1] + [1] * (n - j - 1), [max(j - 1, 1), n - max(j - 1, 1)]):
+            got = feed_in_cuts(eng, "b", other, cuts)
+            e = row_error(got, base)
+            out = torch.cat([e[:lo], e[hi:]])
+            assert out.max() <= ctx.tol, (j, cuts[:3], out.max().item())
+            assert e[lo:hi].min() > 0 and e[lo] > 0.05
+            check(ctx, got, ctx.oracle.forward(cfg, W, other), (j, cuts[:3]))
+    idle(eng)

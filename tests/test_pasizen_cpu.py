@@ -8,8 +8,8 @@ import numpy as np
 import pytest
 import torch
 
+import layered_suite as S
 import pasizen_oracle as O
-import pasizen_suite as S
 from pasizen_models import CONFIGS, config, dense, make_weights, mixer, moe, row_error, save_model, tokens
 
 CTX = S.Ctx("cpu", "float32", 2e-5)

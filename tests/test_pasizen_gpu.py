@@ -2,8 +2,8 @@
 import pytest
 import torch
 
+import layered_suite as S
 import pasizen_oracle as O
-import pasizen_suite as S
 from pasizen_models import CONFIGS, config, dense, far_effect, mixer, moe, row_error, save_model, tokens
 
 pytestmark = pytest.mark.gpu
