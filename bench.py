@@ -17,7 +17,8 @@ cycle with forced cross-GPU resampling, reported under ``fused``.
     python -m torch.distributed.run --nnodes=1 --nproc-per-node 8 --master-addr 127.0.0.1 \
         --master-port 29511 bench.py --gpus 8 --steps 40 --warmup 5
     python bench.py --impl reference        # prints why the reference cannot run here
-    python bench.py --layered 2048,1024     # another workload: Pasizen beside a dense model of equal size, kernel by kernel
+    python bench.py --layered 2048,1024     # another workload: Pasizen (--layered-family makodra: Makodra) beside models of
+                                            # equal size, kernel by kernel
 """
 from __future__ import annotations
 
@@ -115,7 +116,7 @@ def _run_fused_children(rank: int, steps: int, warm: int, dry_run: bool = False,
 
 
 def layered_arm(args) -> int:
-    """Prefill and decode of Pasizen beside the dense family at the given widths (random weights); the kernel tables go to
+    """Prefill and decode of a layer-by-layer family beside the existing ones at the given widths (random weights); the kernel tables go to
     stderr, the whole record is the JSON line."""
     import torch
 
@@ -124,12 +125,13 @@ def layered_arm(args) -> int:
     from smcsd_b200.utils.profiling import ClockSampler
     torch.cuda.set_device(0)
     sampler, l0 = ClockSampler(0).start(), K.launch_count
-    recs = [layered.run(int(w), ctx=args.layered_ctx) for w in args.layered.split(",")]
+    recs = [layered.run(int(w), ctx=args.layered_ctx, family=args.layered_family) for w in args.layered.split(",")]
     for r in recs:
         print(layered.show(r), file=sys.stderr)
     pick = {m["model"]: m for r in recs for m in r["models"]}
-    main_model = pick[f"pasizen-{args.layered.split(',')[0]}-dense"]
-    print(json.dumps({"metric": "decode tokens/s (Pasizen layers, random weights)", "value": main_model["decode_tok_s"],
+    tail = {"pasizen": "dense", "makodra": "heads64"}[args.layered_family]
+    main_model = pick[f"{args.layered_family}-{args.layered.split(',')[0]}-{tail}"]
+    print(json.dumps({"metric": f"decode tokens/s ({args.layered_family.capitalize()} layers, random weights)", "value": main_model["decode_tok_s"],
                       "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
                       "timing": "CUDA events around graph replays; the weights of all layers exceed L2", "records": recs,
                       "clocks": sampler.stop(), "gpu_launches": K.launch_count - l0}))
@@ -162,7 +164,8 @@ def main() -> int:
     ap.add_argument("--no-fp8", action="store_true",
                     help="skip the extra W8A8 (e4m3) measurement reported under the 'fp8' key (one GPU only)")
     ap.add_argument("--layered", default=None, metavar="WIDTHS",
-                    help="run the layer comparison of Pasizen and the dense family at these widths instead of the headline")
+                    help="run the layer comparison of a layer-by-layer family at these widths instead of the headline")
+    ap.add_argument("--layered-family", default="pasizen", choices=["pasizen", "makodra"], help="the family --layered compares")
     ap.add_argument("--layered-ctx", type=int, default=1024, help="cached tokens per sequence of the layer comparison's decode step")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -1,13 +1,15 @@
-"""Prefill and decode of Pasizen beside a dense Llama-style model of equal size, whole forwards and kernel by kernel.
+"""Prefill and decode of a layer-by-layer family beside existing models of equal size, whole forwards and kernel by kernel.
 
-    python -m smcsd_b200.bench.layered --width 2048            (or: python bench.py --layered 2048,1024)
+    python -m smcsd_b200.bench.layered --width 2048 --family makodra
+    (or: python bench.py --layered 2048,1024 --layered-family makodra)
 
-Both models run random weights through their kernel chains: the same width, heads, layer count, head and feed-forward
-weights per layer; the dense model caches as many bytes per token as its KV heads take.  A forward is captured in a CUDA
+Pasizen runs beside a dense Llama-style model, Makodra beside that and a Gated-DeltaNet hybrid with as many attention layers.
+All run random weights through their kernel chains: the same width, heads, layer count, head and feed-forward weights per
+layer; the dense models cache as many bytes per token as their KV heads take.  A forward is captured in a CUDA
 graph and timed with CUDA events (weights of all layers exceed L2; the cached keys come on top).  For the kernel table every
 launch of one forward is recorded and the launches of one kind - the same kernel in all layers, so that the weights rotate -
 are captured and timed together.  Fraction = (the larger of bytes / measured copy bandwidth and FLOPs / measured bf16 rate)
-/ measured time.
+/ measured time; recurrent memories held to fp32 are set against the CUDA cores' fp32 rate instead.
 """
 from __future__ import annotations
 
@@ -19,10 +21,12 @@ from typing import Dict, List, Tuple
 
 import torch
 
-from ..models.config import FeedForwardSpec, GluSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RouterSpec
+from ..models.config import (ChunkAttentionSpec, FeedForwardSpec, GluSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RecurrentSpec,
+                             RouterSpec)
 from ..utils.roofline import measured_peaks
 
 VOCAB = 32768
+F32_TFLOPS = 148 * 128 * 2 * 1.965e-3        # CUDA cores at the highest clock
 
 
 def pasizen_config(width: int, layers: int, kv_rank: int, experts: bool) -> ModelConfig:
@@ -42,6 +46,26 @@ def dense_config(width: int, layers: int) -> ModelConfig:
                        name=f"llama-{width}")
 
 
+def hybrid_config(width: int, layers: int) -> ModelConfig:
+    """Two Gated-DeltaNet layers to one attention layer, the feed-forward of ``makodra_config``."""
+    H = width // 128
+    return ModelConfig(arch="hybrid_gdn", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=H, n_kv_heads=max(1, width // 512),
+                       head_dim=128, ffn_size=2 * width, rms_eps=1e-6, max_position=8192, layer_types=["linear_attention", "linear_attention",
+                       "full_attention"] * (layers // 3), gdn_n_k_heads=H, gdn_n_v_heads=H, gdn_head_k_dim=128, gdn_head_v_dim=128,
+                       gdn_conv_width=4, partial_rotary=0.25, attn_output_gate=True, qk_norm=True, norm_plus_one=True,
+                       name=f"hybrid-gdn-{width}")
+
+
+def makodra_config(width: int, layers: int, memory_dim: int = 64, chunk: int = 8192) -> ModelConfig:
+    """Delta rule, wkv and attention in turn; the chunk holds every sequence of the comparison, so that all keys are seen."""
+    mlp, H = FeedForwardSpec("swiglu", ff=2 * width), width // memory_dim
+    trio = [LayerSpec(RecurrentSpec("general_delta", H, memory_dim), mlp), LayerSpec(RecurrentSpec("wkv", H, memory_dim), mlp),
+            LayerSpec(ChunkAttentionSpec(width // 128, max(1, width // 512), 128, 128, 11.3, chunk, True), mlp)]
+    return ModelConfig(arch="makodra", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=H, n_kv_heads=H, head_dim=memory_dim,
+                       ffn_size=0, rms_eps=1e-6, max_position=1 << 20, tie_embeddings=True, logit_softcap=30.0, layers=trio * (layers // 3),
+                       name=f"makodra-{width}-heads{memory_dim}")
+
+
 class Rig:
     """One model with its chain, caches filled with noise, and step inputs."""
 
@@ -49,6 +73,8 @@ class Rig:
         from ..memory.pools import KVPool, StatePool
         from ..models import build_model
         from ..ops.native_backend import NativeLlama
+        from ..ops.native_hybrid import NativeHybrid
+        from ..ops.native_makodra import NativeMakodra
         from ..ops.native_pasizen import NativePasizen
         dev = self.dev = torch.device("cuda", 0)
         self.cfg, self.bs, self.ctx, self.prompt, self.n_prompts = cfg, bs, ctx, prompt, n_prompts
@@ -62,10 +88,10 @@ class Rig:
         self.bt = perm.view(rows, span).to(dev).contiguous()               # scattered pages: the worst case for both
         self.status = torch.zeros(1, dtype=torch.int32, device=dev)
         T = n_prompts * prompt
-        if cfg.arch == "pasizen":
-            spec = m.state_spec()
-            self.state = StatePool(spec, rows, dev)
-            make = lambda t, lr: NativePasizen(m, kv, self.bt, t, lr, 16, self.status, True, state=self.state)
+        if cfg.arch != "llama":
+            self.state = StatePool(m.state_spec(), rows, dev)
+            Chain = {"pasizen": NativePasizen, "makodra": NativeMakodra, "hybrid_gdn": NativeHybrid}[cfg.arch]
+            make = lambda t, lr: Chain(m, kv, self.bt, t, lr, 16, self.status, True, state=self.state)
         else:
             make = lambda t, lr: NativeLlama(m, kv, self.bt, t, lr, 16, self.status, True)
         self.dec, self.pre = make(bs, bs), make(T, 8)
@@ -76,7 +102,8 @@ class Rig:
         self.locs = self.bt[:bs, ctx].contiguous()
         self.p_ids = torch.randint(0, VOCAB, (T,), generator=g).tolist()
         self.dec.set_context(ctx + 1, bs, (1,))
-        if cfg.arch == "pasizen":
+        self.ragged = getattr(self.pre, "ragged", False)
+        if self.ragged:
             from ..ops.ragged import Portion, pack_ragged
             portions = [Portion(r, 0, self.p_ids[r * prompt:(r + 1) * prompt]) for r in range(n_prompts)]
             self.plan = next(pack_ragged(portions, T, self.pre.BLOCK, self.bt))
@@ -86,15 +113,18 @@ class Rig:
             self.p_args = (i32(self.p_ids), i32(list(range(prompt)) * n_prompts), self.bt[:n_prompts, :prompt].reshape(-1).contiguous(),
                            i32([r for r in range(n_prompts) for _ in range(nb)]), i32([j * B for _ in range(n_prompts) for j in range(nb)]))
             self.pre.set_context(prompt, n_prompts * nb)
+            self.seqs = {} if cfg.arch == "llama" else {"seqs": {
+                "rows": i32(list(range(n_prompts))), "off": i32([r * prompt for r in range(n_prompts)]), "len": i32([prompt] * n_prompts),
+                "n": n_prompts, "max": prompt}}
 
     def decode(self) -> None:
         self.dec.forward(self.ids, self.pos, self.locs, self.rows, self.pref, self.bs, 1)
 
     def prefill(self) -> None:
-        if self.cfg.arch == "pasizen":
+        if self.ragged:
             self.pre.forward_plan(self.plan)
         else:
-            self.pre.forward(*self.p_args, self.n_prompts * self.prompt // 16, 16, two_pass=True)
+            self.pre.forward(*self.p_args, self.n_prompts * self.prompt // 16, 16, two_pass=True, **self.seqs)
 
 
 def timed(fn, reps: int = 20) -> float:
@@ -122,7 +152,9 @@ def timed(fn, reps: int = 20) -> float:
 
 # ---------------------------------------------------------------------------------- kernel by kernel
 RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
-            "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc")
+            "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc", "gdn_step",
+            "rope_kv_write_heads", "post_norm_step", "token_shift", "heads_new", "chunk_attention", "chunk_attention_tc", "memory_scan",
+            "tanh_rows")
 
 
 def record(fn) -> List[Tuple[str, tuple, dict]]:
@@ -173,12 +205,37 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
         H, Hkv, D = kw["Hq"], kw["Hkv"], kw["D"]
         fl = 2.0 * 2 * T * H * keys * D
         return "attention", T * H * D * 6 + seqs * (rig.ctx if T == rig.bs else rig.prompt) * Hkv * D * 4, fl
+    if name in ("chunk_attention", "chunk_attention_tc"):
+        s = a[0]
+        fl = 2.0 * T * s.H * keys * (s.D + s.V)
+        return "attention", T * s.H * (2 * s.D + 6 * s.V) + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.G * (s.D + s.V) * 2, fl
+    if name == "memory_scan":
+        s, is_delta = a[0], a[1]
+        HD = s.H * s.D
+        # fp32 multiply-adds per matrix element and token, as bf16-rate equivalents (the floor divides by the bf16 rate)
+        fl = 2.0 * (5 if is_delta else 3) * T * HD * s.D * measured_peaks()[1] / F32_TFLOPS
+        return "memory " + ("delta" if is_delta else "wkv"), T * HD * (4 * (6 if is_delta else 5) + 2) + seqs * HD * s.D * 8, fl
+    if name == "gdn_step":
+        Hv, dk, dv = kw["Hv"], kw["dk"], kw["dv"]
+        conv = 2 * kw["Hk"] * dk + Hv * dv
+        return "memory gdn + conv", T * (conv * 12 + Hv * dv * 6) + seqs * Hv * dk * dv * 8, 2.0 * 4 * T * Hv * dk * dv
+    if name == "post_norm_step":
+        s = a[0]
+        return "norm + residual" + (" + shift" if s.mu else ""), T * d * (4 + 8 + (2 if s.xa else 0) + (8 + 2 * s.n_mix if s.mu else 0)), 0.0
+    if name == "token_shift":
+        return "token shift", T * d * (4 + 2 * a[1].shape[0]), 0.0
+    if name == "heads_new":
+        s = a[0]
+        return "new heads", T * ((s.H + s.G) * s.D * 6 + s.G * s.V * (6 + 4 * bool(s.v_first))), 0.0
+    if name == "tanh_rows":
+        return "tanh", T * kw["n"] * 6, 0.0
     if name == "hyper_step":
         s = a[0]
         S = s.S
         by = T * d * (4 * S * (1 + (s.w_in is not None)) + 4 * (s.y is not None) + 4 * s.top + 4 * (s.n_out is not None) + 2 * (s.xa is not None))
         return "streams + norm" + (" + conv" if s.conv_w else "") + (" + experts" if s.top else ""), by, 0.0
-    sizes = {"add_rmsnorm": T * d * 10, "short_conv": T * d * 6, "rope_kv_write": T * (cfg.q_size + 2 * cfg.kv_size) * 6}
+    sizes = {"add_rmsnorm": T * d * 10, "short_conv": T * d * 6, "rope_kv_write": T * (cfg.q_size + 2 * cfg.kv_size) * 6,
+             "rope_kv_write_heads": T * (cfg.q_size + 2 * cfg.kv_size) * 6}
     if name == "poly_norm":
         return "PolyNorm", T * kw["ff"] * 6, 0.0
     if name == "latent_new":
@@ -210,11 +267,13 @@ def kernel_table(rig: Rig, fn, T: int, keys: float, seqs: int) -> List[dict]:
 
 
 def run(width: int, layers: int = 12, bs: int = 8, ctx: int = 1024, prompt: int = 1024, n_prompts: int = 4, kv_rank: int = 256,
-        tables: bool = True) -> dict:
+        tables: bool = True, family: str = "pasizen") -> dict:
     import gc
     rec = {"width": width, "layers": layers, "decode": {"sequences": bs, "context": ctx}, "prefill": {"prompts": n_prompts, "tokens": prompt},
-           "kv_rank": kv_rank, "pages": "scattered", "weights": "random, bf16", "models": []}
-    for cfg in (dense_config(width, layers), pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)):
+           "kv_rank": kv_rank if family == "pasizen" else None, "pages": "scattered", "weights": "random, bf16", "models": []}
+    own = [pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)] if family == "pasizen" else \
+        [hybrid_config(width, layers), makodra_config(width, layers), makodra_config(width, layers, 128)]
+    for cfg in [dense_config(width, layers)] + own:
         rig = Rig(cfg, bs, ctx, prompt, n_prompts)
         T = n_prompts * prompt
         dec, pre = timed(rig.decode), timed(rig.prefill, reps=8)
@@ -232,7 +291,7 @@ def run(width: int, layers: int = 12, bs: int = 8, ctx: int = 1024, prompt: int 
 
 
 def show(rec: dict) -> str:
-    lines = [f"width {rec['width']}, {rec['layers']} layers, kv_rank {rec['kv_rank']}; decode {rec['decode']}, prefill {rec['prefill']}, "
+    lines = [f"width {rec['width']}, {rec['layers']} layers{', kv_rank ' + str(rec['kv_rank']) if rec['kv_rank'] else ''}; decode {rec['decode']}, prefill {rec['prefill']}, "
              f"pages {rec['pages']}"]
     for m in rec["models"]:
         lines.append(f"{m['model']}: {m['weight_mb']:.0f} MB  decode {m['decode_us']} us ({m['decode_tok_s']} tok/s)  prefill "
@@ -251,10 +310,11 @@ def main(argv=None) -> None:
     ap.add_argument("--ctx", type=int, default=1024)
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--kv-rank", type=int, default=256)
+    ap.add_argument("--family", default="pasizen", choices=["pasizen", "makodra"])
     ap.add_argument("--no-tables", action="store_true")
     ap.add_argument("--json", default=None)
     ns = ap.parse_args(argv)
-    rec = run(ns.width, ns.layers, ns.bs, ns.ctx, ns.prompt, kv_rank=ns.kv_rank, tables=not ns.no_tables)
+    rec = run(ns.width, ns.layers, ns.bs, ns.ctx, ns.prompt, kv_rank=ns.kv_rank, tables=not ns.no_tables, family=ns.family)
     print(show(rec))
     if ns.json:
         with open(ns.json, "w") as f:

@@ -78,11 +78,13 @@ def make_weights(cfg, seed=0, gain=1.5):
     return {k: v.to(torch.bfloat16) for k, v in W.items()}
 
 
-def save_model(path, name, seed=0):
-    """Writes config.json and model.safetensors; returns (folder, configuration, weights)."""
+def save_model(path, name, seed=0, **changed):
+    """Writes config.json and model.safetensors; returns (folder, configuration, weights).  ``changed`` multiplies all weights
+    with a leaf name by a factor."""
     from smcsd_b200.models.loader import save_safetensors
     cfg = CONFIGS[name] if isinstance(name, str) else name
     W = make_weights(cfg, seed)
+    W = {k: w * changed.get(k.rsplit(".", 1)[-1], 1.0) for k, w in W.items()}
     os.makedirs(path, exist_ok=True)
     with open(os.path.join(path, "config.json"), "w") as f:
         json.dump(cfg, f)
