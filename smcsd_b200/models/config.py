@@ -408,10 +408,11 @@ def preset(name: str) -> ModelConfig:
                            layers=trio * 5, name=n)
     if n in ("tiny-makodra",):
         mlp = FeedForwardSpec("swiglu", ff=200)
-        return ModelConfig(arch="makodra", vocab_size=4096, hidden_size=136, n_layers=3, n_heads=3, n_kv_heads=3, head_dim=40,
+        return ModelConfig(arch="makodra", vocab_size=4096, hidden_size=136, n_layers=4, n_heads=3, n_kv_heads=3, head_dim=40,
                            ffn_size=0, rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, tie_embeddings=True, logit_softcap=20.0,
                            layers=[LayerSpec(RecurrentSpec("wkv", 3, 40), mlp), LayerSpec(ChunkAttentionSpec(4, 2, 24, 40, 3.0, 48, True), None),
-                                   LayerSpec(RecurrentSpec("general_delta", 5, 32), mlp)], name="tiny-makodra")
+                                   LayerSpec(RecurrentSpec("general_delta", 5, 32), mlp),
+                                   LayerSpec(ChunkAttentionSpec(2, 2, 48, 40, 2.0, 80, True), mlp)], name="tiny-makodra")
     raise KeyError(f"unknown preset {name!r}")
 
 

@@ -156,7 +156,7 @@ class MakodraModel(LayeredModel):
         rank = 64 if self.cfg.hidden_size >= 1024 else 16
 
         def get(name, *shape):
-            r = torch.randn(*(rank if n is None else n for n in shape), generator=g, device=self.device, dtype=torch.float32)
+            r = torch.randn([rank if n is None else n for n in shape], generator=g, device=self.device, dtype=torch.float32)
             leaf = name.rsplit(".", 1)[-1]
             if leaf.startswith("norm"):
                 return 1.0 + 0.1 * r

@@ -86,7 +86,7 @@ def test_many_heads_take_one_cta_each(tmp_path):
 
 def test_long_chunk_far_key(tmp_path):
     """A chunk of two thousand positions: the first key still decides the last row, with the prompt and decoded."""
-    cfg = config(96, [(attn(4, 2, 32, 32, 2100, scale=1.0), None)])
+    cfg = config(96, [(attn(4, 2, 32, 32, 2100, scale=0.7), None)])
     folder, cfg, W = save_model(tmp_path / "long", cfg, seed=2, r1=0.1)
     ids = tokens(cfg, 2060)
     ref = O.forward(cfg, W, ids)
