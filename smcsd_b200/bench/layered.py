@@ -154,7 +154,7 @@ def timed(fn, reps: int = 20) -> float:
 RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
             "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc", "gdn_step",
             "rope_kv_write_heads", "post_norm_step", "token_shift", "heads_new", "chunk_attention", "chunk_attention_tc", "memory_scan",
-            "tanh_rows")
+            "tanh_rows", "low_rank")
 
 
 def record(fn) -> List[Tuple[str, tuple, dict]]:
@@ -227,6 +227,9 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
     if name == "heads_new":
         s = a[0]
         return "new heads", T * ((s.H + s.G) * s.D * 6 + s.G * s.V * (6 + 4 * bool(s.v_first))), 0.0
+    if name == "low_rank":
+        W = a[1]
+        return "decay logits", W.numel() * 2 + T * (W.shape[0] + W.shape[1]) * 4, 2.0 * T * W.numel()
     if name == "tanh_rows":
         return "tanh", T * kw["n"] * 6, 0.0
     if name == "hyper_step":

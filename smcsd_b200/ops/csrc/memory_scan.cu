@@ -6,19 +6,21 @@
 //           w = exp(-exp(z + w0)); output gate silu
 //
 // Value columns of a matrix never mix, key rows only in sums.  A CTA therefore keeps some columns of one head's matrix in
-// registers - four threads per column, a quarter of the key rows each - and walks its sequence's tokens in tiles: consumer
-// warps run the recurrence on the tile in shared memory while four producer warps turn the next tile's projections into
-// w, u, a u, ... and finish the outputs of the tile before (division by the head's root mean square, norm weight, gate).
-// With few (sequence, head) pairs the columns of a head are spread over a thread-block cluster that exchanges the sums of
-// squares through distributed shared memory.  Both sums over key rows are taken over the old matrix, so that a token costs
-// one reduction: for delta the read-out is (r w)^T M - (r.a u)(u^T M) + (r.k) v.
+// registers - four threads per pair of columns (one column beyond 128 key rows), a quarter of the key rows each - and walks
+// its sequence's tokens in tiles: consumer warps run the recurrence on the tile in shared memory while eight producer warps
+// turn the next tile's projections into w, u, a u, ... and finish the outputs of the tile before (division by the head's root
+// mean square, norm weight, gate).  Producers fetch a tile ahead of the one they prepare, so a tile's loads have a whole tile
+// of consumer work to land in.  With few (sequence, head) pairs the columns of a head are spread over a thread-block cluster
+// that exchanges the sums of squares through distributed shared memory.  Both sums over key rows are taken over the old
+// matrix, so that a token costs one reduction: for delta the read-out is (r w)^T M - (r.a u)(u^T M) + (r.k) v.
 // The recurrence is held to fp32 (a bf16 or tf32 chunk-parallel form would round the state), so the floor is the CUDA cores'
 // rate; products and sums are issued two at a time (f32x2).
 #include "ragged.cuh"
 
 namespace smc {
 
-constexpr int SCAN_PRODUCERS = 4;        // warps
+constexpr int SCAN_PRODUCERS = 8;        // warps
+constexpr int SCAN_CONSUMERS = 256;      // threads at the most
 
 struct ScanArgs {
   const float* proj;        // [T, ldp]: H * D columns each of r, k, v, gate (and removal rate) at these offsets
@@ -61,20 +63,28 @@ __device__ __forceinline__ f2_t mul2(f2_t a, f2_t b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
+// A store the compiler may move loads across: nobody reads the word before the next barrier.
+__device__ __forceinline__ void store_shared_unordered(uint32_t addr, float v) {
+  asm volatile("st.shared.f32 [%0], %1;" ::"r"(addr), "f"(v));
+}
 __device__ __forceinline__ float sum_of(f2_t a) { const float2 v = unpack2(a); return v.x + v.y; }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 __host__ __device__ constexpr int scan_tokens(int dkp) { return dkp <= 128 ? 16 : 8; }       // tokens of a tile
 __host__ __device__ constexpr int scan_vectors(bool delta) { return delta ? 5 : 3; }
+__host__ __device__ constexpr int scan_columns(int dkp) { return dkp <= 128 ? 2 : 1; }       // of a consumer thread
+__host__ __device__ constexpr int scan_max_columns(int dkp) { return SCAN_CONSUMERS / 4 * scan_columns(dkp); }      // of a CTA
 
 template <bool DELTA, int DKP>
-__global__ void __launch_bounds__(640) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA), NL = (DKP + 31) / 32, NQ = DKP / 16;
+__global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA), NL = (DKP + 31) / 32, NQ = DKP / 16, CP = scan_columns(DKP);
+  constexpr int PT = TB / SCAN_PRODUCERS;                    // tokens of a tile per producer warp
+  constexpr int NC = ((scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;       // columns of a CTA per lane
   extern __shared__ __align__(16) float scan_smem[];
   const int buf_floats = TB * (NVEC * DKP + CC + 2);
   float* obuf = scan_smem + 2 * buf_floats;                  // [3][TB][CC]
   float* ssq = obuf + 3 * TB * CC;                           // [2][TB]
-  const int n_cons = CC * 4, tid = threadIdx.x, lane = tid & 31;
+  const int n_cons = CC / CP * 4, tid = threadIdx.x, lane = tid & 31;
   const bool consumer = tid < n_cons;
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int h = blockIdx.x / CS, rank = blockIdx.x - h * CS, s = blockIdx.y, D = a.D;
@@ -89,192 +99,283 @@ __global__ void __launch_bounds__(640) scan_kernel(const ScanArgs a, int CC, int
     if (CS > 1) cluster_sync(); else __syncthreads();
   };
   const int n_tiles = (len + TB - 1) / TB, c0 = rank * CC;
+  const int last = CS > 1 ? n_tiles + 1 : n_tiles;
 
-  // ---- producers: one warp per token
-  const int pw = (tid - n_cons) >> 5;
-  auto stage = [&](int tile) {
-    float* buf = scan_smem + (tile & 1) * buf_floats;
-    float* val = buf + TB * NVEC * DKP;
-    float* scal = val + TB * CC;
-    const int n = min(TB, len - tile * TB);
-    for (int tb = pw; tb < n; tb += SCAN_PRODUCERS) {
-      const size_t t = (size_t)off + tile * TB + tb;
-      const float* p = a.proj + t * a.ldp + h * D;
-      const float* zr = a.z + t * a.ldz + h * D;
-      float kk[NL], rr[NL], zz[NL], aa[NL], ss = 0.f;
+  if (!consumer) {
+    const int pw = (tid - n_cons) >> 5;
+    float kk[PT][NL], rr[PT][NL], zz[PT][NL], aa[PT][NL], vv[PT][NC], gg[PT][NC];
+    auto fetch = [&](int tile) {                             // projections of a tile into registers
+      const int n = min(TB, len - tile * TB);
 #pragma unroll
-      for (int i = 0; i < NL; ++i) {
-        const int c = lane + 32 * i;
-        const bool ok = c < D;
-        kk[i] = ok ? p[a.k_off + c] : 0.f;
-        rr[i] = ok ? p[a.r_off + c] : 0.f;
-        zz[i] = ok ? zr[c] + a.w0[h * D + c] : 0.f;
-        aa[i] = ok ? (DELTA ? p[a.a_off + c] + a.a_bias[h * D + c] : a.bonus[h * D + c]) : 0.f;
-        ss = fmaf(kk[i], kk[i], ss);
-      }
-      const float inv = DELTA ? 1.0f / sqrtf(warp_sum(ss) + a.unit_eps) : 0.f;
-      float s1 = 0.f, s2 = 0.f;
-      float* d = buf + tb * DKP;
+      for (int j = 0; j < PT; ++j) {
+        const int tb = pw + j * SCAN_PRODUCERS;
+        const size_t t = (size_t)off + tile * TB + tb;
+        const float* p = a.proj + t * a.ldp + h * D;
+        const float* zr = a.z + t * a.ldz + h * D;
 #pragma unroll
-      for (int i = 0; i < NL; ++i) {
-        const int c = lane + 32 * i;
-        if (c >= DKP) continue;
-        const float w = c >= D ? 0.f : DELTA ? expf(-a.log_decay * sigmoid_f(zz[i])) : expf(-expf(zz[i]));
-        d[c] = w;
-        d[TB * DKP + c] = kk[i];
-        if (DELTA) {
-          const float u = kk[i] * inv, au = sigmoid_f(aa[i]) * u;
-          d[2 * TB * DKP + c] = rr[i] * w;
-          d[3 * TB * DKP + c] = u;
-          d[(NVEC - 1) * TB * DKP + c] = au;
-          s1 = fmaf(rr[i], au, s1);
-          s2 = fmaf(rr[i], kk[i], s2);
-        } else {
-          d[2 * TB * DKP + c] = rr[i];
-          s2 = fmaf(rr[i] * aa[i], kk[i], s2);
+        for (int i = 0; i < NL; ++i) {
+          const int c = lane + 32 * i;
+          const bool ok = c < D && tb < n;
+          kk[j][i] = ok ? p[a.k_off + c] : 0.f;
+          rr[j][i] = ok ? p[a.r_off + c] : 0.f;
+          zz[j][i] = ok ? zr[c] : 0.f;
+          if (DELTA) aa[j][i] = ok ? p[a.a_off + c] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const int c = lane + 32 * i;
+          vv[j][i] = c < CC && c0 + c < D && tb < n ? p[a.v_off + c0 + c] : 0.f;
         }
       }
-      for (int c = lane; c < CC; c += 32) val[tb * CC + c] = c0 + c < D ? p[a.v_off + c0 + c] : 0.f;
-      __syncwarp();
-      s1 = DELTA ? warp_sum(s1) : 0.f;
-      s2 = warp_sum(s2);
-      if (lane == 0) { scal[2 * tb] = s1; scal[2 * tb + 1] = s2; }
-    }
-  };
-  auto square = [&](const float* o) {
-    float q = 0.f;
-    for (int c = lane; c < CC; c += 32) q = fmaf(o[c], o[c], q);
-    __syncwarp();
-    return warp_sum(q);                                      // columns beyond D are zero
-  };
-  auto finish = [&](int tile, bool alone) {
-    const int n = min(TB, len - tile * TB);
-    for (int tb = pw; tb < n; tb += SCAN_PRODUCERS) {
-      const size_t t = (size_t)off + tile * TB + tb;
-      const float* o = obuf + ((tile % 3) * TB + tb) * CC;
-      float tot = 0.f;
-      if (alone) {
-        tot = square(o);
-      } else {
-        const uint32_t at = smem_u32(ssq + (tile & 1) * TB + tb);
-        for (int q = 0; q < CS; ++q) tot += ld_dsmem_f32(at, q);
+    };
+    auto stage = [&](int tile) {                             // registers to the consumers' operands
+      float* buf = scan_smem + (tile & 1) * buf_floats;
+      float* val = buf + TB * NVEC * DKP;
+      float* scal = val + TB * CC;
+      const int n = min(TB, len - tile * TB);
+#pragma unroll
+      for (int j = 0; j < PT; ++j) {
+        const int tb = pw + j * SCAN_PRODUCERS;
+        if (tb >= n) continue;
+        float inv = 0.f, s1 = 0.f, s2 = 0.f;
+        if (DELTA) {
+          float ss = 0.f;
+#pragma unroll
+          for (int i = 0; i < NL; ++i) ss = fmaf(kk[j][i], kk[j][i], ss);
+          inv = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
+        }
+        float* d = buf + tb * DKP;
+#pragma unroll
+        for (int i = 0; i < NL; ++i) {
+          const int c = lane + 32 * i;
+          if (c >= DKP) continue;
+          const bool ok = c < D;
+          const float z = ok ? zz[j][i] + a.w0[h * D + c] : 0.f;
+          const float w = !ok ? 0.f : DELTA ? expf(-a.log_decay * sigmoid_f(z)) : expf(-expf(z));
+          d[c] = w;
+          d[TB * DKP + c] = kk[j][i];
+          if (DELTA) {
+            const float u = kk[j][i] * inv, au = ok ? sigmoid_f(aa[j][i] + a.a_bias[h * D + c]) * u : 0.f;
+            d[2 * TB * DKP + c] = rr[j][i] * w;
+            d[3 * TB * DKP + c] = u;
+            d[(NVEC - 1) * TB * DKP + c] = au;
+            s1 = fmaf(rr[j][i], au, s1);
+            s2 = fmaf(rr[j][i], kk[j][i], s2);
+          } else {
+            d[2 * TB * DKP + c] = rr[j][i];
+            s2 = fmaf(rr[j][i] * (ok ? a.bonus[h * D + c] : 0.f), kk[j][i], s2);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < NC; ++i)
+          if (lane + 32 * i < CC) val[tb * CC + lane + 32 * i] = vv[j][i];
+        __syncwarp();
+        s1 = DELTA ? warp_sum(s1) : 0.f;
+        s2 = warp_sum(s2);
+        if (lane == 0) { scal[2 * tb] = s1; scal[2 * tb + 1] = s2; }
       }
-      const float inv = 1.0f / sqrtf(tot / (float)D + a.eps);
-      for (int c = lane; c < CC && c0 + c < D; c += 32) {
-        const int col = h * D + c0 + c;
-        const float g = a.proj[t * a.ldp + a.g_off + col], sg = sigmoid_f(g);
-        const float v = o[c] * inv * a.onorm[col] * (DELTA ? sg : g * sg);
-        if (f32) reinterpret_cast<float*>(a.out)[t * a.ldo + col] = v;
-        else reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + col] = __float2bfloat16(v);
+    };
+    auto gates = [&](int tile) {                             // gate columns of a tile into registers
+      const int n = min(TB, len - tile * TB);
+#pragma unroll
+      for (int j = 0; j < PT; ++j) {
+        const int tb = pw + j * SCAN_PRODUCERS;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const int c = lane + 32 * i;
+          gg[j][i] = c < CC && c0 + c < D && tb < n ? a.proj[((size_t)off + tile * TB + tb) * a.ldp + a.g_off + h * D + c0 + c] : 0.f;
+        }
       }
-      __syncwarp();
+    };
+    auto square = [&](const float* o) {
+      float q = 0.f;
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const float v = lane + 32 * i < CC ? o[lane + 32 * i] : 0.f;       // columns beyond D are zero
+        q = fmaf(v, v, q);
+      }
+      return warp_sum(q);
+    };
+    auto finish = [&](int tile) {
+      const int n = min(TB, len - tile * TB);
+#pragma unroll
+      for (int j = 0; j < PT; ++j) {
+        const int tb = pw + j * SCAN_PRODUCERS;
+        if (tb >= n) continue;
+        const size_t t = (size_t)off + tile * TB + tb;
+        const float* o = obuf + ((tile % 3) * TB + tb) * CC;
+        float tot = 0.f;
+        if (CS == 1) {
+          tot = square(o);
+        } else {
+          const uint32_t at = smem_u32(ssq + (tile & 1) * TB + tb);
+          for (int q = 0; q < CS; ++q) tot += ld_dsmem_f32(at, q);
+        }
+        const float inv = 1.0f / sqrtf(tot / (float)D + a.eps);
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const int c = lane + 32 * i, col = h * D + c0 + c;
+          if (c >= CC || c0 + c >= D) continue;
+          const float g = gg[j][i], sg = sigmoid_f(g);
+          const float v = o[c] * inv * a.onorm[col] * (DELTA ? sg : g * sg);
+          if (f32) reinterpret_cast<float*>(a.out)[t * a.ldo + col] = v;
+          else reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + col] = __float2bfloat16(v);
+        }
+        __syncwarp();
+      }
+    };
+    const int lag = CS > 1 ? 2 : 1;                          // tiles between a tile's recurrence and its outputs
+    if (n_tiles > 0) {
+      fetch(0);
+      stage(0);
+      if (n_tiles > 1) fetch(1);
+      if (lag == 1) gates(0);
     }
-  };
+    barrier();
+    for (int it = 0; it <= last; ++it) {
+      if (it + 1 < n_tiles) stage(it + 1);
+      if (it + 2 < n_tiles) fetch(it + 2);
+      if (CS > 1 && it >= 1 && it - 1 < n_tiles) {
+        const int n = min(TB, len - (it - 1) * TB);
+        for (int tb = pw; tb < n; tb += SCAN_PRODUCERS) {
+          const float q = square(obuf + (((it - 1) % 3) * TB + tb) * CC);
+          if (lane == 0) ssq[((it - 1) & 1) * TB + tb] = q;
+        }
+      }
+      if (it >= lag) finish(it - lag);
+      const int next = it + 1 - lag;                         // the tile the next round finishes
+      if (next >= 0 && next < n_tiles && (lag > 1 || it > 0)) gates(next);
+      barrier();
+    }
+    return;
+  }
 
-  // ---- consumers: a column, and every fourth group of four key rows
-  const int col = tid >> 2, kq = tid & 3, cg = c0 + col;
-  float* sp = a.state + (size_t)row * a.row_stride + ((size_t)h * D + cg) * D;
-  f2_t M[NQ * 2];
-  if (consumer) {
+  // ---- consumers: CP columns, and every fourth group of four key rows
+  const int col = (tid >> 2) * CP, kq = tid & 3;
+  f2_t M[CP][NQ * 2];
+  float* sp[CP];
+#pragma unroll
+  for (int x = 0; x < CP; ++x) {
+    const int cg = c0 + col + x;
     const bool mine = cg < D;
+    sp[x] = a.state + (size_t)row * a.row_stride + ((size_t)h * D + (mine ? cg : 0)) * D;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int k = (kq + 4 * i) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (mine && (D & 3) == 0) {
-        if (k < D) v = *reinterpret_cast<const float4*>(sp + k);
+        if (k < D) v = *reinterpret_cast<const float4*>(sp[x] + k);
       } else if (mine) {
-        if (k < D) v.x = sp[k];
-        if (k + 1 < D) v.y = sp[k + 1];
-        if (k + 2 < D) v.z = sp[k + 2];
-        if (k + 3 < D) v.w = sp[k + 3];
+        if (k < D) v.x = sp[x][k];
+        if (k + 1 < D) v.y = sp[x][k + 1];
+        if (k + 2 < D) v.z = sp[x][k + 2];
+        if (k + 3 < D) v.w = sp[x][k + 3];
       }
-      M[2 * i] = pack2(v.x, v.y);
-      M[2 * i + 1] = pack2(v.z, v.w);
+      M[x][2 * i] = pack2(v.x, v.y);
+      M[x][2 * i + 1] = pack2(v.z, v.w);
     }
-  } else if (n_tiles > 0) {
-    stage(0);
   }
   barrier();
-  const int last = CS > 1 ? n_tiles + 1 : n_tiles;
   for (int it = 0; it <= last; ++it) {
-    if (!consumer) {
-      if (it + 1 < n_tiles) stage(it + 1);
-      if (CS == 1) {
-        if (it >= 1) finish(it - 1, true);
-      } else {
-        if (it >= 1 && it - 1 < n_tiles) {
-          const int n = min(TB, len - (it - 1) * TB);
-          for (int tb = pw; tb < n; tb += SCAN_PRODUCERS) {
-            const float q = square(obuf + (((it - 1) % 3) * TB + tb) * CC);
-            if (lane == 0) ssq[((it - 1) & 1) * TB + tb] = q;
-          }
-        }
-        if (it >= 2) finish(it - 2, false);
-      }
-    } else if (it < n_tiles) {
+    if (it < n_tiles) {
       const float* buf = scan_smem + (it & 1) * buf_floats;
       const float* val = buf + TB * NVEC * DKP;
       const float* scal = val + TB * CC;
-      float* o_out = obuf + (it % 3) * TB * CC;
+      const uint32_t o_out = smem_u32(obuf + (it % 3) * TB * CC);
       const int n = min(TB, len - it * TB);
+#pragma unroll 2
       for (int tb = 0; tb < n; ++tb) {
         const ulonglong2* dw = reinterpret_cast<const ulonglong2*>(buf + tb * DKP);
         const ulonglong2* dk = dw + TB * DKP / 4;
         const ulonglong2* dr = dk + TB * DKP / 4;
         const ulonglong2* du = dr + TB * DKP / 4;
         const ulonglong2* da = du + TB * DKP / 4;
-        const float v = val[tb * CC + col], s2 = scal[2 * tb + 1];
-        f2_t o2[2] = {0, 0}, g2[2] = {0, 0};
+        const float s1 = scal[2 * tb], s2 = scal[2 * tb + 1];
+        float v[CP];
+        f2_t o2[CP][2], g2[CP][2];
+#pragma unroll
+        for (int x = 0; x < CP; ++x) {
+          v[x] = val[tb * CC + col + x];
+          o2[x][0] = o2[x][1] = g2[x][0] = g2[x][1] = 0;
+        }
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+          if (DELTA) {
+            const ulonglong2 u = du[kq + 4 * i];
+#pragma unroll
+            for (int x = 0; x < CP; ++x) {
+              g2[x][0] = fma2(M[x][2 * i], u.x, g2[x][0]);
+              g2[x][1] = fma2(M[x][2 * i + 1], u.y, g2[x][1]);
+            }
+          }
+        }
+        float o[CP], gone[CP];
+#pragma unroll
+        for (int x = 0; x < CP; ++x) {
+          gone[x] = 0.f;
+          if (DELTA) {
+            gone[x] = sum_of(g2[x][0]) + sum_of(g2[x][1]);
+            gone[x] += __shfl_xor_sync(0xffffffffu, gone[x], 1);
+            gone[x] += __shfl_xor_sync(0xffffffffu, gone[x], 2);
+          }
+        }
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
           const ulonglong2 r = dr[kq + 4 * i];
-          o2[0] = fma2(M[2 * i], r.x, o2[0]);
-          o2[1] = fma2(M[2 * i + 1], r.y, o2[1]);
-          if (DELTA) {
-            const ulonglong2 u = du[kq + 4 * i];
-            g2[0] = fma2(M[2 * i], u.x, g2[0]);
-            g2[1] = fma2(M[2 * i + 1], u.y, g2[1]);
+#pragma unroll
+          for (int x = 0; x < CP; ++x) {
+            o2[x][0] = fma2(M[x][2 * i], r.x, o2[x][0]);
+            o2[x][1] = fma2(M[x][2 * i + 1], r.y, o2[x][1]);
           }
         }
-        float o = sum_of(o2[0]) + sum_of(o2[1]), gone = 0.f;
-        if (DELTA) {
-          gone = sum_of(g2[0]) + sum_of(g2[1]);
-          gone += __shfl_xor_sync(0xffffffffu, gone, 1);
-          gone += __shfl_xor_sync(0xffffffffu, gone, 2);
+        f2_t vv[CP], gg[CP];
+#pragma unroll
+        for (int x = 0; x < CP; ++x) {
+          o[x] = sum_of(o2[x][0]) + sum_of(o2[x][1]);
+          vv[x] = pack2(v[x], v[x]);
+          gg[x] = pack2(-gone[x], -gone[x]);
         }
-        const f2_t vv = pack2(v, v), gg = pack2(-gone, -gone);
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
           const ulonglong2 k = dk[kq + 4 * i], w = dw[kq + 4 * i];
-          f2_t x = mul2(k.x, vv), y = mul2(k.y, vv);
-          if (DELTA) {
-            const ulonglong2 au = da[kq + 4 * i];
-            x = fma2(au.x, gg, x);
-            y = fma2(au.y, gg, y);
+          ulonglong2 au;
+          if (DELTA) au = da[kq + 4 * i];
+#pragma unroll
+          for (int x = 0; x < CP; ++x) {
+            f2_t p = mul2(k.x, vv[x]), q = mul2(k.y, vv[x]);
+            if (DELTA) {
+              p = fma2(au.x, gg[x], p);
+              q = fma2(au.y, gg[x], q);
+            }
+            M[x][2 * i] = fma2(w.x, M[x][2 * i], p);
+            M[x][2 * i + 1] = fma2(w.y, M[x][2 * i + 1], q);
           }
-          M[2 * i] = fma2(w.x, M[2 * i], x);
-          M[2 * i + 1] = fma2(w.y, M[2 * i + 1], y);
         }
-        o += __shfl_xor_sync(0xffffffffu, o, 1);
-        o += __shfl_xor_sync(0xffffffffu, o, 2);
-        if (kq == 0) o_out[tb * CC + col] = fmaf(s2, v, DELTA ? fmaf(-scal[2 * tb], gone, o) : o);
+#pragma unroll
+        for (int x = 0; x < CP; ++x) {
+          o[x] += __shfl_xor_sync(0xffffffffu, o[x], 1);
+          o[x] += __shfl_xor_sync(0xffffffffu, o[x], 2);
+          if (kq == 0)
+            store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], DELTA ? fmaf(-s1, gone[x], o[x]) : o[x]));
+        }
       }
     }
     barrier();
   }
-  if (consumer && cg < D) {
+#pragma unroll
+  for (int x = 0; x < CP; ++x) {
+    if (c0 + col + x >= D) continue;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int k = (kq + 4 * i) * 4;
-      const float2 lo = unpack2(M[2 * i]), hi = unpack2(M[2 * i + 1]);
+      const float2 lo = unpack2(M[x][2 * i]), hi = unpack2(M[x][2 * i + 1]);
       if ((D & 3) == 0) {
-        if (k < D) *reinterpret_cast<float4*>(sp + k) = make_float4(lo.x, lo.y, hi.x, hi.y);
+        if (k < D) *reinterpret_cast<float4*>(sp[x] + k) = make_float4(lo.x, lo.y, hi.x, hi.y);
       } else {
-        if (k < D) sp[k] = lo.x;
-        if (k + 1 < D) sp[k + 1] = lo.y;
-        if (k + 2 < D) sp[k + 2] = hi.x;
-        if (k + 3 < D) sp[k + 3] = hi.y;
+        if (k < D) sp[x][k] = lo.x;
+        if (k + 1 < D) sp[x][k + 1] = lo.y;
+        if (k + 2 < D) sp[x][k + 2] = hi.x;
+        if (k + 3 < D) sp[x][k + 3] = hi.y;
       }
     }
   }
@@ -290,47 +391,47 @@ __global__ void __launch_bounds__(128) tanh_rows_kernel(const float* x, int ldx,
   }
 }
 
+// Decay logits of few tokens in one launch: z[t, n] = sum_k W[n, k] tanh(x[t, k]), tanh rounded to the activation type as the
+// GEMM's operand would be; a thread per output.
+template <typename AT>
+__global__ void __launch_bounds__(64) low_rank_kernel(const float* x, int ldx, const AT* W, float* z, int ldz, int N, int K, int pdl) {
+  extern __shared__ __align__(16) float lr_smem[];
+  const int n = blockIdx.x * 64 + threadIdx.x, t = blockIdx.y;
+  const AT* w = W + (size_t)min(n, N - 1) * K;
+  if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  for (int k = threadIdx.x; k < K; k += 64) lr_smem[k] = to_f32<AT>(from_f32<AT>(tanhf(x[(size_t)t * ldx + k])));
+  __syncthreads();
+  float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+  for (int k = 0; k < K; k += 4) {
+    const float4 a = load4(w + k), b = load4((const float*)lr_smem + k);
+    s[0] = fmaf(a.x, b.x, s[0]);
+    s[1] = fmaf(a.y, b.y, s[1]);
+    s[2] = fmaf(a.z, b.z, s[2]);
+    s[3] = fmaf(a.w, b.w, s[3]);
+  }
+  if (n < N) z[(size_t)t * ldz + n] = (s[0] + s[1]) + (s[2] + s[3]);
+}
+
 // Columns per CTA and CTAs per head: a head's columns are cut until the grid fills the machine (16 columns at the least); a
-// CTA takes at most 128.
-static void scan_split(int n_seq, int H, int D, int* CC, int* CS) {
+// CTA takes at most scan_max_columns.  Whole warps of consumers need multiples of 8 (16 in pairs).
+static void scan_split(int n_seq, int H, int D, int most, int unit, int* CC, int* CS) {
   int cs = 1;
-  while ((D + cs - 1) / cs > 128) cs *= 2;
+  while ((D + cs - 1) / cs > most) cs *= 2;
   while (cs < 8 && (long long)n_seq * H * cs * 2 <= 148 && D / (cs * 2) >= 16) cs *= 2;
-  const int cc = ((D + cs - 1) / cs + 7) / 8 * 8;
-  *CC = cc;
+  *CC = ((D + cs - 1) / cs + unit - 1) / unit * unit;
   *CS = cs;
 }
 
 template <bool DELTA, int DKP>
 static int scan_launch(const ScanArgs& a, int f32, cudaStream_t st) {
   int CC, CS;
-  scan_split(a.r.n_seq, a.H, a.D, &CC, &CS);
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA);
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA), CP = scan_columns(DKP);
+  scan_split(a.r.n_seq, a.H, a.D, scan_max_columns(DKP), 8 * CP, &CC, &CS);
   const int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 2 * TB) * 4;
   CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<DELTA, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
-  cudaLaunchAttribute attr[2];
-  int n = 0;
-  if (CS > 1) {
-    attr[n].id = cudaLaunchAttributeClusterDimension;
-    attr[n].val.clusterDim.x = CS;
-    attr[n].val.clusterDim.y = 1;
-    attr[n].val.clusterDim.z = 1;
-    ++n;
-  }
-  if (a.pdl) {
-    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[n].val.programmaticStreamSerializationAllowed = 1;
-    ++n;
-  }
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(a.H * CS, a.r.n_seq);
-  cfg.blockDim = dim3(CC * 4 + SCAN_PRODUCERS * 32);
-  cfg.dynamicSmemBytes = bytes;
-  cfg.stream = st;
-  cfg.attrs = attr;
-  cfg.numAttrs = n;
-  CUDA_CHECK_RET(cudaLaunchKernelEx(&cfg, scan_kernel<DELTA, DKP>, a, CC, CS, f32));
-  return 0;
+  return launch_cluster(scan_kernel<DELTA, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * 4 + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
+                        CS, a, CC, CS, f32);
 }
 
 template <bool DELTA>
@@ -362,4 +463,15 @@ SMC_API int smc_tanh_rows(const float* x, int ldx, void* out, int ldo, int n, in
   const dim3 grid((unsigned)(want < 2368 ? want : 2368)), block(128);
   if (f32) return launch_pdl(tanh_rows_kernel<float>, grid, block, 0, st, pdl, x, ldx, (float*)out, ldo, n, M, pdl);
   return launch_pdl(tanh_rows_kernel<__nv_bfloat16>, grid, block, 0, st, pdl, x, ldx, (__nv_bfloat16*)out, ldo, n, M, pdl);
+}
+
+// z = tanh(x) W^T for a few tokens; W [N, K], K a multiple of 8.
+SMC_API int smc_low_rank(const float* x, int ldx, const void* W, float* z, int ldz, int N, int K, int M, int f32, int pdl,
+                         cudaStream_t st) {
+  using namespace smc;
+  if (M <= 0) return 0;
+  if (K % 8 || K > 8192 || M > 65535) return -121;
+  const dim3 grid((N + 63) / 64, M), block(64);
+  if (f32) return launch_pdl(low_rank_kernel<float>, grid, block, K * 4, st, pdl, x, ldx, (const float*)W, z, ldz, N, K, pdl);
+  return launch_pdl(low_rank_kernel<__nv_bfloat16>, grid, block, K * 4, st, pdl, x, ldx, (const __nv_bfloat16*)W, z, ldz, N, K, pdl);
 }

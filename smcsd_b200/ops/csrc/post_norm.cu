@@ -64,11 +64,38 @@ template <int VEC, typename T> __device__ __forceinline__ void store_cols(T* p, 
   else *p = from_f32<T>(v[0]);
 }
 
-template <typename AT, int VEC>
-__global__ void __launch_bounds__(256) post_norm_kernel(const PostNormArgs a) {
+// AHEAD > 0: AHEAD mixes whose coefficients, and the row before, are read before the sums (two column groups per thread).
+template <typename AT, int VEC, int AHEAD>
+__global__ void __launch_bounds__(AHEAD ? 512 : 256) post_norm_kernel(const PostNormArgs a) {
+  constexpr int POST_MAXV = AHEAD ? 2 : smc::POST_MAXV, NA = AHEAD ? AHEAD : 1, GA = AHEAD ? 2 : 1;
   __shared__ float red[32];
-  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int d = a.d, t = blockIdx.x;
+  float mus[GA][NA][VEC], before[GA][VEC];
+  if constexpr (AHEAD > 0) {
+#pragma unroll
+    for (int i = 0; i < GA; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+      if (c >= d) continue;
+#pragma unroll
+      for (int s = 0; s < NA; ++s) load_cols<VEC>(mus[i][s], a.mu + (size_t)s * d + c);
+    }
+  }
+  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  int row = -1;
+  if (a.mu != nullptr) {
+    row = a.rows[t];
+    if (row < 0 || row >= a.n_rows) {
+      if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
+      row = -1;
+    }
+  }
+  if constexpr (AHEAD > 0) {
+#pragma unroll
+    for (int i = 0; i < GA; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * VEC;
+      if (c < d && row >= 0) load_cols<VEC>(before[i], (const float*)a.hist + (size_t)row * a.ldh + c);
+    }
+  }
   float* x = a.x + (size_t)t * d;
   float v[POST_MAXV][VEC];
   if (a.ids != nullptr) {
@@ -127,14 +154,6 @@ __global__ void __launch_bounds__(256) post_norm_kernel(const PostNormArgs a) {
     }
     inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)d + a.eps);
   }
-  int row = -1;
-  if (a.mu != nullptr) {
-    row = a.rows[t];
-    if (row < 0 || row >= a.n_rows) {
-      if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
-      row = -1;
-    }
-  }
 #pragma unroll
   for (int i = 0; i < POST_MAXV; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * VEC;
@@ -150,10 +169,21 @@ __global__ void __launch_bounds__(256) post_norm_kernel(const PostNormArgs a) {
     if (a.xa != nullptr) store_cols<VEC>(reinterpret_cast<AT*>(a.xa) + (size_t)t * a.ldxa + c, v[i]);
     if (row >= 0) {
       float* hp = a.hist + (size_t)row * a.ldh + c;
+      AT* m = reinterpret_cast<AT*>(a.mix) + (size_t)t * a.n_mix * a.ldxa + c;
+      if constexpr (AHEAD > 0) {
+        store_cols<VEC>(hp, v[i]);
+#pragma unroll
+        for (int s = 0; s < NA; ++s) {
+          float o[VEC];
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) o[k] = fmaf(before[i][k] - v[i][k], mus[i][s][k], v[i][k]);
+          store_cols<VEC>(m + (size_t)s * a.ldxa, o);
+        }
+        continue;
+      }
       float back[VEC];
       load_cols<VEC>(back, (const float*)hp);
       store_cols<VEC>(hp, v[i]);
-      AT* m = reinterpret_cast<AT*>(a.mix) + (size_t)t * a.n_mix * a.ldxa + c;
       for (int s = 0; s < a.n_mix; ++s) {
         float mu[VEC], o[VEC];
         load_cols<VEC>(mu, a.mu + (size_t)s * d + c);
@@ -215,9 +245,11 @@ static int post_norm_launch(const PostNormArgs& a, int T, cudaStream_t st) {
   const bool vec = a.d % 4 == 0 && (a.y == nullptr || a.ldy % 4 == 0) && a.ldxa % 4 == 0 && (a.mu == nullptr || a.ldh % 4 == 0);
   const int groups = vec ? a.d / 4 : a.d;
   const int threads = groups <= 64 ? 64 : groups <= 128 ? 128 : 256;
+  if (a.mu != nullptr && a.n_mix == 5 && vec && groups <= 1024)
+    return launch_pdl(post_norm_kernel<AT, 4, 5>, dim3(T), dim3(groups <= 512 ? threads : 512), 0, st, a.pdl, a);
   if (groups > threads * POST_MAXV) return -91;
-  if (vec) return launch_pdl(post_norm_kernel<AT, 4>, dim3(T), dim3(threads), 0, st, a.pdl, a);
-  return launch_pdl(post_norm_kernel<AT, 1>, dim3(T), dim3(threads), 0, st, a.pdl, a);
+  if (vec) return launch_pdl(post_norm_kernel<AT, 4, 0>, dim3(T), dim3(threads), 0, st, a.pdl, a);
+  return launch_pdl(post_norm_kernel<AT, 1, 0>, dim3(T), dim3(threads), 0, st, a.pdl, a);
 }
 
 template <typename AT>

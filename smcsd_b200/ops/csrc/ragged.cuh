@@ -81,20 +81,34 @@ __device__ __forceinline__ float block_sum_all(float v, float* red) {
 // Launch with an optional programmatic dependency on the previous kernel of the stream.  Kernels launched this way take
 // data of earlier kernels through plain pointers: a const __restrict__ parameter counts as invariant for the compiler, which
 // may then read it ahead of the wait.
+// launch_cluster: the same with `cluster` consecutive CTAs in x as a thread-block cluster.
 template <typename... P, typename... A>
-inline int launch_pdl(void (*kern)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, int pdl, A... args) {
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
+inline int launch_cluster(void (*kern)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, int pdl, int cluster, A... args) {
+  cudaLaunchAttribute attr[2];
+  int n = 0;
+  if (pdl) {
+    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[n++].val.programmaticStreamSerializationAllowed = 1;
+  }
+  if (cluster > 1) {
+    attr[n].id = cudaLaunchAttributeClusterDimension;
+    attr[n].val.clusterDim.x = cluster;
+    attr[n].val.clusterDim.y = 1;
+    attr[n++].val.clusterDim.z = 1;
+  }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = block;
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cfg.attrs = attr;
-  cfg.numAttrs = pdl ? 1 : 0;
+  cfg.numAttrs = n;
   CUDA_CHECK_RET(cudaLaunchKernelEx(&cfg, kern, static_cast<P>(args)...));
   return 0;
+}
+template <typename... P, typename... A>
+inline int launch_pdl(void (*kern)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, int pdl, A... args) {
+  return launch_cluster(kern, grid, block, smem, st, pdl, 1, args...);
 }
 
 }  // namespace smc

@@ -686,14 +686,17 @@ def layered_lib():
         L.smc_post_norm_step.argtypes = [vp, i, i, vp]
         L.smc_token_shift.argtypes = [vp, i, vp, i, vp, i, vp, i, i, vp, vp, i, i, vp]
         L.smc_heads_new.argtypes = [vp, i, i, vp]
-        L.smc_chunk_attn.argtypes = [vp, i, vp]
+        L.smc_chunk_attn.argtypes = [vp, i, i, vp]
+        L.smc_chunk_attn_splits.argtypes = [i, i, i, i, i]
         L.smc_chunk_attn_tc.argtypes = [vp, vp]
         L.smc_memory_scan.argtypes = [vp, i, i, vp]
+        L.smc_low_rank.argtypes = [vp, i, vp, vp, i, i, i, i, i, i, vp]
         L.smc_tanh_rows.argtypes = [vp, i, vp, i, i, i, i, i, vp]
         for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_gated_unit_f32",
                   "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn", "smc_post_norm_step",
-                  "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_tc", "smc_chunk_attn_tc_max_width",
-                  "smc_memory_scan", "smc_tanh_rows"):
+                  "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_splits", "smc_chunk_attn_tc",
+                  "smc_chunk_attn_tc_max_width",
+                  "smc_memory_scan", "smc_tanh_rows", "smc_low_rank"):
             getattr(L, n).restype = C.c_int
         for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
                        (GroupLink, "smc_group_link_size"), (PostNormArgs, "smc_post_norm_args_size"),
@@ -814,8 +817,14 @@ def heads_new(a: HeadsNewArgs, T: int, f32: bool) -> None:
     _check(layered_lib().smc_heads_new(C.byref(a), T, int(f32), _stream()), "smc_heads_new")
 
 
-def chunk_attention(a: ChunkAttnArgs, f32: bool) -> None:
-    _check(layered_lib().smc_chunk_attn(C.byref(a), int(f32), _stream()), "smc_chunk_attn")
+def chunk_attention(a: ChunkAttnArgs, f32: bool, splits: int = 1) -> None:
+    """``splits`` key ranges run as a thread-block cluster and merge on chip."""
+    _check(layered_lib().smc_chunk_attn(C.byref(a), splits, int(f32), _stream()), "smc_chunk_attn")
+
+
+def chunk_attention_splits(tokens: int, H: int, G: int, wide: int, keys: int) -> int:
+    """Key ranges for ``tokens`` tokens (H query heads, G kv heads of up to ``wide`` columns) over about ``keys`` keys."""
+    return layered_lib().smc_chunk_attn_splits(tokens, H, G, wide, int(keys))
 
 
 def chunk_attention_tc(a: ChunkAttnArgs) -> None:
@@ -835,3 +844,9 @@ def memory_scan(a: ScanArgs, delta: bool, f32: bool) -> None:
 
 def tanh_rows(x: torch.Tensor, out: torch.Tensor, *, n: int, M: int, f32: bool, pdl: bool = False) -> None:
     _check(layered_lib().smc_tanh_rows(_p(x), x.stride(0), _p(out), out.stride(0), n, M, int(f32), int(pdl), _stream()), "smc_tanh_rows")
+
+
+def low_rank(x: torch.Tensor, W: torch.Tensor, z: torch.Tensor, *, M: int, f32: bool, pdl: bool = False) -> None:
+    """z = tanh(x) W^T for a few tokens, in one launch (tanh rounded to the activation type)."""
+    _check(layered_lib().smc_low_rank(_p(x), x.stride(0), _p(W), _p(z), z.stride(0), W.shape[0], W.shape[1], M, int(f32), int(pdl),
+                                      _stream()), "smc_low_rank")

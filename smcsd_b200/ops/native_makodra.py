@@ -24,6 +24,7 @@ from .native_layered import NativeLayered, env_flag
 
 class NativeMakodra(NativeLayered):
     TC_MIN_TOKENS = 8                     # portions at least this long take the tensor-core attention
+    LOW_RANK_TOKENS = 32                  # steps up to this long expand the decay logits in one launch
 
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
@@ -79,9 +80,18 @@ class NativeMakodra(NativeLayered):
 
     # ---- planning -----------------------------------------------------------------------
     def set_context(self, ctx: int, bs: int, Es=(1, 2)) -> tuple:
-        """Record the context-length hint (no launch grid depends on it)."""
+        """Record the context-length hint; returns what it decides about the launch grids (part of a graph's identity)."""
         self.ctx_hint = int(ctx)
-        return ()
+        mixers = {L.spec.mixer for L in self.m.layers if L.kind == "attention"}
+        return tuple(sorted((E, m.chunk, m.heads, self._ks(bs * E, m)) for E in Es for m in mixers))
+
+    def _ks(self, tokens: int, m) -> int:
+        """Key ranges of one layer's attention for ``tokens`` tokens."""
+        ks = K.chunk_attention_splits(tokens, m.heads, m.kv_heads, round_up(max(m.dim, m.vdim), 8), min(m.chunk, self.ctx_hint))
+        cap = max(1, int(self.attn_splits))
+        while ks > cap:
+            ks //= 2
+        return ks
 
     # ---- sublayers ----------------------------------------------------------------------
     def _attention(self, L, T: int, locs: torch.Tensor, work: "K.Ragged", longest: int) -> None:
@@ -102,7 +112,7 @@ class NativeMakodra(NativeLayered):
         if self.attn_tc and longest >= self.TC_MIN_TOKENS and max(D, V) <= K.chunk_tc_max_width():
             K.chunk_attention_tc(a)
         else:
-            K.chunk_attention(a, self.f32)
+            K.chunk_attention(a, self.f32, self._ks(T, m))
         self._gemm(L.wo, vo, self._rows("y", T, self.d), T)
 
     def _recurrent(self, L, T: int, work: "K.Ragged", single: bool) -> None:
@@ -127,8 +137,11 @@ class NativeMakodra(NativeLayered):
                                status=self.status, pdl=self.pdl)
             low_in = self._rows("low_in", T, rank)
             self._gemm(L.w1, mix[:, n * d8:], low_in, T, ldx=mix.stride(0))
-        K.tanh_rows(low_in, low, n=rank, M=T, f32=self.f32, pdl=self.pdl)
-        self._gemm(L.w2, low, z, T)
+        if T <= self.LOW_RANK_TOKENS:
+            K.low_rank(low_in, L.w2, z, M=T, f32=self.f32, pdl=self.pdl)
+        else:
+            K.tanh_rows(low_in, low, n=rank, M=T, f32=self.f32, pdl=self.pdl)
+            self._gemm(L.w2, low, z, T)
         S, ldo = self.state.matrix(L.index), L.wo.shape[1]
         vo = self._rows("vo", T, ldo)
         K.memory_scan(K.ScanArgs(proj=K.ptr(proj), ldp=proj.stride(0), r_off=0, k_off=HD, v_off=2 * HD, g_off=3 * HD, a_off=4 * HD,

@@ -130,14 +130,16 @@ def test_new_heads(H, G, dim, vdim, f32):
     assert not kp[0].any() and int(st) == 0
 
 
-SHAPES = [(4, 2, 24, 40, 48), (2, 2, 64, 64, 64), (8, 2, 128, 128, 100), (3, 1, 16, 96, 1000), (2, 2, 200, 256, 33), (6, 2, 80, 8, 1)]
+SHAPES = [(4, 2, 24, 40, 48), (2, 2, 64, 64, 64), (8, 2, 128, 128, 100), (3, 1, 16, 96, 1000), (2, 2, 200, 256, 33), (6, 2, 80, 8, 1), (2, 1, 40, 360, 90)]
 
 
-@pytest.mark.parametrize("form", ["f32", "bf16", "bf16_tc"])
+@pytest.mark.parametrize("form,splits", [("f32", 1), ("f32", 4), ("bf16", 1), ("bf16", 2), ("bf16", 8), ("bf16_tc", 1)])
 @pytest.mark.parametrize("H,G,D,V,chunk", SHAPES)
-def test_chunk_attention(H, G, D, V, chunk, form):
+def test_chunk_attention(H, G, D, V, chunk, form, splits):
     """Portions inside, at and across chunk edges; equal tokens far apart stand out; scattered pages."""
     k, f32 = K(), form == "f32"
+    if form == "bf16_tc" and max(D, V) > k.chunk_tc_max_width():
+        pytest.skip("beyond the tensor-core form")
     dt = torch.float32 if f32 else torch.bfloat16
     prefix, lens = [0, 63, 130, 47, 95], [150, 2, 65, 1, 9]
     total = [p + n for p, n in zip(prefix, lens)]
@@ -167,7 +169,7 @@ def test_chunk_attention(H, G, D, V, chunk, form):
     scale = 6.0 / D
     args = dict(q=k.ptr(qd), kpool=k.ptr(kp), vpool=k.ptr(vp), out=k.ptr(out), block_table=k.ptr(btd), bt_stride=300, bt_rows=7,
                 n_pages=600, H=H, G=G, D=D, V=V, chunk=chunk, scale=scale, r=r, status=k.ptr(st))
-    run = (lambda a: k.chunk_attention_tc(a)) if form == "bf16_tc" else (lambda a: k.chunk_attention(a, f32))
+    run = (lambda a: k.chunk_attention_tc(a)) if form == "bf16_tc" else (lambda a: k.chunk_attention(a, f32, splits))
     run(k.ChunkAttnArgs(gate=k.ptr(gd), ldg=H * V + 4, r1=k.ptr(r1d), r2=k.ptr(r2d), sink=1, **args))
     near = dt if not f32 else torch.float64
     ref = torch.cat([O.chunk_attention(x.to(near).double(), y.to(near).double(), z.to(near).double(), scale, r1.double(), r2.double(), chunk)[p:]
@@ -182,6 +184,21 @@ def test_chunk_attention(H, G, D, V, chunk, form):
     plain = torch.einsum("hij,jhv->ihv", p, vs[0][:n].to(near).double().repeat_interleave(H // G, 1)).reshape(n, -1)
     close(out[:n], plain, 3e-6 if f32 else 1.2e-2)
     assert int(st) == 0
+
+
+@pytest.mark.parametrize("f32", [True, False])
+@pytest.mark.parametrize("N,rank,M", [(2048, 64, 8), (75, 16, 3), (100, 24, 32), (64, 600, 1)])
+def test_decay_logits(N, rank, M, f32):
+    """One launch for few tokens, and the activation of the GEMM form."""
+    k, dt = K(), torch.float32 if f32 else torch.bfloat16
+    x, W = rnd(M, rank + 4), (rnd(N, rank, seed=1) * rank ** -0.5).to(dt)
+    xd, z, low = x.to(DEV), torch.zeros(M, N + 3, device=DEV), torch.zeros(M, rank, dtype=dt, device=DEV)
+    k.low_rank(xd, W.to(DEV).contiguous(), z, M=M, f32=f32)
+    k.tanh_rows(xd, low, n=rank, M=M, f32=f32)
+    want = torch.tanh(x[:, :rank].double())
+    close(low, want, 1e-6 if f32 else 4e-3)
+    close(z[:, :N], want @ W.double().T, 2e-6 if f32 else 6e-3)
+    assert not z[:, N:].any()
 
 
 @pytest.mark.parametrize("f32", [True, False])
