@@ -77,6 +77,9 @@ class NativeLayered:
             K.gated_unit_f32(gu, act, ff=ff2 // 2, blk=blk, limit=link.limit, slope=link.slope, shift=shift, M=M, pdl=self.pdl)
             return
         splits = K.gemm_swiglu_splits(ff2, W.shape[-1], M) if link.mode == 0 else 1
+        if link.mode == 0 and link.act == K.ACT_SILU:        # the plain build of the kernel has this unit
+            K.gemm_skinny(W, X, act, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, ldo=act.stride(0), status=self.status, pdl=self.pdl)
+            return
         K.gemm_grouped(W, X, act, N=ff2, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, link=link, status=self.status, pdl=self.pdl)
 
     # ---- forward ------------------------------------------------------------------------

@@ -33,7 +33,7 @@ def test_chunk_edges(tmp_path, size):
     S.chunk_edges(CTX, tmp_path, config(64, [(attn(4, 2, 16, 24, size), None)]), size, 3 * size + 2)
 
 
-@pytest.mark.parametrize("name", ["all_kinds", "memory_only"])
+@pytest.mark.parametrize("name", ["all_kinds", "attention_only", "memory_only"])
 def test_greedy_generation(tmp_path, name):
     outs = S.greedy_generation(CTX, tmp_path, name)
     assert len({json.dumps(v) for v in outs.values()}) == 1      # whatever the cycle length and the schedule

@@ -44,6 +44,11 @@ def test_greedy_generation(ctx, tmp_path, graph):
     S.greedy_generation(ctx, tmp_path, "all_kinds", cycle_graph=graph)
 
 
+@pytest.mark.parametrize("name", ["attention_only", "memory_only"])
+def test_greedy_generation_without_state_or_cache(tmp_path, name):
+    S.greedy_generation(F32, tmp_path, name, cycle_graph=True)
+
+
 def test_rows_do_not_depend_on_cuts_or_company(tmp_path):
     """bf16 rows of one sequence fed in different cuts, pages and company agree far below the rounding of the model."""
     folder, cfg, W = save_model(tmp_path / "m", "memory_only")
