@@ -334,8 +334,9 @@ SMC_API int smc_heads_new(const smc::HeadsNewArgs* a, int T, int f32, cudaStream
 SMC_API int smc_chunk_attn_splits(int tokens, int H, int G, int wide, int keys) {
   const int rep = H / G, rh = smc::chunk_heads<float>(wide, rep);
   const long long ctas = (long long)tokens * G * ((rep + rh - 1) / rh);
+  const int slots = wide * rh <= 256 ? 296 : 148;             // one CTA per SM where its registers leave room for no second
   int ks = 1;
-  while (ks < 8 && ctas * ks * 2 <= 296 && keys / (ks * 2) >= 64) ks *= 2;
+  while (ks < 8 && ctas * ks * 2 <= slots && keys / (ks * 2) >= 64) ks *= 2;
   return ks;
 }
 
