@@ -1,4 +1,4 @@
-"""Model families: dense Llama-style decoders, Qwen3.5-style Gated-DeltaNet hybrids, Pasizen and Makodra."""
+"""Model families: dense Llama-style decoders, Qwen3.5-style Gated-DeltaNet hybrids, Pasizen, Makodra and Funevik."""
 from __future__ import annotations
 
 import os
@@ -18,6 +18,8 @@ def build_model(spec, dtype=torch.bfloat16, device="cpu", tp_rank: int = 0, tp_s
         from .pasizen import PasizenModel as Cls
     elif cfg.arch == "makodra":
         from .makodra import MakodraModel as Cls
+    elif cfg.arch == "funevik":
+        from .funevik import FunevikModel as Cls
     else:
         from .llama import LlamaModel as Cls
     m = Cls(cfg, dtype=dtype, device=device, tp_rank=tp_rank, tp_size=tp_size, max_positions=max_positions)

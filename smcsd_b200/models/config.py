@@ -1,16 +1,19 @@
 """Architecture descriptions: parsed from a HF ``config.json`` or built from presets.
 
-Four families are served.  Two are the ones the reference runs: dense Llama-style decoders and
+Five families are served.  Two are the ones the reference runs: dense Llama-style decoders and
 Qwen3.5-style hybrids that interleave Gated-DeltaNet layers with gated full attention
 (reference: README.md model list; parameter names checked against the HF
 implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).  The others spell every layer out in config.json.
 Pasizen: latent attention without positions, a short convolution in front of every mixer, hyper-connected residual
 streams, PolyNorm or mixture-of-experts feed-forwards and layers that may be looped.  Makodra: generalized delta rule,
-token-shifted decaying memory and chunked attention in any order, with norms on the sublayers' outputs.
+token-shifted decaying memory and chunked attention in any order, with norms on the sublayers' outputs.  Funevik: matrix
+memories with exponential gates, windowed latent attention with a rotated part and soft-capped attention behind a short
+convolution in any order, mixer and feed-forward side by side in every layer.
 """
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Union
@@ -20,13 +23,38 @@ UNLIMITED_POSITIONS = 1 << 20             # positions of architectures that comp
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` entries of a head, neighbours paired: pair i turns by position / base^(2i / dims)."""
+    dims: int
+    base: float
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Attention over a cached latent: ``kv_rank`` values per token, keys and values of all heads expanded from them."""
     heads: int
-    dim: int                             # query / key size per head
+    dim: int                             # query / key size per head (without the rotated part)
     vdim: int                            # value size per head
     kv_rank: int
     scale: float
+    q_rank: int = 0                      # queries go through a normed latent of this size (0: straight from the input)
+    rot: Optional[RotarySpec] = None     # a rotated part of ``rot.dims`` more query entries; its key is shared by all heads
+    window: int = 0                      # tokens a query sees, itself included (0: all before it)
+    sink: bool = False                   # one learned logit per head in the softmax sum, without a value
+
+
+@dataclass(frozen=True)
+class GroupedAttentionSpec:
+    """Causal grouped-query attention behind a short convolution of queries, keys and values: rotary positions, soft-capped
+    scores, a sink of score 0, a sigmoid gate per head."""
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key size per head
+    vdim: int                            # value size per head
+    scale: float
+    conv: int                            # taps
+    rot: RotarySpec
+    softcap: float
 
 
 @dataclass(frozen=True)
@@ -44,18 +72,25 @@ class ChunkAttentionSpec:
 
 @dataclass(frozen=True)
 class RecurrentSpec:
-    """A memory matrix [dim, dim] per head: "general_delta" (diagonal decay plus a rank-one removal) or "wkv" (diagonal
-    decay, bonus for the current token, token-shifted inputs)."""
+    """A memory matrix [dim, vdim] per head: "general_delta" (diagonal decay plus a rank-one removal), "wkv" (diagonal
+    decay, bonus for the current token, token-shifted inputs) or "mlstm" (one decay per head and token, exponential input
+    gate, read-out divided by a normaliser)."""
     kind: str
     heads: int
     dim: int
+    vdim: int = 0                        # 0: as many as ``dim``
+    gate_cap: float = 0.0                # "mlstm": gate logits are soft-capped at this
+
+    @property
+    def values(self) -> int:
+        return self.vdim or self.dim
 
 
 @dataclass(frozen=True)
 class GluSpec:
-    """Gated unit with clamped inputs (``limit``)."""
+    """Gated unit; with a ``limit`` its inputs are clamped."""
     ff: int
-    limit: float
+    limit: float = math.inf
 
 
 @dataclass(frozen=True)
@@ -65,26 +100,28 @@ class RouterSpec:
     top: int
     groups: int = 1
     keep: int = 1
+    bias: bool = False                   # logits have a bias
 
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    kind: str                            # "dense" (PolyNorm) | "moe" | "swiglu"
+    kind: str                            # "dense" (PolyNorm) | "moe" | "swiglu" | "geglu" (tanh form of gelu)
     ff: int = 0
     expert: Optional[GluSpec] = None
     router: Optional[RouterSpec] = None
     shared: Optional[GluSpec] = None
+    shared_gate: bool = False            # the shared expert is multiplied by a sigmoid gate per token
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[LatentAttentionSpec, ChunkAttentionSpec, RecurrentSpec]
+    mixer: Union[LatentAttentionSpec, ChunkAttentionSpec, GroupedAttentionSpec, RecurrentSpec]
     mlp: Optional[FeedForwardSpec]
 
 
 @dataclass
 class ModelConfig:
-    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen" | "makodra"
+    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen" | "makodra" | "funevik"
     vocab_size: int = 32000
     hidden_size: int = 4096
     n_layers: int = 32
@@ -110,11 +147,12 @@ class ModelConfig:
     attn_output_gate: bool = False
     qk_norm: bool = False
     norm_plus_one: bool = False                    # RMSNorm weight stored as (w - 1)
-    # ---- layer-by-layer description (Pasizen, Makodra) -----------------------
+    # ---- layer-by-layer description (Pasizen, Makodra, Funevik) --------------
     layers: Optional[List[LayerSpec]] = None
     loop: Optional[tuple] = None                   # (start, stop, times): these layers run ``times`` times in a row
     streams: int = 1                               # hyper-connected copies of the residual stream
     conv_taps: int = 1                             # short causal convolution in front of every mixer
+    embed_scale: float = 1.0                       # embedding rows are multiplied by this
     name: str = ""
 
     # ---- derived -------------------------------------------------------------
@@ -163,6 +201,8 @@ class ModelConfig:
             return self._layered_param_count()
         if self.arch == "makodra":
             return self._makodra_param_count()
+        if self.arch == "funevik":
+            return self._funevik_param_count()
         n = self.vocab_size * d * (1 if self.tie_embeddings else 2) + d
         for i in range(self.n_layers):
             n += 3 * d * f + 2 * d
@@ -204,7 +244,70 @@ class ModelConfig:
                 n += m.heads * m.dim * ((6 if delta else 5) * d + 3) + (0 if delta else 5 * d)
         return n
 
+    def _funevik_param_count(self) -> int:
+        d, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + self.hidden_size
+        for L in self.layers:
+            m, f = L.mixer, L.mlp
+            n += 2 * d
+            if isinstance(m, LatentAttentionSpec):
+                r, H = m.rot.dims, m.heads
+                n += m.q_rank * (d + 1 + H * (m.dim + r)) + d * (m.kv_rank + r) + m.kv_rank * (1 + H * (m.dim + m.vdim)) + H * (1 + m.vdim * d)
+            elif isinstance(m, GroupedAttentionSpec):
+                rows = m.heads * m.dim + m.kv_heads * (m.dim + m.vdim)
+                n += rows * (d + m.conv) + m.heads * d * (1 + m.vdim)
+            else:
+                n += m.heads * (d * (2 * m.dim + 3 * m.values + 2) + m.values + 2)
+            if f is None:
+                continue
+            n += 2 * d
+            if f.kind == "moe":
+                n += f.router.experts * (d + 1 + 3 * d * f.expert.ff) + (d + 3 * d * f.shared.ff if f.shared else 0)
+            else:
+                n += 3 * d * f.ff
+        return n
+
     # ---- construction ----------------------------------------------------------
+    @classmethod
+    def from_funevik_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
+        """config.json of a Funevik model: every layer with its mixer and feed-forward."""
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            m, f, mlp = e["mixer"], e.get("mlp"), None
+            rot = RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"])) if "rot" in m else None
+            if e["type"] == "mlstm":
+                mixer = RecurrentSpec("mlstm", int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+            elif e["type"] == "latent_attention":
+                mixer = LatentAttentionSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]),
+                                            int(m["q_rank"]), rot, int(m["mask"]["size"]), True)
+                if rot is None or rot.dims != int(m["rot_dim"]) or mixer.window < 1:
+                    raise ValueError(f"layer {i}: inconsistent latent attention {mixer}")
+            elif e["type"] == "attention":
+                mixer = GroupedAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                             int(m["conv"]), rot, float(m["softcap"]))
+                if mixer.heads % mixer.kv_heads or rot is None or rot.dims > mixer.dim or mixer.conv < 1 or mixer.softcap <= 0.0:
+                    raise ValueError(f"layer {i}: inconsistent attention {mixer}")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            if rot is not None and rot.dims % 2:
+                raise ValueError(f"layer {i}: rotary positions pair entries, {rot.dims} is odd")
+            if f is not None and f["kind"] == "dense":
+                mlp = FeedForwardSpec("geglu", ff=int(f["ff"]))
+            elif f is not None and f["kind"] == "moe":
+                router = RouterSpec(int(f["router"]["experts"]), int(f["router"]["top"]), bias=True)
+                if not 1 <= router.top <= router.experts:
+                    raise ValueError(f"layer {i}: inconsistent router {router}")
+                shared = GluSpec(int(f["shared"]["ff"])) if f.get("shared") else None
+                mlp = FeedForwardSpec("moe", expert=GluSpec(int(f["expert"]["ff"])), router=router, shared=shared, shared_gate=shared is not None)
+            elif f is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(LayerSpec(mixer, mlp))
+        eos = c.get("eos_token_id")
+        m0 = layers[0].mixer
+        return cls(arch="funevik", vocab_size=int(c["vocab"]), hidden_size=int(c["width"]), n_layers=len(layers), n_heads=m0.heads,
+                   n_kv_heads=getattr(m0, "kv_heads", m0.heads), head_dim=m0.dim, ffn_size=0, rms_eps=float(c["norm"]["eps"]),
+                   max_position=UNLIMITED_POSITIONS, layers=layers, embed_scale=float(c["embedding"]["scale"]),
+                   eos_token_ids=[] if eos is None else ([eos] if isinstance(eos, int) else list(eos)))
+
     @classmethod
     def from_makodra_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
         """config.json of a Makodra model: every layer with its mixer and feed-forward."""
@@ -279,6 +382,8 @@ class ModelConfig:
             return cls.from_layered_dict(c)
         if c.get("architecture") == "Makodra":
             return cls.from_makodra_dict(c)
+        if c.get("architecture") == "Funevik":
+            return cls.from_funevik_dict(c)
         archs = c.get("architectures") or []
         mt = (c.get("model_type") or "").lower()
         is_hybrid = "layer_types" in c and any(t == "linear_attention" for t in c["layer_types"])
@@ -413,6 +518,25 @@ def preset(name: str) -> ModelConfig:
                            layers=[LayerSpec(RecurrentSpec("wkv", 3, 40), mlp), LayerSpec(ChunkAttentionSpec(4, 2, 24, 40, 3.0, 48, True), None),
                                    LayerSpec(RecurrentSpec("general_delta", 5, 32), mlp),
                                    LayerSpec(ChunkAttentionSpec(2, 2, 48, 40, 2.0, 80, True), mlp)], name="tiny-makodra")
+    if n in ("funevik-2048", "funevik-1024"):
+        # random-init stand-ins with the layer sizes of a real small model: two memories, one latent and one full attention in turn
+        d, H, ff = (2048, 16, 5632) if n.endswith("2048") else (1024, 8, 2816)
+        dense = FeedForwardSpec("geglu", ff=ff)
+        moe = FeedForwardSpec("moe", expert=GluSpec(ff // 8), router=RouterSpec(32, 4, bias=True), shared=GluSpec(ff // 4), shared_gate=True)
+        mem = RecurrentSpec("mlstm", d // 256, 128, 256, 15.0)
+        four = [mem, mem, LatentAttentionSpec(H, 128, 128, 256, 192 ** -0.5, 768, RotarySpec(64, 10000.0), 1024, True),
+                GroupedAttentionSpec(H, H // 4, 128, 128, 128 ** -0.5, 4, RotarySpec(64, 500000.0), 50.0)]
+        return ModelConfig(arch="funevik", vocab_size=65536, hidden_size=d, n_layers=16, n_heads=H, n_kv_heads=H // 4, head_dim=128,
+                           ffn_size=0, rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, embed_scale=d ** 0.5,
+                           layers=[LayerSpec(m, dense if i % 2 else moe) for i, m in enumerate(four * 4)], name=n)
+    if n in ("tiny-funevik",):
+        moe = FeedForwardSpec("moe", expert=GluSpec(40), router=RouterSpec(6, 2, bias=True), shared=GluSpec(72), shared_gate=True)
+        return ModelConfig(arch="funevik", vocab_size=4096, hidden_size=136, n_layers=4, n_heads=3, n_kv_heads=3, head_dim=40,
+                           ffn_size=0, rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, embed_scale=3.0, name="tiny-funevik", layers=[
+                               LayerSpec(LatentAttentionSpec(3, 40, 24, 48, 0.2, 56, RotarySpec(8, 1000.0), 60, True), moe),
+                               LayerSpec(RecurrentSpec("mlstm", 3, 24, 40, 9.0), FeedForwardSpec("geglu", ff=200)),
+                               LayerSpec(GroupedAttentionSpec(4, 2, 24, 40, 0.3, 4, RotarySpec(12, 2000.0), 20.0), None),
+                               LayerSpec(RecurrentSpec("mlstm", 2, 48, 24, 12.0), moe)])
     raise KeyError(f"unknown preset {name!r}")
 
 

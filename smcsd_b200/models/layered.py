@@ -1,4 +1,4 @@
-"""What the layer-by-layer families (Pasizen, Makodra) have in common: padded weight layouts, checkpoints whose tensors are
+"""What the layer-by-layer families (Pasizen, Makodra, Funevik) have in common: padded weight layouts, checkpoints whose tensors are
 named per layer and checked against the configuration, activations rounded and padded for the GEMMs."""
 from __future__ import annotations
 
@@ -7,6 +7,7 @@ from typing import Iterator, List, Optional
 import torch
 
 from .config import ModelConfig
+from .llama import interleave_gate_up
 from .loader import Checkpoint
 
 GU_BLOCK = 64
@@ -21,6 +22,12 @@ def pad_to(w: torch.Tensor, *shape: int) -> torch.Tensor:
     out = torch.zeros(*shape, dtype=w.dtype, device=w.device)
     out[tuple(slice(0, n) for n in w.shape)] = w
     return out
+
+
+def pad_heads(w: torch.Tensor, heads: int, to: int) -> torch.Tensor:
+    """Rows [heads * size, d] -> [heads * to, d] with zero rows behind every head."""
+    n, d = w.shape
+    return pad_to(w.view(heads, n // heads, d), heads, to, d).view(heads * to, d)
 
 
 class LayeredModel:
@@ -67,7 +74,30 @@ class LayeredModel:
         finally:
             ck.close()
 
+    @staticmethod
+    def _pack_glu(mat, p: str, ff: int, d: int):
+        """Gate / up rows interleaved in blocks of GU_BLOCK channels, and the down matrix, of the gated unit named ``p``."""
+        f, d8 = round_up(ff, GU_BLOCK), round_up(d, 8)
+        gu = interleave_gate_up(pad_to(mat(p + "gate", ff, d), f, d8), pad_to(mat(p + "up", ff, d), f, d8), GU_BLOCK)
+        return gu, pad_to(mat(p + "down", d, ff), d, f)
+
+    def _pack_experts(self, mat, p: str, experts: int, ff: int, d: int):
+        """The same of all experts, stacked."""
+        packed = [self._pack_glu(mat, f"{p}e{e}.", ff, d) for e in range(experts)]
+        return torch.stack([g for g, _ in packed]), torch.stack([w for _, w in packed])
+
     # ---- plain-PyTorch forward ----------------------------------------------------------
+    @staticmethod
+    def _mix_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, run) -> torch.Tensor:
+        """fp32 sum over the chosen experts (ids and weights [T, top]); ``run(expert, rows of x)`` gives an expert's output."""
+        out = None
+        for e in idx.unique().tolist():
+            t, j = (idx == e).nonzero(as_tuple=True)
+            y = run(e, x[t])
+            out = torch.zeros(x.shape[0], y.shape[1], device=x.device) if out is None else out
+            out.index_add_(0, t, w[t, j].unsqueeze(1) * y)
+        return out
+
     def _act(self, h: torch.Tensor) -> torch.Tensor:
         """fp32 rows in the activation dtype, padded to the GEMM operand width."""
         d8 = round_up(h.shape[1], 8)

@@ -149,9 +149,10 @@ def short_conv(h: torch.Tensor, w: torch.Tensor, batch: ExtendBatch, history: to
 
 
 def latent_attention_reference(q: torch.Tensor, pool: torch.Tensor, block_table: torch.Tensor, batch: ExtendBatch,
-                               scale: float) -> torch.Tensor:
+                               scale: float, window: int = 0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention in latent space: q [T, H, R] (queries already multiplied by the key expansion), cached latents
-    ``pool`` [pages, >= R] read through the block table as keys and as values.  Returns fp32 [T, H, R]."""
+    ``pool`` [pages, >= R] read through the block table as keys and as values; with a ``window`` a token sees itself and the
+    window - 1 tokens before it, ``sink`` [H] are logits in the softmax sum without a value.  Returns fp32 [T, H, R]."""
     T, H, R = q.shape
     out = torch.empty(T, H, R, dtype=torch.float32, device=q.device)
     pref = batch.prefix_lens_host if batch.prefix_lens_host is not None else batch.prefix_lens.tolist()
@@ -162,9 +163,12 @@ def latent_attention_reference(q: torch.Tensor, pool: torch.Tensor, block_table:
         L = p + e
         c = pool[block_table[batch.rows[b].long(), :L].long()][:, :R].float()
         s = torch.einsum("ehr,lr->hel", q[t0:t0 + e].float(), c) * scale
-        causal = torch.arange(L, device=q.device).unsqueeze(0) <= (p + torch.arange(e, device=q.device)).unsqueeze(1)
-        s = s.masked_fill(~causal, float("-inf"))
-        out[t0:t0 + e] = torch.einsum("hel,lr->ehr", torch.softmax(s, dim=-1), c)
+        i, j = torch.arange(p, L, device=q.device).unsqueeze(1), torch.arange(L, device=q.device).unsqueeze(0)
+        hidden = (j > i) | (i - j >= window) if window else j > i
+        s = s.masked_fill(hidden, float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink.view(H, 1, 1).expand(H, e, 1)], dim=-1)
+        out[t0:t0 + e] = torch.einsum("hel,lr->ehr", torch.softmax(s, dim=-1)[..., :L], c)
         t0 += e
     return out
 
@@ -211,7 +215,23 @@ def hyper_write(x: torch.Tensor, y: torch.Tensor, w_mix: torch.Tensor, w_out: to
     return torch.einsum("tsd,su->tud", x, w_mix) + w_out.view(1, -1, 1) * y.unsqueeze(1)
 
 
+def route_top(z: torch.Tensor, top: int):
+    """Router logits [T, E] -> (expert ids [T, top], weights [T, top]): the largest logits, softmax over the chosen ones."""
+    best = z.float().topk(top, dim=-1)
+    return best.indices, torch.softmax(best.values, dim=-1)
+
+
 # ---- positions, token shift and memory matrices
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float) -> torch.Tensor:
+    """fp32 x [T, ..., n]: the first ``dims`` entries rotated by position, entries 2i and 2i + 1 paired."""
+    ang = positions.double().unsqueeze(1) * base ** (-torch.arange(0, dims, 2, device=x.device).double() / dims)
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [dims // 2]
+    c, s = ang.cos().float().view(shape), ang.sin().float().view(shape)
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    return torch.cat([torch.stack([u * c - v * s, v * c + u * s], dim=-1).flatten(-2), x[..., dims:]], dim=-1)
+
+
+
 def sinusoidal_positions(positions: torch.Tensor, d: int, base: float = 10000.0) -> torch.Tensor:
     """fp32 [T, d]: entry 2i is sin(p base^(-2i/d)), entry 2i + 1 the cosine of the same angle."""
     c = torch.arange(d, device=positions.device)
@@ -265,16 +285,42 @@ def bonus_memory(state: torch.Tensor, r, w, k, v, bonus) -> torch.Tensor:
     return out
 
 
+def soft_cap(z: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(z / cap)
+
+
+NORMALISER_EPS = 1e-6
+
+
+def gated_memory(state: torch.Tensor, top: torch.Tensor, q, k, v, i, f) -> torch.Tensor:
+    """Matrix memory of one sequence with log input gates i and log forget gates f [T, H]: with the running maximum
+    m <- max(f + m, i), M and the normaliser n decay by exp(f + m_old - m) and gain exp(i - m) times k v^T and k; the read-out
+    M^T q is divided by max(|n q|, exp(-m)) + NORMALISER_EPS.  q, k [T, H, dk], v [T, H, dv]; ``state`` [H, dv + 1, dk] fp32 holds M transposed
+    and n as its last row, ``top`` [H, 1, 1] the maximum; both are advanced in place.  Returns [T, H, dv]."""
+    M, m, out = state.clone(), top[:, 0, 0].clone(), torch.empty_like(v)
+    v1 = torch.cat([v, torch.ones_like(v[..., :1])], dim=-1)
+    for t in range(q.shape[0]):
+        m_new = torch.maximum(f[t] + m, i[t])
+        keep, add = torch.exp(f[t] + m - m_new), torch.exp(i[t] - m_new)
+        m = m_new
+        M = M * keep.view(-1, 1, 1) + (v1[t] * add.unsqueeze(1)).unsqueeze(-1) * k[t].unsqueeze(1)
+        o = (M * q[t].unsqueeze(1)).sum(-1)
+        out[t] = o[:, :-1] / (torch.maximum(o[:, -1].abs(), torch.exp(-m)) + NORMALISER_EPS).unsqueeze(1)
+    state.copy_(M)
+    top[:, 0, 0] = m
+    return out
+
+
 def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
-                              batch: ExtendBatch, kv_heads: int, scale: float, r1: torch.Tensor, r2: torch.Tensor,
-                              chunk: int) -> torch.Tensor:
-    """Causal attention inside chunks of ``chunk`` positions with scores scale q.k - r1 ln(1 + r2 distance) and a sink of
-    score 0.  q [T, H, D]; pools [pages, kv_heads * width]; returns fp32 [T, H, value width]."""
+                              batch: ExtendBatch, kv_heads: int, scale: float, r1: Optional[torch.Tensor],
+                              r2: Optional[torch.Tensor], chunk: int, softcap: float = 0.0) -> torch.Tensor:
+    """Causal attention inside chunks of ``chunk`` positions (0: no chunks) with scores scale q.k - r1 ln(1 + r2 distance), or
+    soft-capped ones, and a sink of score 0.  q [T, H, D]; pools [pages, kv_heads * width]; returns fp32 [T, H, value width]."""
     T, H, D = q.shape
     rep, V = H // kv_heads, v_pool.shape[1] // kv_heads
     out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
     pref = batch.prefix_lens_host if batch.prefix_lens_host is not None else batch.prefix_lens.tolist()
-    t0 = 0
+    chunk, t0 = chunk or 1 << 30, 0
     for b, (p, e) in enumerate(zip(pref, batch.lens())):
         if e == 0:
             continue
@@ -286,7 +332,10 @@ def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
         j = torch.arange(lo, L, device=q.device).unsqueeze(0)
         dist = (i - j).clamp(min=0).float()
         s = torch.einsum("ehd,lhd->hel", q[t0:t0 + e].float(), kk) * scale
-        s = s - r1.view(H, 1, 1) * torch.log1p(r2.view(H, 1, 1) * dist)
+        if softcap:
+            s = soft_cap(s, softcap)
+        if r1 is not None:
+            s = s - r1.view(H, 1, 1) * torch.log1p(r2.view(H, 1, 1) * dist)
         s = s.masked_fill((j > i) | (i // chunk != j // chunk), float("-inf"))
         top = s.amax(-1, keepdim=True).clamp(min=0.0)
         ex = torch.exp(s - top)

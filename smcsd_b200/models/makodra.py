@@ -26,19 +26,13 @@ import torch
 
 from ..memory.pools import KVSpec, StateSpec
 from .config import ChunkAttentionSpec, LayerSpec
-from .layered import GU_BLOCK, LayeredModel, pad_to, round_up
+from .layered import GU_BLOCK, LayeredModel, pad_heads, pad_to, round_up
 from .layers import (ExtendBatch, bonus_memory, chunk_attention_reference, delta_memory, rms_unit, sinusoidal_positions, swiglu,
                      token_shift)
-from .llama import interleave_gate_up, split_gate_up
+from .llama import split_gate_up
 
 SHIFTED = "rkvgw"                            # order of the shifted inputs
 DELTA_LOG_DECAY = math.exp(-0.5)             # largest -ln of a delta-rule decay
-
-
-def pad_heads(w: torch.Tensor, heads: int, to: int) -> torch.Tensor:
-    """Rows [heads * size, d] -> [heads * to, d] with zero rows behind every head."""
-    n, d = w.shape
-    return pad_to(w.view(heads, n // heads, d), heads, to, d).view(heads * to, d)
 
 
 @dataclass
@@ -143,10 +137,8 @@ class MakodraModel(LayeredModel):
                     n_shift += 1
                 n_rec += 1
             if f is not None:
-                ff = round_up(f.ff, GU_BLOCK)
                 L.norm2 = vec(p + "norm2", d)
-                L.wgu = interleave_gate_up(pad_to(mat(p + "mlp.gate", f.ff, d), ff, d8), pad_to(mat(p + "mlp.up", f.ff, d), ff, d8), GU_BLOCK)
-                L.wdown = pad_to(mat(p + "mlp.down", d, f.ff), d, ff)
+                L.wgu, L.wdown = self._pack_glu(mat, p + "mlp.", f.ff, d)
             self.layers.append(L)
         return self
 

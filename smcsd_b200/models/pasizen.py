@@ -29,7 +29,7 @@ from .config import LayerSpec
 from .layered import GU_BLOCK, LayeredModel, pad_to, round_up
 from .layers import (ExtendBatch, clamped_glu, hyper_read, hyper_write, latent_attention_reference, poly_norm, rms_unit,
                      route_grouped, short_conv)
-from .llama import interleave_gate_up, split_gate_up
+from .llama import split_gate_up
 
 
 @dataclass
@@ -97,11 +97,6 @@ class PasizenModel(LayeredModel):
         def hyper(p):
             return HyperWeights(vec(p + "in", S), vec(p + "out", S), vec(p + "mix", S, S))
 
-        def glu(p, ff):
-            f = round_up(ff, GU_BLOCK)
-            gu = interleave_gate_up(pad_to(mat(p + "gate", ff, d), f, d8), pad_to(mat(p + "up", ff, d), f, d8), GU_BLOCK)
-            return gu, pad_to(mat(p + "down", d, ff), d, f)
-
         self.embed, self.pos = mat("embed", c.vocab_size, d), mat("pos", c.max_position, d)
         self.final_norm = vec("final.norm", d)
         self.lm_head = pad_to(mat("head", c.vocab_size, d), c.vocab_size, d8)
@@ -125,10 +120,9 @@ class PasizenModel(LayeredModel):
                     L.poly = vec(p + "mlp.act", 4)
                 else:
                     L.router = pad_to(mat(p + "mlp.router", f.router.experts, d), f.router.experts, d8)
-                    packed = [glu(f"{p}mlp.e{e}.", f.expert.ff) for e in range(f.router.experts)]
-                    L.e_gu, L.e_down = torch.stack([g for g, _ in packed]), torch.stack([w for _, w in packed])
+                    L.e_gu, L.e_down = self._pack_experts(mat, p + "mlp.", f.router.experts, f.expert.ff, d)
                     if f.shared is not None:
-                        L.s_gu, L.s_down = glu(p + "mlp.shared.", f.shared.ff)
+                        L.s_gu, L.s_down = self._pack_glu(mat, p + "mlp.shared.", f.shared.ff, d)
             self.layers.append(L)
         return self
 
@@ -183,11 +177,7 @@ class PasizenModel(LayeredModel):
             return (a @ L.wdown[:, :f.ff].t()).float()
         r = f.router
         idx, w = route_grouped(h @ L.router[:, :h.shape[1]].float().t(), r.top, r.groups, r.keep)
-        out = torch.zeros_like(h)
-        for e in range(r.experts):
-            t, j = (idx == e).nonzero(as_tuple=True)
-            if t.numel():
-                out.index_add_(0, t, w[t, j].unsqueeze(1) * self._glu(x[t], L.e_gu[e], L.e_down[e], f.expert.limit))
+        out = self._mix_experts(x, idx, w, lambda e, rows: self._glu(rows, L.e_gu[e], L.e_down[e], f.expert.limit))
         if f.shared is not None:
             out = out + self._glu(x, L.s_gu, L.s_down, f.shared.limit)
         return out
