@@ -18,8 +18,8 @@ OUT = os.path.join(HERE, "libsmcsd_b200.so")
 OBJ_DIR = os.path.join(HERE, "build")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 # Sources whose fp32 arithmetic serves 32-bit runs: compiled with IEEE division, square root and exponentials.
-PRECISE = {"chunk_attention.cu", "gemm_f32.cu", "hyper.cu", "latent_attention.cu", "memory_scan.cu", "moe.cu",
-           "post_norm.cu"}
+PRECISE = {"chunk_attention.cu", "conv_heads.cu", "gemm_f32.cu", "hyper.cu", "latent_attention.cu", "memory_scan.cu", "moe.cu",
+           "post_norm.cu", "side_norm.cu"}
 
 
 def sources():
@@ -53,15 +53,27 @@ def build(verbose: bool = False, force: bool = False) -> str:
     if verbose:
         flags += ["-Xptxas", "-v"]
 
+    headers = hashlib.sha256()
+    for f in sorted(os.listdir(CSRC)):
+        if not f.endswith(".cu"):
+            with open(os.path.join(CSRC, f), "rb") as fh:
+                headers.update(f.encode() + fh.read())
+
     def compile_one(src: str) -> str:
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
         fast = [] if os.path.basename(src) in PRECISE else ["--use_fast_math"]
+        with open(src, "rb") as fh:
+            made_of = hashlib.sha256(headers.digest() + fh.read() + " ".join([nvcc] + flags + fast).encode()).hexdigest()
+        if not force and os.path.exists(obj) and os.path.exists(obj + ".txt") and open(obj + ".txt").read() == made_of:
+            return obj
         cmd = [nvcc] + flags + fast + ["-c", src, "-o", obj]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if verbose or r.returncode != 0:
             sys.stderr.write(f"$ {' '.join(cmd)}\n{r.stdout}{r.stderr}\n")
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed for {src}")
+        with open(obj + ".txt", "w") as f:
+            f.write(made_of)
         return obj
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:

@@ -1,5 +1,5 @@
-// Attention inside chunks of the sequence, with grouped heads, unit-rms queries and keys, a logarithmic distance bias, a sink
-// in the softmax sum and a gate on the output.
+// Attention inside chunks of the sequence (or over all of it), with grouped heads, unit-rms queries and keys, a logarithmic
+// distance bias or soft-capped scores, a sink in the softmax sum and a gate on the output.
 //
 //   heads_new     per new token: queries and keys divided by their root mean square per head, values mixed with the first
 //                 layer's; keys and values go to the token's cache page
@@ -193,6 +193,7 @@ __global__ void __launch_bounds__(CA_WARPS * 32) chunk_attn_kernel(const ChunkAt
     fetch(next);
     next = page_of(k + 2 * CA_WARPS * 4);
     float sc = scatter_sum<RH>(s, sub) * a.scale;
+    if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
     if (a.r1 != nullptr) sc -= r1 * logf(1.0f + r2 * (float)max(pos - k, 0));
     if (k >= k_end) sc = -INFINITY;
     const float m2 = fmaxf(m, sc), base = m2 == -INFINITY ? 0.f : m2, p = expf(sc - base);
@@ -278,7 +279,7 @@ __global__ void __launch_bounds__(CA_WARPS * 32) chunk_attn_kernel(const ChunkAt
     }
     o /= sum;
     const int col = (h0 + h) * a.V + c;
-    if (a.gate != nullptr) o /= 1.0f + expf(-a.gate[(size_t)tok * a.ldg + col]);
+    if (a.gate != nullptr) o /= 1.0f + expf(-a.gate[(size_t)tok * a.ldg + (a.gate_heads ? h0 + h : col)]);
     reinterpret_cast<AT*>(a.out)[(size_t)tok * a.H * a.V + col] = from_f32<AT>(o);
   }
   __syncwarp();

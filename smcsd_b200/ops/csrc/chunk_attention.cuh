@@ -11,12 +11,14 @@ struct ChunkAttnArgs {
   void* out;                // [T, H * V], already multiplied by the gate
   const float* gate;        // [T, ldg]: H * V logits of the output gate (null: no gate)
   int ldg;
+  int gate_heads;           // the gate has one logit per head instead
   const int* block_table;
   int bt_stride, bt_rows, n_pages, H, G, D, V;
   int chunk;                // positions of one chunk: a token sees its own chunk only
   float scale;
   const float* r1;          // [H] distance bias r1 ln(1 + r2 distance), taken off the score (null: none)
   const float* r2;
+  float softcap;            // score <- softcap tanh(score / softcap) before the bias (0: none)
   int sink;                 // one more term exp(0) in the softmax sum, without a value
   Ragged r;
   int* status;

@@ -76,6 +76,7 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
   fetch(0, 0);
   cp_async_commit();
   const float sc = a.scale * 1.4426950408889634f;
+  const float cap = a.softcap * 1.4426950408889634f, cap_in = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
   const float r1 = a.r1 != nullptr ? a.r1[h] : 0.f, r2 = a.r1 != nullptr ? a.r2[h] : 0.f;
   const int row0 = warp * 16 + (lane >> 2);                // this thread's rows: row0 and row0 + 8
   const int pos[2] = {p0 + row0, p0 + row0 + 8};
@@ -122,6 +123,7 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
         for (int e = 0; e < 4; ++e) {
           const int r = e >> 1, key = k0 + j * 8 + (lane & 3) * 2 + (e & 1);
           float v = s[j][e] * sc;
+          if (a.softcap > 0.f) v = cap * (1.0f - __fdividef(2.0f, 1.0f + exp2f(v * cap_in)));     // cap tanh
           if (a.r1 != nullptr) v = fmaf(-r1, __log2f(fmaf(r2, (float)max(pos[r] - key, 0), 1.0f)), v);
           v = (key > pos[r] || key < lo[r]) ? -INFINITY : v;
           s[j][e] = v;
@@ -174,13 +176,17 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
     const float mm = a.sink ? fmaxf(m[r], 0.f) : m[r];
     const float f = exp2f(m[r] - mm), inv = f / (l[r] * f + (a.sink ? exp2f(-mm) : 0.f));
     const size_t at = (size_t)(t0 + row) * a.H * a.V + (size_t)h * a.V;
-    const float* gate = a.gate != nullptr ? a.gate + (size_t)(t0 + row) * a.ldg + (size_t)h * a.V : nullptr;
+    const float* gate = a.gate != nullptr ? a.gate + (size_t)(t0 + row) * a.ldg + (a.gate_heads ? h : h * a.V) : nullptr;
+    const float head_gate = gate != nullptr && a.gate_heads ? 1.0f / (1.0f + __expf(-gate[0])) : 1.0f;
 #pragma unroll
     for (int j = 0; j < NV * 2; ++j) {
       const int c = j * 8 + (lane & 3) * 2;
       if (c >= a.V) continue;
       float v0 = o[j][r * 2] * inv, v1 = o[j][r * 2 + 1] * inv;
-      if (gate != nullptr) {
+      if (a.gate_heads) {
+        v0 *= head_gate;
+        v1 *= head_gate;
+      } else if (gate != nullptr) {
         v0 /= 1.0f + __expf(-gate[c]);
         v1 /= 1.0f + __expf(-gate[c + 1]);
       }

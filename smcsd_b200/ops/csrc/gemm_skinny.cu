@@ -67,7 +67,8 @@ struct GroupLink {
   int x_cols, out_cols;     // activation / output columns between groups (batched)
   const int4* tiles;        // tiled: {group, first row, end row, -}; entries past the used ones have first == end
   int max_tiles, bn;        // tiled: table length, rows per tile (the token-tile width the table was made for)
-  int act;                  // gated epilogue: 0 silu(g) * u, 1 clamped: min(g, limit) * sigmoid(slope g) * (clamp(u) + 1)
+  int act;                  // gated epilogue: 0 silu(g) * u, 1 clamped: min(g, limit) * sigmoid(slope g) * (clamp(u) + 1),
+                            // 2 gelu(g) * u in the tanh form
   float limit, slope;
 };
 
@@ -109,6 +110,7 @@ __device__ __forceinline__ float gated_unit(const GroupLink& a, float g, float u
     u = fminf(fmaxf(u, -a.limit), a.limit);
     return g / (1.0f + __expf(-a.slope * g)) * (u + 1.0f);
   }
+  if (GRP && a.act == 2) return gelu_tanh(g) * u;
   return g / (1.0f + __expf(-g)) * u;
 }
 

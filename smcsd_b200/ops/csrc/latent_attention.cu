@@ -2,39 +2,71 @@
 // as value.  Queries arrive already multiplied by the key expansion, so a head's score is a dot product of length R with
 // the cached row, and the attended rows go through the value expansion afterwards.
 //
-//   latent_new      per new token: query columns of the projection in the activation type, latent columns divided by their
-//                   root mean square (and weighted) into the token's cache page
+//   latent_new      per new token: query columns of the projection in the activation type (or, for queries that go through a
+//                   latent of their own, that latent normed), latent columns divided by their root mean square (and weighted)
+//                   into the token's cache page, the rotated key behind them
 //   latent_attn     causal attention over the paged rows, one (token, head) per CTA, four warps over the keys: the form
 //                   32-bit runs use; the tensor-core form is in latent_attention_tc.cu
 #include "latent_attention.cuh"
+#include "rotary.cuh"
 
 namespace smc {
 
+struct LatentNewArgs {
+  const float* proj;        // [T, ldp]: nq query columns, latent columns from c_off on, the rotated key behind them
+  int ldp, nq, c_off, R, rot;
+  const float* q_norm;      // [nq_real] the query columns are a latent of nq_real values: normed and weighted (null: copied)
+  int nq_real;
+  const float* c_norm;      // [R]
+  float eps;
+  const double* freq;       // [rot / 2] angles per position
+  const int* positions;
+  void* q;                  // [T, ldq] (optional)
+  int ldq;
+  void* pool;               // [n_pages + 1, ldc]
+  int ldc, n_pages;
+  const int* locs;
+  int* status;
+  int pdl;
+};
+
 template <typename AT>
-__global__ void __launch_bounds__(256) latent_new_kernel(const float* proj, int ldp, int nq, int R,
-                                                         const float* c_norm, float eps, AT* q,
-                                                         int ldq, AT* pool, int ldc, int n_pages,
-                                                         const int* cache_locs, int* status, int pdl) {
+__global__ void __launch_bounds__(256) latent_new_kernel(const LatentNewArgs a) {
   __shared__ float red[32];
-  if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int t = blockIdx.x;
-  const float* row = proj + (size_t)t * ldp;
-  if (q != nullptr) {
-    if (((nq | ldp | ldq) & 3) == 0)
-      for (int i = threadIdx.x * 4; i < nq; i += blockDim.x * 4) store4(q + (size_t)t * ldq + i, load4(row + i));
+  const float* row = a.proj + (size_t)t * a.ldp;
+  AT* q = reinterpret_cast<AT*>(a.q) + (size_t)t * a.ldq;
+  if (a.q != nullptr && a.q_norm != nullptr) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.nq_real; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+    const float inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)a.nq_real + a.eps);
+    for (int i = threadIdx.x; i < a.nq; i += blockDim.x) q[i] = from_f32<AT>(i < a.nq_real ? row[i] * inv * a.q_norm[i] : 0.f);
+  } else if (a.q != nullptr) {
+    if (((a.nq | a.ldp | a.ldq) & 3) == 0)
+      for (int i = threadIdx.x * 4; i < a.nq; i += blockDim.x * 4) store4(q + i, load4(row + i));
     else
-      for (int i = threadIdx.x; i < nq; i += blockDim.x) q[(size_t)t * ldq + i] = from_f32<AT>(row[i]);
+      for (int i = threadIdx.x; i < a.nq; i += blockDim.x) q[i] = from_f32<AT>(row[i]);
   }
-  const float* c = row + nq;
+  const float* c = row + a.c_off;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < R; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
-  const float inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)R + eps);
-  int page = cache_locs[t];
-  if (page < 0 || page > n_pages) {
-    if (threadIdx.x == 0) atomicOr(status, SMC_ERR_BOUNDS);
+  for (int i = threadIdx.x; i < a.R; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
+  const float inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)a.R + a.eps);
+  int page = a.locs[t];
+  if (page < 0 || page > a.n_pages) {
+    if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
     page = 0;
   }
-  for (int i = threadIdx.x; i < R; i += blockDim.x) pool[(size_t)page * ldc + i] = from_f32<AT>(c[i] * inv * c_norm[i]);
+  AT* out = reinterpret_cast<AT*>(a.pool) + (size_t)page * a.ldc;
+  for (int i = threadIdx.x; i < a.R; i += blockDim.x) out[i] = from_f32<AT>(c[i] * inv * a.c_norm[i]);
+  if (a.rot > 0) {
+    const int p = a.positions[t];
+    for (int i = threadIdx.x; i < a.rot / 2; i += blockDim.x) {
+      const float2 v = rotate_pair(make_float2(c[a.R + 2 * i], c[a.R + 2 * i + 1]), a.freq, i, p);
+      out[a.R + 2 * i] = from_f32<AT>(v.x);
+      out[a.R + 2 * i + 1] = from_f32<AT>(v.y);
+    }
+  }
 }
 
 template <int NR, typename AT>      // NR = ldc / 32 values per lane
@@ -56,7 +88,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
   float qv[NR], acc[NR], m = -INFINITY, l = 0.f;
 #pragma unroll
   for (int j = 0; j < NR; ++j) { qv[j] = to_f32<AT>(q[lane + 32 * j]) * a.scale; acc[j] = 0.f; }
-  for (int k = warp; k < n_keys; k += 4) {
+  for (int k = (a.window > 0 ? max(0, n_keys - a.window) : 0) + warp; k < n_keys; k += 4) {
     int page = bt[k];
     if (page < 0 || page > a.n_pages) { atomicOr(a.status, SMC_ERR_BOUNDS); page = 0; }
     const AT* c = pool + (size_t)page * a.ldc;
@@ -74,8 +106,9 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
   for (int j = 0; j < NR; ++j) s_acc[warp][lane + 32 * j] = acc[j];
   if (lane == 0) { s_m[warp] = m; s_l[warp] = l; }
   __syncthreads();
-  const float mm = fmaxf(fmaxf(s_m[0], s_m[1]), fmaxf(s_m[2], s_m[3]));
-  float f[4], lt = 0.f;
+  float mm = fmaxf(fmaxf(s_m[0], s_m[1]), fmaxf(s_m[2], s_m[3]));
+  if (a.sink != nullptr) mm = fmaxf(mm, a.sink[head]);
+  float f[4], lt = a.sink != nullptr ? expf(a.sink[head] - mm) : 0.f;
 #pragma unroll
   for (int w = 0; w < 4; ++w) { f[w] = expf(s_m[w] - mm); lt = fmaf(s_l[w], f[w], lt); }
   AT* o = reinterpret_cast<AT*>(a.out) + ((size_t)tok * a.H + head) * a.ldc;
@@ -87,7 +120,8 @@ template <typename AT>
 static int latent_attn_dispatch(const LatentArgs& a, cudaStream_t st) {
   const dim3 grid((unsigned)(a.r.n_blk * a.r.B), (unsigned)a.H), block(128);
 #define SMC_LA(NR) case NR: return launch_pdl(latent_attn_kernel<NR, AT>, grid, block, 0, st, a.pdl, a);
-  switch (a.ldc / 32) { SMC_LA(2) SMC_LA(4) SMC_LA(6) SMC_LA(8) SMC_LA(10) SMC_LA(12) SMC_LA(14) SMC_LA(16) SMC_LA(20) SMC_LA(24) SMC_LA(32) }
+  switch (a.ldc / 32) { SMC_LA(2) SMC_LA(4) SMC_LA(6) SMC_LA(8) SMC_LA(10) SMC_LA(12) SMC_LA(14) SMC_LA(16) SMC_LA(18)
+                        SMC_LA(20) SMC_LA(22) SMC_LA(24) SMC_LA(26) SMC_LA(28) SMC_LA(30) SMC_LA(32) }
 #undef SMC_LA
   return -99;
 }
@@ -96,17 +130,14 @@ static int latent_attn_dispatch(const LatentArgs& a, cudaStream_t st) {
 
 SMC_API int smc_latent_args_size() { return (int)sizeof(smc::LatentArgs); }
 
-// proj fp32 [M, ldp]: nq query columns, then R latent columns.  q (optional) [M, ldq]; pool [n_pages + 1, ldc].
-SMC_API int smc_latent_new(const float* proj, int ldp, int nq, int R, const float* c_norm, float eps, void* q, int ldq,
-                           void* pool, int ldc, int n_pages, const int* cache_locs, int M, int* status, int f32, int pdl,
-                           cudaStream_t st) {
+SMC_API int smc_latent_new_args_size() { return (int)sizeof(smc::LatentNewArgs); }
+
+SMC_API int smc_latent_new(const smc::LatentNewArgs* a, int T, int f32, cudaStream_t st) {
   using namespace smc;
-  if (M <= 0) return 0;
-  if (f32)
-    return launch_pdl(latent_new_kernel<float>, dim3(M), dim3(256), 0, st, pdl, proj, ldp, nq, R, c_norm, eps, (float*)q, ldq,
-                      (float*)pool, ldc, n_pages, cache_locs, status, pdl);
-  return launch_pdl(latent_new_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, st, pdl, proj, ldp, nq, R, c_norm, eps,
-                    (__nv_bfloat16*)q, ldq, (__nv_bfloat16*)pool, ldc, n_pages, cache_locs, status, pdl);
+  if (T <= 0) return 0;
+  if (a->rot % 2 || a->R + a->rot > a->ldc) return -98;
+  return f32 ? launch_pdl(latent_new_kernel<float>, dim3(T), dim3(256), 0, st, a->pdl, *a)
+             : launch_pdl(latent_new_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, a->pdl, *a);
 }
 
 SMC_API int smc_latent_attn(const smc::LatentArgs* a, int f32, cudaStream_t st) {

@@ -11,6 +11,8 @@ struct LatentArgs {
   const int* block_table;
   int bt_stride, bt_rows, n_pages, H, ldc;
   float scale;
+  int window;               // a token sees itself and the window - 1 tokens before it (0: all)
+  const float* sink;        // [H] logits in the softmax sum without a value (null: none)
   Ragged r;
   int* status;
   int pdl;

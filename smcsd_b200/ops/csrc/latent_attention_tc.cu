@@ -5,7 +5,7 @@
 // as keys and as values from the same shared-memory bytes:
 //     S = Q C^T        UMMA 128 x 64 x R, C taken K-major
 //     softmax          two threads per query row (both take the row's maximum, each exponentiates half of the tile's
-//                      columns), causal limit per row, P as bf16 into a SWIZZLE_128B tile
+//                      columns), causal and window limit per row, an optional sink logit per head in the sum, P as bf16 into a SWIZZLE_128B tile
 //     O += P C         UMMA 128 x R x 64 accumulating in tensor memory, C taken MN-major
 // Two score buffers (64 columns each) and up to 384 output columns live in tensor memory; wider latents split their output
 // columns over two CTAs that both compute the scores.  The exponent reference of a row only moves when its maximum grew by
@@ -30,6 +30,7 @@ constexpr int LT_PANEL_C = LT_BK * 128;
 constexpr int LT_O_COL = 2 * LT_BK;             // first output column in tensor memory
 constexpr int LT_MAX_STAGES = 6;
 constexpr int LT_MAX_SPLITS = 8;                // CTAs of a cluster
+constexpr float LT_LOG2E = 1.4426950408889634f;
 
 // NPAN: panels of 64 values per cached row.  Ring depth within 227 KB next to the Q tile and two P tiles.
 template <int NPAN> struct LtCfg {
@@ -51,6 +52,8 @@ struct LatentTcParams {
   const int* block_table;
   int bt_stride, bt_rows, n_pages, H, ldc, KS, MT, T;
   float scale_log2;
+  int window;                    // 0: all
+  const float* sink;             // [H] (null: none)
   Ragged r;
   int* status;
   int pdl;
@@ -139,9 +142,11 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
   const int pos0 = b.prefix + b.start;                                         // position of the block's first token
   const int lim_min = pos0 + row0 / p.H + 1;                                   // keys the tile's first row sees
   const int n_keys = n_rows > 0 ? pos0 + (row0 + n_rows - 1) / p.H + 1 : 0;
-  int per = (n_keys + p.KS - 1) / p.KS;
+  const int lo_min = p.window > 0 ? max(0, lim_min - p.window) : 0;            // first key the tile's first row sees
+  const int lo_max = p.window > 0 ? max(0, n_keys - p.window) : 0;             // .. the last row
+  int per = (n_keys - lo_min + p.KS - 1) / p.KS;
   per = (per + LT_BK - 1) / LT_BK * LT_BK;
-  const int kb = ks * per, ke = min(n_keys, kb + per);
+  const int kb = lo_min + ks * per, ke = min(n_keys, kb + per);
   const int n_tiles = ke > kb ? (ke - kb + LT_BK - 1) / LT_BK : 0;
   const int vpan = vs * C::OPAN, n_opan = min(C::OPAN, NPAN - vpan);           // this CTA's output panels
 
@@ -192,7 +197,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
         const int base = __shfl_sync(0xffffffffu, pa, 0), key_end = kb + (j + 1) * LT_BK;
         const bool asc = __all_sync(0xffffffffu, pa == base + lane && pb == base + 32 + lane);
         // descending pages reverse the keys inside the tile, which is fine where every row sees all of them
-        const bool desc = __all_sync(0xffffffffu, pa == base - lane && pb == base - 32 - lane) && base >= LT_BK && key_end <= lim_min;
+        const bool desc = __all_sync(0xffffffffu, pa == base - lane && pb == base - 32 - lane) && base >= LT_BK && key_end <= lim_min &&
+                          key_end - LT_BK >= lo_max;
         const bool run = key_end <= ke && base >= 1 && (asc || desc);
         uint8_t* c_ptr = c_s + (size_t)st * C_BYTES;
         if (run) {
@@ -275,16 +281,18 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
     const uint32_t lane_off = ((uint32_t)((warp & 3) * 32)) << 16;
     const bool real = r < n_rows;
     const int lim = real ? pos0 + (row0 + r) / p.H + 1 : ke;             // keys [0, lim) are visible (spare rows: unmasked)
+    const int lo = real && p.window > 0 ? max(0, lim - p.window) : 0;    // .. from here on
     float m_ref = -INFINITY, l = 0.f;                                    // exponent reference (log2 domain), running sum
     bool alive = true;
     const bool idle = (warp & 3) * 32 >= n_rows;                         // no real row in this warp: keep the protocol only
     for (int j = 0; j < n_tiles; ++j) {
-      const int nv = min(lim, ke) - kb - j * LT_BK;                      // visible keys of this tile (may be <= 0)
+      const int nv = min(lim, ke) - kb - j * LT_BK;                      // columns [nl, nv) of this tile are visible (may be none)
+      const int nl = lo - kb - j * LT_BK;
       if (!__all_sync(0xffffffffu, lt_wait(S, p.status, &S.s_full[j & 1], (uint32_t)(j >> 1) & 1u))) { alive = false; break; }
       tc_fence_after();
       uint32_t x[HB];
       float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      const bool full = __all_sync(0xffffffffu, nv >= LT_BK);
+      const bool full = __all_sync(0xffffffffu, nv >= LT_BK && nl <= 0);
       if (!idle) {
         const uint32_t ts = tmem_base + (uint32_t)(j & 1) * LT_BK + lane_off;
         uint32_t y[HB];                               // the other half: only its maximum is needed here
@@ -298,11 +306,11 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
 #pragma unroll
           for (int i = 0; i < HB; ++i) m4[i & 3] = fmaxf(m4[i & 3], fmaxf(__uint_as_float(x[i]), __uint_as_float(y[i])));
         } else {
-          const int nx = nv - half * HB, ny = nv - (half ^ 1) * HB;
+          const int nx = nv - half * HB, ny = nv - (half ^ 1) * HB, lx = nl - half * HB, ly = nl - (half ^ 1) * HB;
 #pragma unroll
           for (int i = 0; i < HB; ++i) {
-            if (i < nx) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(x[i]));
-            if (i < ny) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(y[i]));
+            if (i < nx && i >= lx) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(x[i]));
+            if (i < ny && i >= ly) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(y[i]));
           }
         }
       }
@@ -339,9 +347,9 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       } else {
         const float ref = m_ref == -INFINITY ? 0.f : m_ref;
         if (!full) {                                  // keys the row does not see: exp2 of -inf
-          const int nx = nv - half * HB;
+          const int nx = nv - half * HB, lx = nl - half * HB;
 #pragma unroll
-          for (int i = 0; i < HB; ++i) x[i] = i < nx ? x[i] : 0xff800000u;
+          for (int i = 0; i < HB; ++i) x[i] = i < nx && i >= lx ? x[i] : 0xff800000u;
         }
         float s4[4] = {0.f, 0.f, 0.f, 0.f};
         uint32_t w[HB / 2];
@@ -377,6 +385,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
       st_m[r] = write ? m_ref : -INFINITY;
       st_l[r] = write ? l : 0.f;                       // 0: this split holds nothing for the row
     }
+    if (p.KS == 1 && p.sink != nullptr && write) l += exp2f(p.sink[(row0 + r) % p.H] * LT_LOG2E - m_ref);
     if (n_tiles > 0 && alive && !idle) {
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       float* po = reinterpret_cast<float*>(q_s) + r * C::OLD;       // operands and tiles are no longer needed
@@ -420,9 +429,10 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_tc_kernel(const LatentTc
         ls = ld_dsmem_f32(smem_u32(st_l + r), (uint32_t)lane);
         ms = ld_dsmem_f32(smem_u32(st_m + r), (uint32_t)lane);
       }
-      const float mm = warp_max(ls > 0.f ? ms : -INFINITY);
+      const float snk = p.sink != nullptr ? p.sink[(row0 + r) % p.H] * LT_LOG2E : -INFINITY;
+      const float mm = fmaxf(warp_max(ls > 0.f ? ms : -INFINITY), snk);
       float f = ls > 0.f ? exp2f(ms - mm) : 0.f;
-      f *= 1.0f / warp_sum(ls * f);
+      f *= 1.0f / (warp_sum(ls * f) + (p.sink != nullptr ? exp2f(snk - mm) : 0.f));
       float a0 = 0.f, a1 = 0.f;
 #pragma unroll
       for (int q = 0; q < LT_MAX_SPLITS; ++q) {
@@ -493,7 +503,8 @@ SMC_API int smc_latent_attn_tc(const smc::LatentArgs* a, int tokens, int blk_row
   p.pool = (const __nv_bfloat16*)a->pool; p.out = (__nv_bfloat16*)a->out;
   p.block_table = a->block_table; p.bt_stride = a->bt_stride; p.bt_rows = a->bt_rows; p.n_pages = a->n_pages;
   p.H = a->H; p.ldc = a->ldc; p.KS = KS; p.MT = (blk_rows + 127) / 128; p.T = tokens;
-  p.scale_log2 = a->scale * 1.4426950408889634f;
+  p.scale_log2 = a->scale * LT_LOG2E;
+  p.window = a->window; p.sink = a->sink;
   p.r = a->r; p.status = a->status; p.pdl = a->pdl;
   CUtensorMap tmC, tmQ;
   int rc = pool_tmap(&tmC, a->pool, (long long)a->n_pages + 1, a->ldc);

@@ -4,6 +4,10 @@
 //           w = exp(-log_decay sigmoid(z + w0)); output gate sigmoid
 //   wkv     read out with r before the update, the current k v^T weighted by a bonus; M <- diag(w) M + k v^T,
 //           w = exp(-exp(z + w0)); output gate silu
+//   gated   M <- w M + a k v^T and a normaliser n <- w n + a k, read out with r afterwards and divided by
+//           max(|n.r|, exp(-m)) + unit_eps; log gates i = cap tanh((. + bias) / cap), f = ln sigmoid(cap tanh(..)), running
+//           maximum m <- max(f + m, i), w = exp(f + m_old - m), a = exp(i - m); output gate sigmoid.  The normaliser is one
+//           more value column (of ones), which every CTA of a head keeps for itself.
 //
 // Value columns of a matrix never mix, key rows only in sums.  A CTA therefore keeps some columns of one head's matrix in
 // registers - four threads per pair of columns (one column beyond 128 key rows), a quarter of the key rows each - and walks
@@ -22,21 +26,25 @@ namespace smc {
 constexpr int SCAN_PRODUCERS = 8;        // warps
 constexpr int SCAN_CONSUMERS = 256;      // threads at the most
 
+enum { SCAN_BONUS = 0, SCAN_DELTA = 1, SCAN_GATED = 2 };
+
 struct ScanArgs {
-  const float* proj;        // [T, ldp]: H * D columns each of r, k, v, gate (and removal rate) at these offsets
-  int ldp, r_off, k_off, v_off, g_off, a_off;
+  const float* proj;        // [T, ldp]: H * D columns of r and k, H * V of v and gate at these offsets, from a_off on the removal
+  int ldp, r_off, k_off, v_off, g_off, a_off;        // rates (delta, H * D) or the input and forget gates (gated, 2 H)
   const float* z;           // [T, ldz] decay logits, H * D
   int ldz;
   const float* w0;          // [H * D]
-  const float* a_bias;      // delta
+  const float* a_bias;      // delta [H * D], gated [2 H]
   const float* bonus;       // wkv
-  const float* onorm;       // [H * D]
-  float* state;             // row r: state + r * row_stride, [H, D (value), D (key)]
+  const float* onorm;       // [H * V]
+  float* state;             // row r: state + r * row_stride, [H, V (and one more if gated), D (key)]
   long long row_stride;
   int n_rows;
   void* out;                // [T, ldo]
-  int ldo, H, D;
+  int ldo, H, D, V;
   float eps, unit_eps, log_decay;
+  float* top;               // gated: row r: top + r * row_stride, [H] running maxima
+  float gate_cap, r_scale;  // gated: r is multiplied by r_scale
   Ragged r;
   int* status;
   int pdl;
@@ -71,23 +79,27 @@ __device__ __forceinline__ float sum_of(f2_t a) { const float2 v = unpack2(a); r
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 __host__ __device__ constexpr int scan_tokens(int dkp) { return dkp <= 128 ? 16 : 8; }       // tokens of a tile
-__host__ __device__ constexpr int scan_vectors(bool delta) { return delta ? 5 : 3; }
+__host__ __device__ constexpr int scan_vectors(int kind) { return kind == SCAN_DELTA ? 5 : kind == SCAN_GATED ? 2 : 3; }
 __host__ __device__ constexpr int scan_columns(int dkp) { return dkp <= 128 ? 2 : 1; }       // of a consumer thread
 __host__ __device__ constexpr int scan_max_columns(int dkp) { return SCAN_CONSUMERS / 4 * scan_columns(dkp); }      // of a CTA
 
-template <bool DELTA, int DKP>
+__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
+template <int KIND, int DKP>
 __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA), NL = (DKP + 31) / 32, NQ = DKP / 16, CP = scan_columns(DKP);
+  constexpr bool DELTA = KIND == SCAN_DELTA, GATED = KIND == SCAN_GATED;
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), NL = (DKP + 31) / 32, NQ = DKP / 16, CP = scan_columns(DKP);
   constexpr int PT = TB / SCAN_PRODUCERS;                    // tokens of a tile per producer warp
-  constexpr int NC = ((scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;       // columns of a CTA per lane
+  constexpr int NC = ((GATED || scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;      // columns of a CTA per lane
   extern __shared__ __align__(16) float scan_smem[];
   const int buf_floats = TB * (NVEC * DKP + CC + 2);
   float* obuf = scan_smem + 2 * buf_floats;                  // [3][TB][CC]
   float* ssq = obuf + 3 * TB * CC;                           // [2][TB]
+  float* least = ssq + 2 * TB;                               // [4][TB] exp(-m) (gated)
   const int n_cons = CC / CP * 4, tid = threadIdx.x, lane = tid & 31;
   const bool consumer = tid < n_cons;
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
-  const int h = blockIdx.x / CS, rank = blockIdx.x - h * CS, s = blockIdx.y, D = a.D;
+  const int h = blockIdx.x / CS, rank = blockIdx.x - h * CS, s = blockIdx.y, D = a.D, V = a.V;
   const int row = a.r.seq_row[s];
   const int off = a.r.seq_off != nullptr ? a.r.seq_off[s] : s * a.r.E, len = a.r.seq_len != nullptr ? a.r.seq_len[s] : a.r.E;
   if (row < 0 || row >= a.n_rows) {                          // the same in every CTA of the cluster
@@ -98,12 +110,19 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     __syncwarp();
     if (CS > 1) cluster_sync(); else __syncthreads();
   };
-  const int n_tiles = (len + TB - 1) / TB, c0 = rank * CC;
+  const int own = GATED ? CC - 1 : CC;                       // value columns of this CTA; the last slot is the normaliser's
+  const int n_tiles = (len + TB - 1) / TB, c0 = rank * own;
   const int last = CS > 1 ? n_tiles + 1 : n_tiles;
 
   if (!consumer) {
     const int pw = (tid - n_cons) >> 5;
     float kk[PT][NL], rr[PT][NL], zz[PT][NL], aa[PT][NL], vv[PT][NC], gg[PT][NC];
+    float gi = 0.f, gf = 0.f, m_run = 0.f, bi = 0.f, bf = 0.f;       // gated: gate logits of token `lane` of a tile, running maximum
+    if (GATED) {
+      bi = a.a_bias[h];
+      bf = a.a_bias[a.H + h];
+      m_run = a.top[(size_t)row * a.row_stride + h];
+    }
     auto fetch = [&](int tile) {                             // projections of a tile into registers
       const int n = min(TB, len - tile * TB);
 #pragma unroll
@@ -111,6 +130,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
         const int tb = pw + j * SCAN_PRODUCERS;
         const size_t t = (size_t)off + tile * TB + tb;
         const float* p = a.proj + t * a.ldp + h * D;
+        const float* pv = a.proj + t * a.ldp + h * V;
         const float* zr = a.z + t * a.ldz + h * D;
 #pragma unroll
         for (int i = 0; i < NL; ++i) {
@@ -118,14 +138,19 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           const bool ok = c < D && tb < n;
           kk[j][i] = ok ? p[a.k_off + c] : 0.f;
           rr[j][i] = ok ? p[a.r_off + c] : 0.f;
-          zz[j][i] = ok ? zr[c] : 0.f;
+          if (!GATED) zz[j][i] = ok ? zr[c] : 0.f;
           if (DELTA) aa[j][i] = ok ? p[a.a_off + c] : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
           const int c = lane + 32 * i;
-          vv[j][i] = c < CC && c0 + c < D && tb < n ? p[a.v_off + c0 + c] : 0.f;
+          vv[j][i] = c < own && c0 + c < V && tb < n ? pv[a.v_off + c0 + c] : 0.f;
         }
+      }
+      if (GATED && lane < n) {                               // every producer warp reads the gates of the whole tile
+        const float* p = a.proj + ((size_t)off + tile * TB + lane) * a.ldp + a.a_off + h;
+        gi = p[0];
+        gf = p[a.H];
       }
     };
     auto stage = [&](int tile) {                             // registers to the consumers' operands
@@ -133,6 +158,28 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
       float* val = buf + TB * NVEC * DKP;
       float* scal = val + TB * CC;
       const int n = min(TB, len - tile * TB);
+      float keep = 0.f, add = 0.f, low = 0.f;                // of token `lane`
+      if (GATED) {
+        // running maxima of a tile: a scan over pairs (sum of f, maximum), all in this warp
+        const bool ok = lane < n;
+        const float cap = a.gate_cap, li = ok ? cap * tanhf((gi + bi) / cap) : -INFINITY;
+        const float lf = ok ? log_sigmoid_f(cap * tanhf((gf + bf) / cap)) : 0.f;
+        float sum = lf, most = li;
+#pragma unroll
+        for (int o = 1; o < TB; o <<= 1) {
+          const float s0 = __shfl_up_sync(0xffffffffu, sum, o), m0 = __shfl_up_sync(0xffffffffu, most, o);
+          if (lane >= o) {
+            most = fmaxf(most, m0 + sum);
+            sum += s0;
+          }
+        }
+        const float m = fmaxf(most, m_run + sum), up = __shfl_up_sync(0xffffffffu, m, 1), before = lane == 0 ? m_run : up;
+        keep = expf(lf + before - m);
+        add = expf(li - m);
+        low = expf(-m);
+        m_run = __shfl_sync(0xffffffffu, m, n - 1);
+        if (pw == 0 && lane < n) least[(tile & 3) * TB + lane] = low;
+      }
 #pragma unroll
       for (int j = 0; j < PT; ++j) {
         const int tb = pw + j * SCAN_PRODUCERS;
@@ -150,6 +197,12 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           const int c = lane + 32 * i;
           if (c >= DKP) continue;
           const bool ok = c < D;
+          if (GATED) {
+            d[c] = kk[j][i];
+            d[TB * DKP + c] = rr[j][i] * a.r_scale;
+            s2 = fmaf(rr[j][i] * a.r_scale, kk[j][i], s2);
+            continue;
+          }
           const float z = ok ? zz[j][i] + a.w0[h * D + c] : 0.f;
           const float w = !ok ? 0.f : DELTA ? expf(-a.log_decay * sigmoid_f(z)) : expf(-expf(z));
           d[c] = w;
@@ -169,8 +222,14 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll
         for (int i = 0; i < NC; ++i)
           if (lane + 32 * i < CC) val[tb * CC + lane + 32 * i] = vv[j][i];
+        if (GATED) {
+          const float w = __shfl_sync(0xffffffffu, add, tb);
+#pragma unroll
+          for (int i = 0; i < NC; ++i)
+            if (lane + 32 * i < CC) val[tb * CC + lane + 32 * i] = lane + 32 * i < own ? w * vv[j][i] : w;
+        }
         __syncwarp();
-        s1 = DELTA ? warp_sum(s1) : 0.f;
+        s1 = DELTA ? warp_sum(s1) : GATED ? __shfl_sync(0xffffffffu, keep, tb) : 0.f;
         s2 = warp_sum(s2);
         if (lane == 0) { scal[2 * tb] = s1; scal[2 * tb + 1] = s2; }
       }
@@ -183,7 +242,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
           const int c = lane + 32 * i;
-          gg[j][i] = c < CC && c0 + c < D && tb < n ? a.proj[((size_t)off + tile * TB + tb) * a.ldp + a.g_off + h * D + c0 + c] : 0.f;
+          gg[j][i] = c < own && c0 + c < V && tb < n ? a.proj[((size_t)off + tile * TB + tb) * a.ldp + a.g_off + h * V + c0 + c] : 0.f;
         }
       }
     };
@@ -191,7 +250,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
       float q = 0.f;
 #pragma unroll
       for (int i = 0; i < NC; ++i) {
-        const float v = lane + 32 * i < CC ? o[lane + 32 * i] : 0.f;       // columns beyond D are zero
+        const float v = lane + 32 * i < own ? o[lane + 32 * i] : 0.f;      // columns beyond V are zero
         q = fmaf(v, v, q);
       }
       return warp_sum(q);
@@ -211,13 +270,15 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           const uint32_t at = smem_u32(ssq + (tile & 1) * TB + tb);
           for (int q = 0; q < CS; ++q) tot += ld_dsmem_f32(at, q);
         }
-        const float inv = 1.0f / sqrtf(tot / (float)D + a.eps);
+        float unit = 1.0f;                                   // gated: the read-out's divisor
+        if (GATED) unit = 1.0f / (fmaxf(fabsf(o[CC - 1]), least[(tile & 3) * TB + tb]) + a.unit_eps);
+        const float inv = unit / sqrtf(tot * unit * unit / (float)V + a.eps);
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
-          const int c = lane + 32 * i, col = h * D + c0 + c;
-          if (c >= CC || c0 + c >= D) continue;
+          const int c = lane + 32 * i, col = h * V + c0 + c;
+          if (c >= own || c0 + c >= V) continue;
           const float g = gg[j][i], sg = sigmoid_f(g);
-          const float v = o[c] * inv * a.onorm[col] * (DELTA ? sg : g * sg);
+          const float v = o[c] * inv * a.onorm[col] * (DELTA || GATED ? sg : g * sg);
           if (f32) reinterpret_cast<float*>(a.out)[t * a.ldo + col] = v;
           else reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + col] = __float2bfloat16(v);
         }
@@ -247,18 +308,23 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
       if (next >= 0 && next < n_tiles && (lag > 1 || it > 0)) gates(next);
       barrier();
     }
+    if (GATED && rank == 0 && pw == 0 && lane == 0) a.top[(size_t)row * a.row_stride + h] = m_run;
     return;
   }
 
   // ---- consumers: CP columns, and every fourth group of four key rows
   const int col = (tid >> 2) * CP, kq = tid & 3;
+  auto column = [&](int x) {                                 // row of the transposed matrix (-1: none)
+    if (GATED && col + x == CC - 1) return V;
+    return col + x < own && c0 + col + x < V ? c0 + col + x : -1;
+  };
   f2_t M[CP][NQ * 2];
   float* sp[CP];
 #pragma unroll
   for (int x = 0; x < CP; ++x) {
-    const int cg = c0 + col + x;
-    const bool mine = cg < D;
-    sp[x] = a.state + (size_t)row * a.row_stride + ((size_t)h * D + (mine ? cg : 0)) * D;
+    const int cg = column(x);
+    const bool mine = cg >= 0;
+    sp[x] = a.state + (size_t)row * a.row_stride + ((size_t)h * (V + GATED) + (mine ? cg : 0)) * D;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int k = (kq + 4 * i) * 4;
@@ -286,7 +352,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll 2
       for (int tb = 0; tb < n; ++tb) {
         const ulonglong2* dw = reinterpret_cast<const ulonglong2*>(buf + tb * DKP);
-        const ulonglong2* dk = dw + TB * DKP / 4;
+        const ulonglong2* dk = GATED ? dw : dw + TB * DKP / 4;
         const ulonglong2* dr = dk + TB * DKP / 4;
         const ulonglong2* du = dr + TB * DKP / 4;
         const ulonglong2* da = du + TB * DKP / 4;
@@ -337,7 +403,9 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
         }
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-          const ulonglong2 k = dk[kq + 4 * i], w = dw[kq + 4 * i];
+          const ulonglong2 k = dk[kq + 4 * i];
+          ulonglong2 w;
+          if (GATED) w.x = w.y = pack2(s1, s1); else w = dw[kq + 4 * i];
           ulonglong2 au;
           if (DELTA) au = da[kq + 4 * i];
 #pragma unroll
@@ -356,7 +424,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           o[x] += __shfl_xor_sync(0xffffffffu, o[x], 1);
           o[x] += __shfl_xor_sync(0xffffffffu, o[x], 2);
           if (kq == 0)
-            store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], DELTA ? fmaf(-s1, gone[x], o[x]) : o[x]));
+            store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], DELTA ? fmaf(-s1, gone[x], o[x]) : GATED ? s1 * o[x] : o[x]));
         }
       }
     }
@@ -364,7 +432,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
   }
 #pragma unroll
   for (int x = 0; x < CP; ++x) {
-    if (c0 + col + x >= D) continue;
+    if (column(x) < 0 || (GATED && column(x) == V && rank != 0)) continue;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int k = (kq + 4 * i) * 4;
@@ -414,29 +482,32 @@ __global__ void __launch_bounds__(64) low_rank_kernel(const float* x, int ldx, c
 }
 
 // Columns per CTA and CTAs per head: a head's columns are cut until the grid fills the machine (16 columns at the least); a
-// CTA takes at most scan_max_columns.  Whole warps of consumers need multiples of 8 (16 in pairs).
-static void scan_split(int n_seq, int H, int D, int most, int unit, int* CC, int* CS) {
+// CTA takes at most scan_max_columns, `extra` of them beside its share of the head's.  Whole warps of consumers need multiples
+// of 8 (16 in pairs).
+static void scan_split(int n_seq, int H, int V, int most, int unit, int extra, int* CC, int* CS) {
   int cs = 1;
-  while ((D + cs - 1) / cs > most) cs *= 2;
-  while (cs < 8 && (long long)n_seq * H * cs * 2 <= 148 && D / (cs * 2) >= 16) cs *= 2;
-  *CC = ((D + cs - 1) / cs + unit - 1) / unit * unit;
+  while ((V + cs - 1) / cs + extra > most) cs *= 2;
+  while (cs < 8 && (long long)n_seq * H * cs * 2 <= 148 && V / (cs * 2) >= 16) cs *= 2;
+  *CC = ((V + cs - 1) / cs + extra + unit - 1) / unit * unit;
   *CS = cs;
 }
 
-template <bool DELTA, int DKP>
+template <int KIND, int DKP>
 static int scan_launch(const ScanArgs& a, int f32, cudaStream_t st) {
   int CC, CS;
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(DELTA), CP = scan_columns(DKP);
-  scan_split(a.r.n_seq, a.H, a.D, scan_max_columns(DKP), 8 * CP, &CC, &CS);
-  const int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 2 * TB) * 4;
-  CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<DELTA, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
-  return launch_cluster(scan_kernel<DELTA, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * 4 + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), CP = scan_columns(DKP);
+  scan_split(a.r.n_seq, a.H, a.V, scan_max_columns(DKP), 8 * CP, KIND == SCAN_GATED, &CC, &CS);
+  if (CS > 16) return -122;
+  const int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 6 * TB) * 4;
+  CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
+  if (CS > 8) CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+  return launch_cluster(scan_kernel<KIND, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * 4 + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
                         CS, a, CC, CS, f32);
 }
 
-template <bool DELTA>
+template <int KIND>
 static int scan_dispatch(const ScanArgs& a, int f32, cudaStream_t st) {
-#define SMC_SCAN(N) if (a.D <= N) return scan_launch<DELTA, N>(a, f32, st);
+#define SMC_SCAN(N) if (a.D <= N) return scan_launch<KIND, N>(a, f32, st);
   SMC_SCAN(16) SMC_SCAN(32) SMC_SCAN(48) SMC_SCAN(64) SMC_SCAN(80) SMC_SCAN(96) SMC_SCAN(128) SMC_SCAN(160) SMC_SCAN(192) SMC_SCAN(256)
 #undef SMC_SCAN
   return -120;
@@ -446,13 +517,18 @@ static int scan_dispatch(const ScanArgs& a, int f32, cudaStream_t st) {
 
 SMC_API int smc_scan_args_size() { return (int)sizeof(smc::ScanArgs); }
 
-// One memory layer over the new tokens of every sequence; delta: the generalized delta rule, else the bonus form.  Heads of up
-// to 256 columns.
-SMC_API int smc_memory_scan(const smc::ScanArgs* a, int delta, int f32, cudaStream_t st) {
+// One memory layer over the new tokens of every sequence; kind: 0 the bonus form, 1 the generalized delta rule (both V = D), 2
+// the gated form.  Heads of up to 256 key columns.
+SMC_API int smc_memory_scan(const smc::ScanArgs* a, int kind, int f32, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_seq <= 0) return 0;
-  if (a->D < 1 || a->H < 1 || a->r.n_seq > 65535) return -120;
-  return delta ? scan_dispatch<true>(*a, f32, st) : scan_dispatch<false>(*a, f32, st);
+  if (a->D < 1 || a->H < 1 || a->V < 1 || a->r.n_seq > 65535 || (kind != SCAN_GATED && a->V != a->D)) return -120;
+  switch (kind) {
+    case SCAN_BONUS: return scan_dispatch<SCAN_BONUS>(*a, f32, st);
+    case SCAN_DELTA: return scan_dispatch<SCAN_DELTA>(*a, f32, st);
+    case SCAN_GATED: return scan_dispatch<SCAN_GATED>(*a, f32, st);
+  }
+  return -120;
 }
 
 // out[m, c] = tanh(x[m, c]), c < n.

@@ -1,8 +1,9 @@
 // Feed-forward pieces around the GEMMs of layered architectures:
 //   poly_norm       a N(z) + b N(z^2) + c N(z^3) + e, N dividing the token's row by its root mean square
-//   gated_unit      min(g, limit) sigmoid(slope g) (clamp(u) + shift) on stored gate / up rows (32-bit runs; the bf16 path has
-//                   it in the GEMM epilogue)
-//   route           router logits, softmax over all experts, best groups, best experts, renormalised weights
+//   gated_unit      min(g, limit) sigmoid(slope g) (clamp(u) + shift), or gelu(g) u, on stored gate / up rows (32-bit runs; the
+//                   bf16 path has it in the GEMM epilogue)
+//   route           router logits (with an optional bias), softmax over all experts, best groups, best experts, renormalised
+//                   weights; one more row of the router matrix may give the gate of a shared expert
 //   dispatch        slots of the (token, expert) pairs sorted by expert, and the table of token tiles the grouped GEMMs use
 //   gather_rows     activation rows in slot order
 // Everything the routing decides is fp32.
@@ -55,14 +56,15 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const float* z, int ldz,
 
 // ---------------------------------------------------------------- gated unit on stored rows (an infinite limit: none)
 __global__ void __launch_bounds__(256) gated_unit_kernel(const float* gu, int ldg, float* out, int ldo, int ff, int blk, float limit,
-                                                         float slope, float shift, int M, int pdl) {
+                                                         float slope, float shift, int gelu, int M, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const long long n = (long long)M * ff;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const int m = (int)(i / ff), c = (int)(i % ff), q = c / blk, r = c - q * blk;
     const float* row = gu + (size_t)m * ldg + (size_t)q * 2 * blk + r;
     const float g = fminf(row[0], limit), u = fminf(fmaxf(row[blk], -limit), limit);
-    out[(size_t)m * ldo + c] = g / (1.0f + expf(-slope * g)) * (u + shift);
+    out[(size_t)m * ldo + c] = gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u
+                                    : g / (1.0f + expf(-slope * g)) * (u + shift);
   }
 }
 
@@ -71,12 +73,13 @@ __global__ void __launch_bounds__(256) gated_unit_kernel(const float* gu, int ld
 // and their loads overlap.  Then one warp per token runs the softmax and the two selections.
 template <typename AT, int TM>
 __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const AT* wr, int ldw, int E, int top, int groups,
-                                                    int keep, int T, int* idx, float* wgt, int pdl) {
+                                                    int keep, int T, const float* bias, float* gate, int* idx, float* wgt, int pdl) {
+  const int EL = E + (gate != nullptr);        // rows of the router matrix
   extern __shared__ float rt_smem[];
   const int d4 = (d + 3) & ~3;
   float* sh = rt_smem;                         // [TM][d4]
-  float* sl = sh + (size_t)TM * d4;            // [TM][E] logits, then scores
-  float* sg = sl + TM * E;                     // [TM][groups] best score of every group
+  float* sl = sh + (size_t)TM * d4;            // [TM][EL] logits, then scores
+  float* sg = sl + TM * EL;                    // [TM][groups] best score of every group
   float* sw = sg + TM * groups;                // [TM][top]
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int t0 = blockIdx.x * TM, nt = min(TM, T - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -92,7 +95,7 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
   }
   __syncthreads();
   constexpr int EG = 4;
-  for (int e0 = warp * EG; e0 < E; e0 += nw * EG) {
+  for (int e0 = warp * EG; e0 < EL; e0 += nw * EG) {
     float acc[EG][TM];
 #pragma unroll
     for (int q = 0; q < EG; ++q)
@@ -103,7 +106,7 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
       for (int c = lane * 4; c < d; c += 128) {
         float4 w[EG];
 #pragma unroll
-        for (int q = 0; q < EG; ++q) w[q] = load4(wr + (size_t)min(e0 + q, E - 1) * ldw + c);
+        for (int q = 0; q < EG; ++q) w[q] = load4(wr + (size_t)min(e0 + q, EL - 1) * ldw + c);
 #pragma unroll
         for (int m = 0; m < TM; ++m) {
           const float4 v = load4(sh + (size_t)m * d + c);
@@ -116,7 +119,7 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
       for (int c = lane; c < d; c += 32)
 #pragma unroll
         for (int q = 0; q < EG; ++q) {
-          const float w = to_f32<AT>(wr[(size_t)min(e0 + q, E - 1) * ldw + c]);
+          const float w = to_f32<AT>(wr[(size_t)min(e0 + q, EL - 1) * ldw + c]);
 #pragma unroll
           for (int m = 0; m < TM; ++m) acc[q][m] = fmaf(w, sh[(size_t)m * d4 + c], acc[q][m]);
         }
@@ -126,13 +129,14 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
 #pragma unroll
       for (int m = 0; m < TM; ++m) {
         const float s = warp_sum(acc[q][m]);
-        if (lane == 0 && e0 + q < E) sl[m * E + e0 + q] = s;
+        if (lane == 0 && e0 + q < EL) sl[m * EL + e0 + q] = s + (bias != nullptr && e0 + q < E ? bias[e0 + q] : 0.f);
       }
   }
   __syncthreads();
   const int per = E / groups;
   for (int m = warp; m < nt; m += nw) {
-    float* l = sl + m * E;
+    float* l = sl + m * EL;
+    if (gate != nullptr && lane == 0) gate[t0 + m] = 1.0f / (1.0f + expf(-l[E]));
     float* gs = sg + m * groups;
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, l[e]);
@@ -274,21 +278,22 @@ SMC_API int smc_poly_norm(const float* z, int ldz, const float* coef, float eps,
 }
 
 SMC_API int smc_gated_unit_f32(const float* gu, int ldg, float* out, int ldo, int ff, int blk, float limit, float slope,
-                               float shift, int M, int pdl, cudaStream_t st) {
+                               float shift, int gelu, int M, int pdl, cudaStream_t st) {
   using namespace smc;
   if (M <= 0) return 0;
   const long long n = ((long long)M * ff + 255) / 256;
   return launch_pdl(gated_unit_kernel, dim3((unsigned)(n < 2368 ? n : 2368)), dim3(256), 0, st, pdl, gu, ldg, out, ldo, ff, blk,
-                    limit, slope, shift, M, pdl);
+                    limit, slope, shift, gelu, M, pdl);
 }
 
-// h fp32 [T, d] packed; wr [E, ldw]; idx / wgt [T, top].
-SMC_API int smc_route(const float* h, int d, const void* wr, int ldw, int E, int top, int groups, int keep, int T, int* idx,
-                      float* wgt, int f32, int pdl, cudaStream_t st) {
+// h fp32 [T, d] packed; wr [E, ldw]; idx / wgt [T, top].  bias [E] (optional) is added to the logits; gate [T] (optional): wr has
+// one more row, the sigmoid of whose logit goes there.
+SMC_API int smc_route(const float* h, int d, const void* wr, int ldw, int E, int top, int groups, int keep, int T, const float* bias,
+                      float* gate, int* idx, float* wgt, int f32, int pdl, cudaStream_t st) {
   using namespace smc;
   if (T <= 0) return 0;
   if (E < 1 || top < 1 || groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups)) return -95;
-  auto bytes = [&](int tm) { return (size_t)tm * (((d + 3) & ~3) + E + groups + top) * sizeof(float); };
+  auto bytes = [&](int tm) { return (size_t)tm * (((d + 3) & ~3) + E + 1 + groups + top) * sizeof(float); };
   const bool wide = T > 296 && bytes(8) <= 200 * 1024;      // eight tokens per CTA once there are enough of them
   const int TM = wide ? 8 : 1;
   if (bytes(TM) > 200 * 1024) return -96;
@@ -297,7 +302,7 @@ SMC_API int smc_route(const float* h, int d, const void* wr, int ldw, int E, int
   {                                                                                                                         \
     CUDA_CHECK_RET(cudaFuncSetAttribute(route_kernel<AT, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));     \
     return launch_pdl(route_kernel<AT, N>, grid, dim3(256), bytes(TM), st, pdl, h, d, (const AT*)wr, ldw, E, top, groups,   \
-                      keep, T, idx, wgt, pdl);                                                                              \
+                      keep, T, bias, gate, idx, wgt, pdl);                                                                            \
   }
   if (f32 && wide) SMC_ROUTE(float, 8)
   if (f32) SMC_ROUTE(float, 1)

@@ -7,7 +7,7 @@
 //   token_shift     the shift on its own (several tokens per sequence): every channel of x is mixed with the row before,
 //                   n ways; the thread of a sequence's first tokens, which reads the kept row, also writes the new one.
 // The stream, the norms, the angles and the mixes are computed in fp32 (angles are reduced in fp64).
-#include "ragged.cuh"
+#include "rotary.cuh"
 
 namespace smc {
 
@@ -41,28 +41,6 @@ struct PostNormArgs {
   int* status;
   int pdl;
 };
-
-// {sine, cosine} of position p at frequency index i.
-__device__ __forceinline__ float2 position_pair(const double* freq, int i, int p) {
-  double a = (double)p * freq[i];
-  a -= 6.283185307179586476925 * rint(a * 0.15915494309189533577);
-  float s, c;
-  sincosf((float)a, &s, &c);
-  return make_float2(s, c);
-}
-
-template <int VEC, typename T> __device__ __forceinline__ void load_cols(float (&v)[VEC], const T* p) {
-  if constexpr (VEC == 4) {
-    const float4 a = load4(p);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-  } else {
-    v[0] = to_f32<T>(*p);
-  }
-}
-template <int VEC, typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[VEC]) {
-  if constexpr (VEC == 4) store4(p, make_float4(v[0], v[1], v[2], v[3]));
-  else *p = from_f32<T>(v[0]);
-}
 
 // AHEAD > 0: AHEAD mixes whose coefficients, and the row before, are read before the sums (two column groups per thread).
 template <typename AT, int VEC, int AHEAD>

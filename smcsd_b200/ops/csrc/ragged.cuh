@@ -68,6 +68,20 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = o;
 }
 
+// VEC (1 or 4) consecutive elements.
+template <int VEC, typename T> __device__ __forceinline__ void load_cols(float (&v)[VEC], const T* p) {
+  if constexpr (VEC == 4) {
+    const float4 a = load4(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else {
+    v[0] = to_f32<T>(*p);
+  }
+}
+template <int VEC, typename T> __device__ __forceinline__ void store_cols(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) store4(p, make_float4(v[0], v[1], v[2], v[3]));
+  else *p = from_f32<T>(v[0]);
+}
+
 __device__ __forceinline__ float block_sum_all(float v, float* red) {
   v = warp_sum(v);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;

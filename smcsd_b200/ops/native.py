@@ -625,7 +625,26 @@ class HyperArgs(C.Structure):
 
 class LatentArgs(C.Structure):
     _fields_ = [("q", _VP), ("pool", _VP), ("out", _VP), ("block_table", _VP), ("bt_stride", _I), ("bt_rows", _I), ("n_pages", _I),
-                ("H", _I), ("ldc", _I), ("scale", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+                ("H", _I), ("ldc", _I), ("scale", _F), ("window", _I), ("sink", _VP), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
+class LatentNewArgs(C.Structure):
+    _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "nq", "c_off", "R", "rot")] + \
+               [("q_norm", _VP), ("nq_real", _I), ("c_norm", _VP), ("eps", _F), ("freq", _VP), ("positions", _VP), ("q", _VP), ("ldq", _I),
+                ("pool", _VP), ("ldc", _I), ("n_pages", _I), ("locs", _VP), ("status", _VP), ("pdl", _I)]
+
+
+class ConvHeadsArgs(C.Structure):
+    _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "H", "G", "D", "V", "rot")] + \
+               [("conv", _VP), ("taps", _I), ("hist", _VP), ("row_stride", C.c_longlong), ("n_rows", _I), ("freq", _VP), ("positions", _VP),
+                ("q", _VP), ("kpool", _VP), ("vpool", _VP), ("n_pages", _I), ("locs", _VP), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
+class SideArgs(C.Structure):
+    _fields_ = [("x", _VP), ("d", _I), ("ids", _VP), ("embed", _VP), ("vocab", _I), ("embed_scale", _F), ("y1", _VP), ("s1", _VP),
+                ("y2", _VP), ("gate", _VP), ("ldy", _I), ("ye", _VP), ("ldye", _I), ("top", _I), ("route_slot", _VP), ("route_w", _VP),
+                ("s2", _VP), ("eps", _F), ("w1", _VP), ("w2", _VP), ("xa", _VP), ("xb", _VP), ("n2", _VP), ("ldxa", _I), ("final", _I),
+                ("status", _VP), ("pdl", _I)]
 
 
 class PostNormArgs(C.Structure):
@@ -641,16 +660,17 @@ class HeadsNewArgs(C.Structure):
 
 
 class ChunkAttnArgs(C.Structure):
-    _fields_ = [("q", _VP), ("kpool", _VP), ("vpool", _VP), ("out", _VP), ("gate", _VP), ("ldg", _I), ("block_table", _VP)] + \
+    _fields_ = [("q", _VP), ("kpool", _VP), ("vpool", _VP), ("out", _VP), ("gate", _VP), ("ldg", _I), ("gate_heads", _I),
+                ("block_table", _VP)] + \
                [(n, _I) for n in ("bt_stride", "bt_rows", "n_pages", "H", "G", "D", "V", "chunk")] + \
-               [("scale", _F), ("r1", _VP), ("r2", _VP), ("sink", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+               [("scale", _F), ("r1", _VP), ("r2", _VP), ("softcap", _F), ("sink", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
 class ScanArgs(C.Structure):
     _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "r_off", "k_off", "v_off", "g_off", "a_off")] + \
                [("z", _VP), ("ldz", _I), ("w0", _VP), ("a_bias", _VP), ("bonus", _VP), ("onorm", _VP), ("state", _VP),
-                ("row_stride", C.c_longlong), ("n_rows", _I), ("out", _VP), ("ldo", _I), ("H", _I), ("D", _I), ("eps", _F),
-                ("unit_eps", _F), ("log_decay", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+                ("row_stride", C.c_longlong), ("n_rows", _I), ("out", _VP), ("ldo", _I), ("H", _I), ("D", _I), ("V", _I),
+                ("eps", _F), ("unit_eps", _F), ("log_decay", _F), ("top", _VP), ("gate_cap", _F), ("r_scale", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
 class GroupLink(C.Structure):
@@ -660,7 +680,8 @@ class GroupLink(C.Structure):
 
 
 GROUP_BATCHED, GROUP_TILED = 1, 2
-ACT_SILU, ACT_CLAMPED = 0, 1
+ACT_SILU, ACT_CLAMPED, ACT_GELU = 0, 1, 2
+SCAN_BONUS, SCAN_DELTA, SCAN_GATED = 0, 1, 2
 
 
 def layered_lib():
@@ -672,11 +693,14 @@ def layered_lib():
         L.smc_hyper_step.argtypes = [vp, i, i, vp]
         L.smc_short_conv.argtypes = [vp, vp, i, vp, vp, i, i, i, vp, vp, i, i, vp]
         L.smc_poly_norm.argtypes = [vp, i, vp, f, vp, i, i, i, i, i, vp]
-        L.smc_gated_unit_f32.argtypes = [vp, i, vp, i, i, i, f, f, f, i, i, vp]
-        L.smc_route.argtypes = [vp, i, vp, i, i, i, i, i, i, vp, vp, i, i, vp]
+        L.smc_gated_unit_f32.argtypes = [vp, i, vp, i, i, i, f, f, f, i, i, i, vp]
+        L.smc_route.argtypes = [vp, i, vp, i, i, i, i, i, i, vp, vp, vp, vp, i, i, vp]
         L.smc_dispatch.argtypes = [vp, i, i, i, i, vp, vp, vp, i, vp, i, vp]
         L.smc_gather_rows.argtypes = [vp, i, vp, vp, i, i, i, i, vp, i, vp]
-        L.smc_latent_new.argtypes = [vp, i, i, i, vp, f, vp, i, vp, i, i, vp, i, vp, i, i, vp]
+        L.smc_latent_new.argtypes = [vp, i, i, vp]
+        L.smc_conv_heads.argtypes = [vp, i, vp]
+        L.smc_rotate_heads.argtypes = [vp, i, vp, i, i, i, i, vp, vp, i, i, i, vp]
+        L.smc_side_step.argtypes = [vp, i, i, vp]
         L.smc_latent_attn.argtypes = [vp, i, vp]
         L.smc_latent_attn_tc.argtypes = [vp, i, i, i, vp]
         L.smc_latent_attn_tc.restype = C.c_int
@@ -695,13 +719,14 @@ def layered_lib():
         for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_gated_unit_f32",
                   "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn", "smc_post_norm_step",
                   "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_splits", "smc_chunk_attn_tc",
-                  "smc_chunk_attn_tc_max_width",
+                  "smc_chunk_attn_tc_max_width", "smc_conv_heads", "smc_rotate_heads", "smc_side_step",
                   "smc_memory_scan", "smc_tanh_rows", "smc_low_rank"):
             getattr(L, n).restype = C.c_int
         for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
                        (GroupLink, "smc_group_link_size"), (PostNormArgs, "smc_post_norm_args_size"),
                        (HeadsNewArgs, "smc_heads_new_args_size"), (ChunkAttnArgs, "smc_chunk_attn_args_size"),
-                       (ScanArgs, "smc_scan_args_size")):
+                       (ScanArgs, "smc_scan_args_size"), (LatentNewArgs, "smc_latent_new_args_size"),
+                       (ConvHeadsArgs, "smc_conv_heads_args_size"), (SideArgs, "smc_side_args_size")):
             assert C.sizeof(cls) == getattr(L, n)(), f"{cls.__name__} layout mismatch"
         L._layered_declared = True
     return L
@@ -746,17 +771,18 @@ def poly_norm(z: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, *, ff: int
 
 
 def gated_unit_f32(gu: torch.Tensor, out: torch.Tensor, *, ff: int, blk: int, limit: float, slope: float, shift: float, M: int,
-                   pdl: bool = False) -> None:
-    """min(g, limit) sigmoid(slope g) (clamp(u, limit) + shift) on gate / up columns interleaved in blocks of ``blk``."""
-    _check(layered_lib().smc_gated_unit_f32(_p(gu), gu.stride(0), _p(out), out.stride(0), ff, blk, limit, slope, shift, M, int(pdl),
+                   gelu: bool = False, pdl: bool = False) -> None:
+    """min(g, limit) sigmoid(slope g) (clamp(u, limit) + shift), or gelu(g) u, on gate / up columns interleaved in blocks of ``blk``."""
+    _check(layered_lib().smc_gated_unit_f32(_p(gu), gu.stride(0), _p(out), out.stride(0), ff, blk, limit, slope, shift, int(gelu), M, int(pdl),
                                             _stream()), "smc_gated_unit_f32")
 
 
 def route(h: torch.Tensor, wr: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor, *, d: int, top: int, groups: int, keep: int,
-          T: int, f32: bool, pdl: bool = False) -> None:
-    """Expert choice of T tokens: fp32 logits, softmax over all experts, best groups, best experts, weights summing to one."""
-    _check(layered_lib().smc_route(_p(h), d, _p(wr), wr.stride(0), wr.shape[0], top, groups, keep, T, _p(idx), _p(wgt), int(f32),
-                                   int(pdl), _stream()), "smc_route")
+          T: int, f32: bool, bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """Expert choice of T tokens: fp32 logits (plus ``bias``), softmax over all experts, best groups, best experts, weights
+    summing to one.  With ``gate`` [T] the last row of ``wr`` is no expert: the sigmoid of its logit goes there."""
+    _check(layered_lib().smc_route(_p(h), d, _p(wr), wr.stride(0), wr.shape[0] - (gate is not None), top, groups, keep, T, _p(bias),
+                                   _p(gate), _p(idx), _p(wgt), int(f32), int(pdl), _stream()), "smc_route")
 
 
 def dispatch(idx: torch.Tensor, slot: torch.Tensor, src: torch.Tensor, tiles: torch.Tensor, *, n: int, top: int, experts: int,
@@ -773,12 +799,27 @@ def gather_rows(x: torch.Tensor, src: torch.Tensor, out: torch.Tensor, *, n: int
                                          _p(status), int(pdl), _stream()), "smc_gather_rows")
 
 
-def latent_new(proj: torch.Tensor, q: Optional[torch.Tensor], pool: torch.Tensor, c_norm: torch.Tensor, cache_locs: torch.Tensor, *,
-               nq: int, R: int, eps: float, M: int, status: torch.Tensor, f32: bool, pdl: bool = False) -> None:
-    """New tokens' projections: query columns to ``q``, normalised latent columns to their cache pages."""
-    _check(layered_lib().smc_latent_new(_p(proj), proj.stride(0), nq, R, _p(c_norm), eps, _p(q), q.stride(0) if q is not None else 0,
-                                        _p(pool), pool.stride(0), pool.shape[0] - 1, _p(cache_locs), M, _p(status), int(f32), int(pdl),
-                                        _stream()), "smc_latent_new")
+def latent_new(a: LatentNewArgs, T: int, f32: bool) -> None:
+    """New tokens' projections: query columns (copied, or normed as a latent) to ``q``, normalised latent columns and the rotated
+    key to their cache pages."""
+    _check(layered_lib().smc_latent_new(C.byref(a), T, int(f32), _stream()), "smc_latent_new")
+
+
+def rotate_heads(x: torch.Tensor, out: torch.Tensor, freq: torch.Tensor, positions: torch.Tensor, *, heads: int, width: int, first: int,
+                 rot: int, M: int, f32: bool, pdl: bool = False) -> None:
+    """fp32 heads of ``width`` columns to the activation type, columns [first, first + rot) rotated by position."""
+    _check(layered_lib().smc_rotate_heads(_p(x), x.stride(0), _p(out), heads, width, first, rot, _p(freq), _p(positions), M, int(f32),
+                                          int(pdl), _stream()), "smc_rotate_heads")
+
+
+def conv_heads(a: ConvHeadsArgs, f32: bool) -> None:
+    """New tokens' queries, keys and values: short convolution, rotation, cache pages."""
+    _check(layered_lib().smc_conv_heads(C.byref(a), int(f32), _stream()), "smc_conv_heads")
+
+
+def side_step(a: SideArgs, T: int, f32: bool) -> None:
+    """x <- x + s1 mixer + s2 feed-forward (or the embedding start), and x under the next layer's two norms (or the final one)."""
+    _check(layered_lib().smc_side_step(C.byref(a), T, int(f32), _stream()), "smc_side_step")
 
 
 def latent_attention(a: LatentArgs, f32: bool) -> None:
@@ -837,9 +878,10 @@ def chunk_tc_max_width() -> int:
     return layered_lib().smc_chunk_attn_tc_max_width()
 
 
-def memory_scan(a: ScanArgs, delta: bool, f32: bool) -> None:
-    """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu)."""
-    _check(layered_lib().smc_memory_scan(C.byref(a), int(delta), int(f32), _stream()), "smc_memory_scan")
+def memory_scan(a: ScanArgs, kind: int, f32: bool) -> None:
+    """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu); ``kind``: SCAN_BONUS, SCAN_DELTA or
+    SCAN_GATED."""
+    _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), int(f32), _stream()), "smc_memory_scan")
 
 
 def tanh_rows(x: torch.Tensor, out: torch.Tensor, *, n: int, M: int, f32: bool, pdl: bool = False) -> None:

@@ -4,11 +4,11 @@ can be captured in a graph, and the head."""
 from __future__ import annotations
 
 import os
-from typing import Dict, Optional
+from typing import Dict, List, Optional
 
 import torch
 
-from ..models.layered import round_up
+from ..models.layered import GU_BLOCK, round_up
 from . import native as K
 from .ragged import RaggedPlan, uniform_struct
 
@@ -23,6 +23,8 @@ class NativeLayered:
     ``xa``, and ``set_context``."""
     ragged = True
     BLOCK = 64                            # tokens per block of the work list
+    TC_MIN_TOKENS = 8                     # portions at least this long take the tensor-core form of the attention over heads
+    attn_tc = False
 
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
@@ -74,13 +76,111 @@ class NativeLayered:
         if self.f32:
             gu = self._rows("gu", M, ff2)
             K.gemm_f32(W, X, gu, N=ff2, M=M, link=link, pdl=self.pdl)
-            K.gated_unit_f32(gu, act, ff=ff2 // 2, blk=blk, limit=link.limit, slope=link.slope, shift=shift, M=M, pdl=self.pdl)
+            K.gated_unit_f32(gu, act, ff=ff2 // 2, blk=blk, limit=link.limit, slope=link.slope, shift=shift, M=M,
+                             gelu=link.act == K.ACT_GELU, pdl=self.pdl)
             return
         splits = K.gemm_swiglu_splits(ff2, W.shape[-1], M) if link.mode == 0 else 1
         if link.mode == 0 and link.act == K.ACT_SILU:        # the plain build of the kernel has this unit
             K.gemm_skinny(W, X, act, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, ldo=act.stride(0), status=self.status, pdl=self.pdl)
             return
         K.gemm_grouped(W, X, act, N=ff2, M=M, splits=splits, epi=K.EPI_SWIGLU_BF16, link=link, status=self.status, pdl=self.pdl)
+
+    def _per_head(self, W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, M: int, H: int, x_cols: int, out_cols: int) -> None:
+        """Head h: out[:, h * out_cols ..] = X[:, h * x_cols ..] W_h^T, in the activation type."""
+        link = K.GroupLink(mode=K.GROUP_BATCHED, groups=H, w_rows=out_cols, x_cols=x_cols, out_cols=out_cols)
+        if self.f32:
+            K.gemm_f32(W, X, out, N=out_cols, M=M, link=link, pdl=self.pdl)
+        else:
+            K.gemm_grouped(W, X, out, N=out_cols, M=M, splits=1, epi=K.EPI_BF16, link=link, status=self.status, pdl=self.pdl)
+
+    # ---- mixture of experts -------------------------------------------------------------
+    def _room_experts(self, moe: List) -> None:
+        """Buffers of the expert feed-forwards ``moe`` (specs)."""
+        T, most = self.T, lambda it: max(it, default=0)
+        pairs = T * most(f.router.top for f in moe)
+        self._room("idx", pairs, torch.int32)
+        self._room("wgt", pairs, torch.float32)
+        self._room("slot", pairs, torch.int32)
+        self._room("src", pairs, torch.int32)
+        self._room("tiles", 4 * most(f.router.experts for f in moe) + 4 * (pairs // 16 + 1), torch.int32)
+        self._room("xe", pairs * self.d8, self.dt)
+        self._room("ea", pairs * most(round_up(f.expert.ff, GU_BLOCK) for f in moe), self.dt)
+        self._room("ye", pairs * self.d, torch.float32)
+
+    def _room_gate_up(self, dense: List[int], moe: List) -> None:
+        """32-bit runs store gate / up rows: of gated units of these sizes and of the experts."""
+        if self.f32:
+            pairs = self.T * max((f.router.top for f in moe), default=0)
+            units = list(dense) + [f.shared.ff for f in moe if f.shared]
+            self._room("gu", max([pairs * 2 * round_up(f.expert.ff, GU_BLOCK) for f in moe] + [self.T * 2 * round_up(n, GU_BLOCK) for n in units],
+                                 default=0), torch.float32)
+
+    def _expert_rows(self, L, f, x: torch.Tensor, T: int, unit) -> None:
+        """The chosen experts' outputs, one fp32 row per (token, choice) in "ye" at "slot", from the choices in "idx";
+        ``unit(W, X, out, M, spec, link)`` runs the gated unit."""
+        pdl, E, top, n = self.pdl, f.router.experts, f.router.top, T * f.router.top
+        idx, slot, src, tiles = (self._flat[k] for k in ("idx", "slot", "src", "tiles"))
+        avg = (n + E - 1) // E
+        bn = 64 if self.f32 else 16 if avg <= 16 else 32 if avg <= 32 else 64 if avg <= 64 else 128
+        max_tiles = n // bn + min(E, n)
+        K.dispatch(idx, slot, src, tiles, n=n, top=top, experts=E, rows=bn, max_tiles=max_tiles, status=self.status, pdl=pdl)
+        xe, ffp = self._rows("xe", n, self.d8), L.e_down.shape[-1]
+        K.gather_rows(x, src, xe, n=n, n_src=T, status=self.status, pdl=pdl)
+        ea, ye = self._rows("ea", n, ffp), self._rows("ye", n, self.d)
+        unit(L.e_gu, xe, ea, n, f.expert, K.GroupLink(mode=K.GROUP_TILED, groups=E, w_rows=2 * ffp, tiles=K.ptr(tiles), max_tiles=max_tiles, bn=bn))
+        link = K.GroupLink(mode=K.GROUP_TILED, groups=E, w_rows=self.d, tiles=K.ptr(tiles), max_tiles=max_tiles, bn=bn)
+        if self.f32:
+            K.gemm_f32(L.e_down, ea, ye, N=self.d, M=n, link=link, pdl=pdl)
+            return
+        units, slabs, kb, sp = min(E, n), (self.d + 127) // 128, (ffp + 63) // 64, 1
+        while sp < 8 and units * slabs * sp * 2 <= 256 and kb // (sp * 2) >= 2:
+            sp *= 2
+        K.gemm_grouped(L.e_down, ea, ye, N=self.d, M=n, splits=sp, epi=K.EPI_STORE_F32, link=link, status=self.status, pdl=pdl)
+
+    # ---- attention ----------------------------------------------------------------------
+    def _capped(self, splits: int) -> int:
+        cap = max(1, int(self.attn_splits))
+        while splits > cap:
+            splits //= 2
+        return splits
+
+    def _latent_splits(self, n_blk: int, tokens: int, H: int, Rp: int, window: int = 0) -> int:
+        """Key ranges of a latent attention: ``n_blk`` blocks of at most ``tokens`` tokens."""
+        if not self.attn_tc or Rp > K.latent_tc_max_width():
+            return 1
+        keys = min(self.ctx_hint, window + tokens) if window else self.ctx_hint
+        return self._capped(K.latent_tc_splits(n_blk * ((tokens * H + 127) // 128), Rp, keys))
+
+    def _latent_attention(self, lat: torch.Tensor, pool: torch.Tensor, ctx: torch.Tensor, H: int, scale: float, T: int, work: "K.Ragged",
+                          longest: int, window: int = 0, sink: Optional[torch.Tensor] = None) -> None:
+        Rp = pool.shape[1]
+        a = K.LatentArgs(q=K.ptr(lat), pool=K.ptr(pool), out=K.ptr(ctx), block_table=K.ptr(self.bt), bt_stride=self.bt.stride(0),
+                         bt_rows=self.bt.shape[0], n_pages=pool.shape[0] - 1, H=H, ldc=Rp, scale=scale, window=window, sink=K.ptr(sink),
+                         r=work, status=K.ptr(self.status), pdl=int(self.pdl))
+        if self.attn_tc and Rp <= K.latent_tc_max_width():
+            tokens = min(longest, self.BLOCK)
+            K.latent_attention_tc(a, tokens=T, blk_rows=tokens * H, splits=self._latent_splits(work.n_blk, tokens, H, Rp, window))
+        else:
+            K.latent_attention(a, self.f32)
+
+    def _chunk_splits(self, tokens: int, m, chunk: int) -> int:
+        """Key ranges of one layer's attention over heads for ``tokens`` tokens (``chunk`` 0: all keys)."""
+        keys = min(chunk, self.ctx_hint) if chunk else self.ctx_hint
+        return self._capped(K.chunk_attention_splits(tokens, m.heads, m.kv_heads, round_up(max(m.dim, m.vdim), 8), keys))
+
+    def _chunk_attention(self, a: "K.ChunkAttnArgs", m, chunk: int, T: int, longest: int) -> None:
+        if self.attn_tc and longest >= self.TC_MIN_TOKENS and max(a.D, a.V) <= K.chunk_tc_max_width():
+            K.chunk_attention_tc(a)
+        else:
+            K.chunk_attention(a, self.f32, self._chunk_splits(T, m, chunk))
+
+    @staticmethod
+    def _walk(work: "K.Ragged", longest: int) -> "K.Ragged":
+        """The work list with blocks of ``longest`` tokens where every sequence is one block anyway."""
+        if longest < NativeLayered.BLOCK:
+            work = K.Ragged.from_buffer_copy(work)
+            work.B = longest
+        return work
 
     # ---- forward ------------------------------------------------------------------------
     def _run(self, ids, positions, locs, T: int, work: "K.Ragged", single_rows: Optional[torch.Tensor], longest: int) -> torch.Tensor:

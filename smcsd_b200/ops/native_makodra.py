@@ -23,7 +23,6 @@ from .native_layered import NativeLayered, env_flag
 
 
 class NativeMakodra(NativeLayered):
-    TC_MIN_TOKENS = 8                     # portions at least this long take the tensor-core attention
     LOW_RANK_TOKENS = 32                  # steps up to this long expand the decay logits in one launch
 
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
@@ -83,15 +82,7 @@ class NativeMakodra(NativeLayered):
         """Record the context-length hint; returns what it decides about the launch grids (part of a graph's identity)."""
         self.ctx_hint = int(ctx)
         mixers = {L.spec.mixer for L in self.m.layers if L.kind == "attention"}
-        return tuple(sorted((E, m.chunk, m.heads, self._ks(bs * E, m)) for E in Es for m in mixers))
-
-    def _ks(self, tokens: int, m) -> int:
-        """Key ranges of one layer's attention for ``tokens`` tokens."""
-        ks = K.chunk_attention_splits(tokens, m.heads, m.kv_heads, round_up(max(m.dim, m.vdim), 8), min(m.chunk, self.ctx_hint))
-        cap = max(1, int(self.attn_splits))
-        while ks > cap:
-            ks //= 2
-        return ks
+        return tuple(sorted((E, m.chunk, m.heads, self._chunk_splits(bs * E, m, m.chunk)) for E in Es for m in mixers))
 
     # ---- sublayers ----------------------------------------------------------------------
     def _attention(self, L, T: int, locs: torch.Tensor, work: "K.Ragged", longest: int) -> None:
@@ -109,10 +100,7 @@ class NativeMakodra(NativeLayered):
                             block_table=K.ptr(self.bt), bt_stride=self.bt.stride(0), bt_rows=self.bt.shape[0],
                             n_pages=kp.shape[0] - 1, H=H, G=G, D=D, V=V, chunk=m.chunk, scale=m.scale, r1=K.ptr(L.r1), r2=K.ptr(L.r2),
                             sink=1, r=work, status=st, pdl=pdl)
-        if self.attn_tc and longest >= self.TC_MIN_TOKENS and max(D, V) <= K.chunk_tc_max_width():
-            K.chunk_attention_tc(a)
-        else:
-            K.chunk_attention(a, self.f32, self._ks(T, m))
+        self._chunk_attention(a, m, m.chunk, T, longest)
         self._gemm(L.wo, vo, self._rows("y", T, self.d), T)
 
     def _recurrent(self, L, T: int, work: "K.Ragged", single: bool) -> None:
@@ -146,9 +134,9 @@ class NativeMakodra(NativeLayered):
         vo = self._rows("vo", T, ldo)
         K.memory_scan(K.ScanArgs(proj=K.ptr(proj), ldp=proj.stride(0), r_off=0, k_off=HD, v_off=2 * HD, g_off=3 * HD, a_off=4 * HD,
                                  z=K.ptr(z), ldz=HD, w0=K.ptr(L.w0), a_bias=K.ptr(L.a_bias), bonus=K.ptr(L.bonus), onorm=K.ptr(L.onorm),
-                                 state=K.ptr(S), row_stride=S.stride(0), n_rows=S.shape[0], out=K.ptr(vo), ldo=ldo, H=m.heads, D=m.dim,
+                                 state=K.ptr(S), row_stride=S.stride(0), n_rows=S.shape[0], out=K.ptr(vo), ldo=ldo, H=m.heads, D=m.dim, V=m.dim,
                                  eps=self.c.rms_eps, unit_eps=DELTA_UNIT_EPS, log_decay=DELTA_LOG_DECAY, r=work,
-                                 status=K.ptr(self.status), pdl=pdl), delta, self.f32)
+                                 status=K.ptr(self.status), pdl=pdl), K.SCAN_DELTA if delta else K.SCAN_BONUS, self.f32)
         self._gemm(L.wo, vo, self._rows("y", T, self.d), T)
 
     def _swiglu(self, L, T: int) -> None:
@@ -159,9 +147,7 @@ class NativeMakodra(NativeLayered):
     # ---- forward ------------------------------------------------------------------------
     def _run(self, ids, positions, locs, T: int, work: "K.Ragged", single_rows: Optional[torch.Tensor], longest: int) -> torch.Tensor:
         assert T <= self.T and (self.state is not None or not self.m.has_state)
-        if longest < self.BLOCK:          # every sequence is one block: walk it by its own length
-            work = K.Ragged.from_buffer_copy(work)
-            work.B = longest
+        work = self._walk(work, longest)
         for s in self._steps:
             a, L, kind = s["args"], s["L"], s["kind"]
             if s["prev"] is None:

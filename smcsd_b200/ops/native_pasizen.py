@@ -43,18 +43,8 @@ class NativePasizen(NativeLayered):
         self._room("z", T * most(round_up(f.ff, 8) for f in dense), torch.float32)
         self._room("act", T * most([round_up(f.ff, 8) for f in dense] +
                                    [round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared]), self.dt)
-        pairs = T * most(f.router.top for f in moe)
-        self._room("idx", pairs, torch.int32)
-        self._room("wgt", pairs, torch.float32)
-        self._room("slot", pairs, torch.int32)
-        self._room("src", pairs, torch.int32)
-        self._room("tiles", 4 * most(f.router.experts for f in moe) + 4 * (pairs // 16 + 1), torch.int32)
-        self._room("xe", pairs * self.d8, self.dt)
-        self._room("ea", pairs * most(round_up(f.expert.ff, GU_BLOCK) for f in moe), self.dt)
-        self._room("ye", pairs * self.d, torch.float32)
-        if self.f32:
-            self._room("gu", max([pairs * 2 * round_up(f.expert.ff, GU_BLOCK) for f in moe] +
-                                 [T * 2 * round_up(f.shared.ff, GU_BLOCK) for f in moe if f.shared], default=0), torch.float32)
+        self._room_experts(moe)
+        self._room_gate_up([], moe)
         self.attn_tc = not self.f32 and env_flag("SMC_LATENT_TC", True)
         self._steps = self._build_steps()
 
@@ -95,27 +85,9 @@ class NativePasizen(NativeLayered):
         """Record the context-length hint; returns what it decides about the launch grids (part of a graph's identity)."""
         self.ctx_hint = int(ctx)
         shapes = sorted({(L.mixer.heads, round_up(L.mixer.kv_rank, 64)) for L in self.c.layers})
-        return tuple(self._ks(bs * ((E + self.BLOCK - 1) // self.BLOCK), min(E, self.BLOCK), H, Rp) for E in Es for H, Rp in shapes)
-
-    def _ks(self, n_blk: int, tokens: int, H: int, Rp: int) -> int:
-        """Key splits of one layer's attention: ``n_blk`` blocks of at most ``tokens`` tokens."""
-        if not self.attn_tc or Rp > K.latent_tc_max_width():
-            return 1
-        ks = K.latent_tc_splits(n_blk * ((tokens * H + 127) // 128), Rp, self.ctx_hint)
-        cap = max(1, int(self.attn_splits))
-        while ks > cap:
-            ks //= 2
-        return ks
+        return tuple(self._latent_splits(bs * ((E + self.BLOCK - 1) // self.BLOCK), min(E, self.BLOCK), H, Rp) for E in Es for H, Rp in shapes)
 
     # ---- products -----------------------------------------------------------------------
-    def _per_head(self, W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, M: int, H: int, x_cols: int, out_cols: int) -> None:
-        """Head h: out[:, h * out_cols ..] = X[:, h * x_cols ..] W_h^T, in the activation type."""
-        link = K.GroupLink(mode=K.GROUP_BATCHED, groups=H, w_rows=out_cols, x_cols=x_cols, out_cols=out_cols)
-        if self.f32:
-            K.gemm_f32(W, X, out, N=out_cols, M=M, link=link, pdl=self.pdl)
-        else:
-            K.gemm_grouped(W, X, out, N=out_cols, M=M, splits=1, epi=K.EPI_BF16, link=link, status=self.status, pdl=self.pdl)
-
     def _glu_gemm(self, W: torch.Tensor, X: torch.Tensor, act: torch.Tensor, M: int, limit: float, link: "K.GroupLink") -> None:
         """act = clamped gated unit of the interleaved gate / up product."""
         link.act, link.limit, link.slope = K.ACT_CLAMPED, limit, GLU_SIGMOID_SLOPE
@@ -131,18 +103,12 @@ class NativePasizen(NativeLayered):
         self._gemm(L.wqc, self.xa, proj, T)
         pool = self.kv.k[run]
         q = None if self.f32 else self._rows("q", T, nq)
-        K.latent_new(proj, q, pool, L.c_norm, locs, nq=nq, R=R, eps=self.c.rms_eps, M=T, status=self.status, f32=self.f32, pdl=pdl)
+        K.latent_new(K.LatentNewArgs(proj=K.ptr(proj), ldp=proj.stride(0), nq=nq, c_off=nq, R=R, c_norm=K.ptr(L.c_norm), eps=self.c.rms_eps,
+                                     q=K.ptr(q), ldq=nq, pool=K.ptr(pool), ldc=Rp, n_pages=pool.shape[0] - 1, locs=K.ptr(locs),
+                                     status=K.ptr(self.status), pdl=int(pdl)), T, self.f32)
         lat, ctx, vo = self._rows("lat", T, H * Rp), self._rows("ctx", T, H * Rp), self._rows("vo", T, ov)
         self._per_head(L.wuk_t, proj if q is None else q, lat, T, H, D8, Rp)
-        a = K.LatentArgs(q=K.ptr(lat), pool=K.ptr(pool), out=K.ptr(ctx), block_table=K.ptr(self.bt), bt_stride=self.bt.stride(0),
-                         bt_rows=self.bt.shape[0], n_pages=pool.shape[0] - 1, H=H, ldc=Rp, scale=m.scale, r=work,
-                         status=K.ptr(self.status), pdl=int(pdl))
-        if self.attn_tc and Rp <= K.latent_tc_max_width():
-            tokens = min(longest, self.BLOCK)
-            ks = self._ks(work.n_blk, tokens, H, Rp)
-            K.latent_attention_tc(a, tokens=T, blk_rows=tokens * H, splits=ks)
-        else:
-            K.latent_attention(a, self.f32)
+        self._latent_attention(lat, pool, ctx, H, m.scale, T, work, longest)
         self._per_head(L.wuv, ctx, vo, T, H, Rp, m.vdim)
         self._gemm(L.wo, vo, self._rows("y", T, self.d), T)
 
@@ -156,27 +122,10 @@ class NativePasizen(NativeLayered):
 
     def _experts(self, s: dict, T: int) -> None:
         L, f, pdl = s["L"], s["L"].spec.mlp, self.pdl
-        r, E, top = f.router, f.router.experts, f.router.top
-        n = T * top
-        idx, wgt, slot, src, tiles = (self._flat[k] for k in ("idx", "wgt", "slot", "src", "tiles"))
-        K.route(self.n, L.router, idx, wgt, d=self.d, top=top, groups=r.groups, keep=r.keep, T=T, f32=self.f32, pdl=pdl)
-        avg = (n + E - 1) // E
-        bn = 64 if self.f32 else 16 if avg <= 16 else 32 if avg <= 32 else 64 if avg <= 64 else 128
-        max_tiles = n // bn + min(E, n)
-        K.dispatch(idx, slot, src, tiles, n=n, top=top, experts=E, rows=bn, max_tiles=max_tiles, status=self.status, pdl=pdl)
-        xe, ffp = self._rows("xe", n, self.d8), L.e_down.shape[-1]
-        K.gather_rows(self.xa, src, xe, n=n, n_src=T, status=self.status, pdl=pdl)
-        ea, ye = self._rows("ea", n, ffp), self._rows("ye", n, self.d)
-        link = K.GroupLink(mode=K.GROUP_TILED, groups=E, w_rows=2 * ffp, tiles=K.ptr(tiles), max_tiles=max_tiles, bn=bn)
-        self._glu_gemm(L.e_gu, xe, ea, n, f.expert.limit, link)
-        link = K.GroupLink(mode=K.GROUP_TILED, groups=E, w_rows=self.d, tiles=K.ptr(tiles), max_tiles=max_tiles, bn=bn)
-        if self.f32:
-            K.gemm_f32(L.e_down, ea, ye, N=self.d, M=n, link=link, pdl=pdl)
-        else:
-            units, slabs, kb, sp = min(E, n), (self.d + 127) // 128, (ffp + 63) // 64, 1
-            while sp < 8 and units * slabs * sp * 2 <= 256 and kb // (sp * 2) >= 2:
-                sp *= 2
-            K.gemm_grouped(L.e_down, ea, ye, N=self.d, M=n, splits=sp, epi=K.EPI_STORE_F32, link=link, status=self.status, pdl=pdl)
+        r = f.router
+        K.route(self.n, L.router, self._flat["idx"], self._flat["wgt"], d=self.d, top=r.top, groups=r.groups, keep=r.keep, T=T, f32=self.f32,
+                pdl=pdl)
+        self._expert_rows(L, f, self.xa, T, lambda W, X, out, M, unit, link: self._glu_gemm(W, X, out, M, unit.limit, link))
         if f.shared is not None:
             sa = self._rows("act", T, L.s_down.shape[1])
             self._glu_gemm(L.s_gu, self.xa, sa, T, f.shared.limit, K.GroupLink())

@@ -245,8 +245,8 @@ def test_memory_scan(H, D, rule, f32):
         r, keep = work(lens, at, rows)
         k.memory_scan(k.ScanArgs(proj=k.ptr(p), ldp=p.shape[1], r_off=0, k_off=HD, v_off=2 * HD, g_off=3 * HD, a_off=4 * HD, z=k.ptr(zd),
                                  ldz=HD, w0=k.ptr(w0d), a_bias=k.ptr(bd), bonus=k.ptr(bd), onorm=k.ptr(od), state=k.ptr(state),
-                                 row_stride=stride, n_rows=n_rows, out=k.ptr(out), ldo=ldo, H=H, D=D, eps=eps, unit_eps=1e-6,
-                                 log_decay=math.exp(-0.5), r=r, status=k.ptr(st)), is_delta, f32)
+                                 row_stride=stride, n_rows=n_rows, out=k.ptr(out), ldo=ldo, H=H, D=D, V=D, eps=eps, unit_eps=1e-6,
+                                 log_decay=math.exp(-0.5), r=r, status=k.ptr(st)), k.SCAN_DELTA if is_delta else k.SCAN_BONUS, f32)
         want = torch.cat([ref[s][at[s]:at[s] + m] for s, m in enumerate(lens)])
         close(out[:, :HD], want, 3e-5 if f32 else 8e-3)
         at = [a + m for a, m in zip(at, lens)]

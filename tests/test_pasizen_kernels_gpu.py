@@ -341,7 +341,9 @@ def test_new_latents_reach_their_pages(f32):
     M, nq, R, ldc = 9, 3 * 40, 48, 64
     proj, nw, pool = _rnd(M, nq + R), _rnd(R, seed=1), torch.zeros(31, ldc, dtype=dt, device=DEV)
     q, locs, st = torch.zeros(M, nq, dtype=dt, device=DEV), _ints([5, 1, 30, 2, 17, 9, 8, 3, 4]), _status()
-    K.latent_new(proj, q, pool, nw, locs, nq=nq, R=R, eps=1e-4, M=M, status=st, f32=f32)
+    K.latent_new(K.LatentNewArgs(proj=K.ptr(proj), ldp=proj.stride(0), nq=nq, c_off=nq, R=R, c_norm=K.ptr(nw), eps=1e-4, q=K.ptr(q),
+                                 ldq=q.stride(0), pool=K.ptr(pool), ldc=pool.stride(0), n_pages=pool.shape[0] - 1, locs=K.ptr(locs),
+                                 status=K.ptr(st)), M, f32)
     ref = O.rms_normalise(proj[:, nq:].double(), 1e-4) * nw.double()
     _close(pool[locs.long(), :R], ref, 1e-5 if f32 else 8e-3)
     assert pool[:, R:].abs().sum() == 0 and (q == proj[:, :nq].to(dt)).all() and int(st) == 0
