@@ -8,7 +8,7 @@ import torch
 
 import pasizen_models
 import pasizen_oracle
-from pasizen_models import far_effect, row_error, tokens
+from pasizen_models import far_effect, row_error
 
 
 @dataclass
@@ -56,7 +56,7 @@ def feed_in_cuts(eng, rid, ids, cuts):
 def whole_portions_and_decoding(ctx, tmp_path, name):
     """One sequence whole, in portions of several sizes (two tokens at the least), and token by token."""
     folder, cfg, W = ctx.models.save_model(tmp_path / name, name)
-    ids = tokens(cfg, 150)
+    ids = ctx.models.tokens(cfg, 150)
     ref = ctx.oracle.forward(cfg, W, ids)
     eng = engine(ctx, folder)
     effect = far_effect(lambda x: ctx.oracle.forward(cfg, W, x), cfg, ids, ref)
@@ -77,7 +77,7 @@ def mixed_batches(ctx, tmp_path, name):
     lens = {"a": 130, "b": 40, "c": 70, "d": 5}
     eng = engine(ctx, folder, max_tokens=sum(lens.values()) + 3)
     for gen in range(3):
-        ids = {k: tokens(cfg, n, seed=10 * gen + i) for i, (k, n) in enumerate(lens.items())}
+        ids = {k: ctx.models.tokens(cfg, n, seed=10 * gen + i) for i, (k, n) in enumerate(lens.items())}
         ref = {k: ctx.oracle.forward(cfg, W, v) for k, v in ids.items()}
         at, got = {k: 0 for k in ids}, {k: [] for k in ids}
         plan = [{"a": 64, "b": 1}, {"b": 2, "c": 66}, {"a": 1, "b": 30, "c": 1, "d": 3}, {"a": 62, "d": 1}, {"a": 1, "b": 5, "c": 1, "d": 1},
@@ -99,7 +99,7 @@ def mixed_batches(ctx, tmp_path, name):
 def long_decoding(ctx, tmp_path, name, n=330):
     """Hundreds of single-token steps behind a short prompt, three sequences at once at different lengths."""
     folder, cfg, W = ctx.models.save_model(tmp_path / name, name, seed=5)
-    seqs = {k: tokens(cfg, n + i, seed=20 + i) for i, k in enumerate("xyz")}
+    seqs = {k: ctx.models.tokens(cfg, n + i, seed=20 + i) for i, k in enumerate("xyz")}
     eng = engine(ctx, folder)
     got = {k: [] for k in seqs}
     out = eng.feed([(k, seqs[k][:2 + i], [1 + i]) for i, k in enumerate(seqs)])
@@ -119,7 +119,7 @@ def greedy_generation(ctx, tmp_path, name, gammas=(1, 3), **kw):
     """Greedy output of ``generate``: every token is the oracle's argmax given the tokens before it, or within the tolerance
     of it.  The proposal is the model itself at temperature 0, so the text is the target's own greedy text."""
     folder, cfg, W = ctx.models.save_model(tmp_path / name, name, seed=7)
-    prompts = [tokens(cfg, n, seed=40 + n) for n in (1, 9, 70)]
+    prompts = [ctx.models.tokens(cfg, n, seed=40 + n) for n in (1, 9, 70)]
     outs = {}
     for gamma in gammas:
         for defer in (True, False):
@@ -137,23 +137,54 @@ def greedy_generation(ctx, tmp_path, name, gammas=(1, 3), **kw):
 
 
 def chunk_edges(ctx, tmp_path, cfg, size, n):
-    """One attention layer alone: a changed token moves exactly the rows of its own chunk behind it, whether they come with
-    the prompt or are decoded, and the first rows of every chunk (few keys beside the sink) are right."""
-    folder, cfg, W = ctx.models.save_model(tmp_path / "edges", cfg, seed=4)
+    """One attention layer alone: a changed token moves exactly the rows of its own chunk behind it, and the first rows of every
+    chunk (few keys beside the sink) are right."""
+    seen_by(ctx, tmp_path, cfg, n, (0, size - 2, size - 1, size, 2 * size - 1, 2 * size), lambda j: (j // size + 1) * size)
+
+
+def seen_by(ctx, tmp_path, cfg, n, changed, end, weights_seed=4):
+    """One layer alone: changing the token at j (each of ``changed``) moves rows j up to end(j) and no others, whether they come
+    with the prompt or are decoded."""
+    folder, cfg, W = ctx.models.save_model(tmp_path / "edges", cfg, seed=weights_seed)
     eng = engine(ctx, folder)
-    ids = tokens(cfg, n, seed=6)
+    ids = ctx.models.tokens(cfg, n, seed=6)
     ref = ctx.oracle.forward(cfg, W, ids)
     base = feed_in_cuts(eng, "a", ids, [n])
     check(ctx, base, ref)
-    for j in (0, size - 2, size - 1, size, 2 * size - 1, 2 * size):
+    for j in changed:
         other = list(ids)
         other[j] = (ids[j] + 1) % cfg["vocab"]
-        lo, hi = j, min(n, (j // size + 1) * size)
+        lo, hi = j, min(n, end(j))
         for cuts in ([n], [j + 1] + [1] * (n - j - 1), [max(j - 1, 1), n - max(j - 1, 1)]):
             got = feed_in_cuts(eng, "b", other, cuts)
             e = row_error(got, base)
             out = torch.cat([e[:lo], e[hi:]])
-            assert out.max() <= ctx.tol, (j, cuts[:3], out.max().item())
+            assert out.numel() == 0 or out.max() <= ctx.tol, (j, cuts[:3], out.max().item())
             assert e[lo:hi].min() > 0 and e[lo] > 0.05
             check(ctx, got, ctx.oracle.forward(cfg, W, other), (j, cuts[:3]))
+    idle(eng)
+
+
+def window_ends(ctx, tmp_path, cfg, size):
+    """One layer with a window alone: the seeking token stands just inside and just outside the window of the token it seeks, in
+    the prompt and decoded; inside, it hears it loudly, outside not at all."""
+    folder, cfg, W = ctx.models.save_model(tmp_path / "window", cfg, seed=9)
+    sought, seeker = ctx.models.pair(cfg)
+    eng = engine(ctx, folder)
+    ids = ctx.models.tokens(cfg, 2 * size + 40, seed=8)
+    ids[0] = 1
+    for j in (0, 1, 15, size - 1, size + 3):
+        for inside in (True, False):
+            at = j + size - inside
+            a = list(ids[:at + 3])
+            a[j], a[at] = sought, seeker
+            b = list(a)
+            b[j] = 2
+            ref, other = ctx.oracle.forward(cfg, W, a), ctx.oracle.forward(cfg, W, b)
+            moved = row_error(other[at:at + 1], ref[at:at + 1]).item()
+            assert moved > 0.3 if inside else moved == 0.0
+            for cuts in ([at + 3], [at] + [1] * 3, [j + 1, 2] + [1] * (at - j), [at - 1, 2, 2]):
+                got = feed_in_cuts(eng, "a", a, cuts)
+                check(ctx, got, ref, (j, inside, cuts[:3]))
+                assert row_error(got[at:at + 1], ref[at:at + 1]).item() < 0.1
     idle(eng)
