@@ -87,9 +87,10 @@ def make_weights(cfg, seed=0):
             k = lin(H * D, d)
             slow = torch.rand(H, generator=g) < 0.6            # these heads keep what they hold
             slow[0] = True
+            loud = sought * W[p + "norm1"]                     # and this token enters with more weight
             q = seek(lin(H * D, d).view(H, D, d), k.view(H, D, d), seeker * W[p + "norm1"], sought * W[p + "norm1"])
             W.update({x + "k": k, x + "q": q.reshape(H * D, d), x + "v": lin(H * E, d), x + "g": 0.5 * lin(H * E, d),
-                      x + "i": lin(H, d), x + "i.b": 0.5 * r(H), x + "f": 0.3 * lin(H, d), x + "f.b": torch.where(slow, 30.0, 1.0) + 0.3 * r(H),
+                      x + "i": lin(H, d) + 6.0 * loud / loud.pow(2).sum(), x + "i.b": -2.0 + 0.5 * r(H), x + "f": 0.3 * lin(H, d), x + "f.b": torch.where(slow, 30.0, 1.0) + 0.3 * r(H),
                       x + "norm": gainful(H * E), x + "o": lin(d, H * E)})
         elif L["type"] == "latent_attention":
             R, Q, rot, n1 = m["kv_rank"], m["q_rank"], m["rot_dim"], W[p + "norm1"]
