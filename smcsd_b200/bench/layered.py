@@ -3,7 +3,8 @@
     python -m smcsd_b200.bench.layered --width 2048 --family makodra
     (or: python bench.py --layered 2048,1024 --layered-family makodra)
 
-Pasizen runs beside a dense Llama-style model, Makodra beside that and a Gated-DeltaNet hybrid with as many attention layers.
+Pasizen runs beside a dense Llama-style model, Makodra beside that and a Gated-DeltaNet hybrid with as many attention layers,
+Funevik beside a dense model, Makodra (memories, attention over heads) and Pasizen (latent attention, experts).
 All run random weights through their kernel chains: the same width, heads, layer count, head and feed-forward weights per
 layer; the dense models cache as many bytes per token as their KV heads take.  A forward is captured in a CUDA
 graph and timed with CUDA events (weights of all layers exceed L2; the cached keys come on top).  For the kernel table every
@@ -21,8 +22,8 @@ from typing import Dict, List, Tuple
 
 import torch
 
-from ..models.config import (ChunkAttentionSpec, FeedForwardSpec, GluSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RecurrentSpec,
-                             RouterSpec)
+from ..models.config import (ChunkAttentionSpec, FeedForwardSpec, GluSpec, GroupedAttentionSpec, LatentAttentionSpec, LayerSpec, ModelConfig,
+                             RecurrentSpec, RotarySpec, RouterSpec)
 from ..utils.roofline import measured_peaks
 
 VOCAB = 32768
@@ -66,6 +67,21 @@ def makodra_config(width: int, layers: int, memory_dim: int = 64, chunk: int = 8
                        name=f"makodra-{width}-heads{memory_dim}")
 
 
+def funevik_config(width: int, layers: int, kv_rank: int, experts: bool, window: int = 1024) -> ModelConfig:
+    """Two memories, one latent and one full attention in turn; feed-forwards as in ``makodra_config`` or ``pasizen_config``."""
+    H, rot = width // 128, RotarySpec(64, 10000.0)
+    mlp = FeedForwardSpec("geglu", ff=2 * width)
+    if experts:
+        ff = 3 * width
+        mlp = FeedForwardSpec("moe", expert=GluSpec(ff // 8), router=RouterSpec(32, 4, bias=True), shared=GluSpec(ff // 6), shared_gate=True)
+    mem = RecurrentSpec("mlstm", max(1, width // 256), 128, 256, 15.0)
+    four = [mem, mem, LatentAttentionSpec(H, 128, 128, kv_rank, 192 ** -0.5, 3 * width // 8, rot, window, True),
+            GroupedAttentionSpec(H, max(1, H // 4), 128, 128, 128 ** -0.5, 4, rot, 50.0)]
+    return ModelConfig(arch="funevik", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=H, n_kv_heads=max(1, H // 4), head_dim=128,
+                       ffn_size=0, rms_eps=1e-6, max_position=1 << 20, embed_scale=width ** 0.5, layers=[LayerSpec(m, mlp) for m in four * (layers // 4)],
+                       name=f"funevik-{width}-{'experts' if experts else 'dense'}")
+
+
 class Rig:
     """One model with its chain, caches filled with noise, and step inputs."""
 
@@ -73,6 +89,7 @@ class Rig:
         from ..memory.pools import KVPool, StatePool
         from ..models import build_model
         from ..ops.native_backend import NativeLlama
+        from ..ops.native_funevik import NativeFunevik
         from ..ops.native_hybrid import NativeHybrid
         from ..ops.native_makodra import NativeMakodra
         from ..ops.native_pasizen import NativePasizen
@@ -90,7 +107,7 @@ class Rig:
         T = n_prompts * prompt
         if cfg.arch != "llama":
             self.state = StatePool(m.state_spec(), rows, dev)
-            Chain = {"pasizen": NativePasizen, "makodra": NativeMakodra, "hybrid_gdn": NativeHybrid}[cfg.arch]
+            Chain = {"pasizen": NativePasizen, "makodra": NativeMakodra, "funevik": NativeFunevik, "hybrid_gdn": NativeHybrid}[cfg.arch]
             make = lambda t, lr: Chain(m, kv, self.bt, t, lr, 16, self.status, True, state=self.state)
         else:
             make = lambda t, lr: NativeLlama(m, kv, self.bt, t, lr, 16, self.status, True)
@@ -154,7 +171,7 @@ def timed(fn, reps: int = 20) -> float:
 RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
             "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc", "gdn_step",
             "rope_kv_write_heads", "post_norm_step", "token_shift", "heads_new", "chunk_attention", "chunk_attention_tc", "memory_scan",
-            "tanh_rows", "low_rank")
+            "tanh_rows", "low_rank", "side_step", "conv_heads", "rotate_heads", "gated_step")
 
 
 def record(fn) -> List[Tuple[str, tuple, dict]]:
@@ -199,8 +216,10 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
         return kind, wbytes + M * Kd * 2 * groups + M * N * groups * per_out, flops
     if name == "latent_attention_tc":
         s = a[0]
-        fl = 2.0 * 2 * T * s.H * keys * s.ldc
-        return "attention", T * s.H * s.ldc * 4 + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.ldc * 2, fl
+        seen, held = keys, rig.ctx if T == rig.bs else rig.prompt
+        if s.window:
+            seen, held = min(keys, s.window), min(held, s.window) if T == rig.bs else held
+        return ("latent " if rig.cfg.arch == "funevik" else "") + "attention", T * s.H * s.ldc * 4 + seqs * held * s.ldc * 2, 4.0 * T * s.H * seen * s.ldc
     if name == "attention_fused":
         H, Hkv, D = kw["Hq"], kw["Hkv"], kw["D"]
         fl = 2.0 * 2 * T * H * keys * D
@@ -209,12 +228,22 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
         s = a[0]
         fl = 2.0 * T * s.H * keys * (s.D + s.V)
         return "attention", T * s.H * (2 * s.D + 6 * s.V) + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.G * (s.D + s.V) * 2, fl
-    if name == "memory_scan":
-        s, is_delta = a[0], a[1]
-        HD = s.H * s.D
+    if name in ("memory_scan", "gated_step"):
+        s, kind = a[0], a[1] if name == "memory_scan" else 2
+        HD, HV = s.H * s.D, s.H * s.V
         # fp32 multiply-adds per matrix element and token, as bf16-rate equivalents (the floor divides by the bf16 rate)
-        fl = 2.0 * (5 if is_delta else 3) * T * HD * s.D * measured_peaks()[1] / F32_TFLOPS
-        return "memory " + ("delta" if is_delta else "wkv"), T * HD * (4 * (6 if is_delta else 5) + 2) + seqs * HD * s.D * 8, fl
+        fl = 2.0 * (5 if kind == 1 else 3) * T * HV * s.D * measured_peaks()[1] / F32_TFLOPS
+        name = ("wkv", "delta", "gated")[kind]
+        return "memory " + name, T * (HD * 4 * (3, 4, 2)[kind] + HV * 10) + seqs * HV * s.D * 8, fl
+    if name == "side_step":
+        s = a[0]
+        by = T * d * (4 * (s.ids is None) + 4 * (not s.final) + 4 * bool(s.y1) + 4 * bool(s.y2) + 4 * s.top + 2 + 2 * bool(s.w2) + 4 * bool(s.n2))
+        return ("embedding + norms" if s.ids else "stream + final norm" if s.final else "stream + norms") + (" + experts" if s.top else ""), by, 0.0
+    if name == "conv_heads":
+        s = a[0]
+        return "conv + rotation + new heads", T * ((s.H + s.G) * s.D + s.G * s.V) * 6, 0.0
+    if name == "rotate_heads":
+        return "rotate queries", T * kw["heads"] * kw["width"] * 6, 0.0
     if name == "gdn_step":
         Hv, dk, dv = kw["Hv"], kw["dk"], kw["dv"]
         conv = 2 * kw["Hk"] * dk + Hv * dv
@@ -242,7 +271,8 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
     if name == "poly_norm":
         return "PolyNorm", T * kw["ff"] * 6, 0.0
     if name == "latent_new":
-        return "latent_new", T * (kw["nq"] * 6 + kw["R"] * 6), 0.0
+        s = a[0]
+        return "latent_new", T * (s.nq + s.R + s.rot) * 6, 0.0
     if name == "gather_rows":
         return "gather_rows", kw["n"] * a[2].shape[1] * 4, 0.0
     if name == "route":
@@ -273,9 +303,11 @@ def run(width: int, layers: int = 12, bs: int = 8, ctx: int = 1024, prompt: int 
         tables: bool = True, family: str = "pasizen") -> dict:
     import gc
     rec = {"width": width, "layers": layers, "decode": {"sequences": bs, "context": ctx}, "prefill": {"prompts": n_prompts, "tokens": prompt},
-           "kv_rank": kv_rank if family == "pasizen" else None, "pages": "scattered", "weights": "random, bf16", "models": []}
-    own = [pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)] if family == "pasizen" else \
-        [hybrid_config(width, layers), makodra_config(width, layers), makodra_config(width, layers, 128)]
+           "kv_rank": kv_rank if family != "makodra" else None, "pages": "scattered", "weights": "random, bf16", "models": []}
+    own = {"pasizen": lambda: [pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)],
+           "makodra": lambda: [hybrid_config(width, layers), makodra_config(width, layers), makodra_config(width, layers, 128)],
+           "funevik": lambda: [makodra_config(width, layers, 128), pasizen_config(width, layers, kv_rank, True),
+                               funevik_config(width, layers, kv_rank, False), funevik_config(width, layers, kv_rank, True)]}[family]()
     for cfg in [dense_config(width, layers)] + own:
         rig = Rig(cfg, bs, ctx, prompt, n_prompts)
         T = n_prompts * prompt
@@ -313,7 +345,7 @@ def main(argv=None) -> None:
     ap.add_argument("--ctx", type=int, default=1024)
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--kv-rank", type=int, default=256)
-    ap.add_argument("--family", default="pasizen", choices=["pasizen", "makodra"])
+    ap.add_argument("--family", default="pasizen", choices=["pasizen", "makodra", "funevik"])
     ap.add_argument("--no-tables", action="store_true")
     ap.add_argument("--json", default=None)
     ns = ap.parse_args(argv)

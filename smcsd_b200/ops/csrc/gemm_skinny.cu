@@ -110,7 +110,7 @@ __device__ __forceinline__ float gated_unit(const GroupLink& a, float g, float u
     u = fminf(fmaxf(u, -a.limit), a.limit);
     return g / (1.0f + __expf(-a.slope * g)) * (u + 1.0f);
   }
-  if (GRP && a.act == 2) return gelu_tanh(g) * u;
+  if (a.act == 2) return gelu_tanh(g) * u;
   return g / (1.0f + __expf(-g)) * u;
 }
 
@@ -791,7 +791,7 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
     }
     return -30;
   }
-  if (grp != nullptr) {                       // builds with the group logic compiled in
+  if (grp != nullptr && (gmode != 0 || grp->act == 1)) {       // builds with the group logic and the clamped unit compiled in
     switch (epi) {
       case EPI_BF16: return dispatch_bn<EPI_BF16, true>(bn, tmW, tmX, p, grid, stream);
       case EPI_SWIGLU_BF16: return dispatch_bn<EPI_SWIGLU_BF16, true>(bn, tmW, tmX, p, grid, stream);

@@ -19,36 +19,12 @@
 // matrix, so that a token costs one reduction: for delta the read-out is (r w)^T M - (r.a u)(u^T M) + (r.k) v.
 // The recurrence is held to fp32 (a bf16 or tf32 chunk-parallel form would round the state), so the floor is the CUDA cores'
 // rate; products and sums are issued two at a time (f32x2).
-#include "ragged.cuh"
+#include "memory_scan.cuh"
 
 namespace smc {
 
 constexpr int SCAN_PRODUCERS = 8;        // warps
 constexpr int SCAN_CONSUMERS = 256;      // threads at the most
-
-enum { SCAN_BONUS = 0, SCAN_DELTA = 1, SCAN_GATED = 2 };
-
-struct ScanArgs {
-  const float* proj;        // [T, ldp]: H * D columns of r and k, H * V of v and gate at these offsets, from a_off on the removal
-  int ldp, r_off, k_off, v_off, g_off, a_off;        // rates (delta, H * D) or the input and forget gates (gated, 2 H)
-  const float* z;           // [T, ldz] decay logits, H * D
-  int ldz;
-  const float* w0;          // [H * D]
-  const float* a_bias;      // delta [H * D], gated [2 H]
-  const float* bonus;       // wkv
-  const float* onorm;       // [H * V]
-  float* state;             // row r: state + r * row_stride, [H, V (and one more if gated), D (key)]
-  long long row_stride;
-  int n_rows;
-  void* out;                // [T, ldo]
-  int ldo, H, D, V;
-  float eps, unit_eps, log_decay;
-  float* top;               // gated: row r: top + r * row_stride, [H] running maxima
-  float gate_cap, r_scale;  // gated: r is multiplied by r_scale
-  Ragged r;
-  int* status;
-  int pdl;
-};
 
 typedef unsigned long long f2_t;
 __device__ __forceinline__ f2_t pack2(float a, float b) {
@@ -76,14 +52,11 @@ __device__ __forceinline__ void store_shared_unordered(uint32_t addr, float v) {
   asm volatile("st.shared.f32 [%0], %1;" ::"r"(addr), "f"(v));
 }
 __device__ __forceinline__ float sum_of(f2_t a) { const float2 v = unpack2(a); return v.x + v.y; }
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 __host__ __device__ constexpr int scan_tokens(int dkp) { return dkp <= 128 ? 16 : 8; }       // tokens of a tile
 __host__ __device__ constexpr int scan_vectors(int kind) { return kind == SCAN_DELTA ? 5 : kind == SCAN_GATED ? 2 : 3; }
 __host__ __device__ constexpr int scan_columns(int dkp) { return dkp <= 128 ? 2 : 1; }       // of a consumer thread
 __host__ __device__ constexpr int scan_max_columns(int dkp) { return SCAN_CONSUMERS / 4 * scan_columns(dkp); }      // of a CTA
-
-__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
 template <int KIND, int DKP>
 __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {

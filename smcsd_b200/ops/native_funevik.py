@@ -16,6 +16,7 @@ captured in a graph.
 from __future__ import annotations
 
 import math
+from contextlib import nullcontext
 from typing import Dict, List, Optional
 
 import torch
@@ -25,10 +26,12 @@ from ..models.funevik import conv_channels, latent_row
 from ..models.layered import GU_BLOCK, round_up
 from ..models.layers import NORMALISER_EPS
 from . import native as K
-from .native_layered import NativeLayered
+from .native_layered import NativeLayered, env_flag
 
 
 class NativeFunevik(NativeLayered):
+    BESIDE_TOKENS = 1 << 30               # longest step whose feed-forwards run on a second stream beside the mixers
+
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
         super().__init__(model, kv, block_table, max_tokens, max_logit_rows, attn_splits, status, pdl, state)
@@ -55,6 +58,7 @@ class NativeFunevik(NativeLayered):
         self._room_experts(moe)
         self._room_gate_up(dense, moe)
         self.attn_tc = not self.f32
+        self.beside = env_flag("SMC_BESIDE", True)
         self.freq: Dict[RotarySpec, torch.Tensor] = {}
         for rot in {L.spec.mixer.rot for L in ls if L.kind != "mlstm"}:
             self.freq[rot] = rot.base ** (-torch.arange(0, rot.dims, 2, dtype=torch.float64, device=self.dev) / rot.dims)
@@ -111,11 +115,14 @@ class NativeFunevik(NativeLayered):
         H, D, E, ldo = m.heads, m.dim, m.values, L.wo.shape[1]
         proj, vo = self._rows("proj", T, L.win.shape[0]), self._rows("vo", T, ldo)
         S, top = self.state.matrix(L.state), self.state.matrix(L.state + 1)
-        K.memory_scan(K.ScanArgs(proj=K.ptr(proj), ldp=proj.stride(0), r_off=0, k_off=H * D, v_off=2 * H * D, g_off=H * (2 * D + E),
-                                 a_off=2 * H * (D + E), a_bias=K.ptr(L.gate_bias), onorm=K.ptr(L.onorm), state=K.ptr(S),
-                                 row_stride=S.stride(0), n_rows=S.shape[0], out=K.ptr(vo), ldo=ldo, H=H, D=D, V=E, eps=self.c.rms_eps,
-                                 unit_eps=NORMALISER_EPS, top=K.ptr(top), gate_cap=m.gate_cap, r_scale=D ** -0.5, r=work,
-                                 status=K.ptr(self.status), pdl=int(self.pdl)), K.SCAN_GATED, self.f32)
+        a = K.ScanArgs(proj=K.ptr(proj), ldp=proj.stride(0), r_off=0, k_off=H * D, v_off=2 * H * D, g_off=H * (2 * D + E),
+                       a_off=2 * H * (D + E), a_bias=K.ptr(L.gate_bias), onorm=K.ptr(L.onorm), state=K.ptr(S), row_stride=S.stride(0),
+                       n_rows=S.shape[0], out=K.ptr(vo), ldo=ldo, H=H, D=D, V=E, eps=self.c.rms_eps, unit_eps=NORMALISER_EPS, top=K.ptr(top),
+                       gate_cap=m.gate_cap, r_scale=D ** -0.5, r=work, status=K.ptr(self.status), pdl=int(self.pdl))
+        if longest == 1 and K.gated_step_takes(D, E):
+            K.gated_step(a, self.f32)
+        else:
+            K.memory_scan(a, K.SCAN_GATED, self.f32)
         return vo
 
     def _attention(self, i: int, L, T: int, positions, locs, work: "K.Ragged", longest: int) -> torch.Tensor:
@@ -159,20 +166,25 @@ class NativeFunevik(NativeLayered):
         link.act, link.limit, link.slope = kind, math.inf, 1.0
         self._gated_gemm(W, X, act, M, GU_BLOCK, link, shift=0.0)
 
-    def _feed_forward(self, L, T: int) -> None:
-        f, y = L.spec.mlp, self._rows("y2", T, self.d)
+    def _feed_forward(self, L, T: int, forked: bool) -> None:
+        """All of the feed-forward but a shared expert; ``forked``: first work of a stream that has just been forked."""
+        f = L.spec.mlp
+        first = self._full_order if forked else nullcontext
         if f.kind != "moe":
             act = self._rows("act", T, L.wdown.shape[1])
-            self._unit(L.wgu, self.xb, act, T, K.GroupLink(), K.ACT_GELU)
-            self._gemm(L.wdown, act, y, T)
+            with first():
+                self._unit(L.wgu, self.xb, act, T, K.GroupLink(), K.ACT_GELU)
+            self._gemm(L.wdown, act, self._rows("y2", T, self.d), T)
             return
-        K.route(self._flat["n2"], L.router, self._flat["idx"], self._flat["wgt"], d=self.d, top=f.router.top, groups=1, keep=1, T=T,
-                f32=self.f32, bias=L.router_bias, gate=self._flat["sg"] if f.shared is not None else None, pdl=self.pdl)
+        with first():
+            K.route(self._flat["n2"], L.router, self._flat["idx"], self._flat["wgt"], d=self.d, top=f.router.top, groups=1, keep=1, T=T,
+                    f32=self.f32, bias=L.router_bias, gate=self._flat["sg"] if f.shared is not None else None, pdl=self.pdl)
         self._expert_rows(L, f, self.xb, T, lambda W, X, out, M, spec, link: self._unit(W, X, out, M, link))
-        if f.shared is not None:
-            act = self._rows("act", T, L.s_down.shape[1])
-            self._unit(L.s_gu, self.xb, act, T, K.GroupLink())
-            self._gemm(L.s_down, act, y, T)
+
+    def _shared_expert(self, L, T: int) -> None:
+        act = self._rows("act", T, L.s_down.shape[1])
+        self._unit(L.s_gu, self.xb, act, T, K.GroupLink())
+        self._gemm(L.s_down, act, self._rows("y2", T, self.d), T)
 
     # ---- forward ------------------------------------------------------------------------
     def _run(self, ids, positions, locs, T: int, work: "K.Ragged", single_rows: Optional[torch.Tensor], longest: int) -> torch.Tensor:
@@ -180,12 +192,28 @@ class NativeFunevik(NativeLayered):
         work = self._walk(work, longest)
         self._steps[0].ids = K.ptr(ids)
         mixers = {"mlstm": self._memory, "attention": self._attention, "latent": self._latent}
+        beside = self.beside and T <= self.BESIDE_TOKENS and not self.f32
+        joined = False
         for i, L in enumerate(self.m.layers):
-            K.side_step(self._steps[i], T, self.f32)
+            self._step(i, T, joined)
+            f = L.spec.mlp
+            joined = beside and f is not None
+            if joined:
+                with torch.cuda.stream(self._fork()):
+                    self._feed_forward(L, T, True)
             self._gemm(L.win, self.xa, self._rows("proj", T, L.win.shape[0]), T)
             vo = mixers[L.kind](i, L, T, positions, locs, work, longest)
             self._gemm(L.wo, vo, self._rows("y1", T, self.d), T)
-            if L.spec.mlp is not None:
-                self._feed_forward(L, T)
-        K.side_step(self._steps[-1], T, self.f32)
+            if f is not None and f.shared is not None:
+                self._shared_expert(L, T)
+            if joined:
+                self._join()
+            elif f is not None:
+                self._feed_forward(L, T, False)
+        self._step(len(self.m.layers), T, joined)
         return self.xa
+
+    def _step(self, i: int, T: int, joined: bool) -> None:
+        a = self._steps[i]
+        a.pdl = int(self.pdl and not joined)
+        K.side_step(a, T, self.f32)

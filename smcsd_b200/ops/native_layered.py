@@ -4,6 +4,7 @@ can be captured in a graph, and the head."""
 from __future__ import annotations
 
 import os
+from contextlib import contextmanager
 from typing import Dict, List, Optional
 
 import torch
@@ -41,6 +42,7 @@ class NativeLayered:
         self.ctx_hint = 0
         self._lm_parts = None
         self._splits: Dict = {}
+        self._side = None
         self.xa = torch.zeros(max_tokens, self.d8, dtype=self.dt, device=self.dev)
         # flat buffers, viewed per layer with that layer's own row width
         self._flat: Dict[str, torch.Tensor] = {}
@@ -173,6 +175,30 @@ class NativeLayered:
             K.chunk_attention_tc(a)
         else:
             K.chunk_attention(a, self.f32, self._chunk_splits(T, m, chunk))
+
+    # ---- two streams --------------------------------------------------------------------
+    @contextmanager
+    def _full_order(self):
+        """Launches that depend on work of two streams wait for all of it: no programmatic overlap with the kernel before."""
+        kept, self.pdl = self.pdl, False
+        try:
+            yield
+        finally:
+            self.pdl = kept
+
+    def _fork(self) -> "torch.cuda.Stream":
+        """The second stream, behind everything queued so far (in a capture it joins the same graph)."""
+        if self._side is None:
+            self._side = (torch.cuda.Stream(self.dev), torch.cuda.Event(), torch.cuda.Event())
+        side, forked, _ = self._side
+        forked.record()
+        side.wait_event(forked)
+        return side
+
+    def _join(self) -> None:
+        side, _, done = self._side
+        done.record(side)
+        torch.cuda.current_stream().wait_event(done)
 
     @staticmethod
     def _walk(work: "K.Ragged", longest: int) -> "K.Ragged":

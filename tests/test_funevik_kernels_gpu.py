@@ -241,10 +241,10 @@ def test_soft_capped_attention_with_head_gates(H, G, D, V, cap, form, splits):
 def test_gated_memory_scan(H, D, V, f32):
     """Ragged portions with state, normaliser and maximum carried on between two launches; other rows stay untouched."""
     k, rows, n_rows, eps, cap = K(), [3, 0, 5], 6, 1e-3, 6.0
-    parts = [[1, 17, 40], [33, 2, 1]]
+    parts = [[1, 17, 40], [1, 1, 1], [33, 2, 1], [1, 1, 1]]     # steps of single tokens take the kernel of their own
     total = [sum(p[s] for p in parts) for s in range(3)]
-    cols = H * (2 * D + 2 * V) + 2 * H
-    proj = [rnd(t, cols + 3, seed=s) for s, t in enumerate(total)]
+    cols, ldp = H * (2 * D + 2 * V) + 2 * H, (H * (2 * D + 2 * V) + 2 * H + 7) // 8 * 8
+    proj = [rnd(t, ldp, seed=s) for s, t in enumerate(total)]
     for x in proj:
         x[:, cols - 2 * H:cols] *= 4.0
     bias = torch.cat([rnd(H, seed=30), torch.where(torch.arange(H) % 2 == 0, 20.0, 1.0)])        # half of the heads keep what they hold
@@ -270,10 +270,14 @@ def test_gated_memory_scan(H, D, V, f32):
         p = dev(torch.cat([proj[s][at[s]:at[s] + m] for s, m in enumerate(lens)]))[0]
         out = torch.zeros(p.shape[0], ldo, dtype=torch.float32 if f32 else torch.bfloat16, device=DEV)
         r, keep = work(lens, at, rows)
-        k.memory_scan(k.ScanArgs(proj=k.ptr(p), ldp=p.shape[1], r_off=0, k_off=H * D, v_off=2 * H * D, g_off=H * (2 * D + V), a_off=2 * H * (D + V),
-                                 a_bias=k.ptr(gb), onorm=k.ptr(go), state=k.ptr(state), row_stride=stride, n_rows=n_rows, out=k.ptr(out), ldo=ldo,
-                                 H=H, D=D, V=V, eps=eps, unit_eps=1e-6, top=k.ptr(state[:, at_top:]), gate_cap=cap, r_scale=D ** -0.5, r=r,
-                                 status=k.ptr(st)), k.SCAN_GATED, f32)
+        args = k.ScanArgs(proj=k.ptr(p), ldp=p.shape[1], r_off=0, k_off=H * D, v_off=2 * H * D, g_off=H * (2 * D + V), a_off=2 * H * (D + V),
+                          a_bias=k.ptr(gb), onorm=k.ptr(go), state=k.ptr(state), row_stride=stride, n_rows=n_rows, out=k.ptr(out), ldo=ldo,
+                          H=H, D=D, V=V, eps=eps, unit_eps=1e-6, top=k.ptr(state[:, at_top:]), gate_cap=cap, r_scale=D ** -0.5, r=r,
+                          status=k.ptr(st))
+        if max(lens) == 1 and k.gated_step_takes(D, V):
+            k.gated_step(args, f32)
+        else:
+            k.memory_scan(args, k.SCAN_GATED, f32)
         close(out[:, :H * V], torch.cat([ref[s][at[s]:at[s] + m] for s, m in enumerate(lens)]), 5e-5 if f32 else 8e-3)
         at = [a + m for a, m in zip(at, lens)]
     for row, m in zip(rows, tops):
