@@ -171,7 +171,7 @@ def timed(fn, reps: int = 20) -> float:
 RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
             "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc", "gdn_step",
             "rope_kv_write_heads", "post_norm_step", "token_shift", "heads_new", "chunk_attention", "chunk_attention_tc", "memory_scan",
-            "tanh_rows", "low_rank", "side_step", "conv_heads", "rotate_heads", "gated_step")
+            "tanh_rows", "low_rank", "side_step", "conv_heads", "rotate_heads", "gated_step", "gated_chunk")
 
 
 def record(fn) -> List[Tuple[str, tuple, dict]]:
@@ -228,6 +228,9 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
         s = a[0]
         fl = 2.0 * T * s.H * keys * (s.D + s.V)
         return "attention", T * s.H * (2 * s.D + 6 * s.V) + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.G * (s.D + s.V) * 2, fl
+    if name == "gated_chunk":                    # intra-chunk products and two with the state per token, at the bf16 rate
+        s = a[0]
+        return "memory gated (chunked)", T * s.H * (s.D * 8 + s.V * 10) + seqs * s.H * s.V * s.D * 8, 2.0 * T * s.H * (2 * s.V * s.D + 32 * (s.D + s.V))
     if name in ("memory_scan", "gated_step"):
         s, kind = a[0], a[1] if name == "memory_scan" else 2
         HD, HV = s.H * s.D, s.H * s.V

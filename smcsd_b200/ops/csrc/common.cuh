@@ -314,9 +314,4 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
-// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), the tanh written as a sigmoid.
-__device__ __forceinline__ float gelu_tanh(float z) {
-  return z / (1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));
-}
-
 }  // namespace smc

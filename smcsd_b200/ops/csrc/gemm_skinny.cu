@@ -101,17 +101,18 @@ struct GemmParams {
   const float* w_scale;
   const float* x_scale;
   GroupLink grp;
+  float act_a, act_b;   // gated epilogue: g / (1 + exp(-g (act_a + act_b g^2))) u, silu with 1 and 0, gelu (tanh form) with the constants below
 };
+constexpr float GELU_A = 1.5957691216057308f, GELU_B = 1.5957691216057308f * 0.044715f;      // 2 sqrt(2 / pi), times its cubic's factor
 
 template <bool GRP>
-__device__ __forceinline__ float gated_unit(const GroupLink& a, float g, float u) {
-  if (GRP && a.act == 1) {
-    g = fminf(g, a.limit);
-    u = fminf(fmaxf(u, -a.limit), a.limit);
-    return g / (1.0f + __expf(-a.slope * g)) * (u + 1.0f);
+__device__ __forceinline__ float gated_unit(const GemmParams& p, float g, float u) {
+  if (GRP && p.grp.act == 1) {
+    g = fminf(g, p.grp.limit);
+    u = fminf(fmaxf(u, -p.grp.limit), p.grp.limit);
+    return g / (1.0f + __expf(-p.grp.slope * g)) * (u + 1.0f);
   }
-  if (a.act == 2) return gelu_tanh(g) * u;
-  return g / (1.0f + __expf(-g)) * u;
+  return g / (1.0f + __expf(-g * fmaf(p.act_b * g, g, p.act_a))) * u;
 }
 
 template <int BN, int EPI, bool LEAN>
@@ -342,7 +343,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
             if (m < m_lim && ch * 2 < p.N) {
               const float g = __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
               const float u = sbuf[row_in_tile * LD + c0 + j] * s_rstd[c0 + j];
-              out[(size_t)m * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p.grp, g, u));
+              out[(size_t)m * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p, g, u));
             }
           }
         }
@@ -498,7 +499,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
               const int c = c0 + u * (int)S;
               if (c < BN && m_base + c < m_lim && ch * 2 < p.N) {
                 const float g = prev[u], up = s_pair[u][threadIdx.x];
-                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p.grp, g, up));
+                ob[(size_t)(m_base + c) * p.ldo + ch] = __float2bfloat16(gated_unit<GRP>(p, g, up));
               }
             }
           }
@@ -749,6 +750,8 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
   const int bn = gmode == 2 ? grp->bn : bn_for(M, N * (gmode == 1 ? groups : 1), clustered);
   GemmParams p;
   if (grp != nullptr) p.grp = *grp; else memset(&p.grp, 0, sizeof(p.grp));
+  p.act_a = p.grp.act == 2 ? GELU_A : 1.0f;
+  p.act_b = p.grp.act == 2 ? GELU_B : 0.0f;
   p.N = N; p.K = K; p.M = M;
   p.kblocks = f8 != nullptr ? (K + 127) / 128 : (K + 63) / 64;
   p.fp8 = f8 != nullptr; p.w_scale = f8 ? f8->w_scale : nullptr; p.x_scale = f8 ? f8->x_scale : nullptr;

@@ -30,57 +30,78 @@ struct LatentNewArgs {
   int pdl;
 };
 
-// VEC: all parts start on groups of four columns.  The sums of both parts meet in one round.
-template <typename AT, int VEC>
-__global__ void __launch_bounds__(128) latent_new_kernel(const LatentNewArgs a) {
-  constexpr int W = 4;                                    // groups a thread keeps in registers
-  __shared__ float red[2][4];
+__device__ __forceinline__ int latent_page(const LatentNewArgs& a, int t) {
+  const int page = a.locs[t];
+  if (page >= 0 && page <= a.n_pages) return page;
+  atomicOr(a.status, SMC_ERR_BOUNDS);
+  return 0;
+}
+
+// Queries copied, no rotated key: a CTA per token.
+template <typename AT>
+__global__ void __launch_bounds__(256) latent_new_kernel(const LatentNewArgs a) {
+  __shared__ float red[32];
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x;
+  const float* row = a.proj + (size_t)t * a.ldp;
+  AT* q = reinterpret_cast<AT*>(a.q) + (size_t)t * a.ldq;
+  if (a.q != nullptr) {
+    if (((a.nq | a.ldp | a.ldq) & 3) == 0)
+      for (int i = threadIdx.x * 4; i < a.nq; i += blockDim.x * 4) store4(q + i, load4(row + i));
+    else
+      for (int i = threadIdx.x; i < a.nq; i += blockDim.x) q[i] = from_f32<AT>(row[i]);
+  }
+  const float* c = row + a.c_off;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.R; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
+  const float inv = 1.0f / sqrtf(block_sum_all(ss, red) / (float)a.R + a.eps);
+  AT* out = reinterpret_cast<AT*>(a.pool) + (size_t)latent_page(a, t) * a.ldc;
+  for (int i = threadIdx.x; i < a.R; i += blockDim.x) out[i] = from_f32<AT>(c[i] * inv * a.c_norm[i]);
+}
+
+// Normed query latent and rotated key: a warp per token - or, for few tokens (ROLES), one per part of a token's row -, the values
+// in registers as far as they fit.  VEC: all parts start on groups of four columns.
+template <typename AT, int VEC, bool ROLES>
+__global__ void __launch_bounds__(128) latent_rows_kernel(const LatentNewArgs a, int T) {
+  constexpr int W = 8;                                    // groups per lane and part
+  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = ROLES ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= T) return;
+  const bool query = !ROLES || warp == 0, latent = !ROLES || warp == 1, key = !ROLES || warp == 2;
   const float* row = a.proj + (size_t)t * a.ldp;
   const float* c = row + a.c_off;
   AT* q = reinterpret_cast<AT*>(a.q) + (size_t)t * a.ldq;
-  int page = a.locs[t];
-  if (page < 0 || page > a.n_pages) {
-    if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
-    page = 0;
-  }
-  AT* out = reinterpret_cast<AT*>(a.pool) + (size_t)page * a.ldc;
-  const bool normed = a.q != nullptr && a.q_norm != nullptr;
-  float qv[W][VEC], cv[W][VEC], sums[2] = {0.f, 0.f};
+  AT* out = reinterpret_cast<AT*>(a.pool) + (size_t)latent_page(a, t) * a.ldc;
+  float qv[W][VEC], cv[W][VEC], sq = 0.f, sc = 0.f;
   auto take = [&](float (&v)[W][VEC], const float* src, int n, float& sum) {
 #pragma unroll
     for (int i = 0; i < W; ++i) {
-      const int x = (threadIdx.x + i * 128) * VEC;
+      const int x = (lane + i * 32) * VEC;
       if (x >= n) continue;
       load_cols<VEC>(v[i], src + x);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) sum = x + k < n ? fmaf(v[i][k], v[i][k], sum) : sum;
     }
-    for (int x = threadIdx.x + W * 128 * VEC; x < n; x += 128) sum = fmaf(src[x], src[x], sum);
+    for (int x = lane + W * 32 * VEC; x < n; x += 32) sum = fmaf(src[x], src[x], sum);
   };
-  if (normed) take(qv, row, a.nq_real, sums[0]);
-  take(cv, c, a.R, sums[1]);
-  if (a.rot > 0) {
+  if (query) take(qv, row, a.nq_real, sq);
+  if (latent) take(cv, c, a.R, sc);
+  if (key && a.rot > 0) {
     const int p = a.positions[t];
-    for (int i = threadIdx.x; i < a.rot / 2; i += 128) {
+    for (int i = lane; i < a.rot / 2; i += 32) {
       const float2 v = rotate_pair(make_float2(c[a.R + 2 * i], c[a.R + 2 * i + 1]), a.freq, i, p);
       out[a.R + 2 * i] = from_f32<AT>(v.x);
       out[a.R + 2 * i + 1] = from_f32<AT>(v.y);
     }
   }
   __syncwarp();
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const float v = warp_sum(sums[i]);
-    if (lane == 0) red[i][warp] = v;
-  }
-  __syncthreads();
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
   auto put = [&](AT* dst, float (&v)[W][VEC], const float* src, const float* w, int n, float sum) {
     const float inv = 1.0f / sqrtf(sum / (float)n + a.eps);
 #pragma unroll
     for (int i = 0; i < W; ++i) {
-      const int x = (threadIdx.x + i * 128) * VEC;
+      const int x = (lane + i * 32) * VEC;
       if (x >= n) continue;
       if (VEC == 1 || x + VEC <= n) {
         float g[VEC];
@@ -94,27 +115,26 @@ __global__ void __launch_bounds__(128) latent_new_kernel(const LatentNewArgs a) 
           if (x + k < n) dst[x + k] = from_f32<AT>(v[i][k] * inv * w[x + k]);
       }
     }
-    for (int x = threadIdx.x + W * 128 * VEC; x < n; x += 128) dst[x] = from_f32<AT>(src[x] * inv * w[x]);
+    for (int x = lane + W * 32 * VEC; x < n; x += 32) dst[x] = from_f32<AT>(src[x] * inv * w[x]);
   };
-  put(out, cv, c, a.c_norm, a.R, red[1][0] + red[1][1] + red[1][2] + red[1][3]);
-  if (normed) {
-    put(q, qv, row, a.q_norm, a.nq_real, red[0][0] + red[0][1] + red[0][2] + red[0][3]);
-    for (int x = a.nq_real + threadIdx.x; x < a.nq; x += 128) q[x] = from_f32<AT>(0.f);
-  } else if (a.q != nullptr) {
-    for (int x = threadIdx.x * VEC; x < a.nq; x += 128 * VEC) {
-      float v[VEC];
-      load_cols<VEC>(v, row + x);
-      store_cols<VEC>(q + x, v);
-    }
-  }
+  if (latent) put(out, cv, c, a.c_norm, a.R, sc);
+  if (!query) return;
+  put(q, qv, row, a.q_norm, a.nq_real, sq);
+  for (int x = a.nq_real + lane; x < a.nq; x += 32) q[x] = from_f32<AT>(0.f);
 }
 
 template <typename AT>
 static int latent_new_launch(const LatentNewArgs& a, int T, cudaStream_t st) {
-  // a group may reach beyond the end of the query latent (zero columns) but not of the latent, which the rotated key follows
+  if (a.q_norm == nullptr) return launch_pdl(latent_new_kernel<AT>, dim3(T), dim3(256), 0, st, a.pdl, a);
+  // a group may reach beyond the end of the query latent (zero columns) but not of the cached one, which the rotated key follows
   const bool vec = (a.ldp | a.c_off | a.R | a.ldc | a.ldq | a.nq) % 4 == 0;
-  return vec ? launch_pdl(latent_new_kernel<AT, 4>, dim3(T), dim3(128), 0, st, a.pdl, a)
-             : launch_pdl(latent_new_kernel<AT, 1>, dim3(T), dim3(128), 0, st, a.pdl, a);
+  if (T >= 592) {
+    const dim3 grid((T + 3) / 4), block(128);
+    return vec ? launch_pdl(latent_rows_kernel<AT, 4, false>, grid, block, 0, st, a.pdl, a, T)
+               : launch_pdl(latent_rows_kernel<AT, 1, false>, grid, block, 0, st, a.pdl, a, T);
+  }
+  return vec ? launch_pdl(latent_rows_kernel<AT, 4, true>, dim3(T), dim3(96), 0, st, a.pdl, a, T)
+             : launch_pdl(latent_rows_kernel<AT, 1, true>, dim3(T), dim3(96), 0, st, a.pdl, a, T);
 }
 
 template <int NR, typename AT>      // NR = ldc / 32 values per lane
@@ -183,7 +203,7 @@ SMC_API int smc_latent_new_args_size() { return (int)sizeof(smc::LatentNewArgs);
 SMC_API int smc_latent_new(const smc::LatentNewArgs* a, int T, int f32, cudaStream_t st) {
   using namespace smc;
   if (T <= 0) return 0;
-  if (a->rot % 2 || a->R + a->rot > a->ldc) return -98;
+  if (a->rot % 2 || a->R + a->rot > a->ldc || (a->q_norm == nullptr && a->rot != 0) || (a->q_norm != nullptr && a->q == nullptr)) return -98;
   return f32 ? latent_new_launch<float>(*a, T, st) : latent_new_launch<__nv_bfloat16>(*a, T, st);
 }
 

@@ -70,9 +70,9 @@ __global__ void __launch_bounds__(256) gated_unit_kernel(const float* gu, int ld
 
 // ---------------------------------------------------------------- router
 // A CTA takes TM tokens; a warp takes four experts at a time, so that a value read from shared memory meets four weight rows
-// and their loads overlap.  Then one warp per token runs the softmax and the two selections.
+// and their loads overlap (a CTA with one token has more warps, two experts each and more loads in flight).  Then one warp per token runs the softmax and the two selections.
 template <typename AT, int TM>
-__global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const AT* wr, int ldw, int E, int top, int groups,
+__global__ void __launch_bounds__(TM == 1 ? 1024 : 256) route_kernel(const float* h, int d, const AT* wr, int ldw, int E, int top, int groups,
                                                     int keep, int T, const float* bias, float* gate, int* idx, float* wgt, int pdl) {
   const int EL = E + (gate != nullptr);        // rows of the router matrix
   extern __shared__ float rt_smem[];
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
     }
   }
   __syncthreads();
-  constexpr int EG = 4;
+  constexpr int EG = TM == 1 ? 2 : 4, AHEAD = TM == 1 ? 8 : 2;
   for (int e0 = warp * EG; e0 < EL; e0 += nw * EG) {
     float acc[EG][TM];
 #pragma unroll
@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(256) route_kernel(const float* h, int d, const
 #pragma unroll
       for (int m = 0; m < TM; ++m) acc[q][m] = 0.f;
     if (vec) {
-#pragma unroll 2
+#pragma unroll AHEAD
       for (int c = lane * 4; c < d; c += 128) {
         float4 w[EG];
 #pragma unroll
@@ -301,7 +301,7 @@ SMC_API int smc_route(const float* h, int d, const void* wr, int ldw, int E, int
 #define SMC_ROUTE(AT, N)                                                                                                    \
   {                                                                                                                         \
     CUDA_CHECK_RET(cudaFuncSetAttribute(route_kernel<AT, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));     \
-    return launch_pdl(route_kernel<AT, N>, grid, dim3(256), bytes(TM), st, pdl, h, d, (const AT*)wr, ldw, E, top, groups,   \
+    return launch_pdl(route_kernel<AT, N>, grid, dim3(N == 1 ? 1024 : 256), bytes(TM), st, pdl, h, d, (const AT*)wr, ldw, E, top, groups,   \
                       keep, T, bias, gate, idx, wgt, pdl);                                                                            \
   }
   if (f32 && wide) SMC_ROUTE(float, 8)

@@ -716,12 +716,15 @@ def layered_lib():
         L.smc_memory_scan.argtypes = [vp, i, i, vp]
         L.smc_gated_step.argtypes = [vp, i, vp]
         L.smc_gated_step_takes.argtypes = [i, i]
+        L.smc_gated_chunk.argtypes = [vp, vp]
+        L.smc_gated_chunk_takes.argtypes = [i, i]
         L.smc_low_rank.argtypes = [vp, i, vp, vp, i, i, i, i, i, i, vp]
         L.smc_tanh_rows.argtypes = [vp, i, vp, i, i, i, i, i, vp]
         for n in ("smc_gemm_grouped", "smc_gemm_f32", "smc_hyper_step", "smc_short_conv", "smc_poly_norm", "smc_gated_unit_f32",
                   "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn", "smc_post_norm_step",
                   "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_splits", "smc_chunk_attn_tc",
-                  "smc_chunk_attn_tc_max_width", "smc_conv_heads", "smc_rotate_heads", "smc_side_step", "smc_gated_step", "smc_gated_step_takes",
+                  "smc_chunk_attn_tc_max_width", "smc_conv_heads", "smc_rotate_heads", "smc_side_step", "smc_gated_step", "smc_gated_step_takes", "smc_gated_chunk",
+                  "smc_gated_chunk_takes",
                   "smc_memory_scan", "smc_tanh_rows", "smc_low_rank"):
             getattr(L, n).restype = C.c_int
         for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
@@ -893,6 +896,15 @@ def gated_step_takes(D: int, V: int) -> bool:
 def gated_step(a: ScanArgs, f32: bool) -> None:
     """The SCAN_GATED memory where every sequence brings one token (csrc/gated_memory.cu)."""
     _check(layered_lib().smc_gated_step(C.byref(a), int(f32), _stream()), "smc_gated_step")
+
+
+def gated_chunk_takes(D: int, V: int) -> bool:
+    return bool(layered_lib().smc_gated_chunk_takes(D, V))
+
+
+def gated_chunk(a: ScanArgs) -> None:
+    """The SCAN_GATED memory of prompts in bf16, 64 tokens at a time on the tensor cores (csrc/gated_chunk.cu)."""
+    _check(layered_lib().smc_gated_chunk(C.byref(a), _stream()), "smc_gated_chunk")
 
 
 def tanh_rows(x: torch.Tensor, out: torch.Tensor, *, n: int, M: int, f32: bool, pdl: bool = False) -> None:

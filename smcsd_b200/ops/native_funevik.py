@@ -30,7 +30,7 @@ from .native_layered import NativeLayered, env_flag
 
 
 class NativeFunevik(NativeLayered):
-    BESIDE_TOKENS = 1 << 30               # longest step whose feed-forwards run on a second stream beside the mixers
+    CHUNK_MIN_TOKENS = 32                 # portions at least this long take the chunked form of the memories
 
     def __init__(self, model, kv, block_table: torch.Tensor, max_tokens: int, max_logit_rows: int, attn_splits: int,
                  status: torch.Tensor, pdl: bool, state=None):
@@ -58,6 +58,7 @@ class NativeFunevik(NativeLayered):
         self._room_experts(moe)
         self._room_gate_up(dense, moe)
         self.attn_tc = not self.f32
+        self.memory_tc = not self.f32 and env_flag("SMC_GATED_CHUNK", True)
         self.beside = env_flag("SMC_BESIDE", True)
         self.freq: Dict[RotarySpec, torch.Tensor] = {}
         for rot in {L.spec.mixer.rot for L in ls if L.kind != "mlstm"}:
@@ -121,6 +122,8 @@ class NativeFunevik(NativeLayered):
                        gate_cap=m.gate_cap, r_scale=D ** -0.5, r=work, status=K.ptr(self.status), pdl=int(self.pdl))
         if longest == 1 and K.gated_step_takes(D, E):
             K.gated_step(a, self.f32)
+        elif self.memory_tc and longest >= self.CHUNK_MIN_TOKENS and K.gated_chunk_takes(D, E):
+            K.gated_chunk(a)
         else:
             K.memory_scan(a, K.SCAN_GATED, self.f32)
         return vo
@@ -192,7 +195,7 @@ class NativeFunevik(NativeLayered):
         work = self._walk(work, longest)
         self._steps[0].ids = K.ptr(ids)
         mixers = {"mlstm": self._memory, "attention": self._attention, "latent": self._latent}
-        beside = self.beside and T <= self.BESIDE_TOKENS and not self.f32
+        beside = self.beside and not self.f32
         joined = False
         for i, L in enumerate(self.m.layers):
             self._step(i, T, joined)

@@ -76,7 +76,7 @@ def test_key_splits_in_decoding(tmp_path):
     nm = eng._sched.native_runner._prefill_chain("target")
     got = S.feed_in_cuts(eng, "a", ids, [2090] + [1] * 10)
     nm.ctx_hint = 2100
-    assert nm._ks(1, 1, 3, 128) > 1
+    assert nm._latent_splits(1, 1, 3, 128) > 1
     S.check(BF16, got, ref)
     effect = far_effect(lambda x: O.forward(cfg, W, x), cfg, ids, ref)
     assert effect > 0.05 and row_error(got[-1:], ref[-1:]).item() < 0.4 * effect
