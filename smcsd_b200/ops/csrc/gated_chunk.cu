@@ -18,7 +18,8 @@ constexpr int GC_L = 64;                         // tokens of a chunk
 constexpr int GC_EV = 64;                        // value columns of a CTA
 constexpr int GC_LV = GC_EV + 8;                 // row pitch of value tiles: the columns, the normaliser's, seven of zeros
 constexpr int GC_NT = GC_LV / 8;                 // column tiles
-constexpr int GC_THREADS = 256;
+constexpr int GC_THREADS = 512;
+constexpr int GC_WARPS = GC_THREADS / 32;
 
 __device__ __forceinline__ float gc_ex2(float x) {
   float y;
@@ -32,13 +33,14 @@ template <int DKP> struct GcShared {
   __nv_bfloat16 bq[2][GC_L][DKP + 8], bk[2][GC_L][DKP + 8];              // hi, lo
   __nv_bfloat16 bv[2][GC_L][GC_LV], wv_hi[GC_L][GC_LV], wv_lo[GC_L][GC_LV];
   __nv_bfloat16 s_hi[DKP][GC_LV], s_lo[DKP][GC_LV];
-  float A[GC_L], B[GC_L], carry[GC_L], low[GC_L], w[GC_L];               // A, B in units of ln 2
-  float decay, part[2][GC_L], ssq[2][GC_L];
+  __nv_bfloat16 p_room[DKP >= 64 ? 8 : 2 * GC_L * GC_LV];                // weights inside the chunk; they follow the queries into bq
+  struct Gates { float A[GC_L], B[GC_L], carry[GC_L], low[GC_L], w[GC_L], decay, pad[3]; } gates[2];        // A, B in units of ln 2
+  float nq[GC_L], part[4][GC_L], ssq[2][GC_L];
 };
 
 template <int DKP>
 __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanArgs a, int CS) {
-  constexpr int KD = DKP / 16, GROUPS = 128 / DKP, NTW = (GC_NT + GROUPS - 1) / GROUPS;
+  constexpr int KD = DKP / 16, GROUPS = GC_WARPS / KD, NTW = (GC_NT + GROUPS - 1) / GROUPS;
   constexpr float LOG2E = 1.4426950408889634f;
   extern __shared__ __align__(16) uint8_t gc_smem[];
   GcShared<DKP>& S = *reinterpret_cast<GcShared<DKP>*>(gc_smem);
@@ -56,47 +58,84 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
   float* M = a.state + (size_t)row * a.row_stride + (size_t)h * (V + 1) * D;
   float* top = a.top + (size_t)row * a.row_stride + h;
 
-  // ---- fetching
+  // ---- fetching: a thread stays with its columns
+  constexpr int QSTEP = GC_THREADS / (DKP / 4), VSTEP = GC_THREADS / (GC_EV / 4);
+  const int qt = tid / (DKP / 4), qc = tid % (DKP / 4) * 4, vt = tid / (GC_EV / 4), vc = tid % (GC_EV / 4) * 4;
+  const float* q_src = a.proj + ((size_t)off + qt) * a.ldp + h * D + qc;
+  const float* v_src = a.proj + ((size_t)off + vt) * a.ldp + a.v_off + h * V + c0 + vc;
+  const uint32_t q_dst = smem_u32(&S.q[qt][qc]), k_dst = smem_u32(&S.k[qt][qc]), v_dst = smem_u32(&S.v[vt][vc]);
   auto fetch = [&](int chunk) {
     const int n = min(GC_L, len - chunk * GC_L);
-    const float* p = a.proj + ((size_t)off + chunk * GC_L) * a.ldp;
-    for (int x = tid; x < GC_L * DKP / 4; x += GC_THREADS) {
-      const int t = x / (DKP / 4), c = (x - t * (DKP / 4)) * 4;
-      const bool real = t < n && c < D;
-      const float* src = p + (real ? (size_t)t * a.ldp + h * D + c : 0);
-      cp_async16(smem_u32(&S.q[t][c]), src + (real ? a.r_off : 0), real);
-      cp_async16(smem_u32(&S.k[t][c]), src + (real ? a.k_off : 0), real);
+    const float* p = q_src + (size_t)chunk * GC_L * a.ldp;
+#pragma unroll
+    for (int i = 0; i < GC_L / QSTEP; ++i) {
+      const bool real = qt + i * QSTEP < n && qc < D;
+      const float* src = real ? p + (size_t)i * QSTEP * a.ldp : a.proj;
+      cp_async16(q_dst + i * QSTEP * DKP * 4, src + (real ? a.r_off : 0), real);
+      cp_async16(k_dst + i * QSTEP * DKP * 4, src + (real ? a.k_off : 0), real);
     }
-    for (int x = tid; x < GC_L * GC_EV / 4; x += GC_THREADS) {
-      const int t = x / (GC_EV / 4), c = (x - t * (GC_EV / 4)) * 4;
-      const bool real = t < n && c < nv;
-      cp_async16(smem_u32(&S.v[t][c]), p + (real ? (size_t)t * a.ldp + a.v_off + h * V + c0 + c : 0), real);
+    p = v_src + (size_t)chunk * GC_L * a.ldp;
+#pragma unroll
+    for (int i = 0; i < GC_L / VSTEP; ++i) {
+      const bool real = vt + i * VSTEP < n && vc < nv;
+      cp_async16(v_dst + i * VSTEP * GC_EV * 4, real ? p + (size_t)i * VSTEP * a.ldp : a.proj, real);
     }
     cp_async_commit();
   };
-  float gi[2] = {0.f, 0.f}, gf[2] = {0.f, 0.f};  // warp 0: gate logits of tokens 2 lane and 2 lane + 1 of the next chunk
-  auto fetch_gates = [&](int chunk) {
+  fetch(0);
+
+  // ---- gates: one warp, a chunk ahead; running sums and maxima are a scan over pairs (sum of f, maximum), two tokens per lane
+  const bool gate_warp = warp == GC_WARPS - 1;
+  float m_run = gate_warp ? *top : 0.f;
+  auto gates = [&](int chunk) {
+    typename GcShared<DKP>::Gates& G = S.gates[chunk & 1];
+    const float cap = a.gate_cap, bias_i = a.a_bias[h], bias_f = a.a_bias[H + h];
+    float li[2], lf[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int t = chunk * GC_L + 2 * lane + j;
-      if (t < len) {
-        const float* p = a.proj + ((size_t)off + t) * a.ldp + a.a_off + h;
-        gi[j] = p[0];
-        gf[j] = p[H];
+      const float* p = a.proj + ((size_t)off + min(t, len - 1)) * a.ldp + a.a_off + h;
+      li[j] = t < len ? cap * tanhf((p[0] + bias_i) / cap) : -INFINITY;
+      lf[j] = t < len ? log_sigmoid_f(cap * tanhf((p[H] + bias_f) / cap)) : 0.f;
+    }
+    float sum = lf[0] + lf[1], most = fmaxf(li[1], li[0] + lf[1]);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float s0 = __shfl_up_sync(0xffffffffu, sum, o), m0 = __shfl_up_sync(0xffffffffu, most, o);
+      if (lane >= o) {
+        most = fmaxf(most, m0 + sum);
+        sum += s0;
       }
     }
+    float b = __shfl_up_sync(0xffffffffu, sum, 1), m = __shfl_up_sync(0xffffffffu, most, 1);
+    if (lane == 0) { b = 0.f; m = -INFINITY; }
+    m = fmaxf(m, m_run + b);
+    float A[2], B[2], mt[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      b += lf[j];
+      m = fmaxf(m + lf[j], li[j]);
+      A[j] = b - m;
+      B[j] = li[j] - b;
+      mt[j] = m;
+    }
+    const float a_end = __shfl_sync(0xffffffffu, A[1], 31), m_end = __shfl_sync(0xffffffffu, mt[1], 31);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int t = 2 * lane + j;
+      G.A[t] = A[j] * LOG2E;
+      G.B[t] = B[j] * LOG2E;
+      G.carry[t] = expf(A[j] + m_run);
+      G.low[t] = expf(-mt[j]);
+      G.w[t] = expf(B[j] + a_end);
+    }
+    if (lane == 0) G.decay = expf(a_end + m_run);
+    m_run = m_end;
   };
-  fetch(0);
-  float m_run = 0.f, bias_i = 0.f, bias_f = 0.f;
-  if (warp == 0) {
-    m_run = *top;
-    bias_i = a.a_bias[h];
-    bias_f = a.a_bias[H + h];
-    fetch_gates(0);
-  }
+  if (gate_warp) gates(0);
 
   // ---- state: this warp's 16 key rows, NTW column tiles
-  const int strip = warp % KD, tile0 = KD >= 8 ? 0 : (warp / KD) * NTW;
+  const int strip = warp % KD, tile0 = (warp / KD) * NTW;
   float st[NTW][4];
   auto state_at = [&](int j, int e, bool& real) {            // element e of tile j: where it lives
     const int kr = strip * 16 + (lane >> 2) + (e >> 1) * 8, c = (tile0 + j) * 8 + (lane & 3) * 2 + (e & 1);
@@ -127,86 +166,47 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
     }
   publish();
 
-  // ---- read-out: this warp's 16 tokens, half of the columns and the normaliser's tile
-  const int half = warp >> 2, rs = half ? 3 - (warp & 3) : warp & 3;     // heavy and light token strips share a scheduler
+  // ---- read-out: this warp's 16 tokens and 16 columns, and one of: a 16 x 16 block of the weights on or below the diagonal (ten
+  // warps), the normaliser's read-out for 16 tokens (four), the next chunk's gates (one)
+  const int quarter = warp >> 2, rs = (warp + quarter) & 3;  // token strips of all lengths share a scheduler
   const int r0 = rs * 16 + (lane >> 2);                      // this thread's tokens: r0 and r0 + 8
-  const uint32_t q_addr = smem_u32(&S.bq[0][rs * 16 + (lane & 15)][(lane >> 4) * 8]);
-  const uint32_t k_addr = smem_u32(&S.bk[0][(lane & 7) + ((lane >> 4) << 3)][((lane >> 3) & 1) * 8]);
-  const uint32_t v_addr = smem_u32(&S.bv[0][lane & 15][half * 32 + (lane >> 4) * 8]), v1_addr = smem_u32(&S.bv[0][lane & 15][GC_EV]);
-  const uint32_t s_addr = smem_u32(&S.s_hi[lane & 15][half * 32 + (lane >> 4) * 8]), s1_addr = smem_u32(&S.s_hi[lane & 15][GC_EV]);
-  constexpr uint32_t S_LO = sizeof(S.s_hi), WV_LO = sizeof(S.wv_hi), QK_LO = sizeof(S.bq[0]);
+  constexpr int BLOCKS = 10;
+  const bool has_block = warp < BLOCKS, has_norm = warp >= BLOCKS && warp < BLOCKS + 4;
+  const int rb = has_norm ? warp - BLOCKS : warp >= 6 ? 3 : warp >= 3 ? 2 : warp >= 1 ? 1 : 0, cb = warp - rb * (rb + 1) / 2;
+  const int q_lane = (lane & 15) * (DKP + 8) + (lane >> 4) * 8;
+  const uint32_t q_addr = smem_u32(&S.bq[0][rs * 16][0] + q_lane), qb_addr = smem_u32(&S.bq[0][rb * 16][0] + q_lane);
+  const uint32_t k_addr = smem_u32(&S.bk[0][(has_block ? cb : 0) * 16 + (lane & 7) + ((lane >> 4) << 3)][((lane >> 3) & 1) * 8]);
+  const uint32_t v_addr = smem_u32(&S.bv[0][lane & 15][quarter * 16 + (lane >> 4) * 8]), v1_addr = smem_u32(&S.bv[0][lane & 15][GC_EV]);
+  const uint32_t s_addr = smem_u32(&S.s_hi[lane & 15][quarter * 16 + (lane >> 4) * 8]), s1_addr = smem_u32(&S.s_hi[lane & 15][GC_EV]);
+  constexpr uint32_t S_LO = sizeof(S.s_hi), WV_LO = sizeof(S.wv_hi), QK_LO = sizeof(S.bq[0]), P_LO = GC_L * GC_LV * 2;
+  __nv_bfloat16* P = DKP >= 64 ? &S.bq[0][0][0] : S.p_room;  // [hi, lo][token][token of the chunk], pitch GC_LV
+  const uint32_t p_lane = (uint32_t)(((lane & 15) * GC_LV + (lane >> 4) * 8) * 2);
+  const uint32_t p_addr = smem_u32(P) + rs * 16 * GC_LV * 2 + p_lane, pn_addr = smem_u32(P) + rb * 16 * GC_LV * 2 + p_lane;
   const uint32_t kt_addr = smem_u32(&S.bk[0][(lane & 7) + ((lane >> 4) & 1) * 8][strip * 16 + ((lane >> 3) & 1) * 8]);
   const uint32_t wv_addr = smem_u32(&S.wv_hi[lane & 15][0]);
 
   for (int ch = 0; ch < n_chunks; ++ch) {
     const int n = min(GC_L, len - ch * GC_L);
+    const typename GcShared<DKP>::Gates& G = S.gates[ch & 1];
     cp_async_wait<0>();
     __syncthreads();
-    if (warp == 0) {
-      // running sums and maxima of the chunk: a scan over pairs (sum of f, maximum), two tokens per lane
-      const float cap = a.gate_cap;
-      float li[2], lf[2];
+    // ---- operands
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const bool ok = 2 * lane + j < n;
-        li[j] = ok ? cap * tanhf((gi[j] + bias_i) / cap) : -INFINITY;
-        lf[j] = ok ? log_sigmoid_f(cap * tanhf((gf[j] + bias_f) / cap)) : 0.f;
-      }
-      float sum = lf[0] + lf[1], most = fmaxf(li[1], li[0] + lf[1]);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float s0 = __shfl_up_sync(0xffffffffu, sum, o), m0 = __shfl_up_sync(0xffffffffu, most, o);
-        if (lane >= o) {
-          most = fmaxf(most, m0 + sum);
-          sum += s0;
-        }
-      }
-      float b = __shfl_up_sync(0xffffffffu, sum, 1), m = __shfl_up_sync(0xffffffffu, most, 1);
-      if (lane == 0) { b = 0.f; m = -INFINITY; }
-      m = fmaxf(m, m_run + b);
-      float A[2], B[2], mt[2];
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        b += lf[j];
-        m = fmaxf(m + lf[j], li[j]);
-        A[j] = b - m;
-        B[j] = li[j] - b;
-        mt[j] = m;
-      }
-      const float a_end = __shfl_sync(0xffffffffu, A[1], 31), m_end = __shfl_sync(0xffffffffu, mt[1], 31);
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int t = 2 * lane + j;
-        S.A[t] = A[j] * LOG2E;
-        S.B[t] = B[j] * LOG2E;
-        S.carry[t] = expf(A[j] + m_run);
-        S.low[t] = expf(-mt[j]);
-        S.w[t] = expf(B[j] + a_end);
-      }
-      if (lane == 0) S.decay = expf(a_end + m_run);
-      m_run = m_end;
-      if (ch + 1 < n_chunks) fetch_gates(ch + 1);
-    } else {
-      for (int x = tid - 32; x < GC_L * DKP / 4; x += GC_THREADS - 32) {
-        const int t = x / (DKP / 4), c = (x - t * (DKP / 4)) * 4;
-        const float4 q = load4((const float*)&S.q[t][c]), k = load4((const float*)&S.k[t][c]);
-        uint2 hi, lo;
-        split_bf16(q.x * a.r_scale, q.y * a.r_scale, hi.x, lo.x);
-        split_bf16(q.z * a.r_scale, q.w * a.r_scale, hi.y, lo.y);
-        *reinterpret_cast<uint2*>(&S.bq[0][t][c]) = hi;
-        *reinterpret_cast<uint2*>(&S.bq[1][t][c]) = lo;
-        split_bf16(k.x, k.y, hi.x, lo.x);
-        split_bf16(k.z, k.w, hi.y, lo.y);
-        *reinterpret_cast<uint2*>(&S.bk[0][t][c]) = hi;
-        *reinterpret_cast<uint2*>(&S.bk[1][t][c]) = lo;
-      }
+    for (int i = 0; i < GC_L / QSTEP; ++i) {
+      const int t = qt + i * QSTEP;
+      const float4 q = load4((const float*)&S.q[t][qc]), k = load4((const float*)&S.k[t][qc]);
+      uint2 hi, lo;
+      split_bf16(q.x * a.r_scale, q.y * a.r_scale, hi.x, lo.x);
+      split_bf16(q.z * a.r_scale, q.w * a.r_scale, hi.y, lo.y);
+      *reinterpret_cast<uint2*>(&S.bq[0][t][qc]) = hi;
+      *reinterpret_cast<uint2*>(&S.bq[1][t][qc]) = lo;
+      split_bf16(k.x, k.y, hi.x, lo.x);
+      split_bf16(k.z, k.w, hi.y, lo.y);
+      *reinterpret_cast<uint2*>(&S.bk[0][t][qc]) = hi;
+      *reinterpret_cast<uint2*>(&S.bk[1][t][qc]) = lo;
     }
-    __syncthreads();
-    for (int x = tid; x < GC_L * GC_LV / 4; x += GC_THREADS) {
-      const int t = x / (GC_LV / 4), c = (x - t * (GC_LV / 4)) * 4;
-      float4 v = make_float4(c == GC_EV && t < n ? 1.f : 0.f, 0.f, 0.f, 0.f);
-      if (c < GC_EV) v = load4((const float*)&S.v[t][c]);
-      const float w = S.w[t];
+    auto values = [&](int t, int c, float4 v) {
+      const float w = G.w[t];
       uint2 hi, lo;
       split_bf16(v.x, v.y, hi.x, lo.x);
       split_bf16(v.z, v.w, hi.y, lo.y);
@@ -216,135 +216,157 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
       split_bf16(w * v.z, w * v.w, hi.y, lo.y);
       *reinterpret_cast<uint2*>(&S.wv_hi[t][c]) = hi;
       *reinterpret_cast<uint2*>(&S.wv_lo[t][c]) = lo;
+    };
+#pragma unroll
+    for (int i = 0; i < GC_L / VSTEP; ++i) values(vt + i * VSTEP, vc, load4((const float*)&S.v[vt + i * VSTEP][vc]));
+    if (tid < GC_L * 2) {                                    // the normaliser's columns
+      const int t = tid >> 1;
+      values(t, GC_EV + (tid & 1) * 4, make_float4((tid & 1) == 0 && t < n ? 1.f : 0.f, 0.f, 0.f, 0.f));
     }
     __syncthreads();
     if (ch + 1 < n_chunks) fetch(ch + 1);
 
-    // ---- read-out
-    float acc[5][4];
+    // ---- products with the state, weights
+    float acc[2][4], ex[2][4];                               // read-out; block of weights or the normaliser's read-out
 #pragma unroll
-    for (int j = 0; j < 5; ++j)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
-    float sc[GC_L / 16][2][4];                               // scores against 16 tokens at a time, up to the diagonal
+      for (int e = 0; e < 4; ++e) acc[j][e] = ex[j][e] = 0.f;
 #pragma unroll
-    for (int kk = 0; kk < GC_L / 16; ++kk)
-#pragma unroll
-      for (int e = 0; e < 8; ++e) sc[kk][e >> 2][e & 3] = 0.f;
-#pragma unroll 2
     for (int kd = 0; kd < KD; ++kd) {
-      uint32_t qh[4], ql[4];
+      uint32_t qh[4], ql[4], sb[4];
       ldsm4(qh, q_addr + kd * 32);
       ldsm4(ql, q_addr + QK_LO + kd * 32);
+      const uint32_t at = s_addr + kd * 16 * GC_LV * 2;
+      ldsm4_t(sb, at);
+      mma16816(acc[0], qh, sb[0], sb[1]);
+      mma16816(acc[1], qh, sb[2], sb[3]);
+      mma16816(acc[0], ql, sb[0], sb[1]);
+      mma16816(acc[1], ql, sb[2], sb[3]);
+      ldsm4_t(sb, at + S_LO);
+      mma16816(acc[0], qh, sb[0], sb[1]);
+      mma16816(acc[1], qh, sb[2], sb[3]);
+    }
+    uint32_t ph[4], pl[4];
+    if (has_block) {
 #pragma unroll
-      for (int part = 0; part < 2; ++part) {
-        const uint32_t base = part * S_LO + kd * 16 * GC_LV * 2;
-        uint32_t sb[4], s1[2];
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          ldsm4_t(sb, s_addr + base + j * 32);
-          mma16816(acc[2 * j], qh, sb[0], sb[1]);
-          mma16816(acc[2 * j + 1], qh, sb[2], sb[3]);
-          if (part == 0) {
-            mma16816(acc[2 * j], ql, sb[0], sb[1]);
-            mma16816(acc[2 * j + 1], ql, sb[2], sb[3]);
-          }
-        }
-        ldsm2_t(s1, s1_addr + base);
-        mma16816(acc[4], qh, s1[0], s1[1]);
-        if (part == 0) mma16816(acc[4], ql, s1[0], s1[1]);
-      }
-#pragma unroll
-      for (int kk = 0; kk < GC_L / 16; ++kk) {
-        if (kk > rs) continue;
-        const uint32_t at = k_addr + (uint32_t)(kk * 16 * (DKP + 8) * 2 + kd * 32);
-        uint32_t kh[4], kl[4];
-        ldsm4(kh, at);
-        ldsm4(kl, at + QK_LO);
+      for (int kd = 0; kd < KD; ++kd) {
+        uint32_t qh[4], ql[4], kh[4], kl[4];
+        ldsm4(qh, qb_addr + kd * 32);
+        ldsm4(kh, k_addr + kd * 32);
+        ldsm4(ql, qb_addr + QK_LO + kd * 32);
+        ldsm4(kl, k_addr + QK_LO + kd * 32);
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          mma16816(sc[kk][j], qh, kh[2 * j], kh[2 * j + 1]);
-          mma16816(sc[kk][j], qh, kl[2 * j], kl[2 * j + 1]);
-          mma16816(sc[kk][j], ql, kh[2 * j], kh[2 * j + 1]);
+          mma16816(ex[j], qh, kh[2 * j], kh[2 * j + 1]);
+          mma16816(ex[j], qh, kl[2 * j], kl[2 * j + 1]);
+          mma16816(ex[j], ql, kh[2 * j], kh[2 * j + 1]);
         }
       }
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {                          // {rows, rows + 8} x {tokens 0-7, tokens 8-15}
+        const int j = x >> 1, r = x & 1, key = cb * 16 + j * 8 + (lane & 3) * 2, t = rb * 16 + (lane >> 2) + r * 8;
+        const float At = G.A[t];
+        const float p0 = key <= t ? ex[j][r * 2] * gc_ex2(At + G.B[key]) : 0.f;
+        const float p1 = key + 1 <= t ? ex[j][r * 2 + 1] * gc_ex2(At + G.B[key + 1]) : 0.f;
+        split_bf16(p0, p1, ph[x], pl[x]);
+      }
+    } else if (has_norm) {
+#pragma unroll
+      for (int kd = 0; kd < KD; ++kd) {
+        uint32_t qh[4], ql[4], s1[2];
+        ldsm4(qh, qb_addr + kd * 32);
+        ldsm4(ql, qb_addr + QK_LO + kd * 32);
+        ldsm2_t(s1, s1_addr + kd * 16 * GC_LV * 2);
+        mma16816(ex[0], qh, s1[0], s1[1]);
+        mma16816(ex[0], ql, s1[0], s1[1]);
+        ldsm2_t(s1, s1_addr + S_LO + kd * 16 * GC_LV * 2);
+        mma16816(ex[0], qh, s1[0], s1[1]);
+      }
+      const float g0 = G.carry[rb * 16 + (lane >> 2)], g1 = G.carry[rb * 16 + (lane >> 2) + 8];
+      ex[0][0] *= g0;
+      ex[0][2] *= g1;
+    } else if (gate_warp && ch + 1 < n_chunks) {
+      gates(ch + 1);
     }
     {
-      const float g0 = S.carry[r0], g1 = S.carry[r0 + 8];
+      const float g0 = G.carry[r0], g1 = G.carry[r0 + 8];
 #pragma unroll
-      for (int j = 0; j < 5; ++j) {
+      for (int j = 0; j < 2; ++j) {
         acc[j][0] *= g0; acc[j][1] *= g0;
         acc[j][2] *= g1; acc[j][3] *= g1;
       }
     }
-    const float A0 = S.A[r0], A1 = S.A[r0 + 8];
+    __syncthreads();                                         // the queries have been read
+    if (has_block) {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int at = (rb * 16 + (lane >> 2) + (x & 1) * 8) * GC_LV + cb * 16 + (x >> 1) * 8 + (lane & 3) * 2;
+        *reinterpret_cast<uint32_t*>(P + at) = ph[x];
+        *reinterpret_cast<uint32_t*>(P + GC_L * GC_LV + at) = pl[x];
+      }
+    }
+    __syncthreads();
+    // ---- products with the values
 #pragma unroll
     for (int kk = 0; kk < GC_L / 16; ++kk) {
       if (kk > rs) continue;
-      uint32_t ph[4], pl[4];
-#pragma unroll
-      for (int x = 0; x < 4; ++x) {                          // {rows, rows + 8} x {tokens 0-7, tokens 8-15}
-        const int j = x >> 1, r = x & 1, key = kk * 16 + j * 8 + (lane & 3) * 2, t = r0 + r * 8;
-        const float At = r ? A1 : A0;
-        const float p0 = key <= t ? sc[kk][j][r * 2] * gc_ex2(At + S.B[key]) : 0.f;
-        const float p1 = key + 1 <= t ? sc[kk][j][r * 2 + 1] * gc_ex2(At + S.B[key + 1]) : 0.f;
-        split_bf16(p0, p1, ph[x], pl[x]);
-      }
       const uint32_t base = (uint32_t)(kk * 16 * GC_LV * 2);
-#pragma unroll
-      for (int part = 0; part < 2; ++part) {
-        uint32_t vb[4];
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          ldsm4_t(vb, v_addr + part * WV_LO + base + j * 32);
-          mma16816(acc[2 * j], ph, vb[0], vb[1]);
-          mma16816(acc[2 * j + 1], ph, vb[2], vb[3]);
-          if (part == 0) {
-            mma16816(acc[2 * j], pl, vb[0], vb[1]);
-            mma16816(acc[2 * j + 1], pl, vb[2], vb[3]);
-          }
-        }
-      }
-      uint32_t v1[2];                                        // ones and zeros: no second part
-      ldsm2_t(v1, v1_addr + base);
-      mma16816(acc[4], ph, v1[0], v1[1]);
-      mma16816(acc[4], pl, v1[0], v1[1]);
+      uint32_t vb[4];
+      ldsm4(ph, p_addr + kk * 32);
+      ldsm4(pl, p_addr + P_LO + kk * 32);
+      ldsm4_t(vb, v_addr + base);
+      mma16816(acc[0], ph, vb[0], vb[1]);
+      mma16816(acc[1], ph, vb[2], vb[3]);
+      mma16816(acc[0], pl, vb[0], vb[1]);
+      mma16816(acc[1], pl, vb[2], vb[3]);
+      ldsm4_t(vb, v_addr + WV_LO + base);
+      mma16816(acc[0], ph, vb[0], vb[1]);
+      mma16816(acc[1], ph, vb[2], vb[3]);
     }
-    float sq[2] = {0.f, 0.f};
+    if (has_norm) {                                          // ones and zeros: no second part
+      for (int kk = 0; kk <= rb; ++kk) {
+        uint32_t v1[2];
+        ldsm4(ph, pn_addr + kk * 32);
+        ldsm4(pl, pn_addr + P_LO + kk * 32);
+        ldsm2_t(v1, v1_addr + kk * 16 * GC_LV * 2);
+        mma16816(ex[0], ph, v1[0], v1[1]);
+        mma16816(ex[0], pl, v1[0], v1[1]);
+      }
+      if ((lane & 3) == 0) {
+        S.nq[rb * 16 + (lane >> 2)] = ex[0][0];
+        S.nq[rb * 16 + (lane >> 2) + 8] = ex[0][2];
+      }
+    }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      const float nq = __shfl_sync(0xffffffffu, acc[4][2 * r], lane & ~3);
-      const float unit = 1.0f / (fmaxf(fabsf(nq), S.low[r0 + r * 8]) + a.unit_eps);
+      float sq = 0.f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        acc[j][2 * r] *= unit;
-        acc[j][2 * r + 1] *= unit;
-        sq[r] = fmaf(acc[j][2 * r], acc[j][2 * r], fmaf(acc[j][2 * r + 1], acc[j][2 * r + 1], sq[r]));
-      }
-      sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 1);
-      sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 2);
-      if ((lane & 3) == 0) S.part[half][r0 + r * 8] = sq[r];
+      for (int j = 0; j < 2; ++j) sq = fmaf(acc[j][2 * r], acc[j][2 * r], fmaf(acc[j][2 * r + 1], acc[j][2 * r + 1], sq));
+      sq += __shfl_xor_sync(0xffffffffu, sq, 1);
+      sq += __shfl_xor_sync(0xffffffffu, sq, 2);
+      if ((lane & 3) == 0) S.part[quarter][r0 + r * 8] = sq;
     }
     __syncthreads();                                         // everyone has read the state; the sums are there
     if (CS > 1) {
-      if (tid < GC_L) S.ssq[ch & 1][tid] = S.part[0][tid] + S.part[1][tid];
+      if (tid < GC_L) S.ssq[ch & 1][tid] = (S.part[0][tid] + S.part[1][tid]) + (S.part[2][tid] + S.part[3][tid]);
       __syncwarp();
       asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
     }
     // output gates on their way while the state advances
-    float2 gate[4][2];
+    float2 gate[2][2];
 #pragma unroll
     for (int r = 0; r < 2; ++r)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int t = r0 + r * 8, c = half * 32 + j * 8 + (lane & 3) * 2;
+      for (int j = 0; j < 2; ++j) {
+        const int t = r0 + r * 8, c = quarter * 16 + j * 8 + (lane & 3) * 2;
         gate[j][r] = make_float2(0.f, 0.f);
         if (t < n && c < nv)
           gate[j][r] = *reinterpret_cast<const float2*>(a.proj + ((size_t)off + ch * GC_L + t) * a.ldp + a.g_off + h * V + c0 + c);
       }
 
     // ---- state
-    const float decay = S.decay;
+    const float decay = G.decay;
 #pragma unroll
     for (int j = 0; j < NTW; ++j)
 #pragma unroll
@@ -393,13 +415,13 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
         const uint32_t at = smem_u32(&S.ssq[ch & 1][t]);
         for (int q = 0; q < CS; ++q) tot += ld_dsmem_f32(at, q);
       } else {
-        tot = S.part[0][t] + S.part[1][t];
+        tot = (S.part[0][t] + S.part[1][t]) + (S.part[2][t] + S.part[3][t]);
       }
-      const float inv = 1.0f / sqrtf(tot / (float)V + a.eps);
+      const float unit = 1.0f / (fmaxf(fabsf(S.nq[t]), G.low[t]) + a.unit_eps), inv = unit / sqrtf(tot * unit * unit / (float)V + a.eps);
       if (t >= n) continue;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = half * 32 + j * 8 + (lane & 3) * 2;
+      for (int j = 0; j < 2; ++j) {
+        const int c = quarter * 16 + j * 8 + (lane & 3) * 2;
         if (c >= nv) continue;
         const int col = h * V + c0 + c;
         const float2 w = *reinterpret_cast<const float2*>(a.onorm + col);
@@ -417,7 +439,7 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
       const size_t at = state_at(j, e, real);
       if (real && (rank == 0 || (tile0 + j) * 8 < GC_EV)) M[at] = st[j][e];      // the normaliser once
     }
-  if (rank == 0 && tid == 0) *top = m_run;
+  if (rank == 0 && gate_warp && lane == 0) *top = m_run;
   __syncwarp();
   if (CS > 1) cluster_sync();                                // nobody leaves while its sums are read
 }

@@ -59,21 +59,19 @@ __global__ void __launch_bounds__(256) latent_new_kernel(const LatentNewArgs a) 
   for (int i = threadIdx.x; i < a.R; i += blockDim.x) out[i] = from_f32<AT>(c[i] * inv * a.c_norm[i]);
 }
 
-// Normed query latent and rotated key: a warp per token - or, for few tokens (ROLES), one per part of a token's row -, the values
-// in registers as far as they fit.  VEC: all parts start on groups of four columns.
-template <typename AT, int VEC, bool ROLES>
-__global__ void __launch_bounds__(128) latent_rows_kernel(const LatentNewArgs a, int T) {
+// Normed query latent and rotated key: a warp per part of a token's row, the values in registers as far as they fit.  VEC: all
+// parts start on groups of four columns.
+template <typename AT, int VEC>
+__global__ void __launch_bounds__(96) latent_rows_kernel(const LatentNewArgs a) {
   constexpr int W = 8;                                    // groups per lane and part
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = ROLES ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + warp;
-  if (t >= T) return;
-  const bool query = !ROLES || warp == 0, latent = !ROLES || warp == 1, key = !ROLES || warp == 2;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
   const float* row = a.proj + (size_t)t * a.ldp;
   const float* c = row + a.c_off;
   AT* q = reinterpret_cast<AT*>(a.q) + (size_t)t * a.ldq;
   AT* out = reinterpret_cast<AT*>(a.pool) + (size_t)latent_page(a, t) * a.ldc;
-  float qv[W][VEC], cv[W][VEC], sq = 0.f, sc = 0.f;
-  auto take = [&](float (&v)[W][VEC], const float* src, int n, float& sum) {
+  auto unit = [&](AT* dst, const float* src, const float* w, int n) {
+    float v[W][VEC], sum = 0.f;
 #pragma unroll
     for (int i = 0; i < W; ++i) {
       const int x = (lane + i * 32) * VEC;
@@ -83,21 +81,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentNewArgs a,
       for (int k = 0; k < VEC; ++k) sum = x + k < n ? fmaf(v[i][k], v[i][k], sum) : sum;
     }
     for (int x = lane + W * 32 * VEC; x < n; x += 32) sum = fmaf(src[x], src[x], sum);
-  };
-  if (query) take(qv, row, a.nq_real, sq);
-  if (latent) take(cv, c, a.R, sc);
-  if (key && a.rot > 0) {
-    const int p = a.positions[t];
-    for (int i = lane; i < a.rot / 2; i += 32) {
-      const float2 v = rotate_pair(make_float2(c[a.R + 2 * i], c[a.R + 2 * i + 1]), a.freq, i, p);
-      out[a.R + 2 * i] = from_f32<AT>(v.x);
-      out[a.R + 2 * i + 1] = from_f32<AT>(v.y);
-    }
-  }
-  __syncwarp();
-  sq = warp_sum(sq);
-  sc = warp_sum(sc);
-  auto put = [&](AT* dst, float (&v)[W][VEC], const float* src, const float* w, int n, float sum) {
+    sum = warp_sum(sum);
     const float inv = 1.0f / sqrtf(sum / (float)n + a.eps);
 #pragma unroll
     for (int i = 0; i < W; ++i) {
@@ -117,10 +101,19 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentNewArgs a,
     }
     for (int x = lane + W * 32 * VEC; x < n; x += 32) dst[x] = from_f32<AT>(src[x] * inv * w[x]);
   };
-  if (latent) put(out, cv, c, a.c_norm, a.R, sc);
-  if (!query) return;
-  put(q, qv, row, a.q_norm, a.nq_real, sq);
-  for (int x = a.nq_real + lane; x < a.nq; x += 32) q[x] = from_f32<AT>(0.f);
+  if (warp == 0) {
+    unit(q, row, a.q_norm, a.nq_real);
+    for (int x = a.nq_real + lane; x < a.nq; x += 32) q[x] = from_f32<AT>(0.f);
+  } else if (warp == 1) {
+    unit(out, c, a.c_norm, a.R);
+  } else if (a.rot > 0) {
+    const int p = a.positions[t];
+    for (int i = lane; i < a.rot / 2; i += 32) {
+      const float2 v = rotate_pair(make_float2(c[a.R + 2 * i], c[a.R + 2 * i + 1]), a.freq, i, p);
+      out[a.R + 2 * i] = from_f32<AT>(v.x);
+      out[a.R + 2 * i + 1] = from_f32<AT>(v.y);
+    }
+  }
 }
 
 template <typename AT>
@@ -128,13 +121,8 @@ static int latent_new_launch(const LatentNewArgs& a, int T, cudaStream_t st) {
   if (a.q_norm == nullptr) return launch_pdl(latent_new_kernel<AT>, dim3(T), dim3(256), 0, st, a.pdl, a);
   // a group may reach beyond the end of the query latent (zero columns) but not of the cached one, which the rotated key follows
   const bool vec = (a.ldp | a.c_off | a.R | a.ldc | a.ldq | a.nq) % 4 == 0;
-  if (T >= 592) {
-    const dim3 grid((T + 3) / 4), block(128);
-    return vec ? launch_pdl(latent_rows_kernel<AT, 4, false>, grid, block, 0, st, a.pdl, a, T)
-               : launch_pdl(latent_rows_kernel<AT, 1, false>, grid, block, 0, st, a.pdl, a, T);
-  }
-  return vec ? launch_pdl(latent_rows_kernel<AT, 4, true>, dim3(T), dim3(96), 0, st, a.pdl, a, T)
-             : launch_pdl(latent_rows_kernel<AT, 1, true>, dim3(T), dim3(96), 0, st, a.pdl, a, T);
+  return vec ? launch_pdl(latent_rows_kernel<AT, 4>, dim3(T), dim3(96), 0, st, a.pdl, a)
+             : launch_pdl(latent_rows_kernel<AT, 1>, dim3(T), dim3(96), 0, st, a.pdl, a);
 }
 
 template <int NR, typename AT>      // NR = ldc / 32 values per lane
