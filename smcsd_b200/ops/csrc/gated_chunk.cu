@@ -20,6 +20,7 @@ constexpr int GC_LV = GC_EV + 8;                 // row pitch of value tiles: th
 constexpr int GC_NT = GC_LV / 8;                 // column tiles
 constexpr int GC_THREADS = 512;
 constexpr int GC_WARPS = GC_THREADS / 32;
+constexpr int GC_MAX_CTAS = 8;                   // of a head
 
 __device__ __forceinline__ float gc_ex2(float x) {
   float y;
@@ -86,18 +87,26 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
 
   // ---- gates: one warp, a chunk ahead; running sums and maxima are a scan over pairs (sum of f, maximum), two tokens per lane
   const bool gate_warp = warp == GC_WARPS - 1;
-  float m_run = gate_warp ? *top : 0.f;
+  float m_run = 0.f, gi[2], gf[2];                           // gi, gf: gate logits of the chunk after
+  auto fetch_gates = [&](int chunk) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const float* p = a.proj + ((size_t)off + min(chunk * GC_L + 2 * lane + j, len - 1)) * a.ldp + a.a_off + h;
+      gi[j] = p[0];
+      gf[j] = p[H];
+    }
+  };
   auto gates = [&](int chunk) {
     typename GcShared<DKP>::Gates& G = S.gates[chunk & 1];
     const float cap = a.gate_cap, bias_i = a.a_bias[h], bias_f = a.a_bias[H + h];
     float li[2], lf[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-      const int t = chunk * GC_L + 2 * lane + j;
-      const float* p = a.proj + ((size_t)off + min(t, len - 1)) * a.ldp + a.a_off + h;
-      li[j] = t < len ? cap * tanhf((p[0] + bias_i) / cap) : -INFINITY;
-      lf[j] = t < len ? log_sigmoid_f(cap * tanhf((p[H] + bias_f) / cap)) : 0.f;
+      const bool ok = chunk * GC_L + 2 * lane + j < len;
+      li[j] = ok ? cap * tanhf((gi[j] + bias_i) / cap) : -INFINITY;
+      lf[j] = ok ? log_sigmoid_f(cap * tanhf((gf[j] + bias_f) / cap)) : 0.f;
     }
+    fetch_gates(chunk + 1);
     float sum = lf[0] + lf[1], most = fmaxf(li[1], li[0] + lf[1]);
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -132,7 +141,11 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
     if (lane == 0) G.decay = expf(a_end + m_run);
     m_run = m_end;
   };
-  if (gate_warp) gates(0);
+  if (gate_warp) {
+    m_run = *top;
+    fetch_gates(0);
+    gates(0);
+  }
 
   // ---- state: this warp's 16 key rows, NTW column tiles
   const int strip = warp % KD, tile0 = (warp / KD) * NTW;
@@ -184,6 +197,13 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
   const uint32_t p_addr = smem_u32(P) + rs * 16 * GC_LV * 2 + p_lane, pn_addr = smem_u32(P) + rb * 16 * GC_LV * 2 + p_lane;
   const uint32_t kt_addr = smem_u32(&S.bk[0][(lane & 7) + ((lane >> 4) & 1) * 8][strip * 16 + ((lane >> 3) & 1) * 8]);
   const uint32_t wv_addr = smem_u32(&S.wv_hi[lane & 15][0]);
+
+  float2 onorm[2];
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int c = quarter * 16 + j * 8 + (lane & 3) * 2;
+    onorm[j] = c < nv ? *reinterpret_cast<const float2*>(a.onorm + h * V + c0 + c) : make_float2(0.f, 0.f);
+  }
 
   for (int ch = 0; ch < n_chunks; ++ch) {
     const int n = min(GC_L, len - ch * GC_L);
@@ -406,27 +426,35 @@ __global__ void __launch_bounds__(GC_THREADS, 1) gated_chunk_kernel(const ScanAr
     if (ch + 1 < n_chunks) publish();
 
     // ---- outputs
-    if (CS > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    float tot[2] = {0.f, 0.f};
+    if (CS > 1) {
+      asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+      const uint32_t at = smem_u32(&S.ssq[ch & 1][r0]);
+#pragma unroll
+      for (int q = 0; q < GC_MAX_CTAS; ++q)
+        if (q < CS) {
+          const uint32_t there = dsmem_map(at, (uint32_t)q);
+          tot[0] += ld_dsmem_f32_at(there);
+          tot[1] += ld_dsmem_f32_at(there + 32u);
+        }
+    } else {
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int t = r0 + r * 8;
+        tot[r] = (S.part[0][t] + S.part[1][t]) + (S.part[2][t] + S.part[3][t]);
+      }
+    }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int t = r0 + r * 8;
-      float tot = 0.f;
-      if (CS > 1) {
-        const uint32_t at = smem_u32(&S.ssq[ch & 1][t]);
-        for (int q = 0; q < CS; ++q) tot += ld_dsmem_f32(at, q);
-      } else {
-        tot = (S.part[0][t] + S.part[1][t]) + (S.part[2][t] + S.part[3][t]);
-      }
-      const float unit = 1.0f / (fmaxf(fabsf(S.nq[t]), G.low[t]) + a.unit_eps), inv = unit / sqrtf(tot * unit * unit / (float)V + a.eps);
+      const float unit = 1.0f / (fmaxf(fabsf(S.nq[t]), G.low[t]) + a.unit_eps), inv = unit / sqrtf(tot[r] * unit * unit / (float)V + a.eps);
       if (t >= n) continue;
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int c = quarter * 16 + j * 8 + (lane & 3) * 2;
         if (c >= nv) continue;
-        const int col = h * V + c0 + c;
-        const float2 w = *reinterpret_cast<const float2*>(a.onorm + col);
-        *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)off + ch * GC_L + t) * a.ldo + col) =
-            pack_bf16(acc[j][2 * r] * inv * w.x * gc_sigmoid(gate[j][r].x), acc[j][2 * r + 1] * inv * w.y * gc_sigmoid(gate[j][r].y));
+        *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)off + ch * GC_L + t) * a.ldo + h * V + c0 + c) =
+            pack_bf16(acc[j][2 * r] * inv * onorm[j].x * gc_sigmoid(gate[j][r].x), acc[j][2 * r + 1] * inv * onorm[j].y * gc_sigmoid(gate[j][r].y));
       }
     }
     __syncwarp();
@@ -454,7 +482,7 @@ static int gated_chunk_launch(const ScanArgs& a, cudaStream_t st) {
 }  // namespace smc
 
 // Whether the chunked form takes heads of D key rows and V value columns.
-SMC_API int smc_gated_chunk_takes(int D, int V) { return D % 4 == 0 && D <= 128 && V % 4 == 0 && V <= 8 * smc::GC_EV; }
+SMC_API int smc_gated_chunk_takes(int D, int V) { return D % 4 == 0 && D <= 128 && V % 4 == 0 && V <= smc::GC_MAX_CTAS * smc::GC_EV; }
 
 // The gated form in bf16, 64 tokens at a time; arguments as for smc_memory_scan.
 SMC_API int smc_gated_chunk(const smc::ScanArgs* a, cudaStream_t st) {
