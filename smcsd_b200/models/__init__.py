@@ -1,4 +1,4 @@
-"""Model families: dense Llama-style decoders, Qwen3.5-style Gated-DeltaNet hybrids, Pasizen, Makodra and Funevik."""
+"""Model families: dense Llama-style decoders, Qwen3.5-style Gated-DeltaNet hybrids, Pasizen, Makodra, Funevik and Padadra."""
 from __future__ import annotations
 
 import os
@@ -20,6 +20,8 @@ def build_model(spec, dtype=torch.bfloat16, device="cpu", tp_rank: int = 0, tp_s
         from .makodra import MakodraModel as Cls
     elif cfg.arch == "funevik":
         from .funevik import FunevikModel as Cls
+    elif cfg.arch == "padadra":
+        from .padadra import PadadraModel as Cls
     else:
         from .llama import LlamaModel as Cls
     m = Cls(cfg, dtype=dtype, device=device, tp_rank=tp_rank, tp_size=tp_size, max_positions=max_positions)

@@ -1,6 +1,6 @@
 """Architecture descriptions: parsed from a HF ``config.json`` or built from presets.
 
-Five families are served.  Two are the ones the reference runs: dense Llama-style decoders and
+Six families are served.  Two are the ones the reference runs: dense Llama-style decoders and
 Qwen3.5-style hybrids that interleave Gated-DeltaNet layers with gated full attention
 (reference: README.md model list; parameter names checked against the HF
 implementation, transformers/models/qwen3_5/modeling_qwen3_5.py).  The others spell every layer out in config.json.
@@ -8,7 +8,9 @@ Pasizen: latent attention without positions, a short convolution in front of eve
 streams, PolyNorm or mixture-of-experts feed-forwards and layers that may be looped.  Makodra: generalized delta rule,
 token-shifted decaying memory and chunked attention in any order, with norms on the sublayers' outputs.  Funevik: matrix
 memories with exponential gates, windowed latent attention with a rotated part and soft-capped attention behind a short
-convolution in any order, mixer and feed-forward side by side in every layer.
+convolution in any order, mixer and feed-forward side by side in every layer.  Padadra: a delta rule with a decay per
+channel, and windowed attention with a forget-gated memory side by side behind norms of their own; mixer and feed-forward
+again on the same input, and an embedding of token pairs.
 """
 from __future__ import annotations
 
@@ -16,7 +18,7 @@ import json
 import math
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Union
+from typing import Any, Dict, List, Optional, Tuple, Union
 
 
 UNLIMITED_POSITIONS = 1 << 20             # positions of architectures that compute them instead of looking them up
@@ -24,9 +26,17 @@ UNLIMITED_POSITIONS = 1 << 20             # positions of architectures that comp
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions on the first ``dims`` entries of a head, neighbours paired: pair i turns by position / base^(2i / dims)."""
+    """Rotary positions on the first ``dims`` entries of a head, neighbours paired: pair i turns by position / base^(2i / dims),
+    long waves slowed down by ``scaling`` (factor, low, high, original length)."""
     dims: int
     base: float
+    scaling: Optional[Tuple[float, float, float, float]] = None
+
+    def scaling_dict(self) -> Optional[Dict[str, Any]]:
+        """The scaling in the form of a HF ``rope_scaling`` entry."""
+        if self.scaling is None:
+            return None
+        return dict(zip(("factor", "low_freq_factor", "high_freq_factor", "original_max_position_embeddings"), self.scaling), rope_type="llama3")
 
 
 @dataclass(frozen=True)
@@ -45,8 +55,9 @@ class LatentAttentionSpec:
 
 @dataclass(frozen=True)
 class GroupedAttentionSpec:
-    """Causal grouped-query attention behind a short convolution of queries, keys and values: rotary positions, soft-capped
-    scores, a sink of score 0, a sigmoid gate per head."""
+    """Causal grouped-query attention behind a short convolution of queries, keys and values, with rotary positions: soft-capped
+    scores, a sink of score 0 and a sigmoid gate per head (Funevik), or a window, learned sinks, biased projections, queries and
+    keys normed over all heads at once, and values that turn with their position and back at the reader's (Padadra)."""
     heads: int
     kv_heads: int
     dim: int                             # query / key size per head
@@ -54,7 +65,13 @@ class GroupedAttentionSpec:
     scale: float
     conv: int                            # taps
     rot: RotarySpec
-    softcap: float
+    softcap: float = 0.0                 # 0: scores as they are
+    gate: bool = True                    # sigmoid gate per head
+    window: int = 0                      # tokens a query sees, itself included (0: all before it)
+    learned_sink: bool = False           # one learned sink logit per head instead of 0
+    bias: bool = False                   # of the three projections
+    row_norm: bool = False               # root-mean-square norm of all queries (all keys) of a token together
+    turn_values: Optional[RotarySpec] = None     # rotation of the values
 
 
 @dataclass(frozen=True)
@@ -73,17 +90,39 @@ class ChunkAttentionSpec:
 @dataclass(frozen=True)
 class RecurrentSpec:
     """A memory matrix [dim, vdim] per head: "general_delta" (diagonal decay plus a rank-one removal), "wkv" (diagonal
-    decay, bonus for the current token, token-shifted inputs) or "mlstm" (one decay per head and token, exponential input
-    gate, read-out divided by a normaliser)."""
+    decay, bonus for the current token, token-shifted inputs), "mlstm" (one decay per head and token, exponential input gate,
+    read-out divided by a normaliser), "channel_delta" (decay per channel, then a delta rule with unit keys behind a short
+    convolution) or "hgrn2" (the forget gate of a channel is also what it writes)."""
     kind: str
     heads: int
     dim: int
     vdim: int = 0                        # 0: as many as ``dim``
     gate_cap: float = 0.0                # "mlstm": gate logits are soft-capped at this
+    kv_heads: int = 0                    # "channel_delta": query and key heads, each shared by heads / kv_heads heads
+    conv: int = 1                        # "channel_delta": taps
 
     @property
     def values(self) -> int:
         return self.vdim or self.dim
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers on the same input; half the sum of their outputs, each behind a norm of its own."""
+    left: GroupedAttentionSpec
+    right: RecurrentSpec
+
+    @property
+    def heads(self) -> int:
+        return self.left.heads
+
+    @property
+    def kv_heads(self) -> int:
+        return self.left.kv_heads
+
+    @property
+    def dim(self) -> int:
+        return self.left.dim
 
 
 @dataclass(frozen=True)
@@ -105,7 +144,7 @@ class RouterSpec:
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    kind: str                            # "dense" (PolyNorm) | "moe" | "swiglu" | "geglu" (tanh form of gelu)
+    kind: str                            # "dense" (PolyNorm) | "moe" | "swiglu" | "geglu" (tanh form of gelu) | "relu2" (two matrices)
     ff: int = 0
     expert: Optional[GluSpec] = None
     router: Optional[RouterSpec] = None
@@ -115,13 +154,13 @@ class FeedForwardSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[LatentAttentionSpec, ChunkAttentionSpec, GroupedAttentionSpec, RecurrentSpec]
+    mixer: Union[LatentAttentionSpec, ChunkAttentionSpec, GroupedAttentionSpec, RecurrentSpec, ParallelSpec]
     mlp: Optional[FeedForwardSpec]
 
 
 @dataclass
 class ModelConfig:
-    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen" | "makodra" | "funevik"
+    arch: str = "llama"                  # "llama" | "hybrid_gdn" | "pasizen" | "makodra" | "funevik" | "padadra"
     vocab_size: int = 32000
     hidden_size: int = 4096
     n_layers: int = 32
@@ -147,12 +186,14 @@ class ModelConfig:
     attn_output_gate: bool = False
     qk_norm: bool = False
     norm_plus_one: bool = False                    # RMSNorm weight stored as (w - 1)
-    # ---- layer-by-layer description (Pasizen, Makodra, Funevik) --------------
+    # ---- layer-by-layer description (Pasizen, Makodra, Funevik, Padadra) -----
     layers: Optional[List[LayerSpec]] = None
     loop: Optional[tuple] = None                   # (start, stop, times): these layers run ``times`` times in a row
     streams: int = 1                               # hyper-connected copies of the residual stream
     conv_taps: int = 1                             # short causal convolution in front of every mixer
     embed_scale: float = 1.0                       # embedding rows are multiplied by this
+    bigram: Optional[Tuple[int, int, int]] = None  # embedding of token pairs: buckets, multipliers of the token before and of the token
+    residual_mult: float = 1.0                     # every layer's outputs are multiplied by this
     name: str = ""
 
     # ---- derived -------------------------------------------------------------
@@ -203,6 +244,8 @@ class ModelConfig:
             return self._makodra_param_count()
         if self.arch == "funevik":
             return self._funevik_param_count()
+        if self.arch == "padadra":
+            return self._padadra_param_count()
         n = self.vocab_size * d * (1 if self.tie_embeddings else 2) + d
         for i in range(self.n_layers):
             n += 3 * d * f + 2 * d
@@ -266,7 +309,59 @@ class ModelConfig:
                 n += 3 * d * f.ff
         return n
 
+    def _padadra_param_count(self) -> int:
+        d, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + 1
+        n += (self.bigram[0] + 1) * d if self.bigram else 0
+        for L in self.layers:
+            m, f = L.mixer, L.mlp
+            n += 1 + (0 if f is None else 1 + 2 * d * f.ff)
+            if isinstance(m, ParallelSpec):
+                a, b = m.left, m.right
+                qk, v = (a.heads + a.kv_heads) * a.dim, a.kv_heads * a.vdim
+                n += (qk + v) * (d + 1 + a.conv) + qk + a.heads * (1 + a.vdim * d) + 2 * d
+                n += b.heads * (b.dim * (2 * d + 2) + 2 * b.values * d) + b.values
+            else:                            # without the low-rank maps of decay and gate, whose ranks only the weights tell
+                qk, v = 2 * m.kv_heads * m.dim, m.heads * m.values
+                n += (qk + v) * (d + m.conv) + m.heads * (d + 1 + m.dim) + m.values + v * d
+        return n
+
     # ---- construction ----------------------------------------------------------
+    @classmethod
+    def from_padadra_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
+        """config.json of a Padadra model: every layer with its mixer and feed-forward."""
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            m, f, mlp = e["mixer"], e.get("mlp"), None
+            if e["type"] == "channel_delta":
+                mixer = RecurrentSpec("channel_delta", int(m["heads"]), int(m["dim"]), int(m["vdim"]), kv_heads=int(m["kv_heads"]), conv=int(m["conv"]))
+                if mixer.kv_heads < 1 or mixer.heads % mixer.kv_heads or mixer.conv < 1:
+                    raise ValueError(f"layer {i}: inconsistent delta rule {mixer}")
+            elif e["type"] == "parallel":
+                a, b = m["left"], m["right"]
+                s = a["rot"].get("scaling")
+                scaling = tuple(float(s[k]) for k in ("factor", "low", "high", "original")) if s else None
+                rot = RotarySpec(int(a["rot"]["dims"]), float(a["rot"]["base"]), scaling)
+                left = GroupedAttentionSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]), int(a["conv"]),
+                                            rot, gate=False, window=int(a["mask"]["size"]), learned_sink=True, bias=True, row_norm=True,
+                                            turn_values=RotarySpec(int(a["vdim"]), rot.base))
+                if left.kv_heads < 1 or left.heads % left.kv_heads or rot.dims > left.dim or rot.dims % 2 or left.vdim % 2 or left.conv < 1 or \
+                        left.window < 1:
+                    raise ValueError(f"layer {i}: inconsistent attention {left}")
+                mixer = ParallelSpec(left, RecurrentSpec("hgrn2", int(b["heads"]), int(b["dim"]), int(b["vdim"])))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            if f is not None and f["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(LayerSpec(mixer, None if f is None else FeedForwardSpec("relu2", ff=int(f["ff"]))))
+        eos, g, m0 = c.get("eos_token_id"), c["embedding"].get("bigram"), layers[0].mixer
+        if g and (int(g["buckets"]) < 1 or int(g["mul_prev"]) < 0 or int(g["mul_cur"]) < 0):
+            raise ValueError(f"inconsistent pair embedding {g}")
+        return cls(arch="padadra", vocab_size=int(c["vocab"]), hidden_size=int(c["width"]), n_layers=len(layers), n_heads=m0.heads,
+                   n_kv_heads=m0.kv_heads, head_dim=m0.dim, ffn_size=0, rms_eps=float(c["norm"]["eps"]), max_position=UNLIMITED_POSITIONS,
+                   layers=layers, embed_scale=float(c["embedding"]["scale"]), residual_mult=float(c["residual_mult"]),
+                   bigram=(int(g["buckets"]), int(g["mul_prev"]), int(g["mul_cur"])) if g else None,
+                   eos_token_ids=[] if eos is None else ([eos] if isinstance(eos, int) else list(eos)))
+
     @classmethod
     def from_funevik_dict(cls, c: Dict[str, Any]) -> "ModelConfig":
         """config.json of a Funevik model: every layer with its mixer and feed-forward."""
@@ -384,6 +479,8 @@ class ModelConfig:
             return cls.from_makodra_dict(c)
         if c.get("architecture") == "Funevik":
             return cls.from_funevik_dict(c)
+        if c.get("architecture") == "Padadra":
+            return cls.from_padadra_dict(c)
         archs = c.get("architectures") or []
         mt = (c.get("model_type") or "").lower()
         is_hybrid = "layer_types" in c and any(t == "linear_attention" for t in c["layer_types"])
@@ -537,6 +634,24 @@ def preset(name: str) -> ModelConfig:
                                LayerSpec(RecurrentSpec("mlstm", 3, 24, 40, 9.0), FeedForwardSpec("geglu", ff=200)),
                                LayerSpec(GroupedAttentionSpec(4, 2, 24, 40, 0.3, 4, RotarySpec(12, 2000.0), 20.0), None),
                                LayerSpec(RecurrentSpec("mlstm", 2, 48, 24, 12.0), moe)])
+    if n in ("padadra-2048", "padadra-1024"):
+        # random-init stand-ins with the layer sizes of a real small model: two delta rules to one layer of attention beside a memory
+        d, H = (2048, 16) if n.endswith("2048") else (1024, 8)
+        mlp, delta = FeedForwardSpec("relu2", ff=4 * d), RecurrentSpec("channel_delta", H, 128, 128, kv_heads=H // 2, conv=4)
+        rot = RotarySpec(64, 500000.0, (8.0, 1.0, 4.0, 8192.0))
+        both = ParallelSpec(GroupedAttentionSpec(H, H // 4, 128, 128, 128 ** -0.5, 4, rot, gate=False, window=1024, learned_sink=True, bias=True,
+                                                 row_norm=True, turn_values=RotarySpec(128, rot.base)), RecurrentSpec("hgrn2", H, 128, 128))
+        return ModelConfig(arch="padadra", vocab_size=65536, hidden_size=d, n_layers=15, n_heads=H, n_kv_heads=H // 4, head_dim=128, ffn_size=0,
+                           rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, bigram=(65521, 2654435, 40503), residual_mult=0.4,
+                           layers=[LayerSpec(delta, mlp), LayerSpec(delta, mlp), LayerSpec(both, mlp)] * 5, name=n)
+    if n in ("tiny-padadra",):
+        rot, mlp = RotarySpec(12, 2000.0, (4.0, 1.0, 3.0, 128.0)), FeedForwardSpec("relu2", ff=200)
+        both = ParallelSpec(GroupedAttentionSpec(4, 2, 24, 40, 0.3, 3, rot, gate=False, window=50, learned_sink=True, bias=True, row_norm=True,
+                                                 turn_values=RotarySpec(40, rot.base)), RecurrentSpec("hgrn2", 3, 32, 24))
+        return ModelConfig(arch="padadra", vocab_size=4096, hidden_size=136, n_layers=3, n_heads=4, n_kv_heads=2, head_dim=24, ffn_size=0,
+                           rms_eps=1e-6, max_position=UNLIMITED_POSITIONS, embed_scale=2.0, bigram=(997, 31, 17), residual_mult=0.6,
+                           layers=[LayerSpec(both, mlp), LayerSpec(RecurrentSpec("channel_delta", 4, 24, 40, kv_heads=2, conv=4), None),
+                                   LayerSpec(both, mlp)], name="tiny-padadra")
     raise KeyError(f"unknown preset {name!r}")
 
 

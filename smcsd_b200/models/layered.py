@@ -1,4 +1,4 @@
-"""What the layer-by-layer families (Pasizen, Makodra, Funevik) have in common: padded weight layouts, checkpoints whose tensors are
+"""What the layer-by-layer families (Pasizen, Makodra, Funevik, Padadra) have in common: padded weight layouts, checkpoints whose tensors are
 named per layer and checked against the configuration, activations rounded and padded for the GEMMs."""
 from __future__ import annotations
 

@@ -49,7 +49,8 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, plus_one: bool = False
     return (y * wf).to(x.dtype)
 
 
-def rope_inv_freq(head_dim: int, theta: float, scaling: Optional[dict]) -> torch.Tensor:
+def rope_frequencies(head_dim: int, theta: float, scaling: Optional[dict] = None) -> torch.Tensor:
+    """fp64 angle per position of every pair of a rotation over ``head_dim`` entries."""
     inv = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=torch.float64) / head_dim))
     if scaling:
         kind = scaling.get("rope_type", scaling.get("type", "default"))
@@ -64,7 +65,11 @@ def rope_inv_freq(head_dim: int, theta: float, scaling: Optional[dict]) -> torch
             inv = torch.where(mid, (1 - smooth) * inv / factor + smooth * inv, scaled)
         elif kind == "linear":
             inv = inv / scaling["factor"]
-    return inv.float()
+    return inv
+
+
+def rope_inv_freq(head_dim: int, theta: float, scaling: Optional[dict]) -> torch.Tensor:
+    return rope_frequencies(head_dim, theta, scaling).float()
 
 
 def rope_table(rotary_dim: int, theta: float, scaling: Optional[dict], max_pos: int, device) -> torch.Tensor:
@@ -224,12 +229,18 @@ def route_top(z: torch.Tensor, top: int):
 # ---- positions, token shift and memory matrices
 def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float) -> torch.Tensor:
     """fp32 x [T, ..., n]: the first ``dims`` entries rotated by position, entries 2i and 2i + 1 paired."""
-    ang = positions.double().unsqueeze(1) * base ** (-torch.arange(0, dims, 2, device=x.device).double() / dims)
+    return turn_pairs(x, positions, rope_frequencies(dims, base))
+
+
+def turn_pairs(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, back: bool = False) -> torch.Tensor:
+    """fp32 x [T, ..., n]: entries 2i and 2i + 1 turn by position * freq[i] (fp64), or back by as much; entries behind the pairs
+    pass."""
+    dims = 2 * freq.numel()
+    ang = positions.double().unsqueeze(1) * freq.to(x.device) * (-1.0 if back else 1.0)
     shape = [x.shape[0]] + [1] * (x.dim() - 2) + [dims // 2]
     c, s = ang.cos().float().view(shape), ang.sin().float().view(shape)
     u, v = x[..., 0:dims:2], x[..., 1:dims:2]
     return torch.cat([torch.stack([u * c - v * s, v * c + u * s], dim=-1).flatten(-2), x[..., dims:]], dim=-1)
-
 
 
 def sinusoidal_positions(positions: torch.Tensor, d: int, base: float = 10000.0) -> torch.Tensor:
@@ -285,6 +296,51 @@ def bonus_memory(state: torch.Tensor, r, w, k, v, bonus) -> torch.Tensor:
     return out
 
 
+def channel_delta_memory(state: torch.Tensor, q, k, v, g, beta) -> torch.Tensor:
+    """Delta rule with a decay per channel, one sequence, token by token: M <- diag(g) M, u = beta (v - M^T k), M <- M + k u^T, read
+    out with q.  q, k, g [T, H, dk], v [T, H, dv], beta [T, H]; ``state`` [H, dv, dk] fp32 holds M transposed and is advanced in
+    place.  Returns [T, H, dv]."""
+    M, out = state.clone(), torch.empty_like(v)
+    for t in range(q.shape[0]):
+        M = M * g[t].unsqueeze(1)
+        u = beta[t].unsqueeze(1) * (v[t] - (M * k[t].unsqueeze(1)).sum(-1))
+        M = M + u.unsqueeze(-1) * k[t].unsqueeze(1)
+        out[t] = (M * q[t].unsqueeze(1)).sum(-1)
+    state.copy_(M)
+    return out
+
+
+def forget_memory(state: torch.Tensor, q, v, f, write) -> torch.Tensor:
+    """Forget-gated memory of one sequence: M <- diag(f) M + write v^T with write = 1 - f, read out with q afterwards.  q, f and
+    write [T, H, dk], v [T, H, dv]; layouts as in ``channel_delta_memory``."""
+    M, out = state.clone(), torch.empty_like(v)
+    for t in range(q.shape[0]):
+        M = M * f[t].unsqueeze(1) + v[t].unsqueeze(-1) * write[t].unsqueeze(1)
+        out[t] = (M * q[t].unsqueeze(1)).sum(-1)
+    state.copy_(M)
+    return out
+
+
+def pair_rows(ids: torch.Tensor, batch: ExtendBatch, history: torch.Tensor, rows: torch.Tensor, buckets: int, mul_prev: int,
+              mul_cur: int) -> torch.Tensor:
+    """Rows of an embedding of token pairs: (token before * mul_prev + token * mul_cur) mod buckets, and row ``buckets`` for a
+    sequence's first token.  ``history`` [rows] holds the token before the first new one and is advanced in place."""
+    ids = ids.long()
+    out, t0 = torch.empty_like(ids), 0
+    pref = batch.prefix_lens_host if batch.prefix_lens_host is not None else batch.prefix_lens.tolist()
+    for b, (p, e) in enumerate(zip(pref, batch.lens())):
+        if e == 0:
+            continue
+        mine = ids[t0:t0 + e]
+        prev = torch.cat([history[rows[b]].long().view(1), mine[:-1]])
+        out[t0:t0 + e] = (prev * mul_prev + mine * mul_cur) % buckets
+        if p == 0:
+            out[t0] = buckets
+        history[rows[b]] = mine[-1].to(history.dtype)
+        t0 += e
+    return out
+
+
 def soft_cap(z: torch.Tensor, cap: float) -> torch.Tensor:
     return cap * torch.tanh(z / cap)
 
@@ -313,9 +369,11 @@ def gated_memory(state: torch.Tensor, top: torch.Tensor, q, k, v, i, f) -> torch
 
 def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                               batch: ExtendBatch, kv_heads: int, scale: float, r1: Optional[torch.Tensor],
-                              r2: Optional[torch.Tensor], chunk: int, softcap: float = 0.0) -> torch.Tensor:
-    """Causal attention inside chunks of ``chunk`` positions (0: no chunks) with scores scale q.k - r1 ln(1 + r2 distance), or
-    soft-capped ones, and a sink of score 0.  q [T, H, D]; pools [pages, kv_heads * width]; returns fp32 [T, H, value width]."""
+                              r2: Optional[torch.Tensor], chunk: int, softcap: float = 0.0, window: int = 0,
+                              sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention inside chunks of ``chunk`` positions (0: no chunks) or inside a ``window`` with scores
+    scale q.k - r1 ln(1 + r2 distance), or soft-capped ones, and a sink of score 0 or of the logits ``sink`` [H].  q [T, H, D];
+    pools [pages, kv_heads * width]; returns fp32 [T, H, value width]."""
     T, H, D = q.shape
     rep, V = H // kv_heads, v_pool.shape[1] // kv_heads
     out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
@@ -324,7 +382,7 @@ def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
     for b, (p, e) in enumerate(zip(pref, batch.lens())):
         if e == 0:
             continue
-        lo, L = p // chunk * chunk, p + e
+        lo, L = max(0, p - window + 1) if window else p // chunk * chunk, p + e
         pages = block_table[batch.rows[b].long(), lo:L].long()
         kk = k_pool[pages].view(L - lo, kv_heads, -1)[:, :, :D].float().repeat_interleave(rep, dim=1)
         vv = v_pool[pages].view(L - lo, kv_heads, V).float().repeat_interleave(rep, dim=1)
@@ -336,9 +394,10 @@ def chunk_attention_reference(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
             s = soft_cap(s, softcap)
         if r1 is not None:
             s = s - r1.view(H, 1, 1) * torch.log1p(r2.view(H, 1, 1) * dist)
-        s = s.masked_fill((j > i) | (i // chunk != j // chunk), float("-inf"))
-        top = s.amax(-1, keepdim=True).clamp(min=0.0)
+        s = s.masked_fill((j > i) | ((i - j >= window) if window else (i // chunk != j // chunk)), float("-inf"))
+        extra = torch.zeros(H, 1, 1, device=q.device) if sink is None else sink.view(H, 1, 1)
+        top = torch.maximum(s.amax(-1, keepdim=True), extra)
         ex = torch.exp(s - top)
-        out[t0:t0 + e] = torch.einsum("hel,lhv->ehv", ex / (torch.exp(-top) + ex.sum(-1, keepdim=True)), vv)
+        out[t0:t0 + e] = torch.einsum("hel,lhv->ehv", ex / (torch.exp(extra - top) + ex.sum(-1, keepdim=True)), vv)
         t0 += e
     return out

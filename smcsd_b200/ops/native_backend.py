@@ -563,6 +563,9 @@ class NativeRunner:
         if model.cfg.arch == "funevik":
             from .native_funevik import NativeFunevik
             return NativeFunevik(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, state=state)
+        if model.cfg.arch == "padadra":
+            from .native_padadra import NativePadadra
+            return NativePadadra(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, state=state)
         if model.cfg.arch != "llama":
             from .native_hybrid import NativeHybrid
             return NativeHybrid(model, kv, bt, max_tokens, max_logit_rows, splits, self.status, pdl, runner=self,

@@ -32,7 +32,7 @@ from .worker import PrefillItem, SMCWorker
 
 log = logging.getLogger("smcsd_b200.scheduler")
 
-NATIVE_F32_ARCHS = ("pasizen", "makodra", "funevik")       # architectures whose kernel chain also runs in 32-bit
+NATIVE_F32_ARCHS = ("pasizen", "makodra", "funevik", "padadra")       # architectures whose kernel chain also runs in 32-bit
 
 
 @dataclass
@@ -132,7 +132,7 @@ class SMCScheduler:
             if m.cfg.arch == "pasizen" and self.context_len > m.cfg.max_position:
                 raise ValueError(f"context_length {self.context_len} exceeds the {m.cfg.max_position} learned positions of "
                                  f"{m.cfg.name or 'the model'}")
-            if m.cfg.arch in ("pasizen", "makodra", "funevik") and pp_size > 1:
+            if m.cfg.arch in ("pasizen", "makodra", "funevik", "padadra") and pp_size > 1:
                 raise NotImplementedError("particle-parallel groups do not support caches with a row width per layer")
         # ---- memory -----------------------------------------------------------
         N, G = self.n_local, a.gamma + 1
