@@ -18,8 +18,8 @@ OUT = os.path.join(HERE, "libsmcsd_b200.so")
 OBJ_DIR = os.path.join(HERE, "build")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 # Sources whose fp32 arithmetic serves 32-bit runs: compiled with IEEE division, square root and exponentials.
-PRECISE = {"chunk_attention.cu", "conv_heads.cu", "gated_chunk.cu", "gated_memory.cu", "gemm_f32.cu", "hyper.cu", "latent_attention.cu", "memory_scan.cu",
-           "moe.cu", "post_norm.cu", "side_norm.cu"}
+PRECISE = {"chunk_attention.cu", "conv_act.cu", "conv_heads.cu", "gated_chunk.cu", "gated_memory.cu", "gemm_f32.cu", "hyper.cu", "latent_attention.cu", "memory_scan.cu",
+           "memory_step.cu",            "moe.cu", "post_norm.cu", "side_norm.cu"}
 
 
 def sources():

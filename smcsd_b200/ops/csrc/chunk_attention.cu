@@ -1,5 +1,6 @@
-// Attention inside chunks of the sequence (or over all of it), with grouped heads, unit-rms queries and keys, a logarithmic
-// distance bias or soft-capped scores, a sink in the softmax sum and a gate on the output.
+// Attention inside chunks of the sequence, inside a sliding window or over all of it, with grouped heads, unit-rms queries and
+// keys, a logarithmic distance bias or soft-capped scores, a sink in the softmax sum, a gate on the output or a rotation of it
+// against the token's position.
 //
 //   heads_new     per new token: queries and keys divided by their root mean square per head, values mixed with the first
 //                 layer's; keys and values go to the token's cache page
@@ -141,7 +142,7 @@ __global__ void __launch_bounds__(CA_WARPS * 32) chunk_attn_kernel(const ChunkAt
   const AT* kp = reinterpret_cast<const AT*>(a.kpool) + (size_t)g * a.D;
   const AT* vp = reinterpret_cast<const AT*>(a.vpool) + (size_t)g * a.V;
   const float r1 = a.r1 != nullptr ? a.r1[h0 + mine] : 0.f, r2 = a.r1 != nullptr ? a.r2[h0 + mine] : 0.f;
-  const int lo = chunk_start(pos, a.chunk);
+  const int lo = first_key(a, pos);
   int per = (pos - lo + KS) / KS;
   per = (per + 31) & ~31;
   const int k_begin = lo + rank * per, k_end = min(pos + 1, k_begin + per);
@@ -259,28 +260,37 @@ __global__ void __launch_bounds__(CA_WARPS * 32) chunk_attn_kernel(const ChunkAt
   }
   __syncwarp();
   if (KS > 1) cluster_sync(); else __syncthreads();
-  for (int x = threadIdx.x + rank * CA_WARPS * 32; x < nh * a.V; x += CA_WARPS * 32 * KS) {
+  for (int x = (threadIdx.x + rank * CA_WARPS * 32) * 2; x < nh * a.V; x += CA_WARPS * 32 * KS * 2) {      // pairs of columns
     const int h = x / a.V, c = x - h * a.V;
-    float mm = a.sink ? 0.f : -INFINITY, sum, o = 0.f;
+    const float extra = a.sink_logit != nullptr ? a.sink_logit[h0 + h] : 0.f;
+    float mm = a.sink ? extra : -INFINITY, sum;
+    float2 o = make_float2(0.f, 0.f);
     if (KS == 1) {
       mm = fmaxf(mm, s_ml[0][h]);
       const float fq = expf(s_ml[0][h] - mm);
-      sum = (a.sink ? expf(-mm) : 0.f) + s_ml[1][h] * fq;
-      o = s_o[h][c] * fq;
+      sum = (a.sink ? expf(extra - mm) : 0.f) + s_ml[1][h] * fq;
+      o = make_float2(s_o[h][c] * fq, s_o[h][c + 1] * fq);
     } else {
       const uint32_t am = smem_u32(&s_ml[0][h]), al = smem_u32(&s_ml[1][h]), ao = smem_u32(&s_o[h][c]);
       for (int r = 0; r < KS; ++r) mm = fmaxf(mm, ld_dsmem_f32(am, r));
-      sum = a.sink ? expf(-mm) : 0.f;
+      sum = a.sink ? expf(extra - mm) : 0.f;
       for (int r = 0; r < KS; ++r) {
         const float fq = expf(ld_dsmem_f32(am, r) - mm);
         sum = fmaf(ld_dsmem_f32(al, r), fq, sum);
-        o = fmaf(ld_dsmem_f32(ao, r), fq, o);
+        o.x = fmaf(ld_dsmem_f32(ao, r), fq, o.x);
+        o.y = fmaf(ld_dsmem_f32(ao + 4, r), fq, o.y);
       }
     }
-    o /= sum;
+    o = turn_back(a, tok, c, make_float2(o.x / sum, o.y / sum));
     const int col = (h0 + h) * a.V + c;
-    if (a.gate != nullptr) o /= 1.0f + expf(-a.gate[(size_t)tok * a.ldg + (a.gate_heads ? h0 + h : col)]);
-    reinterpret_cast<AT*>(a.out)[(size_t)tok * a.H * a.V + col] = from_f32<AT>(o);
+    if (a.gate != nullptr) {
+      const float* gate = a.gate + (size_t)tok * a.ldg;
+      o.x /= 1.0f + expf(-gate[a.gate_heads ? h0 + h : col]);
+      o.y /= 1.0f + expf(-gate[a.gate_heads ? h0 + h : col + 1]);
+    }
+    AT* out = reinterpret_cast<AT*>(a.out) + (size_t)tok * a.H * a.V + col;
+    out[0] = from_f32<AT>(o.x);
+    out[1] = from_f32<AT>(o.y);
   }
   __syncwarp();
   if (KS > 1) cluster_sync();                                 // nobody leaves while its shared memory is read
@@ -344,6 +354,6 @@ SMC_API int smc_chunk_attn_splits(int tokens, int H, int G, int wide, int keys) 
 SMC_API int smc_chunk_attn(const smc::ChunkAttnArgs* a, int splits, int f32, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_blk <= 0) return 0;
-  if (a->D % 8 || a->V % 8 || a->H % a->G || a->chunk < 1 || splits < 1 || splits > 8) return -110;
+  if (a->D % 8 || a->V % 8 || a->H % a->G || (a->chunk < 1 && a->window < 1) || a->turn % 2 || splits < 1 || splits > 8) return -110;
   return f32 ? chunk_attn_dispatch<float>(*a, splits, st) : chunk_attn_dispatch<__nv_bfloat16>(*a, splits, st);
 }

@@ -1,7 +1,7 @@
-// Chunked attention of prompts in bf16: one CTA per (block of up to 64 tokens of a sequence, query head), four warps with 16
-// token rows each.  Keys run from the start of the first token's chunk to the last token in tiles of 64, gathered page by
+// Chunked or windowed attention of prompts in bf16: one CTA per (block of up to 64 tokens of a sequence, query head), four warps
+// with 16 token rows each.  Keys run from the first one that the first token sees (the start of its chunk or window) to the last token in tiles of 64, gathered page by
 // page with cp.async into two stages; scores and softmax stay in fp32 registers (base 2), P is rounded to bf16 for the
-// second product and its sum is taken over the rounded values.  The chunk bounds a CTA's work to a handful of tiles: the
+// second product and its sum is taken over the rounded values.  Chunk or window bound a CTA's work to a handful of tiles: the
 // warp-level mma.sync products are short against the gather and the softmax, and a fragment layout in registers lets bias,
 // mask, sink and gate be applied without a trip through tensor memory.
 #include "chunk_attention.cuh"
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
     return;
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, g = h / (a.H / a.G);
-  const int p0 = b.prefix + b.start, t0 = b.off + b.start, k_begin = chunk_start(p0, a.chunk), k_end = p0 + b.n;
+  const int p0 = b.prefix + b.start, t0 = b.off + b.start, k_begin = first_key(a, p0), k_end = p0 + b.n;
   const int* bt = a.block_table + (size_t)b.row * a.bt_stride;
   const __nv_bfloat16* kp = reinterpret_cast<const __nv_bfloat16*>(a.kpool) + (size_t)g * a.D;
   const __nv_bfloat16* vp = reinterpret_cast<const __nv_bfloat16*>(a.vpool) + (size_t)g * a.V;
@@ -63,9 +63,9 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
   const float r1 = a.r1 != nullptr ? a.r1[h] : 0.f, r2 = a.r1 != nullptr ? a.r2[h] : 0.f;
   const int row0 = warp * 16 + (lane >> 2);                // this thread's rows: row0 and row0 + 8
   const int pos[2] = {p0 + row0, p0 + row0 + 8};
-  const int lo[2] = {chunk_start(pos[0], a.chunk), chunk_start(pos[1], a.chunk)};
+  const int lo[2] = {first_key(a, pos[0]), first_key(a, pos[1])};
   const bool active = warp * 16 < b.n;
-  const int w_lo = chunk_start(p0 + warp * 16, a.chunk), w_hi = p0 + warp * 16 + 15;
+  const int w_lo = first_key(a, p0 + warp * 16), w_hi = p0 + warp * 16 + 15;
   float o[NV * 2][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
   for (int j = 0; j < NV * 2; ++j)
@@ -156,8 +156,9 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     const int row = row0 + r * 8;
     if (row >= b.n) continue;
-    const float mm = a.sink ? fmaxf(m[r], 0.f) : m[r];
-    const float f = exp2f(m[r] - mm), inv = f / (l[r] * f + (a.sink ? exp2f(-mm) : 0.f));
+    const float extra = a.sink_logit != nullptr ? a.sink_logit[h] * 1.4426950408889634f : 0.f;
+    const float mm = a.sink ? fmaxf(m[r], extra) : m[r];
+    const float f = exp2f(m[r] - mm), inv = f / (l[r] * f + (a.sink ? exp2f(extra - mm) : 0.f));
     const size_t at = (size_t)(t0 + row) * a.H * a.V + (size_t)h * a.V;
     const float* gate = a.gate != nullptr ? a.gate + (size_t)(t0 + row) * a.ldg + (a.gate_heads ? h : h * a.V) : nullptr;
     const float head_gate = gate != nullptr && a.gate_heads ? 1.0f / (1.0f + __expf(-gate[0])) : 1.0f;
@@ -165,7 +166,8 @@ __global__ void __launch_bounds__(128) chunk_attn_tc_kernel(const ChunkAttnArgs 
     for (int j = 0; j < NV * 2; ++j) {
       const int c = j * 8 + (lane & 3) * 2;
       if (c >= a.V) continue;
-      float v0 = o[j][r * 2] * inv, v1 = o[j][r * 2 + 1] * inv;
+      const float2 back = turn_back(a, t0 + row, c, make_float2(o[j][r * 2] * inv, o[j][r * 2 + 1] * inv));
+      float v0 = back.x, v1 = back.y;
       if (a.gate_heads) {
         v0 *= head_gate;
         v1 *= head_gate;
@@ -201,7 +203,7 @@ SMC_API int smc_chunk_attn_tc_max_width() { return 256; }
 SMC_API int smc_chunk_attn_tc(const smc::ChunkAttnArgs* a, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_blk <= 0) return 0;
-  if (a->D % 8 || a->V % 8 || a->H % a->G || a->chunk < 1 || a->r.B > CT_Q || a->D > 256 || a->V > 256) return -110;
+  if (a->D % 8 || a->V % 8 || a->H % a->G || (a->chunk < 1 && a->window < 1) || a->turn % 2 || a->r.B > CT_Q || a->D > 256 || a->V > 256) return -110;
   if (a->D <= 32) return chunk_tc_values<2>(*a, st);
   if (a->D <= 64) return chunk_tc_values<4>(*a, st);
   if (a->D <= 128) return chunk_tc_values<8>(*a, st);

@@ -4,6 +4,9 @@
 //                  are rotated, and all go to their place (query rows, cache pages).  A thread takes four channels over a run
 //                  of tokens with the window in registers; the thread of a sequence's first tokens, which reads the kept
 //                  projections, also writes the new ones.
+//   normed_heads   the same with biased projections, a norm of all queries (all keys) of a token together before the rotation,
+//                  and rotated values: a CTA takes the queries, the keys or the values of a run of tokens; sine and cosine
+//                  come from a table made once per step
 //   rotate_heads   a range of every head's columns rotated, the rest passed on, in the activation type
 // Convolution, angles and rotation are fp32 (angles are reduced in fp64).
 #include "rotary.cuh"
@@ -28,6 +31,13 @@ struct ConvHeadsArgs {
   void* vpool;              // [n_pages + 1, G * V]
   int n_pages;
   const int* locs;
+  // normed_heads only
+  const float* bias;        // [C]
+  const float* qk_norm;     // [H * D + G * D]
+  int dim;                  // columns of a head the norms count (the rest are zero)
+  float eps;
+  const float2* angles;     // [T, ld_angles] {sine, cosine}: `rot` / 2 pairs from qk_first on, V / 2 from v_first on
+  int ld_angles, qk_first, v_first, turn;            // the first `turn` columns of value heads are rotated
   Ragged r;
   int* status;
   int pdl;
@@ -110,6 +120,129 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeadsArgs a) 
   }
 }
 
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float2 turn_by(float x, float y, float2 sc) { return make_float2(x * sc.y - y * sc.x, y * sc.y + x * sc.x); }
+
+constexpr int NH_THREADS = 512, NH_TOKENS = 8;       // tokens of a run
+
+// NV: groups of four columns per thread.
+template <int TAPS, int NV, typename AT>
+__global__ void __launch_bounds__(NH_THREADS) normed_heads_kernel(const ConvHeadsArgs a) {
+  constexpr int HL = TAPS - 1;
+  __shared__ float red[2][NH_THREADS / 32];
+  const int nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.V, C = nq + nk + nv, part = blockIdx.y;
+  const int base = part == 0 ? 0 : part == 1 ? nq : nq + nk, n = part == 0 ? nq : part == 1 ? nk : nv;
+  const int width = part < 2 ? a.D : a.V, rot = part < 2 ? a.rot : a.turn, first_pair = part < 2 ? a.qk_first : a.v_first;
+  const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x * 4 >= ((n + 127) & ~127)) {       // whole warps without columns; the others meet at a barrier of their own count
+    if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+    return;
+  }
+  const int live = min(nw, ((n + 127) / 128));       // warps that stay
+  float4 w[NV][TAPS], bias[NV], g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    bias[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < n) {
+      bias[i] = load4(a.bias + base + c);
+      if (part < 2) g[i] = load4(a.qk_norm + base + c);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[i][j] = load4(a.conv + (size_t)j * C + base + c);
+    }
+  }
+  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  const RaggedBlock b = ragged_block(a.r, blockIdx.x);
+  const int first = blockIdx.z * NH_TOKENS;
+  if (first >= b.n) return;
+  if (HL > 0 && (b.row < 0 || b.row >= a.n_rows)) {
+    if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
+    return;
+  }
+  const float* src = a.proj + (size_t)b.off * a.ldp + base;
+  const int t0 = b.start + first, t1 = b.start + min(b.n, first + NH_TOKENS);
+  float4 win[NV][HL > 0 ? HL : 1], u[NV];            // win[i][j]: biased projection of token t - HL + j
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    if (c >= n) continue;
+    float* hp = a.hist + (size_t)b.row * a.row_stride + base + c;
+#pragma unroll
+    for (int j = 0; j < HL; ++j) {
+      const int t = t0 - HL + j;
+      win[i][j] = t >= 0 ? add4(load4(src + (size_t)t * a.ldp + c), bias[i]) : load4((const float*)hp + (size_t)(HL + t) * C);
+    }
+    if (t0 == 0) {                                   // the last HL of old and new ones; nobody else reads the old ones
+#pragma unroll
+      for (int j = 0; j < HL; ++j) {
+        const int t = b.len - HL + j;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (t >= 0) {
+          v = add4(load4(src + (size_t)t * a.ldp + c), bias[i]);
+        } else {
+#pragma unroll
+          for (int q = 0; q < HL; ++q)
+            if (q == HL + t) v = win[i][q];
+        }
+        store4(hp + (size_t)j * C, v);
+      }
+    }
+    u[i] = load4(src + (size_t)t0 * a.ldp + c);
+  }
+  const float count = (float)((part == 0 ? a.H : a.G) * a.dim);
+  for (int t = t0; t < t1; ++t) {
+    const int tok = b.off + t;
+    float4 y[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      if (c >= n) continue;
+      const float4 now = add4(u[i], bias[i]);
+      if (t + 1 < t1) u[i] = load4(src + (size_t)(t + 1) * a.ldp + c);
+      y[i] = mul4(w[i][HL], now);
+#pragma unroll
+      for (int j = 0; j < HL; ++j) y[i] = fma4(w[i][j], win[i][j], y[i]);
+#pragma unroll
+      for (int j = 0; j + 1 < HL; ++j) win[i][j] = win[i][j + 1];
+      if (HL > 0) win[i][HL > 0 ? HL - 1 : 0] = now;
+      ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+    }
+    float inv = 1.0f;
+    if (part < 2) {                                  // the same in the whole CTA; the buffers alternate, one barrier per token
+      float* rd = red[t & 1];
+      ss = warp_sum(ss);
+      if (lane == 0) rd[warp] = ss;
+      asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
+      inv = 1.0f / sqrtf(warp_sum(lane < live ? rd[lane] : 0.f) / count + a.eps);
+    }
+    int page = 0;
+    if (part > 0) {
+      page = a.locs[tok];
+      if (page < 0 || page > a.n_pages) { atomicOr(a.status, SMC_ERR_BOUNDS); page = 0; }
+    }
+    AT* out = part == 0 ? reinterpret_cast<AT*>(a.q) + (size_t)tok * nq
+                        : part == 1 ? reinterpret_cast<AT*>(a.kpool) + (size_t)page * nk : reinterpret_cast<AT*>(a.vpool) + (size_t)page * nv;
+    const float2* ang = a.angles + (size_t)tok * a.ld_angles + first_pair;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 4, col = c % width;
+      if (c >= n) continue;
+      float4 v = y[i];
+      if (part < 2) v = make_float4(v.x * inv * g[i].x, v.y * inv * g[i].y, v.z * inv * g[i].z, v.w * inv * g[i].w);
+      if (col < rot) {
+        const float2 lo = turn_by(v.x, v.y, ang[col >> 1]);
+        v.x = lo.x; v.y = lo.y;
+        if (col + 2 < rot) {
+          const float2 hi = turn_by(v.z, v.w, ang[(col >> 1) + 1]);
+          v.z = hi.x; v.w = hi.y;
+        }
+      }
+      store4(out + c, v);
+    }
+  }
+}
+
 // x [T, ldx] -> out [T, heads * width]; columns [first, first + rot) of every head turn.  A thread takes one pair.
 template <typename AT>
 __global__ void __launch_bounds__(128) rotate_heads_kernel(const float* x, int ldx, AT* out, int heads, int width, int first, int rot,
@@ -144,6 +277,26 @@ static int conv_heads_launch(const ConvHeadsArgs& a, cudaStream_t st) {
   return -92;
 }
 
+template <typename AT, int NV>
+static int normed_heads_taps(const ConvHeadsArgs& a, dim3 grid, dim3 block, cudaStream_t st) {
+#define SMC_NH(N) case N: return launch_pdl(normed_heads_kernel<N, NV, AT>, grid, block, 0, st, a.pdl, a);
+  switch (a.taps) { SMC_NH(1) SMC_NH(2) SMC_NH(3) SMC_NH(4) SMC_NH(5) SMC_NH(6) SMC_NH(7) SMC_NH(8) }
+#undef SMC_NH
+  return -92;
+}
+
+template <typename AT>
+static int normed_heads_launch(const ConvHeadsArgs& a, cudaStream_t st) {
+  int most = a.H * a.D;
+  if (a.G * a.V > most) most = a.G * a.V;
+  const int groups = (most / 4 + 31) / 32 * 32;
+  const dim3 grid(a.r.n_blk, 3, (a.r.B + NH_TOKENS - 1) / NH_TOKENS);
+  if (groups <= NH_THREADS) return normed_heads_taps<AT, 1>(a, grid, dim3(groups), st);
+  if (groups <= NH_THREADS * 2) return normed_heads_taps<AT, 2>(a, grid, dim3(NH_THREADS), st);
+  if (groups <= NH_THREADS * 4) return normed_heads_taps<AT, 4>(a, grid, dim3(NH_THREADS), st);
+  return -95;
+}
+
 }  // namespace smc
 
 SMC_API int smc_conv_heads_args_size() { return (int)sizeof(smc::ConvHeadsArgs); }
@@ -153,6 +306,16 @@ SMC_API int smc_conv_heads(const smc::ConvHeadsArgs* a, int f32, cudaStream_t st
   if (a->r.n_blk <= 0) return 0;
   if (a->D % 4 || a->V % 4 || a->ldp % 4 || a->rot % 2 || a->rot > a->D || a->taps < 1 || a->taps > CH_MAX_TAPS) return -92;
   return f32 ? conv_heads_launch<float>(*a, st) : conv_heads_launch<__nv_bfloat16>(*a, st);
+}
+
+// The normed form (see the top): up to 8192 query columns.
+SMC_API int smc_normed_heads(const smc::ConvHeadsArgs* a, int f32, cudaStream_t st) {
+  using namespace smc;
+  if (a->r.n_blk <= 0) return 0;
+  if (a->D % 4 || a->V % 4 || a->ldp % 4 || a->rot % 2 || a->rot > a->D || a->turn % 2 || a->turn > a->V || a->taps < 1 ||
+      a->taps > CH_MAX_TAPS || a->row_stride % 4 || a->angles == nullptr)
+    return -92;
+  return f32 ? normed_heads_launch<float>(*a, st) : normed_heads_launch<__nv_bfloat16>(*a, st);
 }
 
 // Heads of an even number of columns.

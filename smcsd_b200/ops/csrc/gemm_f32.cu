@@ -14,6 +14,7 @@ struct GemmF32Args {
   int N, K, M, ldx, ldo;
   int mode, groups, w_rows, x_cols, out_cols;
   const int4* tiles;        // {group, first row, end row, -}, at most F32_TILE rows each
+  int relu2;                // out = max(., 0)^2
   int pdl;
 };
 
@@ -60,20 +61,21 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args a) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < m_lim && n < a.N) out[(size_t)m * a.ldo + n] = acc[i][j];
+      const float v = a.relu2 ? fmaxf(acc[i][j], 0.f) * fmaxf(acc[i][j], 0.f) : acc[i][j];
+      if (m < m_lim && n < a.N) out[(size_t)m * a.ldo + n] = v;
     }
 }
 
 }  // namespace smc
 
-// mode 0: one product; 1: batched over groups; 2: tiled (max_tiles table entries of at most 64 rows).
+// mode 0: one product; 1: batched over groups; 2: tiled (max_tiles table entries of at most 64 rows).  relu2: squared relu on top.
 SMC_API int smc_gemm_f32(const float* W, const float* X, float* out, int N, int K, int M, int ldx, int ldo, int mode,
-                         int groups, int w_rows, int x_cols, int out_cols, const int4* tiles, int max_tiles, int pdl,
-                         cudaStream_t st) {
+                         int groups, int w_rows, int x_cols, int out_cols, const int4* tiles, int max_tiles, int relu2,
+                         int pdl, cudaStream_t st) {
   using namespace smc;
   if (M <= 0 || N <= 0) return 0;
   if (mode == 2 && (tiles == nullptr || max_tiles < 1)) return -32;
-  GemmF32Args a{W, X, out, N, K, M, ldx, ldo, mode, groups, w_rows, x_cols, out_cols, tiles, pdl};
+  GemmF32Args a{W, X, out, N, K, M, ldx, ldo, mode, groups, w_rows, x_cols, out_cols, tiles, relu2, pdl};
   const int mt = mode == 2 ? max_tiles : (M + F32_TILE - 1) / F32_TILE;
   if (mt > 65535) return -35;
   return launch_pdl(gemm_f32_kernel, dim3((N + F32_TILE - 1) / F32_TILE, mt, mode == 1 ? groups : 1), dim3(256), 0, st, pdl, a);

@@ -8,6 +8,9 @@
 //           max(|n.r|, exp(-m)) + unit_eps; log gates i = cap tanh((. + bias) / cap), f = ln sigmoid(cap tanh(..)), running
 //           maximum m <- max(f + m, i), w = exp(f + m_old - m), a = exp(i - m); output gate sigmoid.  The normaliser is one
 //           more value column (of ones), which every CTA of a head keeps for itself.
+//   channel M <- diag(w) M, then M <- M + b u (v - M^T u)^T, read out with r afterwards; u = k / |k|, r likewise times r_scale (both
+//           shared by groups of heads), b = sigmoid(beta), w = exp(-exp(a_log) softplus(z + w0)); output gate sigmoid
+//   forget  M <- diag(w) M + (1 - w) v^T, read out with silu(r) afterwards; w = lower + (1 - lower) sigmoid(. + bias); no output gate
 //
 // Value columns of a matrix never mix, key rows only in sums.  A CTA therefore keeps some columns of one head's matrix in
 // registers - four threads per pair of columns (one column beyond 128 key rows), a quarter of the key rows each - and walks
@@ -16,7 +19,8 @@
 // mean square, norm weight, gate).  Producers fetch a tile ahead of the one they prepare, so a tile's loads have a whole tile
 // of consumer work to land in.  With few (sequence, head) pairs the columns of a head are spread over a thread-block cluster
 // that exchanges the sums of squares through distributed shared memory.  Both sums over key rows are taken over the old
-// matrix, so that a token costs one reduction: for delta the read-out is (r w)^T M - (r.a u)(u^T M) + (r.k) v.
+// matrix, so that a token costs one reduction: for delta the read-out is (r w)^T M - (r.a u)(u^T M) + (r.k) v, for channel, with g = (w u)^T M,
+// (r w)^T M + (r.b u)(v - g).
 // The recurrence is held to fp32 (a bf16 or tf32 chunk-parallel form would round the state), so the floor is the CUDA cores'
 // rate; products and sums are issued two at a time (f32x2).
 #include "memory_scan.cuh"
@@ -54,16 +58,18 @@ __device__ __forceinline__ void store_shared_unordered(uint32_t addr, float v) {
 __device__ __forceinline__ float sum_of(f2_t a) { const float2 v = unpack2(a); return v.x + v.y; }
 
 __host__ __device__ constexpr int scan_tokens(int dkp) { return dkp <= 128 ? 16 : 8; }       // tokens of a tile
-__host__ __device__ constexpr int scan_vectors(int kind) { return kind == SCAN_DELTA ? 5 : kind == SCAN_GATED ? 2 : 3; }
+__host__ __device__ constexpr int scan_vectors(int kind) { return kind == SCAN_DELTA ? 5 : kind == SCAN_CHANNEL ? 4 : kind == SCAN_GATED ? 2 : 3; }
 __host__ __device__ constexpr int scan_columns(int dkp) { return dkp <= 128 ? 2 : 1; }       // of a consumer thread
 __host__ __device__ constexpr int scan_max_columns(int dkp) { return SCAN_CONSUMERS / 4 * scan_columns(dkp); }      // of a CTA
 
 template <int KIND, int DKP>
 __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {
-  constexpr bool DELTA = KIND == SCAN_DELTA, GATED = KIND == SCAN_GATED;
+  constexpr bool GENERAL = KIND == SCAN_DELTA, GATED = KIND == SCAN_GATED, CHANNEL = KIND == SCAN_CHANNEL, FORGET = KIND == SCAN_FORGET;
+  constexpr bool DELTA = GENERAL || CHANNEL;                 // something is taken off along u
+  constexpr bool SQUARE = GENERAL || KIND == SCAN_BONUS;     // as many values as keys
   constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), NL = (DKP + 31) / 32, NQ = DKP / 16, CP = scan_columns(DKP);
   constexpr int PT = TB / SCAN_PRODUCERS;                    // tokens of a tile per producer warp
-  constexpr int NC = ((GATED || scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;      // columns of a CTA per lane
+  constexpr int NC = ((!SQUARE || scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;      // columns of a CTA per lane
   extern __shared__ __align__(16) float scan_smem[];
   const int buf_floats = TB * (NVEC * DKP + CC + 2);
   float* obuf = scan_smem + 2 * buf_floats;                  // [3][TB][CC]
@@ -91,6 +97,9 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     const int pw = (tid - n_cons) >> 5;
     float kk[PT][NL], rr[PT][NL], zz[PT][NL], aa[PT][NL], vv[PT][NC], gg[PT][NC];
     float gi = 0.f, gf = 0.f, m_run = 0.f, bi = 0.f, bf = 0.f;       // gated: gate logits of token `lane` of a tile, running maximum
+    float bb[PT], rate = 0.f;                                // channel: write strengths, decay rate of the head
+    const int hk = CHANNEL ? h / a.rep : h;
+    if (CHANNEL) rate = expf(a.a_log[h]);
     if (GATED) {
       bi = a.a_bias[h];
       bf = a.a_bias[a.H + h];
@@ -102,18 +111,19 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
       for (int j = 0; j < PT; ++j) {
         const int tb = pw + j * SCAN_PRODUCERS;
         const size_t t = (size_t)off + tile * TB + tb;
-        const float* p = a.proj + t * a.ldp + h * D;
+        const float* p = a.proj + t * a.ldp + hk * D;
         const float* pv = a.proj + t * a.ldp + h * V;
         const float* zr = a.z + t * a.ldz + h * D;
 #pragma unroll
         for (int i = 0; i < NL; ++i) {
           const int c = lane + 32 * i;
           const bool ok = c < D && tb < n;
-          kk[j][i] = ok ? p[a.k_off + c] : 0.f;
+          if (!FORGET) kk[j][i] = ok ? p[a.k_off + c] : 0.f;
           rr[j][i] = ok ? p[a.r_off + c] : 0.f;
-          if (!GATED) zz[j][i] = ok ? zr[c] : 0.f;
-          if (DELTA) aa[j][i] = ok ? p[a.a_off + c] : 0.f;
+          if (!GATED && !FORGET) zz[j][i] = ok ? zr[c] : 0.f;
+          if (GENERAL || FORGET) aa[j][i] = ok ? p[a.a_off + c] : 0.f;
         }
+        if (CHANNEL) bb[j] = tb < n ? a.beta[t * a.ldb + h] : 0.f;
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
           const int c = lane + 32 * i;
@@ -157,12 +167,19 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
       for (int j = 0; j < PT; ++j) {
         const int tb = pw + j * SCAN_PRODUCERS;
         if (tb >= n) continue;
-        float inv = 0.f, s1 = 0.f, s2 = 0.f;
+        float inv = 0.f, s1 = 0.f, s2 = 0.f, rinv = 0.f, b = 0.f;
         if (DELTA) {
           float ss = 0.f;
 #pragma unroll
           for (int i = 0; i < NL; ++i) ss = fmaf(kk[j][i], kk[j][i], ss);
           inv = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
+        }
+        if (CHANNEL) {
+          float ss = 0.f;
+#pragma unroll
+          for (int i = 0; i < NL; ++i) ss = fmaf(rr[j][i], rr[j][i], ss);
+          rinv = a.r_scale / sqrtf(warp_sum(ss) + a.unit_eps);
+          b = sigmoid_f(bb[j]);
         }
         float* d = buf + tb * DKP;
 #pragma unroll
@@ -174,6 +191,25 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
             d[c] = kk[j][i];
             d[TB * DKP + c] = rr[j][i] * a.r_scale;
             s2 = fmaf(rr[j][i] * a.r_scale, kk[j][i], s2);
+            continue;
+          }
+          if (CHANNEL) {
+            const float w = ok ? expf(-rate * softplus_f(zz[j][i] + a.w0[h * D + c])) : 0.f, u = kk[j][i] * inv, r = rr[j][i] * rinv;
+            d[c] = w;
+            d[TB * DKP + c] = b * u;
+            d[2 * TB * DKP + c] = r * w;
+            d[3 * TB * DKP + c] = w * u;
+            s2 = fmaf(r, b * u, s2);
+            continue;
+          }
+          if (FORGET) {
+            const float z = ok ? aa[j][i] + a.a_bias[h * D + c] : 0.f, l = ok ? a.lower[h * D + c] : 0.f;
+            const float w = ok ? fmaf(1.0f - l, sigmoid_f(z), l) : 0.f, k = ok ? (1.0f - l) * sigmoid_f(-z) : 0.f;
+            const float r = rr[j][i] * sigmoid_f(rr[j][i]);
+            d[c] = w;
+            d[TB * DKP + c] = k;
+            d[2 * TB * DKP + c] = r * w;
+            s2 = fmaf(r, k, s2);
             continue;
           }
           const float z = ok ? zz[j][i] + a.w0[h * D + c] : 0.f;
@@ -202,7 +238,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
             if (lane + 32 * i < CC) val[tb * CC + lane + 32 * i] = lane + 32 * i < own ? w * vv[j][i] : w;
         }
         __syncwarp();
-        s1 = DELTA ? warp_sum(s1) : GATED ? __shfl_sync(0xffffffffu, keep, tb) : 0.f;
+        s1 = GENERAL ? warp_sum(s1) : GATED ? __shfl_sync(0xffffffffu, keep, tb) : 0.f;
         s2 = warp_sum(s2);
         if (lane == 0) { scal[2 * tb] = s1; scal[2 * tb + 1] = s2; }
       }
@@ -215,7 +251,9 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
           const int c = lane + 32 * i;
-          gg[j][i] = c < own && c0 + c < V && tb < n ? a.proj[((size_t)off + tile * TB + tb) * a.ldp + a.g_off + h * V + c0 + c] : 0.f;
+          const size_t t = (size_t)off + tile * TB + tb;
+          const float* g = CHANNEL ? a.gate + t * a.ldg : a.proj + t * a.ldp + a.g_off;
+          gg[j][i] = !FORGET && c < own && c0 + c < V && tb < n ? g[h * V + c0 + c] : 0.f;
         }
       }
     };
@@ -251,7 +289,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           const int c = lane + 32 * i, col = h * V + c0 + c;
           if (c >= own || c0 + c >= V) continue;
           const float g = gg[j][i], sg = sigmoid_f(g);
-          const float v = o[c] * inv * a.onorm[col] * (DELTA || GATED ? sg : g * sg);
+          const float v = o[c] * inv * a.onorm[col] * (FORGET ? 1.0f : DELTA || GATED ? sg : g * sg);
           if (f32) reinterpret_cast<float*>(a.out)[t * a.ldo + col] = v;
           else reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + col] = __float2bfloat16(v);
         }
@@ -371,6 +409,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll
         for (int x = 0; x < CP; ++x) {
           o[x] = sum_of(o2[x][0]) + sum_of(o2[x][1]);
+          if (CHANNEL) v[x] -= gone[x];
           vv[x] = pack2(v[x], v[x]);
           gg[x] = pack2(-gone[x], -gone[x]);
         }
@@ -380,11 +419,11 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           ulonglong2 w;
           if (GATED) w.x = w.y = pack2(s1, s1); else w = dw[kq + 4 * i];
           ulonglong2 au;
-          if (DELTA) au = da[kq + 4 * i];
+          if (GENERAL) au = da[kq + 4 * i];
 #pragma unroll
           for (int x = 0; x < CP; ++x) {
             f2_t p = mul2(k.x, vv[x]), q = mul2(k.y, vv[x]);
-            if (DELTA) {
+            if (GENERAL) {
               p = fma2(au.x, gg[x], p);
               q = fma2(au.y, gg[x], q);
             }
@@ -397,7 +436,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           o[x] += __shfl_xor_sync(0xffffffffu, o[x], 1);
           o[x] += __shfl_xor_sync(0xffffffffu, o[x], 2);
           if (kq == 0)
-            store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], DELTA ? fmaf(-s1, gone[x], o[x]) : GATED ? s1 * o[x] : o[x]));
+            store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], GENERAL ? fmaf(-s1, gone[x], o[x]) : GATED ? s1 * o[x] : o[x]));
         }
       }
     }
@@ -491,15 +530,18 @@ static int scan_dispatch(const ScanArgs& a, int f32, cudaStream_t st) {
 SMC_API int smc_scan_args_size() { return (int)sizeof(smc::ScanArgs); }
 
 // One memory layer over the new tokens of every sequence; kind: 0 the bonus form, 1 the generalized delta rule (both V = D), 2
-// the gated form.  Heads of up to 256 key columns.
+// the gated form, 3 the delta rule with a decay per channel, 4 the forget-gated form.  Heads of up to 256 key columns.
 SMC_API int smc_memory_scan(const smc::ScanArgs* a, int kind, int f32, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_seq <= 0) return 0;
-  if (a->D < 1 || a->H < 1 || a->V < 1 || a->r.n_seq > 65535 || (kind != SCAN_GATED && a->V != a->D)) return -120;
+  if (a->D < 1 || a->H < 1 || a->V < 1 || a->r.n_seq > 65535 || (kind < SCAN_GATED && a->V != a->D)) return -120;
+  if (kind == SCAN_CHANNEL && (a->rep < 1 || a->H % a->rep)) return -120;
   switch (kind) {
     case SCAN_BONUS: return scan_dispatch<SCAN_BONUS>(*a, f32, st);
     case SCAN_DELTA: return scan_dispatch<SCAN_DELTA>(*a, f32, st);
     case SCAN_GATED: return scan_dispatch<SCAN_GATED>(*a, f32, st);
+    case SCAN_CHANNEL: return scan_dispatch<SCAN_CHANNEL>(*a, f32, st);
+    case SCAN_FORGET: return scan_dispatch<SCAN_FORGET>(*a, f32, st);
   }
   return -120;
 }

@@ -18,6 +18,7 @@ _LIB_PATH = os.path.join(_HERE, "libsmcsd_b200.so")
 _lib = None
 
 EPI_PARTIAL_F32, EPI_BF16, EPI_SWIGLU_BF16, EPI_STORE_F32, EPI_RESID_F32 = 0, 1, 2, 3, 4
+EPI_RELU2_BF16 = 8
 ERR_BARRIER_TIMEOUT, ERR_PEER_TIMEOUT, ERR_ALLOC_EXHAUSTED, ERR_BOUNDS = 1, 2, 4, 8
 
 
@@ -637,13 +638,17 @@ class LatentNewArgs(C.Structure):
 class ConvHeadsArgs(C.Structure):
     _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "H", "G", "D", "V", "rot")] + \
                [("conv", _VP), ("taps", _I), ("hist", _VP), ("row_stride", C.c_longlong), ("n_rows", _I), ("freq", _VP), ("positions", _VP),
-                ("q", _VP), ("kpool", _VP), ("vpool", _VP), ("n_pages", _I), ("locs", _VP), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+                ("q", _VP), ("kpool", _VP), ("vpool", _VP), ("n_pages", _I), ("locs", _VP), ("bias", _VP), ("qk_norm", _VP), ("dim", _I), ("eps", _F),
+                ("angles", _VP), ("ld_angles", _I), ("qk_first", _I), ("v_first", _I), ("turn", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
 class SideArgs(C.Structure):
-    _fields_ = [("x", _VP), ("d", _I), ("ids", _VP), ("embed", _VP), ("vocab", _I), ("embed_scale", _F), ("y1", _VP), ("s1", _VP),
+    _fields_ = [("x", _VP), ("d", _I), ("ids", _VP), ("embed", _VP), ("vocab", _I), ("embed_scale", _F), ("pairs", _VP), ("buckets", _I),
+                ("mul_prev", C.c_longlong), ("mul_cur", C.c_longlong), ("before", _VP), ("before_stride", C.c_longlong), ("n_rows", _I), ("r", Ragged),
+                ("positions", _VP), ("freq", _VP), ("n_freq", _I), ("angles", _VP), ("y1", _VP), ("s1", _VP),
                 ("y2", _VP), ("gate", _VP), ("ldy", _I), ("ye", _VP), ("ldye", _I), ("top", _I), ("route_slot", _VP), ("route_w", _VP),
-                ("s2", _VP), ("eps", _F), ("w1", _VP), ("w2", _VP), ("xa", _VP), ("xb", _VP), ("n2", _VP), ("ldxa", _I), ("final", _I),
+                ("s2", _VP), ("yb", _VP), ("o1", _VP), ("o2", _VP), ("mult", _F), ("eps", _F), ("w1", _VP), ("w2", _VP), ("one_weight", _I),
+                ("xa", _VP), ("xb", _VP), ("n2", _VP), ("ldxa", _I), ("final", _I),
                 ("status", _VP), ("pdl", _I)]
 
 
@@ -663,14 +668,22 @@ class ChunkAttnArgs(C.Structure):
     _fields_ = [("q", _VP), ("kpool", _VP), ("vpool", _VP), ("out", _VP), ("gate", _VP), ("ldg", _I), ("gate_heads", _I),
                 ("block_table", _VP)] + \
                [(n, _I) for n in ("bt_stride", "bt_rows", "n_pages", "H", "G", "D", "V", "chunk")] + \
-               [("scale", _F), ("r1", _VP), ("r2", _VP), ("softcap", _F), ("sink", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+               [("scale", _F), ("r1", _VP), ("r2", _VP), ("softcap", _F), ("sink", _I), ("sink_logit", _VP), ("window", _I), ("angles", _VP),
+                ("ld_angles", _I), ("angle_first", _I), ("turn", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
 class ScanArgs(C.Structure):
     _fields_ = [("proj", _VP)] + [(n, _I) for n in ("ldp", "r_off", "k_off", "v_off", "g_off", "a_off")] + \
                [("z", _VP), ("ldz", _I), ("w0", _VP), ("a_bias", _VP), ("bonus", _VP), ("onorm", _VP), ("state", _VP),
                 ("row_stride", C.c_longlong), ("n_rows", _I), ("out", _VP), ("ldo", _I), ("H", _I), ("D", _I), ("V", _I),
-                ("eps", _F), ("unit_eps", _F), ("log_decay", _F), ("top", _VP), ("gate_cap", _F), ("r_scale", _F), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+                ("eps", _F), ("unit_eps", _F), ("log_decay", _F), ("top", _VP), ("gate_cap", _F), ("r_scale", _F), ("beta", _VP), ("ldb", _I),
+                ("gate", _VP), ("ldg", _I), ("a_log", _VP), ("rep", _I), ("lower", _VP), ("r", Ragged), ("status", _VP), ("pdl", _I)]
+
+
+class ConvActArgs(C.Structure):
+    _fields_ = [("proj", _VP), ("ldp", _I), ("C", _I), ("conv", _VP), ("taps", _I), ("hist", _VP), ("row_stride", C.c_longlong), ("n_rows", _I),
+                ("out", _VP), ("ldo", _I), ("low_off", _I), ("k1", _I), ("k2", _I), ("low", _VP), ("w1", _VP), ("w2", _VP), ("z1", _VP), ("z2", _VP),
+                ("n1", _I), ("n2", _I), ("r", Ragged), ("status", _VP), ("pdl", _I)]
 
 
 class GroupLink(C.Structure):
@@ -681,7 +694,7 @@ class GroupLink(C.Structure):
 
 GROUP_BATCHED, GROUP_TILED = 1, 2
 ACT_SILU, ACT_CLAMPED, ACT_GELU = 0, 1, 2
-SCAN_BONUS, SCAN_DELTA, SCAN_GATED = 0, 1, 2
+SCAN_BONUS, SCAN_DELTA, SCAN_GATED, SCAN_CHANNEL, SCAN_FORGET = range(5)
 
 
 def layered_lib():
@@ -689,7 +702,7 @@ def layered_lib():
     if not getattr(L, "_layered_declared", False):
         vp, i, f = _VP, _I, _F
         L.smc_gemm_grouped.argtypes = [vp, vp, vp, i, i, i, i, i, i, i, vp, i, vp, vp]
-        L.smc_gemm_f32.argtypes = [vp, vp, vp, i, i, i, i, i, i, i, i, i, i, vp, i, i, vp]
+        L.smc_gemm_f32.argtypes = [vp, vp, vp, i, i, i, i, i, i, i, i, i, i, vp, i, i, i, vp]
         L.smc_hyper_step.argtypes = [vp, i, i, vp]
         L.smc_short_conv.argtypes = [vp, vp, i, vp, vp, i, i, i, vp, vp, i, i, vp]
         L.smc_poly_norm.argtypes = [vp, i, vp, f, vp, i, i, i, i, i, vp]
@@ -715,6 +728,10 @@ def layered_lib():
         L.smc_chunk_attn_tc.argtypes = [vp, vp]
         L.smc_memory_scan.argtypes = [vp, i, i, vp]
         L.smc_gated_step.argtypes = [vp, i, vp]
+        L.smc_memory_step.argtypes = [vp, i, i, vp]
+        L.smc_memory_step_takes.argtypes = [i, i]
+        L.smc_normed_heads.argtypes = [vp, i, vp]
+        L.smc_conv_act.argtypes = [vp, i, vp]
         L.smc_gated_step_takes.argtypes = [i, i]
         L.smc_gated_chunk.argtypes = [vp, vp]
         L.smc_gated_chunk_takes.argtypes = [i, i]
@@ -724,14 +741,14 @@ def layered_lib():
                   "smc_route", "smc_dispatch", "smc_gather_rows", "smc_latent_new", "smc_latent_attn", "smc_post_norm_step",
                   "smc_token_shift", "smc_heads_new", "smc_chunk_attn", "smc_chunk_attn_splits", "smc_chunk_attn_tc",
                   "smc_chunk_attn_tc_max_width", "smc_conv_heads", "smc_rotate_heads", "smc_side_step", "smc_gated_step", "smc_gated_step_takes", "smc_gated_chunk",
-                  "smc_gated_chunk_takes",
+                  "smc_gated_chunk_takes", "smc_memory_step", "smc_memory_step_takes", "smc_normed_heads", "smc_conv_act",
                   "smc_memory_scan", "smc_tanh_rows", "smc_low_rank"):
             getattr(L, n).restype = C.c_int
         for cls, n in ((Ragged, "smc_ragged_size"), (HyperArgs, "smc_hyper_args_size"), (LatentArgs, "smc_latent_args_size"),
                        (GroupLink, "smc_group_link_size"), (PostNormArgs, "smc_post_norm_args_size"),
                        (HeadsNewArgs, "smc_heads_new_args_size"), (ChunkAttnArgs, "smc_chunk_attn_args_size"),
                        (ScanArgs, "smc_scan_args_size"), (LatentNewArgs, "smc_latent_new_args_size"),
-                       (ConvHeadsArgs, "smc_conv_heads_args_size"), (SideArgs, "smc_side_args_size")):
+                       (ConvHeadsArgs, "smc_conv_heads_args_size"), (SideArgs, "smc_side_args_size"), (ConvActArgs, "smc_conv_act_args_size")):
             assert C.sizeof(cls) == getattr(L, n)(), f"{cls.__name__} layout mismatch"
         L._layered_declared = True
     return L
@@ -750,12 +767,12 @@ def gemm_grouped(W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, *, N: int,
 
 
 def gemm_f32(W: torch.Tensor, X: torch.Tensor, out: torch.Tensor, *, N: int, M: int, link: Optional[GroupLink] = None,
-             ldx: Optional[int] = None, pdl: bool = False) -> None:
-    """fp32 product on the CUDA cores, same grouped forms."""
+             ldx: Optional[int] = None, relu2: bool = False, pdl: bool = False) -> None:
+    """fp32 product on the CUDA cores, same grouped forms; ``relu2``: squared relu of it."""
     g = link if link is not None else GroupLink()
     _check(layered_lib().smc_gemm_f32(_p(W), _p(X), _p(out), N, W.shape[-1], M, X.stride(0) if ldx is None else ldx, out.stride(0),
-                                      g.mode, g.groups, g.w_rows, g.x_cols, g.out_cols, g.tiles, g.max_tiles, int(pdl), _stream()),
-           "smc_gemm_f32")
+                                      g.mode, g.groups, g.w_rows, g.x_cols, g.out_cols, g.tiles, g.max_tiles, int(relu2), int(pdl),
+                                      _stream()), "smc_gemm_f32")
 
 
 def hyper_step(a: HyperArgs, T: int, f32: bool) -> None:
@@ -822,8 +839,18 @@ def conv_heads(a: ConvHeadsArgs, f32: bool) -> None:
     _check(layered_lib().smc_conv_heads(C.byref(a), int(f32), _stream()), "smc_conv_heads")
 
 
+def normed_heads(a: ConvHeadsArgs, f32: bool) -> None:
+    """The same with biases, a norm over all queries (all keys) of a token, and rotated values."""
+    _check(layered_lib().smc_normed_heads(C.byref(a), int(f32), _stream()), "smc_normed_heads")
+
+
+def conv_act(a: ConvActArgs, f32: bool) -> None:
+    """Short convolution and silu of a delta rule's queries, keys and values, and its low-rank maps (csrc/conv_act.cu)."""
+    _check(layered_lib().smc_conv_act(C.byref(a), int(f32), _stream()), "smc_conv_act")
+
+
 def side_step(a: SideArgs, T: int, f32: bool) -> None:
-    """x <- x + s1 mixer + s2 feed-forward (or the embedding start), and x under the next layer's two norms (or the final one)."""
+    """x <- x + s1 mixer + s2 feed-forward (or the embedding start, with token pairs and angles), and x under the next layer's two norms (or the final one)."""
     _check(layered_lib().smc_side_step(C.byref(a), T, int(f32), _stream()), "smc_side_step")
 
 
@@ -884,8 +911,8 @@ def chunk_tc_max_width() -> int:
 
 
 def memory_scan(a: ScanArgs, kind: int, f32: bool) -> None:
-    """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu); ``kind``: SCAN_BONUS, SCAN_DELTA or
-    SCAN_GATED."""
+    """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu); ``kind``: SCAN_BONUS, SCAN_DELTA,
+    SCAN_GATED, SCAN_CHANNEL or SCAN_FORGET."""
     _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), int(f32), _stream()), "smc_memory_scan")
 
 
@@ -896,6 +923,15 @@ def gated_step_takes(D: int, V: int) -> bool:
 def gated_step(a: ScanArgs, f32: bool) -> None:
     """The SCAN_GATED memory where every sequence brings one token (csrc/gated_memory.cu)."""
     _check(layered_lib().smc_gated_step(C.byref(a), int(f32), _stream()), "smc_gated_step")
+
+
+def memory_step_takes(D: int, V: int) -> bool:
+    return bool(layered_lib().smc_memory_step_takes(D, V))
+
+
+def memory_step(a: ScanArgs, kind: int, f32: bool) -> None:
+    """SCAN_CHANNEL or SCAN_FORGET where every sequence brings one token (csrc/memory_step.cu)."""
+    _check(layered_lib().smc_memory_step(C.byref(a), int(kind), int(f32), _stream()), "smc_memory_step")
 
 
 def gated_chunk_takes(D: int, V: int) -> bool:

@@ -42,7 +42,7 @@ class NativeLayered:
         self.ctx_hint = 0
         self._lm_parts = None
         self._splits: Dict = {}
-        self._side = None
+        self._side: Dict[int, tuple] = {}
         self.xa = torch.zeros(max_tokens, self.d8, dtype=self.dt, device=self.dev)
         # flat buffers, viewed per layer with that layer's own row width
         self._flat: Dict[str, torch.Tensor] = {}
@@ -70,6 +70,14 @@ class NativeLayered:
         else:
             K.gemm_skinny(W, X, out, M=M, splits=self._cluster(W.shape[0], W.shape[1], M), epi=K.EPI_STORE_F32, ldx=ldx,
                           ldo=out.stride(0), status=self.status, pdl=self.pdl)
+
+    def _relu2_gemm(self, W: torch.Tensor, X: torch.Tensor, act: torch.Tensor, M: int) -> None:
+        """act = max(X W^T, 0)^2 in the activation type."""
+        if self.f32:
+            K.gemm_f32(W, X, act, N=W.shape[0], M=M, relu2=True, pdl=self.pdl)
+        else:
+            K.gemm_skinny(W, X, act, M=M, splits=self._cluster(W.shape[0], W.shape[1], M), epi=K.EPI_RELU2_BF16, ldo=act.stride(0),
+                          status=self.status, pdl=self.pdl)
 
     def _gated_gemm(self, W: torch.Tensor, X: torch.Tensor, act: torch.Tensor, M: int, blk: int, link: "K.GroupLink",
                     shift: float) -> None:
@@ -166,7 +174,7 @@ class NativeLayered:
             K.latent_attention(a, self.f32)
 
     def _chunk_splits(self, tokens: int, m, chunk: int) -> int:
-        """Key ranges of one layer's attention over heads for ``tokens`` tokens (``chunk`` 0: all keys)."""
+        """Key ranges of one layer's attention over heads for ``tokens`` tokens (``chunk``: length of a chunk or window, 0: all keys)."""
         keys = min(chunk, self.ctx_hint) if chunk else self.ctx_hint
         return self._capped(K.chunk_attention_splits(tokens, m.heads, m.kv_heads, round_up(max(m.dim, m.vdim), 8), keys))
 
@@ -176,7 +184,7 @@ class NativeLayered:
         else:
             K.chunk_attention(a, self.f32, self._chunk_splits(T, m, chunk))
 
-    # ---- two streams --------------------------------------------------------------------
+    # ---- streams beside the main one ----------------------------------------------------
     @contextmanager
     def _full_order(self):
         """Launches that depend on work of two streams wait for all of it: no programmatic overlap with the kernel before."""
@@ -186,17 +194,17 @@ class NativeLayered:
         finally:
             self.pdl = kept
 
-    def _fork(self) -> "torch.cuda.Stream":
-        """The second stream, behind everything queued so far (in a capture it joins the same graph)."""
-        if self._side is None:
-            self._side = (torch.cuda.Stream(self.dev), torch.cuda.Event(), torch.cuda.Event())
-        side, forked, _ = self._side
+    def _fork(self, which: int = 0) -> "torch.cuda.Stream":
+        """A second (third, ..) stream, behind everything queued so far (in a capture it joins the same graph)."""
+        if which not in self._side:
+            self._side[which] = (torch.cuda.Stream(self.dev), torch.cuda.Event(), torch.cuda.Event())
+        side, forked, _ = self._side[which]
         forked.record()
         side.wait_event(forked)
         return side
 
-    def _join(self) -> None:
-        side, _, done = self._side
+    def _join(self, which: int = 0) -> None:
+        side, _, done = self._side[which]
         done.record(side)
         torch.cuda.current_stream().wait_event(done)
 
