@@ -17,7 +17,7 @@ cycle with forced cross-GPU resampling, reported under ``fused``.
     python -m torch.distributed.run --nnodes=1 --nproc-per-node 8 --master-addr 127.0.0.1 \
         --master-port 29511 bench.py --gpus 8 --steps 40 --warmup 5
     python bench.py --impl reference        # prints why the reference cannot run here
-    python bench.py --layered 2048,1024     # another workload: Pasizen (--layered-family makodra, funevik: these) beside models of
+    python bench.py --layered 2048,1024     # another workload: Pasizen (--layered-family makodra, funevik, padadra: these) beside models of
                                             # equal size, kernel by kernel
 """
 from __future__ import annotations
@@ -129,8 +129,8 @@ def layered_arm(args) -> int:
     for r in recs:
         print(layered.show(r), file=sys.stderr)
     pick = {m["model"]: m for r in recs for m in r["models"]}
-    tail = {"pasizen": "dense", "makodra": "heads64", "funevik": "dense"}[args.layered_family]
-    main_model = pick[f"{args.layered_family}-{args.layered.split(',')[0]}-{tail}"]
+    tail = {"pasizen": "-dense", "makodra": "-heads64", "funevik": "-dense", "padadra": ""}[args.layered_family]
+    main_model = pick[f"{args.layered_family}-{args.layered.split(',')[0]}{tail}"]
     print(json.dumps({"metric": f"decode tokens/s ({args.layered_family.capitalize()} layers, random weights)", "value": main_model["decode_tok_s"],
                       "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
                       "timing": "CUDA events around graph replays; the weights of all layers exceed L2", "records": recs,
@@ -165,7 +165,7 @@ def main() -> int:
                     help="skip the extra W8A8 (e4m3) measurement reported under the 'fp8' key (one GPU only)")
     ap.add_argument("--layered", default=None, metavar="WIDTHS",
                     help="run the layer comparison of a layer-by-layer family at these widths instead of the headline")
-    ap.add_argument("--layered-family", default="pasizen", choices=["pasizen", "makodra", "funevik"], help="the family --layered compares")
+    ap.add_argument("--layered-family", default="pasizen", choices=["pasizen", "makodra", "funevik", "padadra"], help="the family --layered compares")
     ap.add_argument("--layered-ctx", type=int, default=1024, help="cached tokens per sequence of the layer comparison's decode step")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -4,7 +4,8 @@
     (or: python bench.py --layered 2048,1024 --layered-family makodra)
 
 Pasizen runs beside a dense Llama-style model, Makodra beside that and a Gated-DeltaNet hybrid with as many attention layers,
-Funevik beside a dense model, Makodra (memories, attention over heads) and Pasizen (latent attention, experts).
+Funevik beside a dense model, Makodra (memories, attention over heads) and Pasizen (latent attention, experts), Padadra beside a
+dense model, the hybrid and Makodra.
 All run random weights through their kernel chains: the same width, heads, layer count, head and feed-forward weights per
 layer; the dense models cache as many bytes per token as their KV heads take.  A forward is captured in a CUDA
 graph and timed with CUDA events (weights of all layers exceed L2; the cached keys come on top).  For the kernel table every
@@ -23,7 +24,7 @@ from typing import Dict, List, Tuple
 import torch
 
 from ..models.config import (ChunkAttentionSpec, FeedForwardSpec, GluSpec, GroupedAttentionSpec, LatentAttentionSpec, LayerSpec, ModelConfig,
-                             RecurrentSpec, RotarySpec, RouterSpec)
+                             ParallelSpec, RecurrentSpec, RotarySpec, RouterSpec)
 from ..utils.roofline import measured_peaks
 
 VOCAB = 32768
@@ -82,6 +83,17 @@ def funevik_config(width: int, layers: int, kv_rank: int, experts: bool, window:
                        name=f"funevik-{width}-{'experts' if experts else 'dense'}")
 
 
+def padadra_config(width: int, layers: int, window: int = 1024) -> ModelConfig:
+    """Two delta rules to one layer of attention beside a memory; the feed-forward has as many weights as ``makodra_config``'s."""
+    H, rot = width // 128, RotarySpec(64, 500000.0, (8.0, 1.0, 4.0, 8192.0))
+    mlp, delta = FeedForwardSpec("relu2", ff=3 * width), RecurrentSpec("channel_delta", H, 128, 128, kv_heads=max(1, H // 2), conv=4)
+    both = ParallelSpec(GroupedAttentionSpec(H, max(1, H // 4), 128, 128, 128 ** -0.5, 4, rot, gate=False, window=window, learned_sink=True,
+                                             bias=True, row_norm=True, turn_values=RotarySpec(128, rot.base)), RecurrentSpec("hgrn2", H, 128, 128))
+    return ModelConfig(arch="padadra", vocab_size=VOCAB, hidden_size=width, n_layers=layers, n_heads=H, n_kv_heads=max(1, H // 4), head_dim=128,
+                       ffn_size=0, rms_eps=1e-6, max_position=1 << 20, bigram=(32749, 31013, 4099), residual_mult=0.4,
+                       layers=[LayerSpec(m, mlp) for m in [delta, delta, both] * (layers // 3)], name=f"padadra-{width}")
+
+
 class Rig:
     """One model with its chain, caches filled with noise, and step inputs."""
 
@@ -92,6 +104,7 @@ class Rig:
         from ..ops.native_funevik import NativeFunevik
         from ..ops.native_hybrid import NativeHybrid
         from ..ops.native_makodra import NativeMakodra
+        from ..ops.native_padadra import NativePadadra
         from ..ops.native_pasizen import NativePasizen
         dev = self.dev = torch.device("cuda", 0)
         self.cfg, self.bs, self.ctx, self.prompt, self.n_prompts = cfg, bs, ctx, prompt, n_prompts
@@ -107,7 +120,8 @@ class Rig:
         T = n_prompts * prompt
         if cfg.arch != "llama":
             self.state = StatePool(m.state_spec(), rows, dev)
-            Chain = {"pasizen": NativePasizen, "makodra": NativeMakodra, "funevik": NativeFunevik, "hybrid_gdn": NativeHybrid}[cfg.arch]
+            Chain = {"pasizen": NativePasizen, "makodra": NativeMakodra, "funevik": NativeFunevik, "padadra": NativePadadra,
+                     "hybrid_gdn": NativeHybrid}[cfg.arch]
             make = lambda t, lr: Chain(m, kv, self.bt, t, lr, 16, self.status, True, state=self.state)
         else:
             make = lambda t, lr: NativeLlama(m, kv, self.bt, t, lr, 16, self.status, True)
@@ -171,7 +185,8 @@ def timed(fn, reps: int = 20) -> float:
 RECORDED = ("gemm_skinny", "gemm_skinny_norm", "gemm_grouped", "add_rmsnorm", "attention_fused", "rope_kv_write", "hyper_step",
             "short_conv", "poly_norm", "route", "dispatch", "gather_rows", "latent_new", "latent_attention_tc", "gdn_step",
             "rope_kv_write_heads", "post_norm_step", "token_shift", "heads_new", "chunk_attention", "chunk_attention_tc", "memory_scan",
-            "tanh_rows", "low_rank", "side_step", "conv_heads", "rotate_heads", "gated_step", "gated_chunk")
+            "tanh_rows", "low_rank", "side_step", "conv_heads", "rotate_heads", "gated_step", "gated_chunk",
+            "normed_heads", "conv_act", "memory_step")
 
 
 def record(fn) -> List[Tuple[str, tuple, dict]]:
@@ -211,8 +226,8 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
             wbytes = wbytes * (1.0 - (1.0 - 1.0 / link.groups) ** M)
         flops = 2.0 * M * N * Kd * groups
         epi = kw["epi"]
-        per_out = {1: 2, 2: 1, 3: 4, 4: 8}[epi]                # bytes per product (gated pairs leave half a bf16 value each)
-        kind = f"gemm {N}x{Kd}" + (f" x{groups} heads" if groups > 1 else "") + (" experts" if link is not None and link.mode == 2 else "")
+        per_out = {1: 2, 2: 1, 3: 4, 4: 8, 8: 2}[epi]                # bytes per product (gated pairs leave half a bf16 value each)
+        kind = f"gemm {N}x{Kd}" + (" relu2" if epi == 8 else "") + (f" x{groups} heads" if groups > 1 else "") + (" experts" if link is not None and link.mode == 2 else "")
         return kind, wbytes + M * Kd * 2 * groups + M * N * groups * per_out, flops
     if name == "latent_attention_tc":
         s = a[0]
@@ -226,25 +241,32 @@ def work_of(rig: Rig, name: str, a: tuple, kw: dict, T: int, keys: float, seqs: 
         return "attention", T * H * D * 6 + seqs * (rig.ctx if T == rig.bs else rig.prompt) * Hkv * D * 4, fl
     if name in ("chunk_attention", "chunk_attention_tc"):
         s = a[0]
-        fl = 2.0 * T * s.H * keys * (s.D + s.V)
-        return "attention", T * s.H * (2 * s.D + 6 * s.V) + seqs * (rig.ctx if T == rig.bs else rig.prompt) * s.G * (s.D + s.V) * 2, fl
+        seen, held = keys, rig.ctx if T == rig.bs else rig.prompt
+        if s.window:
+            seen, held = min(keys, s.window), min(held, s.window) if T == rig.bs else held
+        fl = 2.0 * T * s.H * seen * (s.D + s.V)
+        return "attention", T * s.H * (2 * s.D + (6 if s.gate else 2) * s.V) + seqs * held * s.G * (s.D + s.V) * 2, fl
     if name == "gated_chunk":                    # intra-chunk products and two with the state per token, at the bf16 rate
         s = a[0]
         return "memory gated (chunked)", T * s.H * (s.D * 8 + s.V * 10) + seqs * s.H * s.V * s.D * 8, 2.0 * T * s.H * (2 * s.V * s.D + 32 * (s.D + s.V))
-    if name in ("memory_scan", "gated_step"):
-        s, kind = a[0], a[1] if name == "memory_scan" else 2
+    if name in ("memory_scan", "gated_step", "memory_step"):
+        s, kind = a[0], 2 if name == "gated_step" else a[1]
         HD, HV = s.H * s.D, s.H * s.V
         # fp32 multiply-adds per matrix element and token, as bf16-rate equivalents (the floor divides by the bf16 rate)
-        fl = 2.0 * (5 if kind == 1 else 3) * T * HV * s.D * measured_peaks()[1] / F32_TFLOPS
-        name = ("wkv", "delta", "gated")[kind]
-        return "memory " + name, T * (HD * 4 * (3, 4, 2)[kind] + HV * 10) + seqs * HV * s.D * 8, fl
+        fl = 2.0 * (3, 5, 3, 4, 3)[kind] * T * HV * s.D * measured_peaks()[1] / F32_TFLOPS
+        name = ("wkv", "delta", "gated", "channel delta", "hgrn2")[kind]
+        return "memory " + name, T * (HD * 4 * (3, 4, 2, 2, 2)[kind] + HV * (10, 10, 10, 10, 6)[kind]) + seqs * HV * s.D * 8, fl
     if name == "side_step":
         s = a[0]
-        by = T * d * (4 * (s.ids is None) + 4 * (not s.final) + 4 * bool(s.y1) + 4 * bool(s.y2) + 4 * s.top + 2 + 2 * bool(s.w2) + 4 * bool(s.n2))
-        return ("embedding + norms" if s.ids else "stream + final norm" if s.final else "stream + norms") + (" + experts" if s.top else ""), by, 0.0
-    if name == "conv_heads":
+        by = T * d * (4 * (s.ids is None) + 4 * (not s.final) + 4 * bool(s.y1) + 4 * bool(s.y2) + 4 * bool(s.yb) + 4 * s.top + 2 + 2 * bool(s.w2) + 4 * bool(s.n2))
+        return ("embedding + norms" if s.ids else "stream + final norm" if s.final else "stream + norms") + (" + experts" if s.top else "") + (" + pair" if s.yb else ""), by, 0.0
+    if name == "conv_act":
         s = a[0]
-        return "conv + rotation + new heads", T * ((s.H + s.G) * s.D + s.G * s.V) * 6, 0.0
+        low = T * (s.k1 + s.k2) * 6 if s.low else (s.n1 * s.k1 + s.n2 * s.k2) * 2 + T * (s.k1 + s.k2 + s.n1 + s.n2) * 4
+        return "conv + silu" + ("" if s.low else " + low-rank maps"), T * s.C * 8 + low, 0.0 if s.low else 2.0 * T * (s.n1 * s.k1 + s.n2 * s.k2)
+    if name in ("conv_heads", "normed_heads"):
+        s = a[0]
+        return "conv + " + ("norms + " if name == "normed_heads" else "") + "rotation + new heads", T * ((s.H + s.G) * s.D + s.G * s.V) * 6, 0.0
     if name == "rotate_heads":
         return "rotate queries", T * kw["heads"] * kw["width"] * 6, 0.0
     if name == "gdn_step":
@@ -306,11 +328,12 @@ def run(width: int, layers: int = 12, bs: int = 8, ctx: int = 1024, prompt: int 
         tables: bool = True, family: str = "pasizen") -> dict:
     import gc
     rec = {"width": width, "layers": layers, "decode": {"sequences": bs, "context": ctx}, "prefill": {"prompts": n_prompts, "tokens": prompt},
-           "kv_rank": kv_rank if family != "makodra" else None, "pages": "scattered", "weights": "random, bf16", "models": []}
+           "kv_rank": kv_rank if family in ("pasizen", "funevik") else None, "pages": "scattered", "weights": "random, bf16", "models": []}
     own = {"pasizen": lambda: [pasizen_config(width, layers, kv_rank, False), pasizen_config(width, layers, kv_rank, True)],
            "makodra": lambda: [hybrid_config(width, layers), makodra_config(width, layers), makodra_config(width, layers, 128)],
            "funevik": lambda: [makodra_config(width, layers, 128), pasizen_config(width, layers, kv_rank, True),
-                               funevik_config(width, layers, kv_rank, False), funevik_config(width, layers, kv_rank, True)]}[family]()
+                               funevik_config(width, layers, kv_rank, False), funevik_config(width, layers, kv_rank, True)],
+           "padadra": lambda: [hybrid_config(width, layers), makodra_config(width, layers, 128), padadra_config(width, layers)]}[family]()
     for cfg in [dense_config(width, layers)] + own:
         rig = Rig(cfg, bs, ctx, prompt, n_prompts)
         T = n_prompts * prompt
@@ -348,7 +371,7 @@ def main(argv=None) -> None:
     ap.add_argument("--ctx", type=int, default=1024)
     ap.add_argument("--prompt", type=int, default=1024)
     ap.add_argument("--kv-rank", type=int, default=256)
-    ap.add_argument("--family", default="pasizen", choices=["pasizen", "makodra", "funevik"])
+    ap.add_argument("--family", default="pasizen", choices=["pasizen", "makodra", "funevik", "padadra"])
     ap.add_argument("--no-tables", action="store_true")
     ap.add_argument("--json", default=None)
     ns = ap.parse_args(argv)

@@ -165,10 +165,9 @@ class PadadraModel(LayeredModel):
                 n_cache += 1
             else:
                 H, G, D, E = m.heads, m.kv_heads, m.dim, m.values
-                a1, g1 = (pad_to(w, round_up(w.shape[0], 8), d8) for w in (mat(x + "a1", None, d), mat(x + "g1", None, d)))
-                wa, wg = mat(x + "a2", H * D, None), mat(x + "g2", H * E, None)
-                if round_up(wa.shape[1], 8) != a1.shape[0] or round_up(wg.shape[1], 8) != g1.shape[0]:
-                    raise ValueError(f"{x}a1, a2 or {x}g1, g2 do not meet: {tuple(wa.shape)}, {tuple(wg.shape)}")
+                a1, g1 = mat(x + "a1", None, d), mat(x + "g1", None, d)
+                wa, wg = mat(x + "a2", H * D, a1.shape[0]), mat(x + "g2", H * E, g1.shape[0])
+                a1, g1 = (pad_to(w, round_up(w.shape[0], 8), d8) for w in (a1, g1))
                 L = PadadraLayerWeights(
                     win=torch.cat([stack(rows(x + "q", G * D), rows(x + "k", G * D), rows(x + "v", H * E)), stack(rows(x + "b", H)), a1, g1]),
                     conv=torch.cat([vec(f"{x}{n}.conv", w, m.conv) for n, w in (("q", G * D), ("k", G * D), ("v", H * E))]),
