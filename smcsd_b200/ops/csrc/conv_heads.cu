@@ -5,7 +5,7 @@
 //                  of tokens with the window in registers; the thread of a sequence's first tokens, which reads the kept
 //                  projections, also writes the new ones.
 //   normed_heads   the same with biased projections, a norm of all queries (all keys) of a token together before the rotation,
-//                  and rotated values: a CTA takes the queries, the keys or the values of a run of tokens; sine and cosine
+//                  and rotated values: a CTA takes the queries, or keys and values, of a run of tokens; sine and cosine
 //                  come from a table made once per step
 //   rotate_heads   a range of every head's columns rotated, the rest passed on, in the activation type
 // Convolution, angles and rotation are fp32 (angles are reduced in fp64).
@@ -123,22 +123,31 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeadsArgs a) 
 __device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 __device__ __forceinline__ float2 turn_by(float x, float y, float2 sc) { return make_float2(x * sc.y - y * sc.x, y * sc.y + x * sc.x); }
 
-constexpr int NH_THREADS = 512, NH_TOKENS = 8;       // tokens of a run
+constexpr int NH_THREADS = 512, NH_TOKENS = 16;      // tokens of a run
 
 // NV: groups of four columns per thread.
 template <int TAPS, int NV, typename AT>
-__global__ void __launch_bounds__(NH_THREADS) normed_heads_kernel(const ConvHeadsArgs a) {
+__global__ void __launch_bounds__(NH_THREADS, NV == 1 && TAPS <= 4 ? 2 : 1) normed_heads_kernel(const ConvHeadsArgs a) {
   constexpr int HL = TAPS - 1;
   __shared__ float red[2][NH_THREADS / 32];
-  const int nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.V, C = nq + nk + nv, part = blockIdx.y;
-  const int base = part == 0 ? 0 : part == 1 ? nq : nq + nk, n = part == 0 ? nq : part == 1 ? nk : nv;
-  const int width = part < 2 ? a.D : a.V, rot = part < 2 ? a.rot : a.turn, first_pair = part < 2 ? a.qk_first : a.v_first;
+  const int nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.V, C = nq + nk + nv;
+  const bool keys = blockIdx.y == 1;                 // keys and values, else queries
+  const int base = keys ? nq : 0, n = keys ? nk + nv : nq, normed = keys ? nk : nq;      // columns of this CTA, those under the norm
   const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x * 4 >= ((n + 127) & ~127)) {       // whole warps without columns; the others meet at a barrier of their own count
     if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
     return;
   }
   const int live = min(nw, ((n + 127) / 128));       // warps that stay
+  int pair[NV];                                      // first of the columns' pairs in the table of angles (-1: not rotated)
+  bool two[NV];                                      // and the second as well
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4, value = keys && c >= nk;
+    const int col = value ? (c - nk) % a.V : c % a.D, rot = value ? a.turn : a.rot;
+    pair[i] = col < rot ? (value ? a.v_first : a.qk_first) + (col >> 1) : -1;
+    two[i] = col + 2 < rot;
+  }
   float4 w[NV][TAPS], bias[NV], g[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -146,7 +155,7 @@ __global__ void __launch_bounds__(NH_THREADS) normed_heads_kernel(const ConvHead
     bias[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < n) {
       bias[i] = load4(a.bias + base + c);
-      if (part < 2) g[i] = load4(a.qk_norm + base + c);
+      if (c < normed) g[i] = load4(a.qk_norm + base + c);
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) w[i][j] = load4(a.conv + (size_t)j * C + base + c);
     }
@@ -189,11 +198,14 @@ __global__ void __launch_bounds__(NH_THREADS) normed_heads_kernel(const ConvHead
     }
     u[i] = load4(src + (size_t)t0 * a.ldp + c);
   }
-  const float count = (float)((part == 0 ? a.H : a.G) * a.dim);
+  const float count = (float)((keys ? a.G : a.H) * a.dim);
   for (int t = t0; t < t1; ++t) {
     const int tok = b.off + t;
     float4 y[NV];
+    float2 turn[NV][2];                              // sine and cosine, fetched ahead of the barrier
     float ss = 0.f;
+    int page = keys ? a.locs[tok] : 0;
+    const float2* ang = a.angles + (size_t)tok * a.ld_angles;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * 4;
@@ -206,39 +218,27 @@ __global__ void __launch_bounds__(NH_THREADS) normed_heads_kernel(const ConvHead
 #pragma unroll
       for (int j = 0; j + 1 < HL; ++j) win[i][j] = win[i][j + 1];
       if (HL > 0) win[i][HL > 0 ? HL - 1 : 0] = now;
-      ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+      if (c < normed) ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+      turn[i][0] = turn[i][1] = make_float2(0.f, 1.f);
+      if (pair[i] >= 0) turn[i][0] = ang[pair[i]];
+      if (pair[i] >= 0 && two[i]) turn[i][1] = ang[pair[i] + 1];
     }
-    float inv = 1.0f;
-    if (part < 2) {                                  // the same in the whole CTA; the buffers alternate, one barrier per token
-      float* rd = red[t & 1];
-      ss = warp_sum(ss);
-      if (lane == 0) rd[warp] = ss;
-      asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
-      inv = 1.0f / sqrtf(warp_sum(lane < live ? rd[lane] : 0.f) / count + a.eps);
-    }
-    int page = 0;
-    if (part > 0) {
-      page = a.locs[tok];
-      if (page < 0 || page > a.n_pages) { atomicOr(a.status, SMC_ERR_BOUNDS); page = 0; }
-    }
-    AT* out = part == 0 ? reinterpret_cast<AT*>(a.q) + (size_t)tok * nq
-                        : part == 1 ? reinterpret_cast<AT*>(a.kpool) + (size_t)page * nk : reinterpret_cast<AT*>(a.vpool) + (size_t)page * nv;
-    const float2* ang = a.angles + (size_t)tok * a.ld_angles + first_pair;
+    float* rd = red[t & 1];                          // the buffers alternate: one barrier per token
+    ss = warp_sum(ss);
+    if (lane == 0) rd[warp] = ss;
+    asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
+    const float inv = 1.0f / sqrtf(warp_sum(lane < live ? rd[lane] : 0.f) / count + a.eps);
+    if (page < 0 || page > a.n_pages) { atomicOr(a.status, SMC_ERR_BOUNDS); page = 0; }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (threadIdx.x + i * blockDim.x) * 4, col = c % width;
+      const int c = (threadIdx.x + i * blockDim.x) * 4;
       if (c >= n) continue;
       float4 v = y[i];
-      if (part < 2) v = make_float4(v.x * inv * g[i].x, v.y * inv * g[i].y, v.z * inv * g[i].z, v.w * inv * g[i].w);
-      if (col < rot) {
-        const float2 lo = turn_by(v.x, v.y, ang[col >> 1]);
-        v.x = lo.x; v.y = lo.y;
-        if (col + 2 < rot) {
-          const float2 hi = turn_by(v.z, v.w, ang[(col >> 1) + 1]);
-          v.z = hi.x; v.w = hi.y;
-        }
-      }
-      store4(out + c, v);
+      if (c < normed) v = make_float4(v.x * inv * g[i].x, v.y * inv * g[i].y, v.z * inv * g[i].z, v.w * inv * g[i].w);
+      const float2 lo = turn_by(v.x, v.y, turn[i][0]), hi = turn_by(v.z, v.w, turn[i][1]);
+      AT* out = !keys ? reinterpret_cast<AT*>(a.q) + (size_t)tok * nq + c
+                      : c < nk ? reinterpret_cast<AT*>(a.kpool) + (size_t)page * nk + c : reinterpret_cast<AT*>(a.vpool) + (size_t)page * nv + (c - nk);
+      store4(out, make_float4(lo.x, lo.y, hi.x, hi.y));
     }
   }
 }
@@ -288,9 +288,9 @@ static int normed_heads_taps(const ConvHeadsArgs& a, dim3 grid, dim3 block, cuda
 template <typename AT>
 static int normed_heads_launch(const ConvHeadsArgs& a, cudaStream_t st) {
   int most = a.H * a.D;
-  if (a.G * a.V > most) most = a.G * a.V;
+  if (a.G * (a.D + a.V) > most) most = a.G * (a.D + a.V);
   const int groups = (most / 4 + 31) / 32 * 32;
-  const dim3 grid(a.r.n_blk, 3, (a.r.B + NH_TOKENS - 1) / NH_TOKENS);
+  const dim3 grid(a.r.n_blk, 2, (a.r.B + NH_TOKENS - 1) / NH_TOKENS);
   if (groups <= NH_THREADS) return normed_heads_taps<AT, 1>(a, grid, dim3(groups), st);
   if (groups <= NH_THREADS * 2) return normed_heads_taps<AT, 2>(a, grid, dim3(NH_THREADS), st);
   if (groups <= NH_THREADS * 4) return normed_heads_taps<AT, 4>(a, grid, dim3(NH_THREADS), st);
@@ -308,7 +308,7 @@ SMC_API int smc_conv_heads(const smc::ConvHeadsArgs* a, int f32, cudaStream_t st
   return f32 ? conv_heads_launch<float>(*a, st) : conv_heads_launch<__nv_bfloat16>(*a, st);
 }
 
-// The normed form (see the top): up to 8192 query columns.
+// The normed form (see the top): up to 8192 query columns, as many key and value columns.
 SMC_API int smc_normed_heads(const smc::ConvHeadsArgs* a, int f32, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_blk <= 0) return 0;

@@ -42,10 +42,11 @@ namespace smc {
 enum { EPI_PARTIAL_F32 = 0, EPI_BF16 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_F32 = 3, EPI_RESID_F32 = 4, EPI_RS_F32 = 5,
        EPI_SWIGLU_SPLIT = 6,     // 6: SwiGLU after a split-K reduction inside the cluster
        EPI_LMHEAD = 7,           // 7: lm_head: every slab is reduced to per-row sampling partials, logits are not stored
-       EPI_RELU2_BF16 = 8 };     // 8: squared relu, after the split-K reduction inside the cluster
+       EPI_RELU2_BF16 = 8,       // 8: squared relu
+       EPI_RELU2_SPLIT = 9 };    // 9: squared relu after a split-K reduction inside the cluster
 // Epilogues that reduce split-K inside a thread-block cluster (of one CTA, if K is not split).
 __host__ __device__ constexpr bool epi_clustered(int epi) {
-  return epi == EPI_STORE_F32 || epi == EPI_RESID_F32 || epi == EPI_RS_F32 || epi == EPI_SWIGLU_SPLIT || epi == EPI_RELU2_BF16;
+  return epi == EPI_STORE_F32 || epi == EPI_RESID_F32 || epi == EPI_RS_F32 || epi == EPI_SWIGLU_SPLIT || epi == EPI_RELU2_SPLIT;
 }
 
 // Tensor-parallel links of one GEMM.  Consumer side (all-gather -> GEMM): peers store their
@@ -405,8 +406,9 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
                 reinterpret_cast<float*>(p.out)[((size_t)split * p.M + m) * p.N + n] =
                     __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
               } else {
-                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + out_off + n] =
-                    __float2bfloat16(__uint_as_float(r[j]) * wsc * s_rstd[c0 + j]);
+                float v = __uint_as_float(r[j]) * wsc * s_rstd[c0 + j];
+                if constexpr (EPI == EPI_RELU2_BF16) v = v > 0.f ? v * v : 0.f;
+                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + out_off + n] = __float2bfloat16(v);
               }
             }
           }
@@ -474,7 +476,7 @@ __global__ void __launch_bounds__(128) gemm_skinny_kernel(const __grid_constant_
             acc *= s_rstd[c];
             if constexpr (EPI == EPI_SWIGLU_SPLIT) {
               prev[u] = acc;               // paired below: rows 0..63 are gate channels, 64..127 the matching up channels
-            } else if constexpr (EPI == EPI_RELU2_BF16) {
+            } else if constexpr (EPI == EPI_RELU2_SPLIT) {
               const float z = fmaxf(acc, 0.f);
               reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(m_base + c) * p.ldo + n] = __float2bfloat16(z * z);
             } else if constexpr (EPI == EPI_RS_F32) {
@@ -689,8 +691,9 @@ SMC_API int smc_gemm_cluster_splits(int N, int K, int M) {
 }
 
 // W [N, K] bf16 row-major, X [M, ldx] bf16 row-major (ldx >= K).
-// epi 3: out = fp32 [M, ldo] = X W^T;  epi 4: out (fp32 [M, ldo]) += X W^T;  epi 8: out = bf16 [M, ldo] = max(X W^T, 0)^2.
-// These reduce split-K inside a thread-block cluster, so splits must be 1..8.
+// epi 3: out = fp32 [M, ldo] = X W^T;  epi 4: out (fp32 [M, ldo]) += X W^T.  Both reduce split-K inside a
+// thread-block cluster, so splits must be 1..8.
+// epi 8: out = bf16 [M, ldo] = max(X W^T, 0)^2 (splits > 1 reduce split-K inside a cluster first).
 // epi 0: out = fp32 [splits, M, N] partials; epi 1: out = bf16 [M, ldo] (splits must be 1);
 // epi 2: out = bf16 [M, ldo] holding SwiGLU(gate, up) for N/2 channels (N % 128 == 0; splits > 1 reduce split-K
 //        inside a cluster first).
@@ -743,6 +746,7 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
   if ((K * es) % 16 != 0 || (ldx * es) % 16 != 0) return -20;       // row pitch must be a multiple of 16 bytes
   if (f8 != nullptr && nl != nullptr) return -28;
   if (epi == EPI_SWIGLU_BF16 && splits > 1) epi = EPI_SWIGLU_SPLIT;      // split-K reduced in the cluster, then SwiGLU
+  if (epi == EPI_RELU2_BF16 && splits > 1) epi = EPI_RELU2_SPLIT;
   const bool clustered = epi_clustered(epi);
   if (!clustered && epi != EPI_PARTIAL_F32 && splits != 1) return -21;
   if (clustered && (splits < 1 || splits > 8)) return -23;
@@ -821,6 +825,7 @@ static int gemm_entry(const void* W, const void* X, void* out, int N, int K, int
     case EPI_SWIGLU_SPLIT: return dispatch_bn<EPI_SWIGLU_SPLIT>(bn, tmW, tmX, p, grid, stream);
     case EPI_LMHEAD: return dispatch_bn<EPI_LMHEAD>(bn, tmW, tmX, p, grid, stream);
     case EPI_RELU2_BF16: return dispatch_bn<EPI_RELU2_BF16>(bn, tmW, tmX, p, grid, stream);
+    case EPI_RELU2_SPLIT: return dispatch_bn<EPI_RELU2_SPLIT>(bn, tmW, tmX, p, grid, stream);
   }
   return -11;
 }

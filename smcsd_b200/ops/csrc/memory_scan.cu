@@ -13,7 +13,7 @@
 //   forget  M <- diag(w) M + (1 - w) v^T, read out with silu(r) afterwards; w = lower + (1 - lower) sigmoid(. + bias); no output gate
 //
 // Value columns of a matrix never mix, key rows only in sums.  A CTA therefore keeps some columns of one head's matrix in
-// registers - four threads per pair of columns (one column beyond 128 key rows), a quarter of the key rows each - and walks
+// registers - four or eight threads per pair of columns (one column beyond 128 key rows) share the key rows - and walks
 // its sequence's tokens in tiles: consumer warps run the recurrence on the tile in shared memory while eight producer warps
 // turn the next tile's projections into w, u, a u, ... and finish the outputs of the tile before (division by the head's root
 // mean square, norm weight, gate).  Producers fetch a tile ahead of the one they prepare, so a tile's loads have a whole tile
@@ -60,22 +60,27 @@ __device__ __forceinline__ float sum_of(f2_t a) { const float2 v = unpack2(a); r
 __host__ __device__ constexpr int scan_tokens(int dkp) { return dkp <= 128 ? 16 : 8; }       // tokens of a tile
 __host__ __device__ constexpr int scan_vectors(int kind) { return kind == SCAN_DELTA ? 5 : kind == SCAN_CHANNEL ? 4 : kind == SCAN_GATED ? 2 : 3; }
 __host__ __device__ constexpr int scan_columns(int dkp) { return dkp <= 128 ? 2 : 1; }       // of a consumer thread
-__host__ __device__ constexpr int scan_max_columns(int dkp) { return SCAN_CONSUMERS / 4 * scan_columns(dkp); }      // of a CTA
+// Consumer threads that share a column's key rows: eight give a token's chain half the length, at one more exchange per sum.
+__host__ __device__ constexpr int scan_sharers(int kind, int dkp) {
+  return (kind == SCAN_CHANNEL || kind == SCAN_FORGET) && dkp >= 64 && dkp <= 128 && dkp % 32 == 0 ? 8 : 4;
+}
+__host__ __device__ constexpr int scan_max_columns(int kind, int dkp) { return SCAN_CONSUMERS / scan_sharers(kind, dkp) * scan_columns(dkp); }      // of a CTA
 
 template <int KIND, int DKP>
 __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_kernel(const ScanArgs a, int CC, int CS, int f32) {
   constexpr bool GENERAL = KIND == SCAN_DELTA, GATED = KIND == SCAN_GATED, CHANNEL = KIND == SCAN_CHANNEL, FORGET = KIND == SCAN_FORGET;
   constexpr bool DELTA = GENERAL || CHANNEL;                 // something is taken off along u
   constexpr bool SQUARE = GENERAL || KIND == SCAN_BONUS;     // as many values as keys
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), NL = (DKP + 31) / 32, NQ = DKP / 16, CP = scan_columns(DKP);
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), NL = (DKP + 31) / 32, CP = scan_columns(DKP);
+  constexpr int KT = scan_sharers(KIND, DKP), NQ = DKP / (4 * KT), MOST = scan_max_columns(KIND, DKP);
   constexpr int PT = TB / SCAN_PRODUCERS;                    // tokens of a tile per producer warp
-  constexpr int NC = ((!SQUARE || scan_max_columns(DKP) < DKP ? scan_max_columns(DKP) : DKP) + 31) / 32;      // columns of a CTA per lane
+  constexpr int NC = ((!SQUARE || MOST < DKP ? MOST : DKP) + 31) / 32;      // columns of a CTA per lane
   extern __shared__ __align__(16) float scan_smem[];
   const int buf_floats = TB * (NVEC * DKP + CC + 2);
   float* obuf = scan_smem + 2 * buf_floats;                  // [3][TB][CC]
   float* ssq = obuf + 3 * TB * CC;                           // [2][TB]
   float* least = ssq + 2 * TB;                               // [4][TB] exp(-m) (gated)
-  const int n_cons = CC / CP * 4, tid = threadIdx.x, lane = tid & 31;
+  const int n_cons = CC / CP * KT, tid = threadIdx.x, lane = tid & 31;
   const bool consumer = tid < n_cons;
   if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
   const int h = blockIdx.x / CS, rank = blockIdx.x - h * CS, s = blockIdx.y, D = a.D, V = a.V;
@@ -323,8 +328,8 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     return;
   }
 
-  // ---- consumers: CP columns, and every fourth group of four key rows
-  const int col = (tid >> 2) * CP, kq = tid & 3;
+  // ---- consumers: CP columns, and every KT-th group of four key rows
+  const int col = tid / KT * CP, kq = tid % KT;
   auto column = [&](int x) {                                 // row of the transposed matrix (-1: none)
     if (GATED && col + x == CC - 1) return V;
     return col + x < own && c0 + col + x < V ? c0 + col + x : -1;
@@ -338,7 +343,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     sp[x] = a.state + (size_t)row * a.row_stride + ((size_t)h * (V + GATED) + (mine ? cg : 0)) * D;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
-      const int k = (kq + 4 * i) * 4;
+      const int k = (kq + KT * i) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (mine && (D & 3) == 0) {
         if (k < D) v = *reinterpret_cast<const float4*>(sp[x] + k);
@@ -378,7 +383,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
           if (DELTA) {
-            const ulonglong2 u = du[kq + 4 * i];
+            const ulonglong2 u = du[kq + KT * i];
 #pragma unroll
             for (int x = 0; x < CP; ++x) {
               g2[x][0] = fma2(M[x][2 * i], u.x, g2[x][0]);
@@ -392,13 +397,13 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
           gone[x] = 0.f;
           if (DELTA) {
             gone[x] = sum_of(g2[x][0]) + sum_of(g2[x][1]);
-            gone[x] += __shfl_xor_sync(0xffffffffu, gone[x], 1);
-            gone[x] += __shfl_xor_sync(0xffffffffu, gone[x], 2);
+#pragma unroll
+            for (int s = 1; s < KT; s <<= 1) gone[x] += __shfl_xor_sync(0xffffffffu, gone[x], s);
           }
         }
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-          const ulonglong2 r = dr[kq + 4 * i];
+          const ulonglong2 r = dr[kq + KT * i];
 #pragma unroll
           for (int x = 0; x < CP; ++x) {
             o2[x][0] = fma2(M[x][2 * i], r.x, o2[x][0]);
@@ -415,11 +420,11 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
         }
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-          const ulonglong2 k = dk[kq + 4 * i];
+          const ulonglong2 k = dk[kq + KT * i];
           ulonglong2 w;
-          if (GATED) w.x = w.y = pack2(s1, s1); else w = dw[kq + 4 * i];
+          if (GATED) w.x = w.y = pack2(s1, s1); else w = dw[kq + KT * i];
           ulonglong2 au;
-          if (GENERAL) au = da[kq + 4 * i];
+          if (GENERAL) au = da[kq + KT * i];
 #pragma unroll
           for (int x = 0; x < CP; ++x) {
             f2_t p = mul2(k.x, vv[x]), q = mul2(k.y, vv[x]);
@@ -433,8 +438,8 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
         }
 #pragma unroll
         for (int x = 0; x < CP; ++x) {
-          o[x] += __shfl_xor_sync(0xffffffffu, o[x], 1);
-          o[x] += __shfl_xor_sync(0xffffffffu, o[x], 2);
+#pragma unroll
+          for (int s = 1; s < KT; s <<= 1) o[x] += __shfl_xor_sync(0xffffffffu, o[x], s);
           if (kq == 0)
             store_shared_unordered(o_out + (tb * CC + col + x) * 4, fmaf(s2, v[x], GENERAL ? fmaf(-s1, gone[x], o[x]) : GATED ? s1 * o[x] : o[x]));
         }
@@ -447,7 +452,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     if (column(x) < 0 || (GATED && column(x) == V && rank != 0)) continue;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
-      const int k = (kq + 4 * i) * 4;
+      const int k = (kq + KT * i) * 4;
       const float2 lo = unpack2(M[x][2 * i]), hi = unpack2(M[x][2 * i + 1]);
       if ((D & 3) == 0) {
         if (k < D) *reinterpret_cast<float4*>(sp[x] + k) = make_float4(lo.x, lo.y, hi.x, hi.y);
@@ -495,7 +500,7 @@ __global__ void __launch_bounds__(64) low_rank_kernel(const float* x, int ldx, c
 
 // Columns per CTA and CTAs per head: a head's columns are cut until the grid fills the machine (16 columns at the least); a
 // CTA takes at most scan_max_columns, `extra` of them beside its share of the head's.  Whole warps of consumers need multiples
-// of 8 (16 in pairs).
+// of 8 (16 in pairs), half of that with eight threads per pair.
 static void scan_split(int n_seq, int H, int V, int most, int unit, int extra, int* CC, int* CS) {
   int cs = 1;
   while ((V + cs - 1) / cs + extra > most) cs *= 2;
@@ -507,13 +512,13 @@ static void scan_split(int n_seq, int H, int V, int most, int unit, int extra, i
 template <int KIND, int DKP>
 static int scan_launch(const ScanArgs& a, int f32, cudaStream_t st) {
   int CC, CS;
-  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), CP = scan_columns(DKP);
-  scan_split(a.r.n_seq, a.H, a.V, scan_max_columns(DKP), 8 * CP, KIND == SCAN_GATED, &CC, &CS);
+  constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), CP = scan_columns(DKP), KT = scan_sharers(KIND, DKP);
+  scan_split(a.r.n_seq, a.H, a.V, scan_max_columns(KIND, DKP), 32 / KT * CP, KIND == SCAN_GATED, &CC, &CS);
   if (CS > 16) return -122;
   const int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 6 * TB) * 4;
   CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
   if (CS > 8) CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
-  return launch_cluster(scan_kernel<KIND, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * 4 + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
+  return launch_cluster(scan_kernel<KIND, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * KT + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
                         CS, a, CC, CS, f32);
 }
 

@@ -12,7 +12,7 @@ from test_padadra_cpu import alone
 pytestmark = pytest.mark.gpu
 
 F32 = S.Ctx("cuda", "float32", 3e-5, models=M, oracle=O)
-BF16 = S.Ctx("cuda", "bfloat16", 0.06, models=M, oracle=O)
+BF16 = S.Ctx("cuda", "bfloat16", 0.06, slack=0.01, models=M, oracle=O)
 BOTH = pytest.mark.parametrize("ctx", [F32, BF16], ids=["f32", "bf16"])
 
 
