@@ -11,6 +11,8 @@
 //   channel M <- diag(w) M, then M <- M + b u (v - M^T u)^T, read out with r afterwards; u = k / |k|, r likewise times r_scale (both
 //           shared by groups of heads), b = sigmoid(beta), w = exp(-exp(a_log) softplus(z + w0)); output gate sigmoid
 //   forget  M <- diag(w) M + (1 - w) v^T, read out with silu(r) afterwards; w = lower + (1 - lower) sigmoid(. + bias); no output gate
+// The elementwise functions of the last two are taken by a kernel of its own ahead of the scan, in place (scan_operands): the
+// columns of a head are spread over CTAs, each of which would take them again, and the producers would not keep up.
 //
 // Value columns of a matrix never mix, key rows only in sums.  A CTA therefore keeps some columns of one head's matrix in
 // registers - four or eight threads per pair of columns (one column beyond 128 key rows) share the key rows - and walks
@@ -29,6 +31,7 @@ namespace smc {
 
 constexpr int SCAN_PRODUCERS = 8;        // warps
 constexpr int SCAN_CONSUMERS = 256;      // threads at the most
+constexpr int SCAN_ALONE_BYTES = 118 * 1024;          // shared memory that leaves no room for a second CTA
 
 typedef unsigned long long f2_t;
 __device__ __forceinline__ f2_t pack2(float a, float b) {
@@ -102,9 +105,8 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
     const int pw = (tid - n_cons) >> 5;
     float kk[PT][NL], rr[PT][NL], zz[PT][NL], aa[PT][NL], vv[PT][NC], gg[PT][NC];
     float gi = 0.f, gf = 0.f, m_run = 0.f, bi = 0.f, bf = 0.f;       // gated: gate logits of token `lane` of a tile, running maximum
-    float bb[PT], rate = 0.f;                                // channel: write strengths, decay rate of the head
+    float bb[PT];                                            // channel: write strengths
     const int hk = CHANNEL ? h / a.rep : h;
-    if (CHANNEL) rate = expf(a.a_log[h]);
     if (GATED) {
       bi = a.a_bias[h];
       bf = a.a_bias[a.H + h];
@@ -199,7 +201,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
             continue;
           }
           if (CHANNEL) {
-            const float w = ok ? expf(-rate * softplus_f(zz[j][i] + a.w0[h * D + c])) : 0.f, u = kk[j][i] * inv, r = rr[j][i] * rinv;
+            const float w = zz[j][i], u = kk[j][i] * inv, r = rr[j][i] * rinv;
             d[c] = w;
             d[TB * DKP + c] = b * u;
             d[2 * TB * DKP + c] = r * w;
@@ -208,9 +210,7 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
             continue;
           }
           if (FORGET) {
-            const float z = ok ? aa[j][i] + a.a_bias[h * D + c] : 0.f, l = ok ? a.lower[h * D + c] : 0.f;
-            const float w = ok ? fmaf(1.0f - l, sigmoid_f(z), l) : 0.f, k = ok ? (1.0f - l) * sigmoid_f(-z) : 0.f;
-            const float r = rr[j][i] * sigmoid_f(rr[j][i]);
+            const float k = aa[j][i], w = ok ? 1.0f - k : 0.f, r = rr[j][i];
             d[c] = w;
             d[TB * DKP + c] = k;
             d[2 * TB * DKP + c] = r * w;
@@ -293,8 +293,8 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
         for (int i = 0; i < NC; ++i) {
           const int c = lane + 32 * i, col = h * V + c0 + c;
           if (c >= own || c0 + c >= V) continue;
-          const float g = gg[j][i], sg = sigmoid_f(g);
-          const float v = o[c] * inv * a.onorm[col] * (FORGET ? 1.0f : DELTA || GATED ? sg : g * sg);
+          const float g = gg[j][i], sg = CHANNEL || FORGET ? 1.0f : sigmoid_f(g);
+          const float v = o[c] * inv * (CHANNEL ? g : a.onorm[col] * (FORGET || GENERAL || GATED ? sg : g * sg));
           if (f32) reinterpret_cast<float*>(a.out)[t * a.ldo + col] = v;
           else reinterpret_cast<__nv_bfloat16*>(a.out)[t * a.ldo + col] = __float2bfloat16(v);
         }
@@ -466,6 +466,46 @@ __global__ void __launch_bounds__(SCAN_CONSUMERS + SCAN_PRODUCERS * 32) scan_ker
   }
 }
 
+// Elementwise operands of the kinds channel and forget, in place, four (or one) columns per thread:
+//   channel  z <- exp(-exp(a_log) softplus(z + w0)), gate <- sigmoid(gate) onorm
+//   forget   r <- silu(r), forget gate <- 1 - w = (1 - lower) sigmoid(-(. + bias)): what is written keeps its relative accuracy
+template <int KIND, int VEC>
+__global__ void __launch_bounds__(128) scan_operands_kernel(const ScanArgs a, int T) {
+  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  const int HD = a.H * a.D, n2 = KIND == SCAN_CHANNEL ? a.H * a.V : HD, c = (blockIdx.x * 128 + threadIdx.x) * VEC;
+  if (c >= HD + n2) return;
+  const bool second = c >= HD;                               // VEC divides HD
+  const int at = second ? c - HD : c;
+  float w[VEC], l[VEC];
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) {
+    w[k] = KIND == SCAN_CHANNEL ? (second ? a.onorm[at + k] : a.w0[at + k]) : a.a_bias[at + k];
+    l[k] = KIND == SCAN_CHANNEL ? (second ? 0.f : -expf(a.a_log[(at + k) / a.D])) : 1.0f - a.lower[at + k];
+  }
+  for (int t = blockIdx.y; t < T; t += gridDim.y) {
+    float* p = const_cast<float*>(KIND == SCAN_CHANNEL ? (second ? a.gate + (size_t)t * a.ldg : a.z + (size_t)t * a.ldz)
+                                                       : a.proj + (size_t)t * a.ldp + (second ? a.a_off : a.r_off)) + at;
+    float v[VEC];
+    load_cols<VEC>(v, (const float*)p);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+      if (KIND == SCAN_CHANNEL) v[k] = second ? sigmoid_f(v[k]) * w[k] : expf(l[k] * softplus_f(v[k] + w[k]));
+      else v[k] = second ? l[k] * sigmoid_f(-(v[k] + w[k])) : v[k] * sigmoid_f(v[k]);
+    }
+    store_cols<VEC>(p, v);
+  }
+}
+
+template <int KIND>
+static int scan_operands(const ScanArgs& a, int T, cudaStream_t st) {
+  const int HD = a.H * a.D, n = HD + (KIND == SCAN_CHANNEL ? a.H * a.V : HD);
+  const bool vec = HD % 4 == 0 && n % 4 == 0 && a.D % 4 == 0 &&
+                   (KIND == SCAN_CHANNEL ? a.ldz % 4 == 0 && a.ldg % 4 == 0 : (a.ldp | a.r_off | a.a_off) % 4 == 0);
+  const dim3 grid((n / (vec ? 4 : 1) + 127) / 128, T < 1024 ? T : 1024), block(128);
+  return vec ? launch_pdl(scan_operands_kernel<KIND, 4>, grid, block, 0, st, a.pdl, a, T)
+             : launch_pdl(scan_operands_kernel<KIND, 1>, grid, block, 0, st, a.pdl, a, T);
+}
+
 template <typename AT>
 __global__ void __launch_bounds__(128) tanh_rows_kernel(const float* x, int ldx, AT* out, int ldo, int n, int M, int pdl) {
   if (pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
@@ -515,7 +555,9 @@ static int scan_launch(const ScanArgs& a, int f32, cudaStream_t st) {
   constexpr int TB = scan_tokens(DKP), NVEC = scan_vectors(KIND), CP = scan_columns(DKP), KT = scan_sharers(KIND, DKP);
   scan_split(a.r.n_seq, a.H, a.V, scan_max_columns(KIND, DKP), 32 / KT * CP, KIND == SCAN_GATED, &CC, &CS);
   if (CS > 16) return -122;
-  const int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 6 * TB) * 4;
+  int bytes = (2 * TB * (NVEC * DKP + CC + 2) + 3 * TB * CC + 6 * TB) * 4;
+  // a grid of no more CTAs than SMs: one each, also where the launch overlaps the kernel before and SMs are unevenly free
+  if ((KIND == SCAN_CHANNEL || KIND == SCAN_FORGET) && (long long)a.H * CS * a.r.n_seq <= 148 && bytes < SCAN_ALONE_BYTES) bytes = SCAN_ALONE_BYTES;
   CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes));
   if (CS > 8) CUDA_CHECK_RET(cudaFuncSetAttribute(scan_kernel<KIND, DKP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
   return launch_cluster(scan_kernel<KIND, DKP>, dim3(a.H * CS, a.r.n_seq), dim3(CC / CP * KT + SCAN_PRODUCERS * 32), bytes, st, a.pdl,
@@ -535,8 +577,9 @@ static int scan_dispatch(const ScanArgs& a, int f32, cudaStream_t st) {
 SMC_API int smc_scan_args_size() { return (int)sizeof(smc::ScanArgs); }
 
 // One memory layer over the new tokens of every sequence; kind: 0 the bonus form, 1 the generalized delta rule (both V = D), 2
-// the gated form, 3 the delta rule with a decay per channel, 4 the forget-gated form.  Heads of up to 256 key columns.
-SMC_API int smc_memory_scan(const smc::ScanArgs* a, int kind, int f32, cudaStream_t st) {
+// the gated form, 3 the delta rule with a decay per channel, 4 the forget-gated form (the last two overwrite their operands, T
+// rows in all).  Heads of up to 256 key columns.
+SMC_API int smc_memory_scan(const smc::ScanArgs* a, int kind, int T, int f32, cudaStream_t st) {
   using namespace smc;
   if (a->r.n_seq <= 0) return 0;
   if (a->D < 1 || a->H < 1 || a->V < 1 || a->r.n_seq > 65535 || (kind < SCAN_GATED && a->V != a->D)) return -120;
@@ -545,8 +588,12 @@ SMC_API int smc_memory_scan(const smc::ScanArgs* a, int kind, int f32, cudaStrea
     case SCAN_BONUS: return scan_dispatch<SCAN_BONUS>(*a, f32, st);
     case SCAN_DELTA: return scan_dispatch<SCAN_DELTA>(*a, f32, st);
     case SCAN_GATED: return scan_dispatch<SCAN_GATED>(*a, f32, st);
-    case SCAN_CHANNEL: return scan_dispatch<SCAN_CHANNEL>(*a, f32, st);
-    case SCAN_FORGET: return scan_dispatch<SCAN_FORGET>(*a, f32, st);
+    case SCAN_CHANNEL:
+      if (const int rc = scan_operands<SCAN_CHANNEL>(*a, T, st)) return rc;
+      return scan_dispatch<SCAN_CHANNEL>(*a, f32, st);
+    case SCAN_FORGET:
+      if (const int rc = scan_operands<SCAN_FORGET>(*a, T, st)) return rc;
+      return scan_dispatch<SCAN_FORGET>(*a, f32, st);
   }
   return -120;
 }

@@ -726,7 +726,7 @@ def layered_lib():
         L.smc_chunk_attn.argtypes = [vp, i, i, vp]
         L.smc_chunk_attn_splits.argtypes = [i, i, i, i, i]
         L.smc_chunk_attn_tc.argtypes = [vp, vp]
-        L.smc_memory_scan.argtypes = [vp, i, i, vp]
+        L.smc_memory_scan.argtypes = [vp, i, i, i, vp]
         L.smc_gated_step.argtypes = [vp, i, vp]
         L.smc_memory_step.argtypes = [vp, i, i, vp]
         L.smc_memory_step_takes.argtypes = [i, i]
@@ -910,10 +910,12 @@ def chunk_tc_max_width() -> int:
     return layered_lib().smc_chunk_attn_tc_max_width()
 
 
-def memory_scan(a: ScanArgs, kind: int, f32: bool) -> None:
+def memory_scan(a: ScanArgs, kind: int, f32: bool, T: int = 0) -> None:
     """A recurrent memory layer over the new tokens of every sequence (csrc/memory_scan.cu); ``kind``: SCAN_BONUS, SCAN_DELTA,
-    SCAN_GATED, SCAN_CHANNEL or SCAN_FORGET."""
-    _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), int(f32), _stream()), "smc_memory_scan")
+    SCAN_GATED, SCAN_CHANNEL or SCAN_FORGET; the last two run over ``T`` tokens in all and overwrite their operands."""
+    if kind in (SCAN_CHANNEL, SCAN_FORGET) and T < 1:
+        raise ValueError("the number of tokens is missing")
+    _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), T, int(f32), _stream()), "smc_memory_scan")
 
 
 def gated_step_takes(D: int, V: int) -> bool:

@@ -102,11 +102,11 @@ class NativePadadra(NativeLayered):
         return tuple(sorted((E, m.window, m.heads, self._chunk_splits(bs * E, m, m.window)) for E in Es for m in mixers))
 
     # ---- mixers -------------------------------------------------------------------------
-    def _memory(self, a: "K.ScanArgs", kind: int, longest: int) -> None:
+    def _memory(self, a: "K.ScanArgs", kind: int, T: int, longest: int) -> None:
         if longest == 1 and K.memory_step_takes(a.D, a.V):
             K.memory_step(a, kind, self.f32)
         else:
-            K.memory_scan(a, kind, self.f32)
+            K.memory_scan(a, kind, self.f32, T)
 
     def _scan_args(self, L, m, proj: torch.Tensor, out: torch.Tensor, work: "K.Ragged", **kw) -> "K.ScanArgs":
         S = self.state.matrix(L.state + 1)
@@ -133,7 +133,7 @@ class NativePadadra(NativeLayered):
             self._gemm(L.wg, low[:, ra:], gate, T, ldx=ra + rg)
         self._memory(self._scan_args(L, m, u, vo, work, r_off=0, k_off=G * D, v_off=2 * G * D, z=K.ptr(z), ldz=HD, w0=K.ptr(L.dt_bias),
                                      r_scale=D ** -0.5, beta=K.ptr(proj[:, C8:]), ldb=proj.stride(0), gate=K.ptr(gate), ldg=HE, a_log=K.ptr(L.a_log),
-                                     rep=H // G), K.SCAN_CHANNEL, longest)
+                                     rep=H // G), K.SCAN_CHANNEL, T, longest)
         return vo
 
     def _attention(self, i: int, L, T: int, locs, work: "K.Ragged", longest: int) -> torch.Tensor:
@@ -157,7 +157,7 @@ class NativePadadra(NativeLayered):
         m, C = L.spec.mixer.right, attention_columns(L.spec.mixer.left)
         proj, vo, HD = self._rows("proj", T, L.win.shape[0]), self._rows("vo2", T, L.wo2.shape[1]), m.heads * m.dim
         self._memory(self._scan_args(L, m, proj, vo, work, r_off=C, a_off=C + HD, v_off=C + 2 * HD, a_bias=K.ptr(L.f_bias), lower=K.ptr(L.lower)),
-                     K.SCAN_FORGET, longest)
+                     K.SCAN_FORGET, T, longest)
         return vo
 
     # ---- forward ------------------------------------------------------------------------

@@ -248,7 +248,7 @@ def run_memory(kind, args_of, columns, ref, H, D, V, f32):
         if max(lens) == 1 and k.memory_step_takes(D, V):
             k.memory_step(args, kind, f32)
         else:
-            k.memory_scan(args, kind, f32)
+            k.memory_scan(args, kind, f32, sum(lens))
         close(out[:, :H * V], torch.cat([want[s][at[s]:at[s] + m] for s, m in enumerate(lens)]), 5e-5 if f32 else 8e-3)
         at = [a + m for a, m in zip(at, lens)]
     assert (state[1] == 7).all() and not state[2].any() and not state[:, H * V * D:][[0, 3, 5]].any() and int(st) == 0
