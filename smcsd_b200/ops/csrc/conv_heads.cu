@@ -123,62 +123,55 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeadsArgs a) 
 __device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 __device__ __forceinline__ float2 turn_by(float x, float y, float2 sc) { return make_float2(x * sc.y - y * sc.x, y * sc.y + x * sc.x); }
 
-constexpr int NH_THREADS = 512, NH_TOKENS = 16;      // tokens of a run
+constexpr int NH_THREADS = 512, NH_TOKENS = 8;       // most tokens of a run
+constexpr int NH_SMEM = 224 * 1024;                  // seven tokens of the widest rows
 
-// NV: groups of four columns per thread.
+// A run of tokens in two passes: convolved columns to shared memory with a sum of squares per token and warp, then norm, rotation and
+// stores.  Short runs, so that many CTAs share an SM: the kernel lives from loads in flight.  NV: groups of four columns per thread.
 template <int TAPS, int NV, typename AT>
-__global__ void __launch_bounds__(NH_THREADS, NV == 1 && TAPS <= 4 ? 2 : 1) normed_heads_kernel(const ConvHeadsArgs a) {
+__global__ void __launch_bounds__(NH_THREADS, NV == 1 && TAPS <= 4 ? 2 : 1) normed_heads_kernel(const ConvHeadsArgs a, int run) {
   constexpr int HL = TAPS - 1;
-  __shared__ float red[2][NH_THREADS / 32];
-  const int nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.V, C = nq + nk + nv;
+  extern __shared__ __align__(16) float4 nh_y[];     // [run][NV][blockDim.x], every thread reads what it has written
+  __shared__ float red[NH_TOKENS][NH_THREADS / 32], scale[NH_TOKENS];
+  const int nq = a.H * a.D, nk = a.G * a.D, nv = a.G * a.V, C = nq + nk + nv, nt = blockDim.x;
   const bool keys = blockIdx.y == 1;                 // keys and values, else queries
   const int base = keys ? nq : 0, n = keys ? nk + nv : nq, normed = keys ? nk : nq;      // columns of this CTA, those under the norm
-  const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (threadIdx.x * 4 >= ((n + 127) & ~127)) {       // whole warps without columns; the others meet at a barrier of their own count
-    if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, live = min(nt >> 5, (n + 127) / 128);
+  if (a.pdl) pdl_launch_dependents();
+  if (warp >= live) {                                // whole warps without columns; the others meet at a barrier of their own count
+    if (a.pdl) pdl_wait_prior_grid();
     return;
   }
-  const int live = min(nw, ((n + 127) / 128));       // warps that stay
-  int pair[NV];                                      // first of the columns' pairs in the table of angles (-1: not rotated)
-  bool two[NV];                                      // and the second as well
+  float4 w[NV][TAPS], bias[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (threadIdx.x + i * blockDim.x) * 4, value = keys && c >= nk;
-    const int col = value ? (c - nk) % a.V : c % a.D, rot = value ? a.turn : a.rot;
-    pair[i] = col < rot ? (value ? a.v_first : a.qk_first) + (col >> 1) : -1;
-    two[i] = col + 2 < rot;
-  }
-  float4 w[NV][TAPS], bias[NV], g[NV];
-#pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int c = (threadIdx.x + i * blockDim.x) * 4;
-    bias[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int c = (tid + i * nt) * 4;
+    bias[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < n) {
       bias[i] = load4(a.bias + base + c);
-      if (c < normed) g[i] = load4(a.qk_norm + base + c);
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) w[i][j] = load4(a.conv + (size_t)j * C + base + c);
     }
   }
-  if (a.pdl) { pdl_launch_dependents(); pdl_wait_prior_grid(); }
+  if (a.pdl) pdl_wait_prior_grid();
   const RaggedBlock b = ragged_block(a.r, blockIdx.x);
-  const int first = blockIdx.z * NH_TOKENS;
+  const int first = blockIdx.z * run;
   if (first >= b.n) return;
   if (HL > 0 && (b.row < 0 || b.row >= a.n_rows)) {
-    if (threadIdx.x == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
+    if (tid == 0) atomicOr(a.status, SMC_ERR_BOUNDS);
     return;
   }
   const float* src = a.proj + (size_t)b.off * a.ldp + base;
-  const int t0 = b.start + first, t1 = b.start + min(b.n, first + NH_TOKENS);
-  float4 win[NV][HL > 0 ? HL : 1], u[NV];            // win[i][j]: biased projection of token t - HL + j
+  const int t0 = b.start + first, m = min(b.n - first, run);
+  float4 win[NV][HL > 0 ? HL : 1];                   // win[i][j]: biased projection of token t - HL + j
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    const int c = (tid + i * nt) * 4;
     if (c >= n) continue;
     float* hp = a.hist + (size_t)b.row * a.row_stride + base + c;
 #pragma unroll
     for (int j = 0; j < HL; ++j) {
-      const int t = t0 - HL + j;
+      const int t = t0 - HL + j;                     // a run is no shorter than the history: only the sequence's first one reads it
       win[i][j] = t >= 0 ? add4(load4(src + (size_t)t * a.ldp + c), bias[i]) : load4((const float*)hp + (size_t)(HL + t) * C);
     }
     if (t0 == 0) {                                   // the last HL of old and new ones; nobody else reads the old ones
@@ -196,49 +189,69 @@ __global__ void __launch_bounds__(NH_THREADS, NV == 1 && TAPS <= 4 ? 2 : 1) norm
         store4(hp + (size_t)j * C, v);
       }
     }
-    u[i] = load4(src + (size_t)t0 * a.ldp + c);
   }
-  const float count = (float)((keys ? a.G : a.H) * a.dim);
-  for (int t = t0; t < t1; ++t) {
-    const int tok = b.off + t;
-    float4 y[NV];
-    float2 turn[NV][2];                              // sine and cosine, fetched ahead of the barrier
+#pragma unroll 4
+  for (int k = 0; k < m; ++k) {
     float ss = 0.f;
-    int page = keys ? a.locs[tok] : 0;
-    const float2* ang = a.angles + (size_t)tok * a.ld_angles;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      const int c = (tid + i * nt) * 4;
       if (c >= n) continue;
-      const float4 now = add4(u[i], bias[i]);
-      if (t + 1 < t1) u[i] = load4(src + (size_t)(t + 1) * a.ldp + c);
-      y[i] = mul4(w[i][HL], now);
+      const float4 now = add4(load4(src + (size_t)(t0 + k) * a.ldp + c), bias[i]);
+      float4 y = mul4(w[i][HL], now);
 #pragma unroll
-      for (int j = 0; j < HL; ++j) y[i] = fma4(w[i][j], win[i][j], y[i]);
+      for (int j = 0; j < HL; ++j) y = fma4(w[i][j], win[i][j], y);
 #pragma unroll
       for (int j = 0; j + 1 < HL; ++j) win[i][j] = win[i][j + 1];
       if (HL > 0) win[i][HL > 0 ? HL - 1 : 0] = now;
-      if (c < normed) ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
-      turn[i][0] = turn[i][1] = make_float2(0.f, 1.f);
-      if (pair[i] >= 0) turn[i][0] = ang[pair[i]];
-      if (pair[i] >= 0 && two[i]) turn[i][1] = ang[pair[i] + 1];
+      nh_y[(k * NV + i) * nt + tid] = y;
+      if (c < normed) ss = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, fmaf(y.w, y.w, ss))));
     }
-    float* rd = red[t & 1];                          // the buffers alternate: one barrier per token
     ss = warp_sum(ss);
-    if (lane == 0) rd[warp] = ss;
-    asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
-    const float inv = 1.0f / sqrtf(warp_sum(lane < live ? rd[lane] : 0.f) / count + a.eps);
+    if (lane == 0) red[k][warp] = ss;
+  }
+  asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
+  const float count = (float)((keys ? a.G : a.H) * a.dim);
+  for (int k = warp; k < m; k += live) {
+    const float ss = warp_sum(lane < live ? red[k][lane] : 0.f);
+    if (lane == 0) scale[k] = 1.0f / sqrtf(ss / count + a.eps);
+  }
+  int pair[NV];                                      // first of the columns' pairs in the table of angles (-1: not rotated)
+  bool two[NV];                                      // and the second as well
+  float4 g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (tid + i * nt) * 4, value = keys && c >= nk;
+    const int col = value ? (c - nk) % a.V : c % a.D, rot = value ? a.turn : a.rot;
+    pair[i] = col < rot ? (value ? a.v_first : a.qk_first) + (col >> 1) : -1;
+    two[i] = col + 2 < rot;
+    g[i] = c < normed ? load4(a.qk_norm + base + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  asm volatile("bar.sync 1, %0;" ::"r"(live * 32) : "memory");
+#pragma unroll 4
+  for (int k = 0; k < m; ++k) {
+    const int tok = b.off + t0 + k;
+    const float inv = scale[k];
+    const float2* ang = a.angles + (size_t)tok * a.ld_angles;
+    int page = keys ? a.locs[tok] : 0;
     if (page < 0 || page > a.n_pages) { atomicOr(a.status, SMC_ERR_BOUNDS); page = 0; }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      const int c = (tid + i * nt) * 4;
       if (c >= n) continue;
-      float4 v = y[i];
+      float4 v = nh_y[(k * NV + i) * nt + tid];
       if (c < normed) v = make_float4(v.x * inv * g[i].x, v.y * inv * g[i].y, v.z * inv * g[i].z, v.w * inv * g[i].w);
-      const float2 lo = turn_by(v.x, v.y, turn[i][0]), hi = turn_by(v.z, v.w, turn[i][1]);
+      if (pair[i] >= 0) {
+        const float2 lo = turn_by(v.x, v.y, ang[pair[i]]);
+        v.x = lo.x; v.y = lo.y;
+        if (two[i]) {
+          const float2 hi = turn_by(v.z, v.w, ang[pair[i] + 1]);
+          v.z = hi.x; v.w = hi.y;
+        }
+      }
       AT* out = !keys ? reinterpret_cast<AT*>(a.q) + (size_t)tok * nq + c
                       : c < nk ? reinterpret_cast<AT*>(a.kpool) + (size_t)page * nk + c : reinterpret_cast<AT*>(a.vpool) + (size_t)page * nv + (c - nk);
-      store4(out, make_float4(lo.x, lo.y, hi.x, hi.y));
+      store4(out, v);
     }
   }
 }
@@ -278,8 +291,15 @@ static int conv_heads_launch(const ConvHeadsArgs& a, cudaStream_t st) {
 }
 
 template <typename AT, int NV>
-static int normed_heads_taps(const ConvHeadsArgs& a, dim3 grid, dim3 block, cudaStream_t st) {
-#define SMC_NH(N) case N: return launch_pdl(normed_heads_kernel<N, NV, AT>, grid, block, 0, st, a.pdl, a);
+static int normed_heads_taps(const ConvHeadsArgs& a, int threads, cudaStream_t st) {
+  int run = a.r.B < NH_TOKENS ? a.r.B : NH_TOKENS;
+  if (run > NH_SMEM / (NV * threads * 16)) run = NH_SMEM / (NV * threads * 16);      // seven at the least: as long as any history
+  const int smem = run * NV * threads * 16;
+  const dim3 grid(a.r.n_blk, 2, (a.r.B + run - 1) / run), block(threads);
+#define SMC_NH(N)                                                                                                              \
+  case N:                                                                                                                      \
+    CUDA_CHECK_RET(cudaFuncSetAttribute(normed_heads_kernel<N, NV, AT>, cudaFuncAttributeMaxDynamicSharedMemorySize, NH_SMEM)); \
+    return launch_pdl(normed_heads_kernel<N, NV, AT>, grid, block, smem, st, a.pdl, a, run);
   switch (a.taps) { SMC_NH(1) SMC_NH(2) SMC_NH(3) SMC_NH(4) SMC_NH(5) SMC_NH(6) SMC_NH(7) SMC_NH(8) }
 #undef SMC_NH
   return -92;
@@ -290,10 +310,9 @@ static int normed_heads_launch(const ConvHeadsArgs& a, cudaStream_t st) {
   int most = a.H * a.D;
   if (a.G * (a.D + a.V) > most) most = a.G * (a.D + a.V);
   const int groups = (most / 4 + 31) / 32 * 32;
-  const dim3 grid(a.r.n_blk, 2, (a.r.B + NH_TOKENS - 1) / NH_TOKENS);
-  if (groups <= NH_THREADS) return normed_heads_taps<AT, 1>(a, grid, dim3(groups), st);
-  if (groups <= NH_THREADS * 2) return normed_heads_taps<AT, 2>(a, grid, dim3(NH_THREADS), st);
-  if (groups <= NH_THREADS * 4) return normed_heads_taps<AT, 4>(a, grid, dim3(NH_THREADS), st);
+  if (groups <= NH_THREADS) return normed_heads_taps<AT, 1>(a, groups, st);
+  if (groups <= NH_THREADS * 2) return normed_heads_taps<AT, 2>(a, NH_THREADS, st);
+  if (groups <= NH_THREADS * 4) return normed_heads_taps<AT, 4>(a, NH_THREADS, st);
   return -95;
 }
 
