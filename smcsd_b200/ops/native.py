@@ -604,6 +604,7 @@ def gdn_chunked_supported(dk: int, dv: int) -> bool:
 
 
 _KERNELS_PER_CALL["smc_gdn_step"] = 2
+_KERNELS_PER_CALL["smc_memory_scan with operands"] = 2
 
 
 # ----------------------------------------------------------------------------- layered architectures
@@ -915,7 +916,8 @@ def memory_scan(a: ScanArgs, kind: int, f32: bool, T: int = 0) -> None:
     SCAN_GATED, SCAN_CHANNEL or SCAN_FORGET; the last two run over ``T`` tokens in all and overwrite their operands."""
     if kind in (SCAN_CHANNEL, SCAN_FORGET) and T < 1:
         raise ValueError("the number of tokens is missing")
-    _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), T, int(f32), _stream()), "smc_memory_scan")
+    _check(layered_lib().smc_memory_scan(C.byref(a), int(kind), T, int(f32), _stream()),
+           "smc_memory_scan with operands" if kind in (SCAN_CHANNEL, SCAN_FORGET) else "smc_memory_scan")
 
 
 def gated_step_takes(D: int, V: int) -> bool:
